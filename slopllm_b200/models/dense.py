@@ -11,6 +11,7 @@ Reference: `src/qwen3_model.ts:1-187`, `src/qwen35_model.ts:1-467`.
 """
 from __future__ import annotations
 
+import functools
 import json
 import os
 from dataclasses import dataclass, field
@@ -18,11 +19,12 @@ from typing import Dict, List, Optional
 
 import torch
 
-from ..config import PAGE_SIZE
+from ..kv.hybrid import CacheSpec, HybridCache
 from ..ops import dense as D
 from ..ops import get_ops, recurrent as RC
 from ..parallel.dist import Comm, ParallelContext
 from ..utils.tracing import traced
+from .stack import DecoderStack, Sublayer, token_ranges
 from .weights import LinearWeight
 
 
@@ -145,107 +147,46 @@ class DenseWeights:
     vocab_offset: int = 0
 
 
-class DenseCache:
-    """Paged bf16 K/V per full-attention layer; conv + recurrent state per linear-attention layer
-    (indexed by a per-sequence state slot).  Reference: `PagedKVCache` dense layout and recurrent
-    layers (`src/paged_kv.ts:82-106`, `Qwen35ChatCache`)."""
+def dense_cache_specs(cfg: DenseConfig, tp: int = 1) -> List[CacheSpec]:
+    """Paged K/V rows per full-attention layer; conv + recurrent state per linear-attention layer."""
+    n_kv = max(1, cfg.num_key_value_heads // tp)
+    lh = max(1, cfg.linear_num_key_heads // tp)
+    cdim = lh * (2 * cfg.linear_key_head_dim + cfg.linear_value_head_dim)
+    full = CacheSpec(rows={"k": (n_kv, cfg.head_dim), "v": (n_kv, cfg.head_dim)})
+    lin = CacheSpec(state={"conv": (cdim, cfg.linear_conv_kernel_dim - 1),
+                           "rec": (lh, cfg.linear_key_head_dim, cfg.linear_value_head_dim)})
+    return [full if kind == "full_attention" else lin for kind in cfg.layer_types]
+
+
+class DenseCache(HybridCache):
+    """:class:`HybridCache` of a Qwen3 / Qwen3.5 decoder, with the tensors by layer number."""
 
     def __init__(self, cfg: DenseConfig, num_pages: int, device, tp: int = 1, max_states: int = 64, dtype=torch.bfloat16):
-        self.num_pages, self.page_size = num_pages, PAGE_SIZE
-        n_kv = max(1, cfg.num_key_value_heads // tp)
-        lh = max(1, cfg.linear_num_key_heads // tp)
-        self.k, self.v, self.conv, self.rec = {}, {}, {}, {}
-        for i, kind in enumerate(cfg.layer_types):
-            if kind == "full_attention":
-                self.k[i] = torch.zeros(num_pages * PAGE_SIZE, n_kv, cfg.head_dim, dtype=dtype, device=device)
-                self.v[i] = torch.zeros_like(self.k[i])
-            else:
-                cdim = lh * (2 * cfg.linear_key_head_dim + cfg.linear_value_head_dim)
-                self.conv[i] = torch.zeros(max_states, cdim, cfg.linear_conv_kernel_dim - 1, dtype=torch.float32, device=device)
-                self.rec[i] = torch.zeros(max_states, lh, cfg.linear_key_head_dim, cfg.linear_value_head_dim, dtype=torch.float32,
-                                          device=device)
-        self.layers = list(range(len(cfg.layer_types)))
-        self.max_states = max_states
-
-    def copy_page(self, src: int, dst: int) -> None:
-        a, b = slice(src * PAGE_SIZE, (src + 1) * PAGE_SIZE), slice(dst * PAGE_SIZE, (dst + 1) * PAGE_SIZE)
-        for i in self.k:
-            self.k[i][b] = self.k[i][a]
-            self.v[i][b] = self.v[i][a]
-
-    def page_tensors(self):
-        """Slot-indexed tensors in a fixed order (host prefix tier); None for hybrid models, whose recurrent and
-        convolution state belongs to a sequence, not to its pages."""
-        if self.conv:
-            return None
-        return [t for i in sorted(self.k) for t in (self.k[i], self.v[i])]
-
-    def reset_state(self, slot: int) -> None:
-        for i in self.conv:
-            self.conv[i][slot].zero_()
-            self.rec[i][slot].zero_()
-
-    def nbytes(self) -> int:
-        t = list(self.k.values()) + list(self.v.values()) + list(self.conv.values()) + list(self.rec.values())
-        return sum(x.numel() * x.element_size() for x in t)
+        super().__init__(dense_cache_specs(cfg, tp), num_pages, device, max_states, dtype)
+        self.k, self.v = ({i: r[n] for i, r in enumerate(self.rows) if n in r} for n in ("k", "v"))
+        self.conv, self.rec = ({i: r[n] for i, r in enumerate(self.state) if n in r} for n in ("conv", "rec"))
 
 
-class DenseModel:
+class DenseModel(DecoderStack):
     """Forward pass of the Qwen3 / Qwen3.5 decoders over the paged cache."""
 
     def __init__(self, cfg: DenseConfig, weights: DenseWeights, ctx: Optional[ParallelContext] = None, ops=None,
                  comm: Optional[Comm] = None):
         self.cfg, self.w = cfg, weights
-        self.ctx = ctx or ParallelContext()
-        self.ops = ops or get_ops(cfg, self.ctx.device, self.ctx)
-        self.comm = comm or Comm(self.ctx)
-        # linear-attention state needs one slot per live sequence; prefix sharing cannot restore it
-        self.supports_prefix_sharing = "linear_attention" not in cfg.layer_types
-        self._slot_of: Dict[int, int] = {}
-        self._free_slots: List[int] = []
-        self._state_idx: Optional[torch.Tensor] = None
-        self._cache: Optional[DenseCache] = None
+        ctx = ctx or ParallelContext()
+        self.specs = dense_cache_specs(cfg, ctx.world)
+        self.sublayers = []
+        for i, lw in enumerate(weights.layers):
+            mixer = self._full_attention if lw.kind == "full_attention" else self._linear_attention
+            self.sublayers.append(Sublayer(functools.partial(mixer, i, lw), lw.input_norm))
+            self.sublayers.append(Sublayer(functools.partial(self._mlp, lw), lw.post_attn_norm))
+        self._init_stack(ctx, ops or get_ops(cfg, ctx.device, ctx), comm,
+                         torch.bfloat16 if ctx.device.type == "cuda" else torch.float32)
 
-    # ---- engine hooks ----------------------------------------------------------------------------------
-    def allocate_cache(self, num_pages: int, max_states: int = 64) -> DenseCache:
-        self._cache = DenseCache(self.cfg, num_pages, self.ctx.device, self.ctx.world, max_states,
-                                 dtype=torch.bfloat16 if self.ctx.device.type == "cuda" else torch.float32)
-        self._free_slots = list(range(max_states - 1, -1, -1))
-        self._state_idx = torch.zeros(max_states, dtype=torch.int32, device=self.ctx.device)
-        return self._cache
-
-    def prepare_step(self, st, seqs) -> None:
-        """Host-side, outside any graph capture: give every sequence a recurrent-state slot (zeroed
-        on first use) and upload the slot of each batch row."""
-        if self.supports_prefix_sharing or self._cache is None:
-            return
-        slots = []
-        for s in seqs:
-            if s.seq_id not in self._slot_of:
-                if not self._free_slots:
-                    raise RuntimeError("out of recurrent-state slots")
-                self._slot_of[s.seq_id] = self._free_slots.pop()
-                self._cache.reset_state(self._slot_of[s.seq_id])
-            slots.append(self._slot_of[s.seq_id])
-        self._state_idx[: len(slots)].copy_(torch.tensor(slots, dtype=torch.int32), non_blocking=True)
-
-    def release_sequence(self, seq_id: int) -> None:
-        slot = self._slot_of.pop(seq_id, None)
-        if slot is not None:
-            self._free_slots.append(slot)
+    def _make_cache(self, num_pages: int, max_states: int) -> DenseCache:
+        return DenseCache(self.cfg, num_pages, self.ctx.device, self.ctx.world, max_states, dtype=self.cache_dtype)
 
     # ---- layers -------------------------------------------------------------------------------------------
-    def _qo_indptr(self, st):
-        """Token ranges of the step's sequences: one token per page-table row in a decode step,
-        otherwise one sequence holding every token (the engine prefills one sequence per chunk)."""
-        q = st.extra.get("qo_indptr")
-        if q is not None:
-            return q, st.extra.get("max_q", st.num_tokens)
-        T, B = st.num_tokens, st.page_table.shape[0]
-        if T == B:
-            return None, 1
-        return torch.tensor([0, T], dtype=torch.int32, device=st.input_ids.device), T
-
     @traced(lambda self, i, *a, **k: f"layer{i}.attention")
     def _full_attention(self, i: int, lw: DenseLayer, x, st, cache: DenseCache):
         cfg, ops = self.cfg, self.ops
@@ -258,7 +199,7 @@ class DenseModel:
         q_out = D.qk_norm_rope_cache(q, k, v, lw.q_norm, lw.k_norm, st.positions, st.batch_idx, st.page_table, st.page_size,
                                      cache.k[i], cache.v[i], hl, kvl, cfg.head_dim, cfg.rope_dim, cfg.rope_theta,
                                      cfg.rms_norm_eps, q_stride=qs)
-        qo, max_q = self._qo_indptr(st)
+        qo, max_q = token_ranges(st)
         o = D.paged_attention(q_out, cache.k[i], cache.v[i], st.positions, st.batch_idx, st.page_table, st.page_size,
                               cfg.scaling, qo_indptr=qo, max_q=max_q, max_kv_len=st.max_kv_len)
         if cfg.attn_output_gate:
@@ -275,36 +216,15 @@ class DenseModel:
         cdim, zdim = lh * (2 * dk + dv), lh * dv
         proj = ops.linear(x, lw.w_in)
         qkv, z, a, b = proj[:, :cdim], proj[:, cdim:cdim + zdim], proj[:, cdim + zdim:cdim + zdim + lh], proj[:, cdim + zdim + lh:]
-        qo, _ = self._qo_indptr(st)
-        if qo is None:
-            qo = torch.arange(T + 1, dtype=torch.int32, device=x.device)
-        sidx = self._state_idx if self._state_idx is not None else torch.zeros(qo.numel() - 1, dtype=torch.int32, device=x.device)
+        qo, sidx = self.scan_ranges(st)
         conv = RC.causal_conv1d(qkv, lw.conv_w, None, cache.conv[i], qo, sidx, activation=True)
         o = RC.gdn_scan(conv, a.contiguous(), b.contiguous(), lw.A_log, lw.dt_bias, cache.rec[i], qo, sidx, lh, dk, dv)
         gated = RC.rmsnorm_gated(o.reshape(T * lh, dv), z.reshape(T * lh, dv), lw.gdn_norm, cfg.rms_norm_eps)
         return ops.linear(gated.reshape(T, zdim), lw.out_proj, out_f32=True)
 
     @traced("mlp")
-    def _mlp(self, lw: DenseLayer, y):
+    def _mlp(self, lw: DenseLayer, y, st, cache):
         return self.ops.dense_mlp(y, lw)
-
-    def forward_hidden(self, st, cache: DenseCache) -> torch.Tensor:
-        ops, comm, cfg = self.ops, self.comm, self.cfg
-        partial, residual = ops.embed(st.input_ids, self.w.embed), None
-        x, residual = ops.add_rmsnorm(partial, residual, self.w.layers[0].input_norm, cfg.rms_norm_eps)
-        for i, lw in enumerate(self.w.layers):
-            attn = self._full_attention(i, lw, x, st, cache) if lw.kind == "full_attention" else self._linear_attention(i, lw, x, st, cache)
-            y, residual = comm.allreduce_add_rmsnorm(ops, attn, residual, lw.post_attn_norm, cfg.rms_norm_eps)
-            mlp = self._mlp(lw, y)
-            nxt = self.w.layers[i + 1].input_norm if i + 1 < len(self.w.layers) else self.w.final_norm
-            x, residual = comm.allreduce_add_rmsnorm(ops, mlp, residual, nxt, cfg.rms_norm_eps)
-        return x
-
-    def compute_logits(self, hidden: torch.Tensor) -> torch.Tensor:
-        local = self.ops.logits(hidden, self.w.lm_head)
-        if self.ctx.world == 1:
-            return local
-        return self.comm.all_gather(local, dim=-1)
 
 
 # ---- weights: random init (tests, benchmarks) and HF safetensors loading ------------------------------------

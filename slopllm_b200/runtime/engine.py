@@ -69,7 +69,7 @@ class StepBuffers:
 class Engine:
     def __init__(self, cfg: GlmMoeDsaConfig, model: GlmMoeDsaModel, num_pages: int, max_batch: int = 8,
                  max_seq_len: int = 16384, cuda_graph: bool = True, mtp: int = 0, sampler=None, phased_prefill: bool = False,
-                 phased_min_tokens: int = 2048):
+                 phased_min_tokens: int = 2048, max_states: int = 0):
         self.cfg = cfg
         self.model = model
         self.ctx: ParallelContext = model.ctx
@@ -77,7 +77,8 @@ class Engine:
         self.kv = PagedKVCache(num_pages, self.ctx.cp_world, copy_page=self._copy_page)
         self.kv.prefix_sharing = getattr(model, "supports_prefix_sharing", True)
         # model families bring their own cache layout (dense K/V, recurrent state); the flagship uses packed MLA rows
-        self.cache = (model.allocate_cache(num_pages) if hasattr(model, "allocate_cache")
+        # (state slots: one per live sequence; prefilling rows beyond the decode batch hold one too)
+        self.cache = (model.allocate_cache(num_pages, max_states or max(64, max_batch)) if hasattr(model, "allocate_cache")
                       else KVCacheTensors.allocate(cfg, num_pages, self.device, len(model.w.layers)))
         self.max_batch = max_batch
         self.pt_width = -(-max_seq_len // (PAGE_SIZE * self.ctx.cp_world)) + 1
@@ -241,18 +242,8 @@ class Engine:
                 budget -= n
             if not spans:
                 break
-            ids: List[int] = []
-            positions: List[int] = []
-            bidx: List[int] = []
             group = [seqs[b] for b, _, _ in spans]
-            for gi, (b, start, n) in enumerate(spans):
-                tok = list(prompts[b][start:start + n])
-                self.kv.append_tokens(seqs[b], tok)
-                ids += tok
-                positions += range(start, start + n)
-                bidx += [gi] * n
-            st = self._eager_state(ids, positions, bidx, group, max_kv_len=max(start + n for _, start, n in spans))
-            self._prepare(st, group)
+            st, ids, positions = self._pack(group, [list(prompts[b][start:start + n]) for b, start, n in spans])
             if len(spans) == 1 and self.phased_prefill and spans[0][2] >= self.phased_min_tokens:
                 _, start, n = spans[0]
                 hidden = self._forward_phased(ids, positions, group[0], start, n)
@@ -279,6 +270,51 @@ class Engine:
             hiddens.append(last_hidden[b])
         self.check_device_errors()           # (the token reads above already synchronised the stream)
         return tokens, (hiddens if want_hidden else None)
+
+    def _pack(self, seqs: Seq[Sequence], tokens: Seq[Seq[int]]):
+        """Append each sequence's next tokens and lay the portions out as one batch.  Returns (state, ids, positions)."""
+        ids: List[int] = []
+        positions: List[int] = []
+        bidx: List[int] = []
+        for i, (s, tok) in enumerate(zip(seqs, tokens)):
+            start = s.length
+            self.kv.append_tokens(s, tok)
+            ids += tok
+            positions += range(start, start + len(tok))
+            bidx += [i] * len(tok)
+        st = self._eager_state(ids, positions, bidx, seqs, max_kv_len=max(s.length for s in seqs))
+        self._prepare(st, seqs)
+        return st, ids, positions
+
+    @traced("step")
+    def step(self, seqs: Seq[Sequence], tokens: Seq[Seq[int]], want: Optional[Seq[Seq[int]]] = None) -> Optional[torch.Tensor]:
+        """Advance several sequences by given tokens in one forward pass: portions of prompts beside single decoded tokens.
+        `want[b]` are places among `tokens[b]`; returns their logits [wanted, vocab] (fp32, in order) or None.
+
+        Prefill batches and eager steps share `_pack`; a step of single tokens takes the captured decode graph of
+        :meth:`decode_step` with the logits as its result."""
+        if any(not t for t in tokens):
+            raise ValueError("every sequence of a step brings at least one token")
+        rows: List[int] = []
+        off = 0
+        for b, t in enumerate(tokens):
+            rows += [off + w for w in (want[b] if want is not None else ())]
+            off += len(t)
+        if all(len(t) == 1 for t in tokens) and all(s.length > 0 for s in seqs):
+            logits = self._decode_graph(seqs, [t[0] for t in tokens], "decode_logits", None,
+                                        lambda hidden: self.model.compute_logits(hidden).to(torch.float32))
+            out = logits[rows] if rows else None
+        else:
+            st, _, _ = self._pack(seqs, [list(t) for t in tokens])
+            hidden = self.model.forward_hidden(st, self.cache)
+            out = None
+            if rows:
+                idx = torch.as_tensor(rows, dtype=torch.int64, device=self.device)
+                out = self.model.compute_logits(hidden.index_select(0, idx)).to(torch.float32)
+        for s in seqs:
+            self.kv.report_tokens(s)
+        self.check_device_errors()
+        return out
 
     def _forward_phased(self, ids, positions, s: Sequence, start: int, n: int) -> torch.Tensor:
         half = (n // 2 + 63) // 64 * 64
@@ -326,6 +362,11 @@ class Engine:
         if hasattr(self.model, "release_sequence"):
             self.model.release_sequence(s.seq_id)
 
+    def finish(self, s: Sequence) -> None:
+        """Give back everything a sequence holds: its pages and its per-sequence state."""
+        self.kv.free_sequence(s)
+        self.release(s)
+
     def _eager_state(self, ids, positions, batch_idx, seqs, max_kv_len, logits_idx=None) -> StepState:
         dev = self.device
         width = max(self.pt_width, max(len(s.pages) for s in seqs))
@@ -337,6 +378,20 @@ class Engine:
                        max_kv_len=max_kv_len)
         # rows of one sequence share one page table: the prefill index scorer on the tensor cores takes that case
         st.extra["one_sequence"] = len(batch_idx) > 0 and min(batch_idx) == max(batch_idx)
+        # (first position, tokens) of every sequence in batch order, and the same as token ranges on the device; a step of
+        # single tokens is left to the decode kernels
+        spans: List[List[int]] = []
+        for i, b in enumerate(batch_idx):
+            if i == 0 or b != batch_idx[i - 1]:
+                spans.append([positions[i], 0])
+            spans[-1][1] += 1
+        if len(spans) == len(seqs) and any(n > 1 for _, n in spans):
+            ends = [0]
+            for _, n in spans:
+                ends.append(ends[-1] + n)
+            st.extra["spans"] = spans
+            st.extra["qo_indptr"] = torch.tensor(ends, dtype=torch.int32, device=dev)
+            st.extra["max_q"] = max(n for _, n in spans)
         return st
 
     # ---- plain decode -----------------------------------------------------------------------------------------
@@ -348,21 +403,8 @@ class Engine:
         B = len(seqs)
         rows = list(range(B)) if rows is None else list(rows)
         sampled = self.sampler is not None and not self.sampler.all_greedy(rows)
-        positions = []
-        for s, t in zip(seqs, last_tokens):
-            positions.append(s.length)
-            self.kv.append_tokens(s, [t])
-        buf = self._buffers(B, 1)
-        self._upload(buf, list(last_tokens), positions, list(range(B)), seqs)
-        bucket = R.padded_kv_len(max(positions) + 1)
-        st = self._state(buf, bucket)
-        self._prepare(st, seqs)
-
-        def run():
-            hidden = self.model.forward_hidden(st, self.cache)
-            return self._select(hidden, rows if sampled else None)
-
-        out = self.graphs.execute(("decode", B, bucket, tuple(rows) if sampled else None), run)
+        out = self._decode_graph(seqs, last_tokens, "decode", tuple(rows) if sampled else None,
+                                 lambda hidden: self._select(hidden, rows if sampled else None))
         host = self._readback(("decode", B), out)
         for s in seqs:
             self.kv.report_tokens(s)
@@ -370,6 +412,21 @@ class Engine:
         if sampled and self.sampler.uses_penalties(rows):
             self.sampler.record(rows, toks)
         return toks
+
+    def _decode_graph(self, seqs: Seq[Sequence], tokens: Seq[int], kind: str, variant, finish):
+        """Append one token per sequence and run the captured step of this batch size and KV bucket; `finish(hidden)` is
+        its last part (`kind` and `variant` name it in the graph's key).  Returns the graph's static output."""
+        B = len(seqs)
+        positions = []
+        for s, t in zip(seqs, tokens):
+            positions.append(s.length)
+            self.kv.append_tokens(s, [t])
+        buf = self._buffers(B, 1)
+        self._upload(buf, list(tokens), positions, list(range(B)), seqs)
+        bucket = R.padded_kv_len(max(positions) + 1)
+        st = self._state(buf, bucket)
+        self._prepare(st, seqs)
+        return self.graphs.execute((kind, B, bucket, variant), lambda: finish(self.model.forward_hidden(st, self.cache)))
 
     def _select(self, hidden: torch.Tensor, rows: Optional[Seq[int]], stream: int = 0) -> torch.Tensor:
         """Next tokens from hidden states: greedy arg-max, or the sampling kernel over the

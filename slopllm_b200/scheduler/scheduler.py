@@ -304,12 +304,20 @@ class GenerationScheduler:
                 req.finish_reason = req.cancel_reason or "cancelled"
             req.retired = True
             self.engine.kv.stage(r.seq)           # keep the pages for prefix reuse
+            self._release(r.seq)
             self._free_rows.append(r.row)
             if req.finish_reason in ("stop", "length"):
                 self.metrics.request_success_total += 1
             if req.on_finish:
                 req.on_finish(req)
         self.rows = keep
+
+    def _release(self, seq: Sequence) -> None:
+        """Per-sequence state outside the page pool (recurrent-state slots) goes back when its request ends; a staged
+        sequence of such a model keeps no pages, so nothing can resume it."""
+        release = getattr(self.engine, "release", None)
+        if release is not None:
+            release(seq)
 
     def _drain_events(self) -> None:
         while len(self.rows) < self.max_batch or not self.events.empty():
@@ -523,6 +531,7 @@ class GenerationScheduler:
             self._free_rows.append(r.row)
             try:
                 self.engine.kv.free_sequence(r.seq)
+                self._release(r.seq)
             except Exception:  # noqa: BLE001
                 pass
         self.rows = []
