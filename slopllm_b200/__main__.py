@@ -13,6 +13,7 @@ COMMANDS = {
     "weights-doc": "slopllm_b200.cli.weights_doc",
     "plan": "slopllm_b200.cli.plan",
     "kernel-bench": "slopllm_b200.cli.kernel_bench",
+    "trace-run": "slopllm_b200.cli.trace_run",
     "profile-step": "slopllm_b200.cli.profile_step",
     "collective-bench": "slopllm_b200.cli.collective_bench",
     "build": "slopllm_b200.build_native",

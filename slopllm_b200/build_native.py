@@ -8,8 +8,10 @@ Run `python -m slopllm_b200.build_native` (or `__graft_entry__.build()`).
 """
 from __future__ import annotations
 
+import fcntl
 import glob
 import os
+import shutil
 import subprocess
 import sys
 from concurrent.futures import ThreadPoolExecutor
@@ -43,9 +45,32 @@ def _run(cmd, log_path=None):
     return p.stdout + p.stderr
 
 
-def build_kernels(force: bool = False, verbose: bool = False) -> str:
+def _nvcc() -> str:
+    return shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
+
+
+def family_library(name: str) -> str:
+    """Library that holds one model family's kernels only."""
+    return os.path.join(LIB, f"libslopllm_kernels_{name}.so")
+
+
+def ensure_kernels(name: str, sources=None) -> str:
+    """A loadable kernel library for a model family: the complete in-tree build when it is there and current, else a library
+    of the family's own sources (`csrc/<source>.cu`), built now if need be.  Processes that get here together build once."""
+    os.makedirs(LIB, exist_ok=True)
+    with open(os.path.join(LIB, ".lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        files = glob.glob(os.path.join(CSRC, "*.cu")) + glob.glob(os.path.join(CSRC, "*.cuh")) + glob.glob(os.path.join(CSRC, "*.h"))
+        if not _newer(KERNELS_SO, files):
+            return KERNELS_SO
+        return build_kernels() if sources is None else build_kernels(sources=sources, target=family_library(name))
+
+
+def build_kernels(force: bool = False, verbose: bool = False, sources=None, target: str = KERNELS_SO) -> str:
     os.makedirs(LIB, exist_ok=True)
     cus = sorted(glob.glob(os.path.join(CSRC, "*.cu")))
+    if sources is not None:
+        cus = [cu for cu in cus if os.path.basename(cu)[:-3] in sources]
     hdrs = glob.glob(os.path.join(CSRC, "*.cuh")) + glob.glob(os.path.join(CSRC, "*.h"))
     objs = []
     jobs = []
@@ -57,15 +82,15 @@ def build_kernels(force: bool = False, verbose: bool = False) -> str:
 
     def compile_one(job):
         cu, obj = job
-        out = _run(["nvcc", *NVCC_FLAGS, "-I", CSRC, "-c", cu, "-o", obj], obj + ".log")
+        out = _run([_nvcc(), *NVCC_FLAGS, "-I", CSRC, "-c", cu, "-o", obj], obj + ".log")
         if verbose:
             print(out)
 
     with ThreadPoolExecutor(max_workers=min(8, max(1, len(jobs)))) as ex:
         list(ex.map(compile_one, jobs))
-    if jobs or force or _newer(KERNELS_SO, objs):
-        _run(["nvcc", "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", KERNELS_SO, *objs])
-    return KERNELS_SO
+    if jobs or force or _newer(target, objs):
+        _run([_nvcc(), "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", target, *objs])
+    return target
 
 
 def build_runtime(force: bool = False) -> str:

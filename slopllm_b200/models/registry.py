@@ -4,7 +4,7 @@ from __future__ import annotations
 import json
 import os
 from dataclasses import dataclass
-from typing import Callable, Dict, Optional
+from typing import Callable, Dict, Optional, Tuple
 
 import torch
 
@@ -17,7 +17,9 @@ class ModelRegistration:
     context_parallel: bool
     mtp: bool
     persistent_loader: bool
-    load: Callable            # (model_dir, ctx, mtp) -> (cfg, model)
+    load: Callable            # (model_dir, ctx, mtp[, dtype]) -> (cfg, model)
+    float32: bool = False     # also runs entirely in fp32 on a GPU (`load` then takes `dtype`)
+    kernel_sources: Optional[Tuple[str, ...]] = None     # csrc/*.cu that serve the family (None: the complete library)
 
 
 def _load_glm_moe_dsa(model_dir: str, ctx: ParallelContext, mtp: int = 0):
@@ -41,11 +43,21 @@ def _load_glm5_next(model_dir: str, ctx: ParallelContext, mtp: int = 0):
     return m.cfg, m
 
 
+def _load_gidisun(model_dir: str, ctx: ParallelContext, mtp: int = 0, dtype=None):
+    from .gidisun import load_gidisun_model
+    if dtype is None:
+        dtype = torch.bfloat16 if ctx.device.type == "cuda" else torch.float32
+    return load_gidisun_model(model_dir, ctx, dtype)
+
+
 MODEL_REGISTRY: Dict[str, ModelRegistration] = {
     "glm_moe_dsa": ModelRegistration(True, True, True, True, _load_glm_moe_dsa),
     "glm5_next": ModelRegistration(False, False, False, True, _load_glm5_next),
     "qwen3": ModelRegistration(False, False, False, True, _load_dense),
     "qwen3_5": ModelRegistration(False, False, False, False, _load_dense),
+    "gidisun": ModelRegistration(False, False, False, False, _load_gidisun, float32=True,
+                                 kernel_sources=("elementwise", "gated_scan", "gemm_tcgen05", "gemv", "latent_attn", "linear_simt",
+                                                 "sampling", "sandwich_norm", "sparse_mla")),
 }
 
 
@@ -62,6 +74,8 @@ def inspect_model(model_dir: str, cp: bool = False, mtp: int = 0):
     with open(path) as f:
         config = json.load(f)
     mt = config.get("model_type")
+    if mt is None and isinstance(config.get("architecture"), str):
+        mt = config["architecture"].lower()
     if not isinstance(mt, str) or mt not in MODEL_REGISTRY:
         raise ValueError(f"unsupported model_type {mt!r} in {path}; supported types: {', '.join(MODEL_REGISTRY)}")
     reg = MODEL_REGISTRY[mt]
@@ -72,7 +86,16 @@ def inspect_model(model_dir: str, cp: bool = False, mtp: int = 0):
     return mt, reg, config
 
 
-def load_any(model_dir: str, ctx: Optional[ParallelContext] = None, mtp: int = 0):
+def load_registered(reg: ModelRegistration, model_dir: str, ctx: ParallelContext, mtp: int = 0, dtype: Optional[str] = None):
+    """`dtype`: "bfloat16" / "float32" (None: bfloat16 on a GPU, float32 on the CPU)."""
+    if dtype is None or (dtype == "bfloat16") == (ctx.device.type == "cuda"):
+        return reg.load(model_dir, ctx, mtp)
+    if not reg.float32:
+        raise ValueError(f"{model_dir}: this model family does not run in {dtype} on {ctx.device.type}")
+    return reg.load(model_dir, ctx, mtp, dtype=getattr(torch, dtype))
+
+
+def load_any(model_dir: str, ctx: Optional[ParallelContext] = None, mtp: int = 0, dtype: Optional[str] = None):
     ctx = ctx or ParallelContext()
     _, reg, _ = inspect_model(model_dir, cp=ctx.cp, mtp=mtp)
-    return reg.load(model_dir, ctx, mtp)
+    return load_registered(reg, model_dir, ctx, mtp, dtype)

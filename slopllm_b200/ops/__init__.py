@@ -39,6 +39,14 @@ class RefOps:
     def add_rmsnorm(self, x, residual, w, eps=None, want_perm: bool = False):
         return R.add_rmsnorm(x, residual, w, self.cfg.rms_norm_eps if eps is None else eps)
 
+    def embed_norm(self, ids, table, w_next, eps):
+        r = self.embed(ids, table)
+        return R.rmsnorm(r, w_next, eps), r
+
+    def post_norm(self, y, residual, w_post, w_next, eps):
+        r = residual + R.rmsnorm(y, w_post, eps)
+        return R.rmsnorm(r, w_next, eps), r
+
     def linear(self, x, w, out_f32: bool = False, sink=None, defer_reduce: bool = False):
         return R.linear(x, w)
 
@@ -150,11 +158,12 @@ class RefOps:
         return logits.argmax(-1)
 
 
-def get_ops(cfg, device, ctx=None):
+def get_ops(cfg, device, ctx=None, dtype=torch.bfloat16):
+    """`dtype`: activation type on a GPU (the CPU definitions always compute in fp32)."""
     device = torch.device(device)
     if device.type == "cuda":
         from .cuda_ops import CudaOps
-        return CudaOps(cfg, ctx)
+        return CudaOps(cfg, ctx, dtype)
     return RefOps(cfg, ctx)
 
 

@@ -48,9 +48,10 @@ class CudaOps:
     name = "cuda"
     act_dtype = torch.bfloat16
 
-    def __init__(self, cfg, ctx=None):
+    def __init__(self, cfg, ctx=None, act_dtype=torch.bfloat16):
         self.cfg = cfg
         self.ctx = ctx
+        self.act_dtype = act_dtype      # fp32: families whose kernels exist in both types (every product on the CUDA cores)
         N.kernels()            # fail loudly when the native library is missing
         self._counters = {}
         from ..config import env_str
@@ -92,6 +93,29 @@ class CudaOps:
                float(eps), int(x.dtype == torch.float32), N.ptr(xp), N.stream())
         return out, res
 
+    def _post_norm(self, T: int, H: int, w_next, eps, dev, **src):
+        out = torch.empty(T, H, dtype=self.act_dtype, device=dev)
+        res = torch.empty(T, H, dtype=torch.float32, device=dev)
+        p = N.PostNormParams(out=out.data_ptr(), out_f32=int(self.act_dtype == torch.float32), res_out=res.data_ptr(),
+                             w_next=w_next.data_ptr(), H=H, eps=float(eps), **src)
+        N.call("sl_post_norm", C.byref(p), T, N.stream())
+        return out, res
+
+    def embed_norm(self, ids, table, w_next, eps):
+        """Residual stream from the embedding table and its RMS norm (fp32 weight).  Returns (normed, residual)."""
+        T, H = ids.shape[0], table.shape[1]
+        ids = ids.to(torch.int64).contiguous()
+        return self._post_norm(T, H, w_next, eps, table.device, ids=ids.data_ptr(), table=table.data_ptr(),
+                               table_f32=int(table.dtype == torch.float32), vocab=table.shape[0])
+
+    def post_norm(self, y, residual, w_post, w_next, eps):
+        """residual' = residual + rms(y) * w_post; returns (rms(residual') * w_next, residual').  fp32 weights and sums."""
+        if y.dtype != torch.float32 or y.stride(-1) != 1:
+            y = y.to(torch.float32).contiguous()
+        T, H = y.shape
+        return self._post_norm(T, H, w_next, eps, y.device, y=y.data_ptr(), ldy=y.stride(0), w_post=w_post.data_ptr(),
+                               res_in=residual.data_ptr())
+
     @staticmethod
     def _perm_of(x, T: int, K: int):
         """The permuted f16 copy that x's producer left with it, if it has the shape this consumer needs."""
@@ -112,6 +136,8 @@ class CudaOps:
         stored straight into the peers' memory by the producing kernel and the sink is returned.
         With `defer_reduce` a split-K product may come back as `SplitKSlabs` (fp32 partial sums the
         consumer adds up while it loads them); only `attn_pre` and `q_post` accept that form."""
+        if w.weight.dtype == torch.float32:
+            return self._linear_simt(x.to(torch.float32), w, True)
         x = self._bf16(x)
         if x.stride(-1) != 1:
             x = x.contiguous()
@@ -119,6 +145,9 @@ class CudaOps:
         Nn = w.out_features
         if getattr(w, "is_fp8", False):
             return self._linear_fp8(x, w, out_f32, sink)
+        if sink is None and not w.is_nvfp4 and (K % 8 or x.stride(0) % 8 or w.weight.stride(0) % 8 or x.data_ptr() % 16
+                                                or w.weight.data_ptr() % 16):
+            return self._linear_simt(x, w, out_f32)      # rows that TMA and 16-byte loads cannot address
         if sink is not None and hasattr(sink, "rs"):
             # prefill-sized partial sum: the GEMM's epilogue sends each tile row to the rank that owns it
             from . import tcgen05
@@ -175,6 +204,18 @@ class CudaOps:
         else:
             N.call("sl_gemv_bf16", y.data_ptr(), x.data_ptr(), w.weight.data_ptr(), T, Nn, K, x.stride(0), int(out_f32),
                    N.stream())
+        return y
+
+    def _linear_simt(self, x, w, out_f32: bool):
+        """y = x @ W^T on the CUDA cores, fp32 accumulation: fp32 weights, or bf16 rows of any alignment."""
+        if x.stride(-1) != 1:
+            x = x.contiguous()
+        T, K = x.shape
+        wt = w.weight
+        y = torch.empty(T, wt.shape[0], dtype=torch.float32 if out_f32 else torch.bfloat16, device=x.device)
+        p = N.SimtLinearParams(y=y.data_ptr(), x=x.data_ptr(), w=wt.data_ptr(), T=T, N=wt.shape[0], K=K, batch=1, y_t=y.stride(0),
+                               x_t=x.stride(0), w_n=wt.stride(0), w_k=wt.stride(1))
+        N.call("sl_linear_simt", C.byref(p), int(wt.dtype == torch.float32), int(out_f32), N.stream())
         return y
 
     FP8_GEMV_MAX_T = 8         # token rows served by the FP8 weight-streaming kernel in one pass over the weights
@@ -473,8 +514,8 @@ class CudaOps:
         if gu.stride(0) != gu.shape[1]:
             gu = gu.contiguous()
         T, I2 = gu.shape
-        act = torch.empty(T, I2 // 2, dtype=torch.bfloat16, device=x.device)
-        N.call("sl_silu_mul", act.data_ptr(), gu.data_ptr(), T, I2 // 2, N.stream())
+        act = torch.empty(T, I2 // 2, dtype=gu.dtype, device=x.device)
+        N.call("sl_silu_mul_f32" if gu.dtype == torch.float32 else "sl_silu_mul", act.data_ptr(), gu.data_ptr(), T, I2 // 2, N.stream())
         return self.linear(act, lw.mlp_w2, out_f32=True, sink=sink)
 
     def route(self, x, lw):

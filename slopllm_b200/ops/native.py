@@ -29,34 +29,51 @@ class CollectiveTimeout(RuntimeError):
     """A device-side bounded wait expired (a peer did not publish its flag in time)."""
 
 
+_chosen = None
+
+
+def use_library(path: str) -> None:
+    """Load this kernel library (a family's own build) instead of the complete one; call before the first kernel."""
+    global _chosen
+    _chosen = path
+
+
+def _library_path() -> str:
+    """The kernel library to load: an explicit choice (`use_library`, `SLOPLLM_B200_KERNELS_SO`), else the complete in-tree
+    build."""
+    path = os.environ.get("SLOPLLM_B200_KERNELS_SO") or _chosen or KERNELS_SO
+    if not os.path.exists(path):
+        raise NativeError(f"{path} is missing: run `python -m slopllm_b200.build_native` "
+                          "(the CUDA path has no PyTorch fallback)")
+    return path
+
+
+# kernel choices that can be switched for comparison runs: setter -> value.  A library built for one model family may lack some.
+def _switches():
+    off = lambda name: 0 if os.environ.get("SLOPLLM_B200_" + name, "1") == "0" else 1
+    return {
+        "sl_set_pdl": off("PDL"),                  # programmatic dependent launch between the library's kernels
+        "sl_indexer_set_tiled": off("INDEXER_TILED"),
+        "sl_indexer_set_tcgen05": off("INDEXER_TCGEN05"),
+        "sl_sparse_mla_set_transposed": off("MLA_TRANSPOSED"),
+        # 0 = mma.sync everywhere, prefill = tcgen05 only where the kernel writes the final output, anything else (default) =
+        # also the key-split launches of decode
+        "sl_sparse_mla_set_tcgen05": {"0": 0, "prefill": 1}.get(os.environ.get("SLOPLLM_B200_MLA_TCGEN05", "1"), 3),
+    }
+
+
 @lru_cache(maxsize=None)
 def kernels() -> C.CDLL:
-    if not os.path.exists(KERNELS_SO):
-        raise NativeError(f"{KERNELS_SO} is missing: run `python -m slopllm_b200.build_native` "
-                          "(the CUDA path has no PyTorch fallback)")
-    lib = C.CDLL(os.environ.get("SLOPLLM_B200_KERNELS_SO", KERNELS_SO))
-    # programmatic dependent launch between the library's kernels; SLOPLLM_B200_PDL=0 turns it off
-    lib.sl_set_pdl.argtypes = [i32]
-    lib.sl_set_pdl.restype = None
-    lib.sl_set_pdl(0 if os.environ.get("SLOPLLM_B200_PDL", "1") == "0" else 1)
-    lib.sl_indexer_set_tiled.argtypes = [i32]
-    lib.sl_indexer_set_tiled.restype = None
-    lib.sl_indexer_set_tiled(0 if os.environ.get("SLOPLLM_B200_INDEXER_TILED", "1") == "0" else 1)
-    lib.sl_indexer_set_tcgen05.argtypes = [i32]
-    lib.sl_indexer_set_tcgen05.restype = None
-    lib.sl_indexer_set_tcgen05(0 if os.environ.get("SLOPLLM_B200_INDEXER_TCGEN05", "1") == "0" else 1)
-    lib.sl_sparse_mla_direct_ok.argtypes = [i32, i32, i32]
-    lib.sl_sparse_mla_direct_ok.restype = i32
-    lib.sl_sparse_mla_set_transposed.argtypes = [i32]
-    lib.sl_sparse_mla_set_transposed.restype = None
-    lib.sl_sparse_mla_set_transposed(0 if os.environ.get("SLOPLLM_B200_MLA_TRANSPOSED", "1") == "0" else 1)
-    lib.sl_sparse_mla_set_tcgen05.argtypes = [i32]
-    lib.sl_sparse_mla_set_tcgen05.restype = None
-    # SLOPLLM_B200_MLA_TCGEN05: 0 = mma.sync everywhere, prefill = tcgen05 only where the kernel writes the final output,
-    # anything else (default) = also the key-split launches of decode
-    lib.sl_sparse_mla_set_tcgen05({"0": 0, "prefill": 1}.get(os.environ.get("SLOPLLM_B200_MLA_TCGEN05", "1"), 3))
-    lib.sl_sparse_mla_tcgen05_decode_ok.argtypes = [i32, i32, i32, i32, i32]
-    lib.sl_sparse_mla_tcgen05_decode_ok.restype = i32
+    lib = C.CDLL(_library_path())
+    for name, value in _switches().items():
+        if hasattr(lib, name):
+            f = getattr(lib, name)
+            f.argtypes, f.restype = [i32], None
+            f(value)
+    for name, n_args in (("sl_sparse_mla_direct_ok", 3), ("sl_sparse_mla_tcgen05_decode_ok", 5)):
+        if hasattr(lib, name):
+            getattr(lib, name).argtypes = [i32] * n_args
+            getattr(lib, name).restype = i32
     return lib
 
 
@@ -178,9 +195,25 @@ class SpecRejectParams(C.Structure):
                 ("D", i32), ("C", i32), ("counter", vp), ("out_tokens", vp), ("num_accepted", vp)]
 
 
+class SimtLinearParams(C.Structure):
+    _fields_ = [("y", vp), ("x", vp), ("w", vp), ("T", i32), ("N", i32), ("K", i32), ("batch", i32), ("y_t", i64), ("y_b", i64),
+                ("x_t", i64), ("x_b", i64), ("w_n", i64), ("w_k", i64), ("w_b", i64)]
+
+
+class PostNormParams(C.Structure):
+    _fields_ = [("out", vp), ("out_f32", i32), ("res_out", vp), ("y", vp), ("ldy", i32), ("w_post", vp), ("res_in", vp), ("ids", vp),
+                ("table", vp), ("table_f32", i32), ("vocab", i32), ("w_next", vp), ("H", i32), ("eps", f32)]
+
+
 # ---- function signatures ----------------------------------------------------------------------------------
 
 _SIGS = {
+    "sl_linear_simt": [C.POINTER(SimtLinearParams), i32, i32, vp],
+    "sl_silu_mul_f32": [vp, vp, i32, i32, vp],
+    "sl_post_norm": [C.POINTER(PostNormParams), i32, vp],
+    "sl_latent_pre": [vp, i32, i32, vp],
+    "sl_latent_rows": [vp, i32, i32, vp],
+    "sl_gated_step": [vp, i32, i32, i32, i32, vp],
     "sl_embed": [vp, vp, vp, i32, i32, i32, vp],
     "sl_add_rmsnorm": [vp, vp, vp, vp, vp, i32, i32, f32, i32, vp, vp],
     "sl_attn_pre": [C.POINTER(AttnPreParams), i32, vp],

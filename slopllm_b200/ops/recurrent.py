@@ -1,5 +1,6 @@
 """Recurrent sub-layer ops of the hybrid families: Gated DeltaNet (Qwen3.5), KDA and manifold
-hyper-connections (glm5_next).  CUDA tensors run the sm_100a kernels of `csrc/recurrent.cu`;
+hyper-connections (glm5_next), GLA and mLSTM (Gidisun).  CUDA tensors run the sm_100a kernels of
+`csrc/recurrent.cu` and `csrc/gated_scan.cu`;
 CPU tensors run the fp32 definitions in `ops/reference.py` (the oracle of the GPU tests).
 """
 from __future__ import annotations
@@ -90,6 +91,94 @@ def kda_scan(qkv, forget, b, A_log, dt_bias, state, qo_indptr, state_idx, h: int
             out[lo:hi], state[slot] = R.kda_scan(q[lo:hi], k[lo:hi], v[lo:hi], forget[lo:hi].reshape(hi - lo, h, dk), b[lo:hi], A_log,
                                                  dt_bias.reshape(h, dk), state[slot], lower_bound)
     return out.to(torch.bfloat16)
+
+
+# ---- gated outer-product recurrences: GLA and mLSTM --------------------------------------------------------------------------
+
+class GatedScanParams(C.Structure):
+    _fields_ = [("out", C.c_void_p), ("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("g", C.c_void_p), ("ld", C.c_int),
+                ("gates", C.c_void_p), ("ld_gates", C.c_int), ("a2", C.c_void_p), ("a2_b", C.c_void_p), ("rank", C.c_int),
+                ("inv_tau", C.c_float), ("i_b", C.c_void_p), ("f_b", C.c_void_p), ("cap", C.c_float), ("norm_w", C.c_void_p),
+                ("eps", C.c_float), ("S", C.c_void_p), ("n", C.c_void_p), ("m", C.c_void_p), ("qo_indptr", C.c_void_p),
+                ("state_idx", C.c_void_p), ("h", C.c_int), ("dk", C.c_int), ("dv", C.c_int)]
+
+
+KIND_GLA, KIND_MLSTM = 0, 1
+
+
+def _gated_params(p_in, h, dk, dv, out, norm_w, eps, qo_indptr, state_idx) -> GatedScanParams:
+    esz = p_in.element_size()
+    base = p_in.data_ptr()
+    return GatedScanParams(out=out.data_ptr(), q=base, k=base + h * dk * esz, v=base + 2 * h * dk * esz,
+                           g=base + (2 * h * dk + h * dv) * esz, ld=p_in.stride(0), norm_w=norm_w.data_ptr(), eps=float(eps),
+                           qo_indptr=qo_indptr.data_ptr(), state_idx=state_idx.data_ptr(), h=h, dk=dk, dv=dv)
+
+
+def _run_gated(kind: int, p: GatedScanParams, proj, out, qo_indptr) -> torch.Tensor:
+    N = _native()
+    N.call("sl_gated_step", C.byref(p), qo_indptr.numel() - 1, kind, int(proj.dtype == torch.float32), int(out.dtype == torch.float32),
+           N.stream())
+    return out
+
+
+def _qkvg(proj, h, dk, dv):
+    T = proj.shape[0]
+    q, k, v, g = torch.split(proj[:, :h * (2 * dk + 2 * dv)].to(torch.float32), [h * dk, h * dk, h * dv, h * dv], dim=1)
+    return q.reshape(T, h, dk) * dk ** -0.5, k.reshape(T, h, dk), v.reshape(T, h, dv), g.reshape(T, h, dv)
+
+
+def gla_mix(proj, low, a2, a2_b, tau: float, norm_w, eps: float, state, qo_indptr, state_idx, h: int, dk: int, dv: int, out_dtype):
+    """Gated linear attention over the token ranges of B sequences, up to the output projection.
+
+    proj [T, h*dk (q) | h*dk (k) | h*dv (v) | h*dv (output gate)], low fp32 [T, rank] the low-rank decay input, a2 [h*dk, rank],
+    a2_b fp32 [h*dk], norm_w fp32 [dv] shared by the heads, state [slots, h, dk, dv] fp32 updated in place.
+    S = diag(sigmoid(a2 low + b)^(1/tau)) S + k v^T, o = S^T q dk^-0.5; returns rms(o) * norm_w * silu(gate) [T, h*dv]."""
+    T = proj.shape[0]
+    if proj.is_cuda:
+        out = torch.empty(T, h * dv, dtype=out_dtype, device=proj.device)
+        p = _gated_params(proj, h, dk, dv, out, norm_w, eps, qo_indptr, state_idx)
+        p.gates, p.ld_gates, p.a2, p.a2_b, p.rank, p.inv_tau = low.data_ptr(), low.stride(0), a2.data_ptr(), a2_b.data_ptr(), a2.shape[1], 1.0 / tau
+        p.S = state.data_ptr()
+        return _run_gated(KIND_GLA, p, proj, out, qo_indptr)
+    q, k, v, g = _qkvg(proj, h, dk, dv)
+    z = low.to(torch.float32) @ a2.to(torch.float32).t() + a2_b
+    decay = torch.exp(torch.nn.functional.logsigmoid(z) / tau).view(T, h, dk)
+    o = torch.empty(T, h, dv, dtype=torch.float32)
+    ind = qo_indptr.tolist()
+    for b in range(len(ind) - 1):
+        if ind[b + 1] > ind[b]:
+            o[ind[b]:ind[b + 1]] = R.gla_scan(q[ind[b]:ind[b + 1]], k[ind[b]:ind[b + 1]], v[ind[b]:ind[b + 1]], decay[ind[b]:ind[b + 1]],
+                                              state[int(state_idx[b])])
+    o = R.rmsnorm(o, norm_w, eps) * torch.nn.functional.silu(g)
+    return o.reshape(T, h * dv).to(out_dtype)
+
+
+def mlstm_mix(proj, gates, i_b, f_b, cap: float, norm_w, eps: float, state, qo_indptr, state_idx, h: int, dk: int, dv: int, out_dtype):
+    """mLSTM matrix memory over the token ranges of B sequences, up to the output projection.
+
+    proj as in :func:`gla_mix`, gates fp32 [T, i_raw h | f_raw h], i_b / f_b fp32 [h], norm_w fp32 [h*dv], state = (S
+    [slots, h, dk, dv], n [slots, h, dk], m [slots, h]) fp32 updated in place.  Both gates pass a soft cap cap*tanh(x/cap), the
+    forget gate then a log-sigmoid; the running maximum m keeps the exponentials below one.  Returns
+    rms(o) * norm_w * sigmoid(gate) [T, h*dv]."""
+    T = proj.shape[0]
+    S, n, m = state
+    if proj.is_cuda:
+        out = torch.empty(T, h * dv, dtype=out_dtype, device=proj.device)
+        p = _gated_params(proj, h, dk, dv, out, norm_w, eps, qo_indptr, state_idx)
+        p.gates, p.ld_gates, p.i_b, p.f_b, p.cap = gates.data_ptr(), gates.stride(0), i_b.data_ptr(), f_b.data_ptr(), float(cap)
+        p.S, p.n, p.m = S.data_ptr(), n.data_ptr(), m.data_ptr()
+        return _run_gated(KIND_MLSTM, p, proj, out, qo_indptr)
+    q, k, v, g = _qkvg(proj, h, dk, dv)
+    gi = cap * torch.tanh((gates[:, :h].to(torch.float32) + i_b) / cap)
+    gf = torch.nn.functional.logsigmoid(cap * torch.tanh((gates[:, h:2 * h].to(torch.float32) + f_b) / cap))
+    o = torch.empty(T, h, dv, dtype=torch.float32)
+    ind = qo_indptr.tolist()
+    for b in range(len(ind) - 1):
+        r, sl = slice(ind[b], ind[b + 1]), int(state_idx[b])
+        if ind[b + 1] > ind[b]:
+            o[r] = R.mlstm_scan(q[r], k[r], v[r], gi[r], gf[r], S[sl], n[sl], m[sl])
+    o = R.rmsnorm(o, torch.ones(dv), eps).reshape(T, h * dv) * norm_w * torch.sigmoid(g.reshape(T, h * dv))
+    return o.to(out_dtype)
 
 
 def causal_conv1d(x, weight, bias, state, qo_indptr, state_idx, activation: bool = True):

@@ -500,6 +500,30 @@ def kda_scan(q, k, v, forget, beta, A_log, dt_bias, state, lower_bound: float):
     return out, S
 
 
+def gla_scan(q, k, v, decay, state):
+    """Per-channel gated linear attention.  q, k, decay [T, h, dk], v [T, h, dv]; state [h, dk, dv] advanced in place."""
+    out = []
+    for t in range(q.shape[0]):
+        state.mul_(decay[t].unsqueeze(-1)).add_(k[t].unsqueeze(-1) * v[t].unsqueeze(-2))
+        out.append(torch.einsum("hkv,hk->hv", state, q[t]))
+    return torch.stack(out)
+
+
+def mlstm_scan(q, k, v, gi, gf, S, n, m):
+    """Exponentially gated matrix memory with a running maximum m of the log scale.  gi, gf [T, h] log gates;
+    S [h, dk, dv], n [h, dk], m [h] advanced in place."""
+    out = []
+    for t in range(q.shape[0]):
+        top = torch.maximum(gf[t] + m, gi[t])
+        keep, add = torch.exp(gf[t] + m - top), torch.exp(gi[t] - top)
+        S.mul_(keep[:, None, None]).add_((add[:, None] * k[t]).unsqueeze(-1) * v[t].unsqueeze(-2))
+        n.mul_(keep[:, None]).add_(add[:, None] * k[t])
+        m.copy_(top)
+        den = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+        out.append(torch.einsum("hkv,hk->hv", S, q[t]) / den[:, None])
+    return torch.stack(out)
+
+
 def kda_norm(x, gate, weight, eps):
     """Sigmoid-gated RMSNorm (`csrc/glm_flash_hybrid.cu:73-83`)."""
     return rmsnorm(x, weight, eps) * torch.sigmoid(gate.to(torch.float32))
