@@ -1,0 +1,574 @@
+// Chunked form of the gated outer-product recurrences (see gated_scan.cu) for portions of prompts, on the tensor cores.
+//
+// A sequence's tokens are cut into chunks of 64.  With b_t the running sum of the log decay inside a chunk,
+//
+//   GLA    o_t = (q_t e^{b_t}) . S_in + sum_{s<=t} [sum_c q_t[c] k_s[c] e^{b_t[c] - b_s[c]}] v_s
+//          S_out = diag(e^{b_C}) S_in + sum_s (k_s e^{b_C - b_s}) v_s^T
+//   mLSTM  with a_s = i_s - b_s, M_t = max_{s<=t} a_s, x_t = max(m_in, M_t), m_t = b_t + x_t:
+//          S_t^T q_t = e^{m_in - x_t} S_in^T q_t + sum_{s<=t} e^{a_s - x_t} (q_t . k_s) v_s   (n_t . q_t likewise without v)
+//          S_out = e^{m_in - x_C} S_in + e^{M_C - x_C} sum_s (k_s e^{a_s - M_C}) v_s^T
+//
+// in three launches:
+//   1 chunk_state_kernel   (chunk, head): decays, the chunk's own state contribution
+//   2 chunk_scan_kernel    (elements, head, sequence): carries the fp32 state over the chunks and leaves each chunk's S_in
+//   3 chunk_output_kernel  (chunk, head): intra-chunk and S_in parts, normaliser, head norm, output gate
+//
+// No exponent is ever positive: the products e^{b_t - b_s} of GLA are taken directly inside 16-token diagonal blocks and
+// through an anchor between the blocks otherwise.  q, k, v come as bf16; every other operand of a tensor-core product (decayed
+// keys and queries, scores, the state) is split into two bf16 terms, so the results keep fp32-like accuracy.
+#include "gated_scan.cuh"
+#include "mma_sync.cuh"
+
+namespace {
+
+constexpr int CT = 64;                       // tokens per chunk
+
+struct GatedChunkParams {
+    GatedScanParams s;
+    const int* chunks;                       // [chunks][4]: sequence, first token, tokens, 1 if the sequence's last chunk
+    const int* seq_chunks;                   // [B + 1]
+    int c0, c1;                              // chunk range of this pass
+    float* b;                                // GLA: running log decays [T, h * dk]
+    float* loc;                              // [chunks of the pass, h, dk, dv]: own contribution, then S_in as (hi, lo) bf16 words
+    float* nloc;                             // mLSTM: [chunks of the pass, h, dk], then n_in
+    float* scal;                             // mLSTM: [chunks of the pass, h, 4]: b_C, M_C, m_in
+};
+
+// rows [n][dim] (bf16, 16-byte chunks) -> shared [CT][ld], zero beyond n rows and beyond dim columns up to `padded`
+__device__ __forceinline__ void load_rows(bf16* dst, int ld, const bf16* src, size_t stride, int n, int dim, int padded) {
+    const int per = padded / 8;
+    for (int i = threadIdx.x; i < CT * per; i += blockDim.x) {
+        const int r = i / per, c = (i % per) * 8;
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (r < n && c < dim) v = *reinterpret_cast<const uint4*>(src + (size_t)r * stride + c);
+        *reinterpret_cast<uint4*>(dst + r * ld + c) = v;
+    }
+}
+
+// One warp: a_s = i_s - b_s, b_s, and the running maximum M_s of a over the chunk's tokens (two tokens per lane).
+__device__ __forceinline__ void mlstm_gates(const GatedScanParams& p, int t0, int n, int h, float* a_s, float* b_s, float* mx_s) {
+    const int lane = threadIdx.x & 31;
+    float gi[2], gf[2];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+        const int s = lane * 2 + j;
+        gi[j] = -INFINITY;
+        gf[j] = 0.f;
+        if (s < n) {
+            const float* gr = p.gates + (size_t)(t0 + s) * p.ld_gates;
+            gi[j] = p.cap * tanhf((gr[h] + p.i_b[h]) / p.cap);
+            gf[j] = logsigmoid_f(p.cap * tanhf((gr[p.h + h] + p.f_b[h]) / p.cap));
+        }
+    }
+    float sum = gf[0] + gf[1];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const float x = __shfl_up_sync(0xffffffffu, sum, o);
+        if (lane >= o) sum += x;
+    }
+    float before = __shfl_up_sync(0xffffffffu, sum, 1);
+    if (lane == 0) before = 0.f;
+    const float b0 = before + gf[0], b1 = b0 + gf[1];
+    const float a0 = gi[0] - b0, a1 = gi[1] - b1;
+    float mx = fmaxf(a0, a1);
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const float x = __shfl_up_sync(0xffffffffu, mx, o);
+        if (lane >= o) mx = fmaxf(mx, x);
+    }
+    float mb = __shfl_up_sync(0xffffffffu, mx, 1);
+    if (lane == 0) mb = -INFINITY;
+    a_s[lane * 2] = a0; a_s[lane * 2 + 1] = a1;
+    b_s[lane * 2] = b0; b_s[lane * 2 + 1] = b1;
+    mx_s[lane * 2] = fmaxf(mb, a0); mx_s[lane * 2 + 1] = fmaxf(fmaxf(mb, a0), a1);
+}
+
+// ---- 1: decays and the chunk's own state contribution -----------------------------------------------------------------------
+// grid (chunks of the pass, h), block 256
+template <int KIND>
+__global__ void __launch_bounds__(256) chunk_state_kernel(GatedChunkParams cp) {
+    pdl_grid_sync();
+    extern __shared__ __align__(16) unsigned char smraw[];
+    const GatedScanParams& p = cp.s;
+    const int ci = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int* ch = cp.chunks + (size_t)(cp.c0 + ci) * 4;
+    const int t0 = ch[1], n = ch[2], dk = p.dk, dv = p.dv;
+    const int dkp = (dk + 15) / 16 * 16, ldk = dkp + 8, ldv = dv + 8;
+    bf16* kh = reinterpret_cast<bf16*>(smraw);           // [CT][ldk] decayed keys, high and low terms
+    bf16* kl = kh + CT * ldk;
+    bf16* vs = kl + CT * ldk;                            // [CT][ldv]
+    float* fs = reinterpret_cast<float*>(vs + CT * ldv); // GLA: log decays [CT][dk] | low-rank rows [CT][rank]; mLSTM: a, b, M
+    load_rows(vs, ldv, (const bf16*)p.v + (size_t)t0 * p.ld + h * dv, p.ld, n, dv, dv);
+    if (KIND == KIND_GLA) {
+        float* low = fs + CT * dk;
+        for (int i = tid; i < n * p.rank; i += 256) low[i] = p.gates[(size_t)(t0 + i / p.rank) * p.ld_gates + i % p.rank];
+        __syncthreads();
+        for (int i = tid; i < dk * (CT / 8); i += 256) {                 // a channel, eight tokens
+            const int c = i % dk, s0 = i / dk * 8;
+            if (s0 >= n) continue;
+            const bf16* a2 = (const bf16*)p.a2 + (size_t)(h * dk + c) * p.rank;
+            float z[8];
+#pragma unroll
+            for (int j = 0; j < 8; ++j) z[j] = p.a2_b[h * dk + c];
+            for (int r = 0; r < p.rank; ++r) {
+                const float w = __bfloat162float(a2[r]);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) z[j] += w * (s0 + j < n ? low[(s0 + j) * p.rank + r] : 0.f);
+            }
+#pragma unroll
+            for (int j = 0; j < 8; ++j) fs[(s0 + j) * dk + c] = logsigmoid_f(z[j]) * p.inv_tau;
+        }
+        __syncthreads();
+        for (int c = tid; c < dk; c += 256) {
+            float run = 0.f;
+#pragma unroll 8
+            for (int s = 0; s < n; ++s) {
+                run += fs[s * dk + c];
+                fs[s * dk + c] = run;
+                cp.b[(size_t)(t0 + s) * (p.h * dk) + h * dk + c] = run;
+            }
+        }
+    } else if (warp == 0) {
+        mlstm_gates(p, t0, n, h, fs, fs + CT, fs + 2 * CT);
+    }
+    __syncthreads();
+    const float top = KIND == KIND_MLSTM ? fs[2 * CT + n - 1] : 0.f;
+    const bf16* kg = (const bf16*)p.k + (size_t)t0 * p.ld + h * dk;
+    for (int i = tid; i < CT * (dkp / 2); i += 256) {
+        const int s = i / (dkp / 2), c = (i % (dkp / 2)) * 2;
+        uint32_t hi = 0, lo = 0;
+        if (s < n && c < dk) {
+            const float2 k = bf162_to_f2(*reinterpret_cast<const uint32_t*>(kg + (size_t)s * p.ld + c));
+            float w0, w1;
+            if (KIND == KIND_GLA) {
+                w0 = __expf(fs[(n - 1) * dk + c] - fs[s * dk + c]);
+                w1 = __expf(fs[(n - 1) * dk + c + 1] - fs[s * dk + c + 1]);
+            } else {
+                w0 = w1 = __expf(fs[s] - top);
+            }
+            split_bf162(k.x * w0, k.y * w1, hi, lo);
+        }
+        *reinterpret_cast<uint32_t*>(kh + s * ldk + c) = hi;
+        *reinterpret_cast<uint32_t*>(kl + s * ldk + c) = lo;
+    }
+    __syncthreads();
+    const size_t base = (size_t)ci * p.h + h;
+    if (KIND == KIND_MLSTM) {
+        for (int c = tid; c < dk; c += 256) {
+            float a = 0.f;
+            for (int s = 0; s < n; ++s) a += __bfloat162float(kh[s * ldk + c]) + __bfloat162float(kl[s * ldk + c]);
+            cp.nloc[base * dk + c] = a;
+        }
+        if (tid == 0) { cp.scal[base * 4] = fs[CT + n - 1]; cp.scal[base * 4 + 1] = top; }
+    }
+    // loc[c, j] = sum_s k~[s, c] v[s, j]: units of 16 channels x 64 values over the warps
+    float* loc = cp.loc + base * dk * dv;
+    const int cols = (dv + 63) / 64, units = dkp / 16 * cols, ksteps = (n + 15) / 16, g = lane >> 2, q = lane & 3;
+    for (int u = warp; u < units; u += 8) {
+        const int m0 = u / cols * 16, j0 = u % cols * 64, nt = min(8, (dv - j0) / 8);
+        float acc[8][4] = {};
+        for (int ks = 0; ks < ksteps; ++ks) {
+            const int off = (ks * 16 + (lane & 7) + ((lane >> 4) & 1) * 8) * ldk + m0 + ((lane >> 3) & 1) * 8;
+            uint32_t ah[4], al[4];
+            ldsm_x4_trans(ah, kh + off);
+            ldsm_x4_trans(al, kl + off);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                if (i >= nt) break;
+                uint32_t b0, b1;
+                ldsm_x2_trans(b0, b1, vs + (ks * 16 + (lane & 15)) * ldv + j0 + i * 8);
+                mma_bf16_16816(acc[i], ah, b0, b1);
+                mma_bf16_16816(acc[i], al, b0, b1);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            if (i >= nt) break;
+            const int j = j0 + i * 8 + q * 2;
+            if (m0 + g < dk) *reinterpret_cast<float2*>(loc + (size_t)(m0 + g) * dv + j) = make_float2(acc[i][0], acc[i][1]);
+            if (m0 + g + 8 < dk) *reinterpret_cast<float2*>(loc + (size_t)(m0 + g + 8) * dv + j) = make_float2(acc[i][2], acc[i][3]);
+        }
+    }
+}
+
+// ---- 2: the state over the chunks --------------------------------------------------------------------------------------------
+__device__ __forceinline__ uint32_t pack_split(float x) {
+    const bf16 hi = __float2bfloat16(x);
+    const bf16 lo = __float2bfloat16(x - __bfloat162float(hi));
+    return (uint32_t)*reinterpret_cast<const unsigned short*>(&hi) | ((uint32_t)*reinterpret_cast<const unsigned short*>(&lo) << 16);
+}
+
+// grid (ceil(dk * dv / 1024), h, B), block 256: four consecutive values of a state row per thread
+template <int KIND>
+__global__ void __launch_bounds__(256) chunk_scan_kernel(GatedChunkParams cp) {
+    pdl_grid_sync();
+    const GatedScanParams& p = cp.s;
+    const int h = blockIdx.y, seq = blockIdx.z, dk = p.dk, dv = p.dv;
+    const int lo = max(cp.seq_chunks[seq], cp.c0), hi = min(cp.seq_chunks[seq + 1], cp.c1);
+    if (lo >= hi) return;
+    const size_t slot = (size_t)p.state_idx[seq] * p.h + h, size = (size_t)dk * dv;
+    const int e = (blockIdx.x * 256 + threadIdx.x) * 4;
+    const float m0 = KIND == KIND_MLSTM ? p.m[slot] : 0.f;
+    if (e < (int)size) {
+        const int c = e / dv;
+        float4 S = *reinterpret_cast<const float4*>(p.S + slot * size + e);
+        float m = m0;
+        constexpr int U = 4;                              // chunks whose contributions are in flight
+        for (int i0 = lo; i0 < hi; i0 += U) {
+            float4 x[U];
+            float d[U];
+#pragma unroll
+            for (int j = 0; j < U; ++j) {
+                const int i = i0 + j;
+                if (i >= hi) continue;
+                x[j] = *reinterpret_cast<const float4*>(cp.loc + ((size_t)(i - cp.c0) * p.h + h) * size + e);
+                if (KIND == KIND_GLA) {
+                    const int* ch = cp.chunks + (size_t)i * 4;
+                    d[j] = expf(cp.b[(size_t)(ch[1] + ch[2] - 1) * (p.h * dk) + h * dk + c]);
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < U; ++j) {
+                const int i = i0 + j;
+                if (i >= hi) continue;
+                float add = 1.f, keep = d[j];
+                if (KIND == KIND_MLSTM) {
+                    const float* sc = cp.scal + ((size_t)(i - cp.c0) * p.h + h) * 4;
+                    const float top = fmaxf(m, sc[1]);
+                    keep = expf(m - top);
+                    add = expf(sc[1] - top);
+                    m = sc[0] + top;
+                }
+                uint4 w;
+                w.x = pack_split(S.x); w.y = pack_split(S.y); w.z = pack_split(S.z); w.w = pack_split(S.w);
+                *reinterpret_cast<uint4*>(cp.loc + ((size_t)(i - cp.c0) * p.h + h) * size + e) = w;
+                S.x = keep * S.x + add * x[j].x; S.y = keep * S.y + add * x[j].y;
+                S.z = keep * S.z + add * x[j].z; S.w = keep * S.w + add * x[j].w;
+            }
+        }
+        *reinterpret_cast<float4*>(p.S + slot * size + e) = S;
+    }
+    if (KIND == KIND_MLSTM && blockIdx.x == 0) {
+        // normaliser and running maximum; m itself is stored by the output kernel (other blocks of this grid still read it)
+        for (int c = threadIdx.x; c < dk; c += 256) {
+            float nn = p.n[slot * dk + c], m = m0;
+            for (int i = lo; i < hi; ++i) {
+                const size_t at = (size_t)(i - cp.c0) * p.h + h;
+                const float* sc = cp.scal + at * 4;
+                const float top = fmaxf(m, sc[1]), x = cp.nloc[at * dk + c];
+                cp.nloc[at * dk + c] = nn;
+                nn = expf(m - top) * nn + expf(sc[1] - top) * x;
+                m = sc[0] + top;
+            }
+            p.n[slot * dk + c] = nn;
+        }
+        if (threadIdx.x == 0) {
+            float m = m0;
+            for (int i = lo; i < hi; ++i) {
+                float* sc = cp.scal + ((size_t)(i - cp.c0) * p.h + h) * 4;
+                sc[2] = m;
+                m = sc[0] + fmaxf(m, sc[1]);
+                sc[3] = m;
+            }
+        }
+    }
+}
+
+// ---- 3: outputs --------------------------------------------------------------------------------------------------------------
+constexpr int OUT_THREADS = 512;             // 16 warps: 4 row tiles of 16 tokens x 4 column quarters
+constexpr int LDA = CT + 8;
+constexpr int SLAB = 64;                     // state rows in shared memory at a time
+
+template <int KIND>
+size_t output_smem(int dk, int dv) {
+    const int dkp = (dk + 15) / 16 * 16;
+    size_t b = (size_t)CT * (dkp + 8) * 2 * 2 + (size_t)CT * (dv + 8) * 2 + (size_t)2 * SLAB * (dv + 8) * 2 + (size_t)2 * CT * LDA * 2;
+    b += KIND == KIND_GLA ? (size_t)CT * (dkp + 4) * 4 : 0;
+    return b + (size_t)CT * 12 * 4;
+}
+
+// grid (chunks of the pass, h).  NT: 8-wide value tiles per column quarter (dv <= 32 * NT).
+template <int KIND, int NT>
+__global__ void __launch_bounds__(OUT_THREADS) chunk_output_kernel(GatedChunkParams cp) {
+    pdl_grid_sync();
+    extern __shared__ __align__(16) unsigned char smraw[];
+    const GatedScanParams& p = cp.s;
+    const int ci = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, c4 = lane & 3;
+    const int rt = warp & 3, quarter = warp >> 2;
+    const int* ch = cp.chunks + (size_t)(cp.c0 + ci) * 4;
+    const int seq = ch[0], t0 = ch[1], n = ch[2], last = ch[3], dk = p.dk, dv = p.dv;
+    const int dkp = (dk + 15) / 16 * 16, ldk = dkp + 8, ldv = dv + 8, ldb = dkp + 4;
+    bf16* qs = reinterpret_cast<bf16*>(smraw);           // [CT][ldk]
+    bf16* ks = qs + CT * ldk;
+    bf16* vs = ks + CT * ldk;                            // [CT][ldv]
+    bf16* sh = vs + CT * ldv;                            // [SLAB][ldv] state rows, high and low terms
+    bf16* sl = sh + SLAB * ldv;
+    bf16* ah = sl + SLAB * ldv;                          // [CT][LDA] scores
+    bf16* al = ah + CT * LDA;
+    float* fs = reinterpret_cast<float*>(al + CT * LDA);
+    float* bs = fs;                                      // GLA: [CT][ldb]
+    float* rows = fs + (KIND == KIND_GLA ? CT * ldb : 0);
+    float *ga = rows, *gb = rows + CT, *gx = rows + 2 * CT, *qn = rows + 3 * CT, *nq = rows + 4 * CT, *ssq = rows + 8 * CT;
+    const float qscale = rsqrtf((float)dk);
+    const size_t base = (size_t)ci * p.h + h;
+    load_rows(qs, ldk, (const bf16*)p.q + (size_t)t0 * p.ld + h * dk, p.ld, n, dk, dkp);
+    load_rows(ks, ldk, (const bf16*)p.k + (size_t)t0 * p.ld + h * dk, p.ld, n, dk, dkp);
+    load_rows(vs, ldv, (const bf16*)p.v + (size_t)t0 * p.ld + h * dv, p.ld, n, dv, dv);
+    const float m_in = KIND == KIND_MLSTM ? cp.scal[base * 4 + 2] : 0.f;
+    if (KIND == KIND_GLA) {
+        for (int i = tid; i < CT * dkp; i += OUT_THREADS) {
+            const int s = i / dkp, c = i % dkp;
+            bs[s * ldb + c] = (s < n && c < dk) ? cp.b[(size_t)(t0 + s) * (p.h * dk) + h * dk + c] : 0.f;
+        }
+    } else if (warp == 0) {
+        mlstm_gates(p, t0, n, h, ga, gb, gx);
+    }
+    __syncthreads();
+    if (KIND == KIND_MLSTM) {
+        if (tid < CT) gx[tid] = fmaxf(gx[tid], m_in);
+        // q_t . n_in: eight lanes per token
+        float a = 0.f;
+        const float* nin = cp.nloc + base * dk;
+        const int r = tid >> 3;
+        for (int c = tid & 7; c < dk; c += 8) a += __bfloat162float(qs[r * ldk + c]) * nin[c];
+#pragma unroll
+        for (int o = 1; o < 8; o <<= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
+        if ((tid & 7) == 0) qn[r] = a;
+        __syncthreads();
+    }
+    // ---- scores of (row tile rt, key tile J = quarter) ----
+    {
+        const int J = quarter, r0 = rt * 16 + g, r1 = r0 + 8;
+        float sc[2][4] = {};
+        if (KIND == KIND_MLSTM ? J <= rt : J < rt) {
+            for (int kk = 0; kk < dkp; kk += 16) {
+                uint32_t a[4], a2[4];
+                if (KIND == KIND_MLSTM) {
+                    ldsm_x4(a, qs + (rt * 16 + (lane & 15)) * ldk + kk + (lane >> 4) * 8);
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        const int r = (i & 1) ? r1 : r0, c = kk + c4 * 2 + (i >> 1) * 8;
+                        const float2 x = bf162_to_f2(*reinterpret_cast<const uint32_t*>(qs + r * ldk + c));
+                        const float2 b = *reinterpret_cast<const float2*>(bs + r * ldb + c);
+                        const float2 an = *reinterpret_cast<const float2*>(bs + (rt * 16 - 1) * ldb + c);
+                        split_bf162(x.x * __expf(fminf(b.x - an.x, 0.f)), x.y * __expf(fminf(b.y - an.y, 0.f)), a[i], a2[i]);
+                    }
+                }
+#pragma unroll
+                for (int t = 0; t < 2; ++t) {
+                    const int s = J * 16 + t * 8;
+                    if (KIND == KIND_MLSTM) {
+                        uint32_t b0, b1;
+                        ldsm_x2(b0, b1, ks + (s + (lane & 7)) * ldk + kk + ((lane >> 3) & 1) * 8);
+                        mma_bf16_16816(sc[t], a, b0, b1);
+                    } else {
+                        uint32_t bh[2], bl[2];
+#pragma unroll
+                        for (int i = 0; i < 2; ++i) {
+                            const int c = kk + c4 * 2 + i * 8;
+                            const float2 x = bf162_to_f2(*reinterpret_cast<const uint32_t*>(ks + (s + g) * ldk + c));
+                            const float2 b = *reinterpret_cast<const float2*>(bs + (s + g) * ldb + c);
+                            const float2 an = *reinterpret_cast<const float2*>(bs + (rt * 16 - 1) * ldb + c);
+                            split_bf162(x.x * __expf(fminf(an.x - b.x, 0.f)), x.y * __expf(fminf(an.y - b.y, 0.f)), bh[i], bl[i]);
+                        }
+                        mma_bf16_16816(sc[t], a, bh[0], bh[1]);
+                        mma_bf16_16816(sc[t], a, bl[0], bl[1]);
+                        mma_bf16_16816(sc[t], a2, bh[0], bh[1]);
+                    }
+                }
+            }
+        }
+        if (KIND == KIND_MLSTM || J != rt) {
+            float sum0 = 0.f, sum1 = 0.f;
+#pragma unroll
+            for (int t = 0; t < 2; ++t) {
+                float v[4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const int r = i < 2 ? r0 : r1, s = J * 16 + t * 8 + c4 * 2 + (i & 1);
+                    float w = qscale;
+                    if (KIND == KIND_MLSTM) w *= s < n ? __expf(ga[s] - gx[r]) : 0.f;
+                    v[i] = s <= r ? sc[t][i] * w : 0.f;
+                }
+                sum0 += v[0] + v[1];
+                sum1 += v[2] + v[3];
+                uint32_t hi, lo;
+                const int s = J * 16 + t * 8 + c4 * 2;
+                split_bf162(v[0], v[1], hi, lo);
+                *reinterpret_cast<uint32_t*>(ah + r0 * LDA + s) = hi;
+                *reinterpret_cast<uint32_t*>(al + r0 * LDA + s) = lo;
+                split_bf162(v[2], v[3], hi, lo);
+                *reinterpret_cast<uint32_t*>(ah + r1 * LDA + s) = hi;
+                *reinterpret_cast<uint32_t*>(al + r1 * LDA + s) = lo;
+            }
+            if (KIND == KIND_MLSTM) {
+                sum0 += __shfl_xor_sync(0xffffffffu, sum0, 1); sum0 += __shfl_xor_sync(0xffffffffu, sum0, 2);
+                sum1 += __shfl_xor_sync(0xffffffffu, sum1, 1); sum1 += __shfl_xor_sync(0xffffffffu, sum1, 2);
+                if (c4 == 0) { nq[r0 * 4 + J] = sum0; nq[r1 * 4 + J] = sum1; }
+            }
+        }
+    }
+    if (KIND == KIND_GLA) {
+        // diagonal blocks: a quad of lanes per (t, s) pair, channels interleaved over the quad
+        for (int it = tid >> 2; it < 4 * 256; it += OUT_THREADS / 4) {
+            const int r = (it >> 8) * 16 + ((it >> 4) & 15), s = (it >> 8) * 16 + (it & 15);
+            float a = 0.f;
+            if (s <= r && r < n) {
+                for (int c = tid & 3; c < dk; c += 4)
+                    a += __bfloat162float(qs[r * ldk + c]) * __bfloat162float(ks[s * ldk + c]) * __expf(bs[r * ldb + c] - bs[s * ldb + c]);
+            }
+            a += __shfl_xor_sync(0xffffffffu, a, 1);
+            a += __shfl_xor_sync(0xffffffffu, a, 2);
+            if ((tid & 3) == 0) {
+                a *= qscale;
+                const bf16 hi = __float2bfloat16(a);
+                ah[r * LDA + s] = hi;
+                al[r * LDA + s] = __float2bfloat16(a - __bfloat162float(hi));
+            }
+        }
+    }
+    // ---- S_in part: rows of the state in slabs ----
+    const int ntiles = dv / 8, tq = (ntiles + 3) / 4, nt0 = quarter * tq, ntn = max(0, min(tq, ntiles - nt0));
+    const int r0 = rt * 16 + g, r1 = r0 + 8;
+    float acc[NT][4];
+#pragma unroll
+    for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    const uint32_t* sin = reinterpret_cast<const uint32_t*>(cp.loc) + base * dk * dv;
+    for (int k0 = 0; k0 < dkp; k0 += SLAB) {
+        const int rowsn = min(SLAB, dkp - k0);
+        __syncthreads();
+        for (int i = tid; i < rowsn * (dv / 4); i += OUT_THREADS) {
+            const int r = i / (dv / 4), c = (i % (dv / 4)) * 4;
+            uint4 w = make_uint4(0, 0, 0, 0);
+            if (k0 + r < dk) w = *reinterpret_cast<const uint4*>(sin + (size_t)(k0 + r) * dv + c);
+            *reinterpret_cast<uint2*>(sh + r * ldv + c) = make_uint2(__byte_perm(w.x, w.y, 0x5410), __byte_perm(w.z, w.w, 0x5410));
+            *reinterpret_cast<uint2*>(sl + r * ldv + c) = make_uint2(__byte_perm(w.x, w.y, 0x7632), __byte_perm(w.z, w.w, 0x7632));
+        }
+        __syncthreads();
+        for (int kk = 0; kk < rowsn; kk += 16) {
+            uint32_t a[4], a2[4];
+            if (KIND == KIND_MLSTM) {
+                ldsm_x4(a, qs + (rt * 16 + (lane & 15)) * ldk + k0 + kk + (lane >> 4) * 8);
+            } else {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const int r = (i & 1) ? r1 : r0, c = k0 + kk + c4 * 2 + (i >> 1) * 8;
+                    const float2 x = bf162_to_f2(*reinterpret_cast<const uint32_t*>(qs + r * ldk + c));
+                    const float2 b = *reinterpret_cast<const float2*>(bs + r * ldb + c);
+                    split_bf162(x.x * qscale * __expf(b.x), x.y * qscale * __expf(b.y), a[i], a2[i]);
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < NT; ++i) {
+                if (i >= ntn) break;
+                uint32_t b0, b1, l0, l1;
+                ldsm_x2_trans(b0, b1, sh + (kk + (lane & 15)) * ldv + (nt0 + i) * 8);
+                ldsm_x2_trans(l0, l1, sl + (kk + (lane & 15)) * ldv + (nt0 + i) * 8);
+                mma_bf16_16816(acc[i], a, b0, b1);
+                mma_bf16_16816(acc[i], a, l0, l1);
+                if (KIND == KIND_GLA) mma_bf16_16816(acc[i], a2, b0, b1);
+            }
+        }
+    }
+    float e0 = 1.f, e1 = 1.f;
+    if (KIND == KIND_MLSTM) {
+        e0 = __expf(m_in - gx[r0]) * qscale;
+        e1 = __expf(m_in - gx[r1]) * qscale;
+#pragma unroll
+        for (int i = 0; i < NT; ++i) { acc[i][0] *= e0; acc[i][1] *= e0; acc[i][2] *= e1; acc[i][3] *= e1; }
+    }
+    // ---- intra-chunk part ----
+    for (int kk = 0; kk <= rt * 16; kk += 16) {
+        uint32_t a[4], a2[4];
+        ldsm_x4(a, ah + (rt * 16 + (lane & 15)) * LDA + kk + (lane >> 4) * 8);
+        ldsm_x4(a2, al + (rt * 16 + (lane & 15)) * LDA + kk + (lane >> 4) * 8);
+#pragma unroll
+        for (int i = 0; i < NT; ++i) {
+            if (i >= ntn) break;
+            uint32_t b0, b1;
+            ldsm_x2_trans(b0, b1, vs + (kk + (lane & 15)) * ldv + (nt0 + i) * 8);
+            mma_bf16_16816(acc[i], a, b0, b1);
+            mma_bf16_16816(acc[i], a2, b0, b1);
+        }
+    }
+    if (KIND == KIND_MLSTM) {
+        const float q0 = e0 * qn[r0] + nq[r0 * 4] + nq[r0 * 4 + 1] + nq[r0 * 4 + 2] + nq[r0 * 4 + 3];
+        const float q1 = e1 * qn[r1] + nq[r1 * 4] + nq[r1 * 4 + 1] + nq[r1 * 4 + 2] + nq[r1 * 4 + 3];
+        const float d0 = 1.f / (fmaxf(fabsf(q0), expf(-(gb[r0] + gx[r0]))) + 1e-6f), d1 = 1.f / (fmaxf(fabsf(q1), expf(-(gb[r1] + gx[r1]))) + 1e-6f);
+#pragma unroll
+        for (int i = 0; i < NT; ++i) { acc[i][0] *= d0; acc[i][1] *= d0; acc[i][2] *= d1; acc[i][3] *= d1; }
+        if ((last || cp.c0 + ci + 1 == cp.c1) && tid == 0) p.m[(size_t)p.state_idx[seq] * p.h + h] = cp.scal[base * 4 + 3];
+    }
+    float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+        s0 += acc[i][0] * acc[i][0] + acc[i][1] * acc[i][1];
+        s1 += acc[i][2] * acc[i][2] + acc[i][3] * acc[i][3];
+    }
+    s0 += __shfl_xor_sync(0xffffffffu, s0, 1); s0 += __shfl_xor_sync(0xffffffffu, s0, 2);
+    s1 += __shfl_xor_sync(0xffffffffu, s1, 1); s1 += __shfl_xor_sync(0xffffffffu, s1, 2);
+    if (c4 == 0) { ssq[r0 * 4 + quarter] = s0; ssq[r1 * 4 + quarter] = s1; }
+    __syncthreads();
+    const float i0 = rsqrtf((ssq[r0 * 4] + ssq[r0 * 4 + 1] + ssq[r0 * 4 + 2] + ssq[r0 * 4 + 3]) / (float)dv + p.eps);
+    const float i1 = rsqrtf((ssq[r1 * 4] + ssq[r1 * 4 + 1] + ssq[r1 * 4 + 2] + ssq[r1 * 4 + 3]) / (float)dv + p.eps);
+    const float* nw = p.norm_w + (KIND == KIND_MLSTM ? (size_t)h * dv : 0);
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+        if (i >= ntn) break;
+        const int j = (nt0 + i) * 8 + c4 * 2;
+        const float2 w = make_float2(nw[j], nw[j + 1]);
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+            const int r = u ? r1 : r0;
+            if (r >= n) continue;
+            const float inv = u ? i1 : i0;
+            const float2 gt = bf162_to_f2(*reinterpret_cast<const uint32_t*>((const bf16*)p.g + (size_t)(t0 + r) * p.ld + h * dv + j));
+            const float x = 1.f / (1.f + __expf(-gt.x)), y = 1.f / (1.f + __expf(-gt.y));
+            const float gx0 = KIND == KIND_GLA ? gt.x * x : x, gy0 = KIND == KIND_GLA ? gt.y * y : y;
+            *reinterpret_cast<uint32_t*>((bf16*)p.out + ((size_t)(t0 + r) * p.h + h) * dv + j) =
+                f2_to_bf162(acc[i][u * 2] * inv * w.x * gx0, acc[i][u * 2 + 1] * inv * w.y * gy0);
+        }
+    }
+}
+
+size_t state_smem(int kind, int dk, int dv, int rank) {
+    const int dkp = (dk + 15) / 16 * 16;
+    return (size_t)CT * (dkp + 8) * 4 + (size_t)CT * (dv + 8) * 2 + (kind == KIND_GLA ? (size_t)CT * (dk + rank) * 4 : (size_t)3 * CT * 4);
+}
+
+template <int KIND>
+int run_chunks(const GatedChunkParams* p, int B, cudaStream_t s) {
+    const int dk = p->s.dk, dv = p->s.dv, h = p->s.h, nc = p->c1 - p->c0;
+    const size_t s1 = state_smem(KIND, dk, dv, p->s.rank), s3 = output_smem<KIND>(dk, dv);
+    auto k1 = chunk_state_kernel<KIND>;
+    if (s1 > 48 * 1024) cudaFuncSetAttribute(k1, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1);
+    sl_launch(k1, dim3(nc, h), 256, s1, s, *p);
+    sl_launch(chunk_scan_kernel<KIND>, dim3((dk * dv + 1023) / 1024, h, B), 256, 0, s, *p);
+    if (dv <= 128) {
+        auto k3 = chunk_output_kernel<KIND, 4>;
+        cudaFuncSetAttribute(k3, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s3);
+        sl_launch(k3, dim3(nc, h), OUT_THREADS, s3, s, *p);
+    } else {
+        auto k3 = chunk_output_kernel<KIND, 8>;
+        cudaFuncSetAttribute(k3, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s3);
+        sl_launch(k3, dim3(nc, h), OUT_THREADS, s3, s, *p);
+    }
+    return SL_LAUNCH_CHECK();
+}
+
+}  // namespace
+
+// 1 when the chunked kernels take these sizes (head rows of whole 16-byte pieces, tiles that fit in shared memory).
+SL_API int sl_gated_chunk_ok(int kind, int dk, int dv, int rank) {
+    if (dk < 8 || dv < 8 || dk % 8 != 0 || dv % 8 != 0 || dv > 256) return 0;
+    const size_t s3 = kind == KIND_GLA ? output_smem<KIND_GLA>(dk, dv) : output_smem<KIND_MLSTM>(dk, dv);
+    return state_smem(kind, dk, dv, rank) <= 220 * 1024 && s3 <= 220 * 1024;
+}
+
+// One pass over the chunks [c0, c1) of B sequences (bf16 rows in and out).  Passes of one step run in order on one stream.
+SL_API int sl_gated_chunks(const GatedChunkParams* p, int B, int kind, cudaStream_t s) {
+    if (B == 0 || p->c1 <= p->c0) return 0;
+    if (!sl_gated_chunk_ok(kind, p->s.dk, p->s.dv, p->s.rank) || p->s.ld % 8 != 0 || B > 65535 || p->s.h > 65535) return -1;
+    return kind == KIND_GLA ? run_chunks<KIND_GLA>(p, B, s) : kind == KIND_MLSTM ? run_chunks<KIND_MLSTM>(p, B, s) : -1;
+}

@@ -80,7 +80,7 @@ class GatedLinearAttention(_GatedRecurrence):
         proj, low = self._project(model.ops, x)
         qo, sidx = model.scan_ranges(st)
         o = RC.gla_mix(proj, low, self.a2, self.a2_b, self.tau, self.norm, self.eps, cache.state[self.index]["S"], qo, sidx,
-                       self.heads, self.dk, self.dv, x.dtype)
+                       self.heads, self.dk, self.dv, x.dtype, RC.ChunkPlan.of(st))
         return model.ops.linear(o, self.o_proj, out_f32=True)
 
 
@@ -110,5 +110,5 @@ class MLstm(_GatedRecurrence):
         qo, sidx = model.scan_ranges(st)
         s = cache.state[self.index]
         o = RC.mlstm_mix(proj, gates, self.i_b, self.f_b, self.cap, self.norm, self.eps, (s["S"], s["n"], s["m"]), qo, sidx,
-                         self.heads, self.dk, self.dv, x.dtype)
+                         self.heads, self.dk, self.dv, x.dtype, RC.ChunkPlan.of(st))
         return model.ops.linear(o, self.o_proj, out_f32=True)

@@ -214,6 +214,8 @@ _SIGS = {
     "sl_latent_pre": [vp, i32, i32, vp],
     "sl_latent_rows": [vp, i32, i32, vp],
     "sl_gated_step": [vp, i32, i32, i32, i32, vp],
+    "sl_gated_chunk_ok": [i32, i32, i32, i32],
+    "sl_gated_chunks": [vp, i32, i32, vp],
     "sl_embed": [vp, vp, vp, i32, i32, i32, vp],
     "sl_add_rmsnorm": [vp, vp, vp, vp, vp, i32, i32, f32, i32, vp, vp],
     "sl_attn_pre": [C.POINTER(AttnPreParams), i32, vp],

@@ -104,6 +104,41 @@ class GatedScanParams(C.Structure):
 
 
 KIND_GLA, KIND_MLSTM = 0, 1
+CHUNK = 64                          # tokens per chunk of the chunked kernels
+CHUNK_MIN_Q = 16                    # longest portion of a step from which on they are used
+CHUNK_SCRATCH_BYTES = 96 << 20      # chunk states of one pass (they stay in L2); longer steps run in several passes
+
+
+class GatedChunkParams(C.Structure):
+    _fields_ = [("s", GatedScanParams), ("chunks", C.c_void_p), ("seq_chunks", C.c_void_p), ("c0", C.c_int), ("c1", C.c_int),
+                ("b", C.c_void_p), ("loc", C.c_void_p), ("nloc", C.c_void_p), ("scal", C.c_void_p)]
+
+
+class ChunkPlan:
+    """The chunks of a step's portions: table [chunks, 4] of (sequence, first token, tokens, last chunk of its sequence) and
+    the chunk range of every sequence, on the device."""
+
+    def __init__(self, lengths, device):
+        rows, ends, t0 = [], [0], 0
+        for b, n in enumerate(lengths):
+            for o in range(0, n, CHUNK):
+                rows.append((b, t0 + o, min(CHUNK, n - o), int(o + CHUNK >= n)))
+            ends.append(len(rows))
+            t0 += n
+        self.count, self.longest = len(rows), max(lengths)
+        flat = [x for r in rows for x in r] + ends
+        t = torch.tensor(flat, dtype=torch.int32, device=device)
+        self.table, self.seq_chunks = t[:4 * self.count], t[4 * self.count:]
+
+    @staticmethod
+    def of(st):
+        """The plan of a step that holds portions of prompts (made once per step), else None."""
+        spans = st.extra.get("spans")
+        if spans is None or not st.input_ids.is_cuda:
+            return None
+        if "chunk_plan" not in st.extra:
+            st.extra["chunk_plan"] = ChunkPlan([n for _, n in spans], st.input_ids.device)
+        return st.extra["chunk_plan"]
 
 
 def _gated_params(p_in, h, dk, dv, out, norm_w, eps, qo_indptr, state_idx) -> GatedScanParams:
@@ -114,10 +149,23 @@ def _gated_params(p_in, h, dk, dv, out, norm_w, eps, qo_indptr, state_idx) -> Ga
                            qo_indptr=qo_indptr.data_ptr(), state_idx=state_idx.data_ptr(), h=h, dk=dk, dv=dv)
 
 
-def _run_gated(kind: int, p: GatedScanParams, proj, out, qo_indptr) -> torch.Tensor:
+def _run_gated(kind: int, p: GatedScanParams, proj, out, qo_indptr, plan=None) -> torch.Tensor:
     N = _native()
-    N.call("sl_gated_step", C.byref(p), qo_indptr.numel() - 1, kind, int(proj.dtype == torch.float32), int(out.dtype == torch.float32),
-           N.stream())
+    B = qo_indptr.numel() - 1
+    h, dk, dv, dev = p.h, p.dk, p.dv, proj.device
+    if (plan is None or plan.longest < CHUNK_MIN_Q or proj.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or p.ld % 8
+            or p.q % 16 or not N.fn("sl_gated_chunk_ok")(kind, dk, dv, p.rank)):
+        N.call("sl_gated_step", C.byref(p), B, kind, int(proj.dtype == torch.float32), int(out.dtype == torch.float32), N.stream())
+        return out
+    per_pass = min(plan.count, max(1, CHUNK_SCRATCH_BYTES // (h * dk * dv * 4)))
+    loc = torch.empty(per_pass * h * dk * dv, dtype=torch.float32, device=dev)
+    b = torch.empty(out.shape[0] * h * dk if kind == KIND_GLA else 1, dtype=torch.float32, device=dev)
+    aux = torch.empty(per_pass * h * (dk + 4) if kind == KIND_MLSTM else 1, dtype=torch.float32, device=dev)
+    cp = GatedChunkParams(s=p, chunks=plan.table.data_ptr(), seq_chunks=plan.seq_chunks.data_ptr(), b=b.data_ptr(), loc=loc.data_ptr(),
+                          nloc=aux.data_ptr(), scal=aux.data_ptr() + per_pass * h * dk * 4)
+    for c0 in range(0, plan.count, per_pass):
+        cp.c0, cp.c1 = c0, min(plan.count, c0 + per_pass)
+        N.call("sl_gated_chunks", C.byref(cp), B, kind, N.stream())
     return out
 
 
@@ -127,19 +175,21 @@ def _qkvg(proj, h, dk, dv):
     return q.reshape(T, h, dk) * dk ** -0.5, k.reshape(T, h, dk), v.reshape(T, h, dv), g.reshape(T, h, dv)
 
 
-def gla_mix(proj, low, a2, a2_b, tau: float, norm_w, eps: float, state, qo_indptr, state_idx, h: int, dk: int, dv: int, out_dtype):
+def gla_mix(proj, low, a2, a2_b, tau: float, norm_w, eps: float, state, qo_indptr, state_idx, h: int, dk: int, dv: int, out_dtype,
+            plan=None):
     """Gated linear attention over the token ranges of B sequences, up to the output projection.
 
     proj [T, h*dk (q) | h*dk (k) | h*dv (v) | h*dv (output gate)], low fp32 [T, rank] the low-rank decay input, a2 [h*dk, rank],
     a2_b fp32 [h*dk], norm_w fp32 [dv] shared by the heads, state [slots, h, dk, dv] fp32 updated in place.
-    S = diag(sigmoid(a2 low + b)^(1/tau)) S + k v^T, o = S^T q dk^-0.5; returns rms(o) * norm_w * silu(gate) [T, h*dv]."""
+    S = diag(sigmoid(a2 low + b)^(1/tau)) S + k v^T, o = S^T q dk^-0.5; returns rms(o) * norm_w * silu(gate) [T, h*dv].
+    With a :class:`ChunkPlan` longer portions run in chunks on the tensor cores (`csrc/gated_chunk.cu`)."""
     T = proj.shape[0]
     if proj.is_cuda:
         out = torch.empty(T, h * dv, dtype=out_dtype, device=proj.device)
         p = _gated_params(proj, h, dk, dv, out, norm_w, eps, qo_indptr, state_idx)
         p.gates, p.ld_gates, p.a2, p.a2_b, p.rank, p.inv_tau = low.data_ptr(), low.stride(0), a2.data_ptr(), a2_b.data_ptr(), a2.shape[1], 1.0 / tau
         p.S = state.data_ptr()
-        return _run_gated(KIND_GLA, p, proj, out, qo_indptr)
+        return _run_gated(KIND_GLA, p, proj, out, qo_indptr, plan)
     q, k, v, g = _qkvg(proj, h, dk, dv)
     z = low.to(torch.float32) @ a2.to(torch.float32).t() + a2_b
     decay = torch.exp(torch.nn.functional.logsigmoid(z) / tau).view(T, h, dk)
@@ -153,7 +203,8 @@ def gla_mix(proj, low, a2, a2_b, tau: float, norm_w, eps: float, state, qo_indpt
     return o.reshape(T, h * dv).to(out_dtype)
 
 
-def mlstm_mix(proj, gates, i_b, f_b, cap: float, norm_w, eps: float, state, qo_indptr, state_idx, h: int, dk: int, dv: int, out_dtype):
+def mlstm_mix(proj, gates, i_b, f_b, cap: float, norm_w, eps: float, state, qo_indptr, state_idx, h: int, dk: int, dv: int, out_dtype,
+            plan=None):
     """mLSTM matrix memory over the token ranges of B sequences, up to the output projection.
 
     proj as in :func:`gla_mix`, gates fp32 [T, i_raw h | f_raw h], i_b / f_b fp32 [h], norm_w fp32 [h*dv], state = (S
@@ -167,7 +218,7 @@ def mlstm_mix(proj, gates, i_b, f_b, cap: float, norm_w, eps: float, state, qo_i
         p = _gated_params(proj, h, dk, dv, out, norm_w, eps, qo_indptr, state_idx)
         p.gates, p.ld_gates, p.i_b, p.f_b, p.cap = gates.data_ptr(), gates.stride(0), i_b.data_ptr(), f_b.data_ptr(), float(cap)
         p.S, p.n, p.m = S.data_ptr(), n.data_ptr(), m.data_ptr()
-        return _run_gated(KIND_MLSTM, p, proj, out, qo_indptr)
+        return _run_gated(KIND_MLSTM, p, proj, out, qo_indptr, plan)
     q, k, v, g = _qkvg(proj, h, dk, dv)
     gi = cap * torch.tanh((gates[:, :h].to(torch.float32) + i_b) / cap)
     gf = torch.nn.functional.logsigmoid(cap * torch.tanh((gates[:, h:2 * h].to(torch.float32) + f_b) / cap))
