@@ -56,7 +56,7 @@ MODEL_REGISTRY: Dict[str, ModelRegistration] = {
     "qwen3": ModelRegistration(False, False, False, True, _load_dense),
     "qwen3_5": ModelRegistration(False, False, False, False, _load_dense),
     "gidisun": ModelRegistration(False, False, False, False, _load_gidisun, float32=True,
-                                 kernel_sources=("elementwise", "gated_chunk", "gated_scan", "gemm_tcgen05", "gemv", "latent_attn", "linear_simt",
+                                 kernel_sources=("elementwise", "gated_chunk", "gated_scan", "gemm_tcgen05", "gemv", "latent_attn", "latent_mma", "linear_simt",
                                                  "sampling", "sandwich_norm", "sparse_mla")),
 }
 

@@ -214,6 +214,10 @@ _SIGS = {
     "sl_latent_pre": [vp, i32, i32, vp],
     "sl_latent_rows": [vp, i32, i32, vp],
     "sl_gated_step": [vp, i32, i32, i32, i32, vp],
+    "sl_latent_gather": [vp, i32, i32, vp],
+    "sl_latent_mma_ok": [i32, i32, i32, i32],
+    "sl_latent_prefill": [vp, i32, i32, vp],
+    "sl_latent_decode": [vp, i32, vp],
     "sl_gated_chunk_ok": [i32, i32, i32, i32],
     "sl_gated_chunks": [vp, i32, i32, vp],
     "sl_embed": [vp, vp, vp, i32, i32, i32, vp],
