@@ -54,6 +54,8 @@ def parse():
     ap.add_argument("--serving-decode", type=int, default=512, help="tokens each request of the scheduler run decodes")
     ap.add_argument("--cp-context", type=int, default=131072)
     ap.add_argument("--tiny", action="store_true", help="small model (smoke runs)")
+    ap.add_argument("--hybrid", nargs="?", const="small,medium,large", default="", metavar="SIZES",
+                    help="instead of the headline: prefill / decode throughput of the hybrid families (Gidisun beside Qwen3.5), one GPU")
     return ap.parse_args()
 
 
@@ -124,6 +126,10 @@ def main():
         print(json.dumps({"impl": "reference", "unavailable": "reference is a Node.js/N-API addon compiled only for sm_120a "
                           "with an empty vendor/flashinfer submodule; `pip install` of the reference tree fails: no setup.py/pyproject.toml"}))
         return 0
+
+    if args.hybrid:
+        from slopllm_b200.cli.hybrid_bench import main as hybrid_main
+        return hybrid_main(["--sizes", args.hybrid, "--iters", str(args.steps)])
 
     # the contract is ONE line on stdout: libraries that print there (NCCL's version banner) are sent to stderr for the
     # whole run, the JSON line goes to the saved descriptor at the end

@@ -15,6 +15,7 @@ COMMANDS = {
     "kernel-bench": "slopllm_b200.cli.kernel_bench",
     "trace-run": "slopllm_b200.cli.trace_run",
     "profile-step": "slopllm_b200.cli.profile_step",
+    "hybrid-bench": "slopllm_b200.cli.hybrid_bench",
     "collective-bench": "slopllm_b200.cli.collective_bench",
     "build": "slopllm_b200.build_native",
 }

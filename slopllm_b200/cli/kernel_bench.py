@@ -1,6 +1,6 @@
 """Kernel micro-benchmarks at the production shapes of one rank of a TP-8 GLM-5-class model.
 
-    python -m slopllm_b200.cli.kernel_bench [--cases linear,mlp,moe,gemm,fp8] [--tokens 1,8,32,4096] [--iters 20]
+    python -m slopllm_b200.cli.kernel_bench [--cases linear,mlp,moe,gemm,fp8,mixers] [--tokens 1,8,32,4096] [--iters 20]
 
 For every (kernel, token count) it prints one JSON line with the device time (CUDA events, median of `--iters`
 runs, three warm-up runs, a 256 MB write between runs so that no operand is served from L2), the algorithmic
@@ -80,6 +80,86 @@ def time_op(fn: Callable[[], object], iters: int, flush: torch.Tensor) -> float:
     return statistics.median(times)
 
 
+def mixer_rows(emit, tokens, iters: int, flush, peaks, dev, h: int = 16, dk: int = 128, dv: int = 128, rank: int = 512, rot: int = 64,
+               window: int = 1024, context: int = 2048, n_kv: int = 4) -> None:
+    """Token mixers of the hybrid families at 16 heads of 128: GLA, mLSTM and latent attention beside Gated DeltaNet and paged
+    grouped-query attention.  More than 64 tokens: one prompt; fewer: that many sequences of `context` tokens decode one each."""
+    import types
+    from ..models.glm_moe_dsa import StepState
+    from ..ops import dense as D, get_ops, latent as L, recurrent as RC
+    from ..ops.rotary import rotary_table
+    ops = get_ops(types.SimpleNamespace(rms_norm_eps=1e-6), dev)
+    g = torch.Generator(device=dev).manual_seed(3)
+    rnd = lambda *s, k=1.0: torch.randn(*s, device=dev, generator=g) * k
+    bf = lambda *s, k=1.0: rnd(*s, k=k).to(torch.bfloat16)
+    for T in tokens:
+        prompt = T > 64
+        B = 1 if prompt else T
+        start = 0 if prompt else context - 1
+        kv = T if prompt else context
+        width = -(-kv // 64)
+        i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+        pt = torch.arange(B * width, dtype=torch.int32, device=dev).view(B, width)
+        st = StepState(input_ids=torch.zeros(T, dtype=torch.int64, device=dev), positions=i32([start + i if prompt else start for i in range(T)]),
+                       batch_idx=i32([0 if prompt else i for i in range(T)]), page_table=pt, max_kv_len=kv)
+        qo = i32([0, T] if prompt else list(range(T + 1)))
+        if prompt:
+            st.extra.update(spans=[[0, T]], qo_indptr=qo, max_q=T)
+        sidx, plan = i32(list(range(B))), RC.ChunkPlan.of(st)
+        low16, S = rnd(T, 16), rnd(B, h, dk, dv)
+        io = T * h * (2 * dk + 3 * dv) * 2 + 2 * B * h * dk * dv * 4
+        flops = 4.0 * T * h * dk * dv
+        a2, a2b, nw, nwh = bf(h * dk, 16), rnd(h * dk), rnd(dv), rnd(h * dv)
+        proj, projf = bf(T, h * 2 * (dk + dv)), rnd(T, h * 2 * (dk + dv))
+        pr = proj if prompt else projf                        # decoding rows arrive in fp32
+        io += 0 if prompt else T * h * (2 * dk + 2 * dv) * 2
+        us = time_op(lambda: RC.gla_mix(pr, low16, a2, a2b, 16.0, nw, 1e-6, S, qo, sidx, h, dk, dv, torch.bfloat16, plan), iters, flush)
+        emit(roofline_row("gla", T, us, io, flops, peaks))
+        gates, ib, fb = rnd(T, 2 * h), rnd(h), rnd(h) + 4
+        state = (S, rnd(B, h, dk), torch.zeros(B, h, device=dev))
+        us = time_op(lambda: RC.mlstm_mix(pr, gates, ib, fb, 15.0, nwh, 1e-6, state, qo, sidx, h, dk, dv, torch.bfloat16, plan), iters, flush)
+        emit(roofline_row("mlstm", T, us, io, flops, peaks))
+        qkv, ab = bf(T, h * (2 * dk + dv)), bf(T, h)
+        us = time_op(lambda: RC.gdn_scan(qkv, ab, ab, ib, fb, S, qo, sidx, h, dk, dv), iters, flush)
+        emit(roofline_row("gdn (scan alone)", T, us, T * h * (2 * dk + 2 * dv) * 2 + 2 * B * h * dk * dv * 4, flops, peaks))
+        # attention
+        sh = L.LatentShape(h, dk, rot, dv, rank, (dk + rot) ** -0.5, window)
+        uv = bf(h, dv, rank, k=rank ** -0.5)
+        w = L.LatentWeights(rnd(rank), bf(h, dk, rank, k=rank ** -0.5), uv, uv.transpose(1, 2).contiguous(), rnd(h))
+        rt = rotary_table(rot, 1e6).to(dev)
+        cache, qd = bf(B * width * 64, sh.row), bf(T, h * (dk + rot) + sh.row)
+        us = time_op(lambda: L.latent_pre(qd, sh, w, rt, st, cache), iters, flush)
+        emit(roofline_row("latent_pre", T, us, 2 * T * (2 * h * rot + 2 * sh.row), 0.0, peaks))
+        q_rot = L.latent_pre(qd, sh, w, rt, st, cache)
+        pairs = sum(min(start + i + 1, window) for i in range(T)) if prompt else T * min(kv, window)
+        if prompt:
+            us = time_op(lambda: L.latent_prefill(qd, q_rot, sh, w, st, cache, ops), iters, flush)
+            fl = 2.0 * pairs * h * (dk + rot + dv) + 2.0 * T * rank * h * (dk + dv)
+            emit(roofline_row("latent_prefill (gather, expand, attend)", T, us, 2.0 * T * (sh.row + h * (dk + rot + dv)), fl, peaks))
+            rows, k, v = bf(T, sh.row), bf(T, h * dk), bf(T, h * dv)
+            out, pp = bf(T, h * dv), L.PortionPlan.of(st, window)
+            us = time_op(lambda: L.latent_prefill_kernel(qd, q_rot, sh, w, rows, k, v, pp, 0, h, out), iters, flush)
+            emit(roofline_row("latent_prefill kernel", T, us, 2.0 * T * h * (2 * (dk + dv) + rot), 2.0 * pairs * h * (dk + rot + dv), peaks))
+        else:
+            us = time_op(lambda: L.latent_attention(qd, q_rot, sh, w, st, cache, ops), iters, flush)
+            nb = 2.0 * T * min(kv, window) * sh.row + 2.0 * h * rank * (dk + dv)
+            emit(roofline_row("latent_decode (absorb, attend, expand)", T, us, nb, 2.0 * pairs * h * (2 * rank + rot), peaks))
+        kc, vc = bf(B * width * 64, n_kv, 128), bf(B * width * 64, n_kv, 128)
+        q = bf(T, h, 128)
+        us = time_op(lambda: D.paged_attention(q, kc, vc, st.positions, st.batch_idx, pt, 64, 128 ** -0.5, qo_indptr=qo if prompt else None,
+                                               max_q=T, max_kv_len=kv), iters, flush)
+        full = T * (T + 1) / 2 if prompt else T * kv
+        emit(roofline_row("paged_attention (full context)", T, us, 2.0 * (T if prompt else T * kv) * n_kv * 256 + 4.0 * T * h * 128,
+                          4.0 * full * h * 128, peaks))
+        # norms
+        H = h * 128
+        y, res, wf, wb = rnd(T, H), rnd(T, H), rnd(H), bf(H)
+        us = time_op(lambda: ops.post_norm(y, res, wf, wf, 1e-6), iters, flush)
+        emit(roofline_row("post_norm", T, us, T * H * 14.0, 0.0, peaks))
+        us = time_op(lambda: ops.add_rmsnorm(y, res, wb, 1e-6), iters, flush)
+        emit(roofline_row("add_rmsnorm", T, us, T * H * 14.0, 0.0, peaks))
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="slopllm_b200.cli.kernel_bench")
     ap.add_argument("--cases", default="linear,mlp,moe")
@@ -151,6 +231,8 @@ def main(argv=None) -> int:
                 us = time_op(lambda: ops.linear(x, w), args.iters, flush)
                 emit(roofline_row(name, T, us, n * k + 4 * sc.numel() + 2 * T * (n + k), 2.0 * T * n * k, peaks))
             del w, q
+    if "mixers" in cases:
+        mixer_rows(emit, tokens, args.iters, flush, peaks, dev)
     H = cfg.hidden_size
     if "mlp" in cases:
         lw = random_layer(cfg, 0, 0, dev, torch.bfloat16, 0, args.tp_shape, exact=False)

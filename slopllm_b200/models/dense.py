@@ -236,20 +236,21 @@ def _lin(t: torch.Tensor) -> LinearWeight:
     return LinearWeight(t.contiguous())
 
 
-def random_dense_model(cfg: DenseConfig, seed: int = 0, device="cpu", dtype=torch.bfloat16, rank: int = 0, world: int = 1) -> DenseWeights:
+def random_dense_model(cfg: DenseConfig, seed: int = 0, device="cpu", dtype=torch.bfloat16, rank: int = 0, world: int = 1,
+                       draw_device="cpu") -> DenseWeights:
     """Random weights with the checkpoint's shapes, sharded for `rank` of `world`: the full
-    matrices are drawn from the seed on every rank and sliced, so shards agree."""
-    g = torch.Generator().manual_seed(seed)
+    matrices are drawn from the seed on every rank and sliced, so shards agree.  `draw_device`: where they are drawn."""
+    g = torch.Generator(device=draw_device).manual_seed(seed)
     H, I, hd = cfg.hidden_size, cfg.intermediate_size, cfg.head_dim
     tensors: Dict[str, torch.Tensor] = {}
     pfx = cfg.weight_prefix
 
     def rnd(*shape, scale=None):
         s = scale if scale is not None else shape[-1] ** -0.5
-        return (torch.randn(*shape, generator=g) * s).to(torch.bfloat16)
+        return (torch.randn(*shape, generator=g, device=draw_device) * s).to(torch.bfloat16)
 
     def norm_w(n):
-        w = 1.0 + 0.1 * torch.randn(n, generator=g)
+        w = 1.0 + 0.1 * torch.randn(n, generator=g, device=draw_device)
         return (w - 1.0 if cfg.gemma_norm else w).to(torch.bfloat16)
 
     tensors[pfx + "embed_tokens.weight"] = rnd(cfg.vocab_size, H, scale=1.0)
@@ -275,9 +276,9 @@ def random_dense_model(cfg: DenseConfig, seed: int = 0, device="cpu", dtype=torc
             tensors[lp + "linear_attn.in_proj_a.weight"] = rnd(lh, H)
             tensors[lp + "linear_attn.in_proj_b.weight"] = rnd(lh, H)
             tensors[lp + "linear_attn.conv1d.weight"] = rnd(cfg.conv_dim, 1, kw, scale=0.5)
-            tensors[lp + "linear_attn.A_log"] = torch.log(torch.rand(lh, generator=g) * 2 + 0.5)
-            tensors[lp + "linear_attn.dt_bias"] = torch.randn(lh, generator=g) * 0.1
-            tensors[lp + "linear_attn.norm.weight"] = (1.0 + 0.1 * torch.randn(dv, generator=g)).to(torch.bfloat16)
+            tensors[lp + "linear_attn.A_log"] = torch.log(torch.rand(lh, generator=g, device=draw_device) * 2 + 0.5)
+            tensors[lp + "linear_attn.dt_bias"] = torch.randn(lh, generator=g, device=draw_device) * 0.1
+            tensors[lp + "linear_attn.norm.weight"] = (1.0 + 0.1 * torch.randn(dv, generator=g, device=draw_device)).to(torch.bfloat16)
             tensors[lp + "linear_attn.out_proj.weight"] = rnd(H, lh * dv)
     tensors[pfx + "norm.weight"] = norm_w(H)
     if not cfg.tie_word_embeddings:

@@ -201,12 +201,18 @@ def latent_prefill(qd, q_rot, s: LatentShape, w: LatentWeights, st, cache, ops) 
         hn = min(group, s.heads - h0)
         k = ops.linear(lat, LinearWeight(uk[h0 * s.dim:(h0 + hn) * s.dim]))
         v = ops.linear(lat, LinearWeight(uv[h0 * s.vdim:(h0 + hn) * s.vdim]))
-        p = LatentPrefillParams(q=qd.data_ptr(), ldq=qd.stride(0), q_head=s.dim + s.rot_dim, q_rot=q_rot.data_ptr(), k=k.data_ptr(),
-                                ldk=k.stride(0), v=v.data_ptr(), ldv=v.stride(0), rows=rows.data_ptr(), row=s.row, rank=s.rank,
-                                tiles=plan.tiles.data_ptr(), heads=s.heads, h0=h0, dim=s.dim, rot_dim=s.rot_dim, vdim=s.vdim,
-                                window=s.window, scale=s.scale, sink=N.ptr(w.sink), out=out.data_ptr())
-        N.call("sl_latent_prefill", C.byref(p), hn, plan.tile_count, N.stream())
+        latent_prefill_kernel(qd, q_rot, s, w, rows, k, v, plan, h0, hn, out)
     return out
+
+
+def latent_prefill_kernel(qd, q_rot, s: LatentShape, w: LatentWeights, rows, k, v, plan: PortionPlan, h0: int, heads: int, out) -> None:
+    """Attention of heads h0 .. h0 + heads - 1 over their expanded keys k [rows, heads * dim] and values v [rows, heads * vdim]."""
+    N = _native()
+    p = LatentPrefillParams(q=qd.data_ptr(), ldq=qd.stride(0), q_head=s.dim + s.rot_dim, q_rot=q_rot.data_ptr(), k=k.data_ptr(),
+                            ldk=k.stride(0), v=v.data_ptr(), ldv=v.stride(0), rows=rows.data_ptr(), row=s.row, rank=s.rank,
+                            tiles=plan.tiles.data_ptr(), heads=s.heads, h0=h0, dim=s.dim, rot_dim=s.rot_dim, vdim=s.vdim,
+                            window=s.window, scale=s.scale, sink=N.ptr(w.sink), out=out.data_ptr())
+    N.call("sl_latent_prefill", C.byref(p), heads, plan.tile_count, N.stream())
 
 
 def decode_splits(T: int, heads: int, keys: int) -> int:
