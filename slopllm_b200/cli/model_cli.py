@@ -23,7 +23,10 @@ from ..parallel.dist import ParallelContext, init_from_env
 def add_model_args(ap: argparse.ArgumentParser) -> None:
     ap.add_argument("--model", default="", help="checkpoint directory or Hugging Face hub id (local cache only)")
     ap.add_argument("--random-init", default="", metavar="SPEC",
-                    help="no checkpoint: random weights of 'tiny', 'glm5[:layers]', 'qwen3-tiny' or 'qwen35-tiny'")
+                    help="no checkpoint: random weights of 'tiny', 'glm5[:layers]', 'qwen3-tiny', 'qwen35-tiny' or 'gidisun-tiny'")
+    ap.add_argument("--dtype", choices=("bfloat16", "float32"), default=None,
+                    help="activation and weight type; default bfloat16 on a GPU.  float32 (no reduced-precision products) for the "
+                         "families that have it")
     ap.add_argument("--gpus", default="", help="comma-separated device list; its length must equal the number of ranks")
     ap.add_argument("--arena", type=float, default=0.0,
                     help="GiB of device memory this process may allocate per GPU (weights + KV cache + step buffers); a larger "
@@ -102,7 +105,7 @@ def check_memory_plan(args, ctx: ParallelContext, model_dir: str, model_type: st
     """Before the weights are read: does this rank's share of the model plus the KV pages asked for fit the memory the
     process may use?  A plan that does not fit is reported on stderr (rank 0) and returned; loading still goes ahead, the
     estimate of the workspace is deliberately generous."""
-    if model_type not in ("glm_moe_dsa", "qwen3", "qwen3_5") or ctx.device.type != "cuda":
+    if model_type not in ("glm_moe_dsa", "qwen3", "qwen3_5", "gidisun") or ctx.device.type != "cuda":
         return None
     import sys
     from ..utils.sizing import GIB, plan_dense, plan_memory
@@ -111,6 +114,14 @@ def check_memory_plan(args, ctx: ParallelContext, model_dir: str, model_type: st
         from ..checkpoint.loader import load_config
         p = plan_memory(load_config(model_dir), world=ctx.world, cp=args.cp, ep=args.ep, mtp=args.mtp, batch_size=args.batch_size,
                         chunk_size=args.chunk_size, max_pages=args.max_pages, arena_gb=args.arena, device_gb=total / GIB)
+    elif model_type == "gidisun":
+        import json
+        from ..models.gidisun import GidisunConfig
+        from ..utils.sizing import plan_gidisun
+        with open(os.path.join(model_dir, "config.json")) as f:
+            gcfg = GidisunConfig.from_dict(json.load(f))
+        p = plan_gidisun(gcfg, world=ctx.world, batch_size=args.batch_size, chunk_size=args.chunk_size, max_pages=args.max_pages,
+                         arena_gb=args.arena, device_gb=total / GIB, elem=4 if getattr(args, "dtype", None) == "float32" else 2)
     else:
         import json
         from ..models.dense import DenseConfig
@@ -128,9 +139,15 @@ def check_memory_plan(args, ctx: ParallelContext, model_dir: str, model_type: st
     return msg
 
 
-def _random_model(spec: str, ctx: ParallelContext, mtp: int):
+def _random_model(spec: str, ctx: ParallelContext, mtp: int, dtype_name: Optional[str] = None):
     from ..parallel.fused import make_comm
     dtype = torch.bfloat16 if ctx.device.type == "cuda" else torch.float32
+    if spec.startswith("gidisun"):
+        from ..models.gidisun import GidisunConfig, GidisunModel, random_gidisun_tensors
+        cfg = GidisunConfig.tiny()
+        return cfg, GidisunModel.from_tensors(cfg, random_gidisun_tensors(cfg), ctx, getattr(torch, dtype_name) if dtype_name else dtype), cfg.model_type
+    if dtype_name is not None and getattr(torch, dtype_name) != dtype:
+        raise SystemExit(f"--random-init {spec} does not run in {dtype_name} on {ctx.device.type}")
     tp_world = ctx.world          # weights stay tensor-parallel under context parallelism too
     tp_rank = ctx.rank if tp_world > 1 else 0
     if spec.startswith("qwen"):
@@ -151,7 +168,7 @@ def _random_model(spec: str, ctx: ParallelContext, mtp: int):
 
 
 def build_runtime(args, with_scheduler: bool = True) -> Runtime:
-    from ..models.registry import inspect_model
+    from ..models.registry import inspect_model, load_registered
     from ..runtime.engine import Engine
     from ..sampling.workspace import SamplingWorkspace
     from ..scheduler.replicated import make_channel
@@ -165,7 +182,7 @@ def build_runtime(args, with_scheduler: bool = True) -> Runtime:
         os.environ["SLOPLLM_B200_FUSED"] = "0"
     model_dir: Optional[str] = None
     if args.random_init:
-        cfg, model, model_type = _random_model(args.random_init, ctx, args.mtp)
+        cfg, model, model_type = _random_model(args.random_init, ctx, args.mtp, getattr(args, "dtype", None))
     else:
         if not args.model:
             raise SystemExit("give --model DIR|HUB_ID or --random-init SPEC")
@@ -175,7 +192,7 @@ def build_runtime(args, with_scheduler: bool = True) -> Runtime:
             args.max_model_len = max_position_embeddings(model_dir)
         model_type, reg, _ = inspect_model(model_dir, cp=args.cp, mtp=args.mtp)
         check_memory_plan(args, ctx, model_dir, model_type)
-        cfg, model = reg.load(model_dir, ctx, args.mtp)
+        cfg, model = load_registered(reg, model_dir, ctx, args.mtp, getattr(args, "dtype", None))
     if getattr(args, "max_model_len", None) is None:
         args.max_model_len = 65536
     ecfg = EngineConfig(model=args.model or args.random_init, gpus=list(range(ctx.world)), arena_gb=args.arena, cp=args.cp, ep=args.ep,

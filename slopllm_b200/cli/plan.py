@@ -26,13 +26,19 @@ def _config(args) -> GlmMoeDsaConfig:
         if model_type in ("qwen3", "qwen3_5"):
             from ..models.dense import DenseConfig
             return DenseConfig.from_hf_dict(raw)
+        if model_type == "gidisun":
+            from ..models.gidisun import GidisunConfig
+            return GidisunConfig.from_dict(raw)
         if model_type != "glm_moe_dsa":
-            raise SystemExit(f"plan: the sizing arithmetic covers glm_moe_dsa, qwen3 and qwen3_5; {args.model} is {model_type}")
+            raise SystemExit(f"plan: the sizing arithmetic covers glm_moe_dsa, qwen3, qwen3_5 and gidisun; {args.model} is {model_type}")
         return load_config(model_dir)
     spec = args.random_init or "glm5"
     if spec.startswith("qwen"):
         from ..models.dense import DenseConfig
         return DenseConfig.tiny(hybrid=spec.startswith("qwen35"))
+    if spec.startswith("gidisun"):
+        from ..models.gidisun import GidisunConfig
+        return GidisunConfig.tiny()
     if spec.startswith("glm5"):
         return GlmMoeDsaConfig.glm5(num_layers=int(spec.split(":")[1]) if ":" in spec else 78)
     return GlmMoeDsaConfig.tiny()
@@ -41,7 +47,7 @@ def _config(args) -> GlmMoeDsaConfig:
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="slopllm_b200.cli.plan", description=__doc__.split("\n")[0])
     ap.add_argument("--model", default="", help="checkpoint directory or hub id (only config.json is read)")
-    ap.add_argument("--random-init", default="", help="glm5[:layers], tiny, qwen3 or qwen35 instead of a checkpoint")
+    ap.add_argument("--random-init", default="", help="glm5[:layers], tiny, qwen3, qwen35 or gidisun instead of a checkpoint")
     ap.add_argument("--world", type=int, default=1, help="GPUs of one replica")
     ap.add_argument("--cp", action="store_true")
     ap.add_argument("--ep", action="store_true")
@@ -55,8 +61,9 @@ def main(argv=None) -> int:
     args = ap.parse_args(argv)
     cfg = _config(args)
     if not isinstance(cfg, GlmMoeDsaConfig):
-        from ..utils.sizing import plan_dense
-        p = plan_dense(cfg, world=args.world, batch_size=args.batch_size, chunk_size=args.chunk_size, max_pages=args.max_pages,
+        from ..utils.sizing import plan_dense, plan_gidisun
+        planner = plan_gidisun if cfg.model_type == "gidisun" else plan_dense
+        p = planner(cfg, world=args.world, batch_size=args.batch_size, chunk_size=args.chunk_size, max_pages=args.max_pages,
                        arena_gb=args.arena, device_gb=args.device_gb)
     else:
         p = plan_memory(cfg, world=args.world, cp=args.cp, ep=args.ep, mtp=args.mtp, batch_size=args.batch_size,

@@ -188,3 +188,54 @@ def plan_dense(cfg, world: int = 1, batch_size: int = 8, chunk_size: int = 8192,
     return MemoryPlan(tp=world, cp=1, ep=False, weights_bytes=weights, page_bytes=page, tokens_per_page=PAGE_SIZE,
                       workspace_bytes=work, budget_bytes=budget, max_pages=int(fit), max_tokens=int(fit) * PAGE_SIZE,
                       requested_pages=requested, requested_fits=requested <= fit)
+
+
+# ---- Gidisun --------------------------------------------------------------------------------------------------------------
+
+def gidisun_weight_bytes(cfg, tp: int = 1, elem: int = 2, low_rank: int = 16) -> int:
+    """Per-rank weight bytes: projections head-sharded, feed-forward sharded, embedding whole, head vocabulary-sharded; norm
+    weights, biases and sinks are fp32.  `low_rank`: width of the GLA decay projection (a tensor shape, not in the
+    configuration)."""
+    H = cfg.hidden_size
+    b = cfg.vocab_size * H * elem + (cfg.vocab_size // tp) * H * elem + 4 * H
+    for l in cfg.layers:
+        c, h = l.mixer, l.mixer["heads"] // tp
+        dk, dv = c["dim"], c["vdim"]
+        b += h * dv * H * elem + 4 * 2 * H * (2 if l.ff else 1) + 3 * (l.ff // tp) * H * elem
+        if l.type == "latent_attention":
+            R, dr = c["kv_rank"], c["rot_dim"]
+            b += (h * (dk + dr) + R + dr) * H * elem + h * (dk + 2 * dv) * R * elem + 4 * (R + h)     # (values in two layouts)
+        elif l.type == "gla":
+            b += (h * 2 * (dk + dv) + low_rank) * H * elem + h * dk * (low_rank * elem + 4) + 4 * dv
+        else:
+            b += (h * 2 * (dk + dv) + 2 * h) * H * elem + 4 * (2 * h + h * dv)
+    return b
+
+
+def gidisun_cache_bytes(cfg, tp: int = 1, elem: int = 2):
+    """(bytes of one 64-token page, bytes of one sequence's recurrent state) on one rank."""
+    page = state = 0
+    for l in cfg.layers:
+        c = l.mixer
+        if l.type == "latent_attention":
+            page += (c["kv_rank"] + c["rot_dim"]) * elem * PAGE_SIZE
+        else:
+            h = c["heads"] // tp
+            state += 4 * h * (c["dim"] * c["vdim"] + (c["dim"] + 1 if l.type == "mlstm" else 0))
+    return page, state
+
+
+def plan_gidisun(cfg, world: int = 1, batch_size: int = 8, chunk_size: int = 8192, max_pages: int = 0, arena_gb: float = 0.0,
+                 device_gb: float = 180.0, elem: int = 2, reserve_gb: float = 4.0) -> MemoryPlan:
+    """`plan_memory` for Gidisun (tensor parallel only).  The workspace estimate is the widest layer's rows of one chunk, the
+    recurrent state of every slot, and the transient keys, values and chunk states of a prefill."""
+    weights = gidisun_weight_bytes(cfg, world, elem)
+    page, state = gidisun_cache_bytes(cfg, world, elem)
+    requested = max_pages if max_pages > 0 else batch_size * -(-chunk_size // PAGE_SIZE)
+    row = max(max(3 * l.ff, 6 * l.mixer["heads"] * (l.mixer["dim"] + l.mixer["vdim"])) for l in cfg.layers) // world
+    work = chunk_size * (cfg.hidden_size * 12 + row * elem) + state * max(64, batch_size) + (1 << 30)
+    budget = int(((arena_gb if arena_gb > 0 else device_gb) - reserve_gb) * GIB)
+    fit = max(0, (budget - weights - work) // max(1, page))
+    return MemoryPlan(tp=world, cp=1, ep=False, weights_bytes=weights, page_bytes=page, tokens_per_page=PAGE_SIZE,
+                      workspace_bytes=work, budget_bytes=budget, max_pages=int(fit), max_tokens=int(fit) * PAGE_SIZE,
+                      requested_pages=requested, requested_fits=requested <= fit)

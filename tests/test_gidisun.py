@@ -219,3 +219,52 @@ def test_registry_and_trace_replay(tmp_path, monkeypatch, capsys):
     assert not (tmp_path / "o" / "1.f32").exists()
     assert row_error(read(2), torch.stack([wa[69], wb[11]])).max() < 1e-5
     assert row_error(read(3), wa[69:70]).max() < 1e-5
+
+
+def _tensor_bytes(obj) -> int:
+    seen, total, stack = set(), 0, [obj]
+    while stack:
+        x = stack.pop()
+        if isinstance(x, torch.Tensor):
+            if x.data_ptr() not in seen:
+                seen.add(x.data_ptr())
+                total += x.numel() * x.element_size()
+        elif isinstance(x, (list, tuple)):
+            stack += x
+        elif hasattr(x, "__dataclass_fields__"):
+            stack += [getattr(x, f) for f in x.__dataclass_fields__]
+    return total
+
+
+@pytest.mark.parametrize("world", [1, 2])
+def test_memory_plan_matches_the_built_model(world, capsys):
+    from slopllm_b200.cli import plan as plan_cli
+    from slopllm_b200.models.gidisun import assemble_gidisun_weights, random_gidisun_tensors
+    from slopllm_b200.utils.sizing import gidisun_cache_bytes, gidisun_weight_bytes
+    cfg = GidisunConfig.tiny()
+    w = assemble_gidisun_weights(cfg, random_gidisun_tensors(cfg), "cpu", torch.float32, 0, world)
+    table = sum(t.numel() * 4 for t in {id(m.rot.freq): m.rot.freq for m in w.mixers if hasattr(m, "rot")}.values())
+    assert _tensor_bytes(w) == gidisun_weight_bytes(cfg, world, 4) + table
+    page, state = gidisun_cache_bytes(cfg, world, 4)
+    assert page == sum(m.spec.row_values() for m in w.mixers) * 4 * 64 and state == sum(m.spec.state_values() for m in w.mixers) * 4
+    assert plan_cli.main(["--random-init", "gidisun", "--max-pages", "64"]) == 0
+    capsys.readouterr()
+
+
+def test_command_line_runtime():
+    """The shared entry-point code builds the family, and a request runs through its scheduler with sampling."""
+    import argparse
+    from slopllm_b200.cli.model_cli import add_model_args, build_runtime
+    from slopllm_b200.config import SamplingParams
+    from slopllm_b200.scheduler.scheduler import GenerationRequest
+    ap = argparse.ArgumentParser()
+    add_model_args(ap)
+    rt = build_runtime(ap.parse_args(["--cpu", "--random-init", "gidisun-tiny", "--no-cuda-graph", "--batch-size", "2", "--chunk-size", "32",
+                                      "--max-pages", "16"]))
+    assert rt.model_type == "gidisun"
+    reqs = [GenerationRequest(id=str(i), input_ids=[5 + i] * 40, max_tokens=4, sampling=SamplingParams(temperature=0.8)) for i in range(3)]
+    for r in reqs:
+        rt.scheduler.submit(r)
+    for _ in range(40):
+        rt.scheduler.step()
+    assert all(r.retired and r.error is None and len(r.generated) == 4 for r in reqs)
