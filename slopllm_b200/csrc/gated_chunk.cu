@@ -28,21 +28,29 @@ struct GatedChunkParams {
     const int* chunks;                       // [chunks][4]: sequence, first token, tokens, 1 if the sequence's last chunk
     const int* seq_chunks;                   // [B + 1]
     int c0, c1;                              // chunk range of this pass
-    float* b;                                // GLA: running log decays [T, h * dk]
-    float* loc;                              // [chunks of the pass, h, dk, dv]: own contribution, then S_in as (hi, lo) bf16 words
+    float* b;                                // GLA: running log2 decays [T, h * dk]
+    float* loc;                              // [chunks of the pass, h, dk, dv]: own contribution, then S_in: eight high bf16 terms,
+                                             // then their eight low terms, in the place of every eight values
     float* nloc;                             // mLSTM: [chunks of the pass, h, dk], then n_in
-    float* scal;                             // mLSTM: [chunks of the pass, h, 4]: b_C, M_C, m_in
+    float* scal;                             // mLSTM: [chunks of the pass, h, 4]: b_C, M_C, m_in, m after the chunk
+    int slab_bufs;                           // set by the launcher: state slabs in shared memory at a time (1 or 2)
 };
 
-// rows [n][dim] (bf16, 16-byte chunks) -> shared [CT][ld], zero beyond n rows and beyond dim columns up to `padded`
+// rows [n][dim] (bf16, 16-byte pieces) -> shared [CT][ld] with cp.async, zero beyond n rows and beyond dim columns up to `padded`
 __device__ __forceinline__ void load_rows(bf16* dst, int ld, const bf16* src, size_t stride, int n, int dim, int padded) {
     const int per = padded / 8;
     for (int i = threadIdx.x; i < CT * per; i += blockDim.x) {
         const int r = i / per, c = (i % per) * 8;
-        uint4 v = make_uint4(0, 0, 0, 0);
-        if (r < n && c < dim) v = *reinterpret_cast<const uint4*>(src + (size_t)r * stride + c);
-        *reinterpret_cast<uint4*>(dst + r * ld + c) = v;
+        if (r < n && c < dim) cp_async16(dst + r * ld + c, src + (size_t)r * stride + c);
+        else *reinterpret_cast<uint4*>(dst + r * ld + c) = make_uint4(0, 0, 0, 0);
     }
+}
+
+constexpr float LOG2E = 1.4426950408889634f;
+__device__ __forceinline__ float exp2_fast(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
 }
 
 // One warp: a_s = i_s - b_s, b_s, and the running maximum M_s of a over the chunk's tokens (two tokens per lane).
@@ -94,29 +102,38 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(GatedChunkParams cp) {
     const int* ch = cp.chunks + (size_t)(cp.c0 + ci) * 4;
     const int t0 = ch[1], n = ch[2], dk = p.dk, dv = p.dv;
     const int dkp = (dk + 15) / 16 * 16, ldk = dkp + 8, ldv = dv + 8;
-    bf16* kh = reinterpret_cast<bf16*>(smraw);           // [CT][ldk] decayed keys, high and low terms
+    bf16* kh = reinterpret_cast<bf16*>(smraw);           // [CT][ldk] keys, then decayed keys: high and low terms
     bf16* kl = kh + CT * ldk;
     bf16* vs = kl + CT * ldk;                            // [CT][ldv]
-    float* fs = reinterpret_cast<float*>(vs + CT * ldv); // GLA: log decays [CT][dk] | low-rank rows [CT][rank]; mLSTM: a, b, M
+    float* fs = reinterpret_cast<float*>(vs + CT * ldv); // GLA: log2 decays [CT][dk], then the inputs; mLSTM: a, b, M
+    load_rows(kh, ldk, (const bf16*)p.k + (size_t)t0 * p.ld + h * dk, p.ld, n, dk, dkp);
     load_rows(vs, ldv, (const bf16*)p.v + (size_t)t0 * p.ld + h * dv, p.ld, n, dv, dv);
+    cp_async_commit();
     if (KIND == KIND_GLA) {
-        float* low = fs + CT * dk;
-        for (int i = tid; i < n * p.rank; i += 256) low[i] = p.gates[(size_t)(t0 + i / p.rank) * p.ld_gates + i % p.rank];
+        float* low = fs + CT * dk;                       // [CT][rank]
+        bf16* a2 = reinterpret_cast<bf16*>(low + CT * p.rank);       // [dk][rank]
+        const bf16* a2g = (const bf16*)p.a2 + (size_t)h * dk * p.rank;
+#pragma unroll 4
+        for (int i = tid; i < dk * p.rank; i += 256) a2[i] = a2g[i];
+#pragma unroll 4
+        for (int i = tid; i < CT * p.rank; i += 256)
+            low[i] = i < n * p.rank ? p.gates[(size_t)(t0 + i / p.rank) * p.ld_gates + i % p.rank] : 0.f;
         __syncthreads();
         for (int i = tid; i < dk * (CT / 8); i += 256) {                 // a channel, eight tokens
             const int c = i % dk, s0 = i / dk * 8;
             if (s0 >= n) continue;
-            const bf16* a2 = (const bf16*)p.a2 + (size_t)(h * dk + c) * p.rank;
             float z[8];
 #pragma unroll
             for (int j = 0; j < 8; ++j) z[j] = p.a2_b[h * dk + c];
+#pragma unroll 4
             for (int r = 0; r < p.rank; ++r) {
-                const float w = __bfloat162float(a2[r]);
+                const float w = __bfloat162float(a2[c * p.rank + r]);
 #pragma unroll
-                for (int j = 0; j < 8; ++j) z[j] += w * (s0 + j < n ? low[(s0 + j) * p.rank + r] : 0.f);
+                for (int j = 0; j < 8; ++j) z[j] += w * low[(s0 + j) * p.rank + r];
             }
+            const float scale = p.inv_tau * LOG2E;
 #pragma unroll
-            for (int j = 0; j < 8; ++j) fs[(s0 + j) * dk + c] = logsigmoid_f(z[j]) * p.inv_tau;
+            for (int j = 0; j < 8; ++j) fs[(s0 + j) * dk + c] = logsigmoid_f(z[j]) * scale;
         }
         __syncthreads();
         for (int c = tid; c < dk; c += 256) {
@@ -125,24 +142,28 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(GatedChunkParams cp) {
             for (int s = 0; s < n; ++s) {
                 run += fs[s * dk + c];
                 fs[s * dk + c] = run;
-                cp.b[(size_t)(t0 + s) * (p.h * dk) + h * dk + c] = run;
             }
+        }
+        __syncthreads();
+        for (int i = tid; i < n * (dk / 4); i += 256) {
+            const int s = i / (dk / 4), c = (i % (dk / 4)) * 4;
+            *reinterpret_cast<float4*>(cp.b + (size_t)(t0 + s) * (p.h * dk) + h * dk + c) = *reinterpret_cast<const float4*>(fs + s * dk + c);
         }
     } else if (warp == 0) {
         mlstm_gates(p, t0, n, h, fs, fs + CT, fs + 2 * CT);
     }
+    cp_async_wait<0>();
     __syncthreads();
     const float top = KIND == KIND_MLSTM ? fs[2 * CT + n - 1] : 0.f;
-    const bf16* kg = (const bf16*)p.k + (size_t)t0 * p.ld + h * dk;
     for (int i = tid; i < CT * (dkp / 2); i += 256) {
         const int s = i / (dkp / 2), c = (i % (dkp / 2)) * 2;
         uint32_t hi = 0, lo = 0;
         if (s < n && c < dk) {
-            const float2 k = bf162_to_f2(*reinterpret_cast<const uint32_t*>(kg + (size_t)s * p.ld + c));
+            const float2 k = bf162_to_f2(*reinterpret_cast<const uint32_t*>(kh + s * ldk + c));
             float w0, w1;
             if (KIND == KIND_GLA) {
-                w0 = __expf(fs[(n - 1) * dk + c] - fs[s * dk + c]);
-                w1 = __expf(fs[(n - 1) * dk + c + 1] - fs[s * dk + c + 1]);
+                w0 = exp2_fast(fs[(n - 1) * dk + c] - fs[s * dk + c]);
+                w1 = exp2_fast(fs[(n - 1) * dk + c + 1] - fs[s * dk + c + 1]);
             } else {
                 w0 = w1 = __expf(fs[s] - top);
             }
@@ -156,6 +177,7 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(GatedChunkParams cp) {
     if (KIND == KIND_MLSTM) {
         for (int c = tid; c < dk; c += 256) {
             float a = 0.f;
+#pragma unroll 8
             for (int s = 0; s < n; ++s) a += __bfloat162float(kh[s * ldk + c]) + __bfloat162float(kl[s * ldk + c]);
             cp.nloc[base * dk + c] = a;
         }
@@ -192,13 +214,7 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(GatedChunkParams cp) {
 }
 
 // ---- 2: the state over the chunks --------------------------------------------------------------------------------------------
-__device__ __forceinline__ uint32_t pack_split(float x) {
-    const bf16 hi = __float2bfloat16(x);
-    const bf16 lo = __float2bfloat16(x - __bfloat162float(hi));
-    return (uint32_t)*reinterpret_cast<const unsigned short*>(&hi) | ((uint32_t)*reinterpret_cast<const unsigned short*>(&lo) << 16);
-}
-
-// grid (ceil(dk * dv / 1024), h, B), block 256: four consecutive values of a state row per thread
+// grid (ceil(dk * dv / 2048), h, B), block 256: eight consecutive values of a state row per thread
 template <int KIND>
 __global__ void __launch_bounds__(256) chunk_scan_kernel(GatedChunkParams cp) {
     pdl_grid_sync();
@@ -207,31 +223,33 @@ __global__ void __launch_bounds__(256) chunk_scan_kernel(GatedChunkParams cp) {
     const int lo = max(cp.seq_chunks[seq], cp.c0), hi = min(cp.seq_chunks[seq + 1], cp.c1);
     if (lo >= hi) return;
     const size_t slot = (size_t)p.state_idx[seq] * p.h + h, size = (size_t)dk * dv;
-    const int e = (blockIdx.x * 256 + threadIdx.x) * 4;
+    const int e = (blockIdx.x * 256 + threadIdx.x) * 8;
     const float m0 = KIND == KIND_MLSTM ? p.m[slot] : 0.f;
     if (e < (int)size) {
         const int c = e / dv;
-        float4 S = *reinterpret_cast<const float4*>(p.S + slot * size + e);
+        float S[8];
+        *reinterpret_cast<float4*>(S) = *reinterpret_cast<const float4*>(p.S + slot * size + e);
+        *reinterpret_cast<float4*>(S + 4) = *reinterpret_cast<const float4*>(p.S + slot * size + e + 4);
         float m = m0;
         constexpr int U = 4;                              // chunks whose contributions are in flight
         for (int i0 = lo; i0 < hi; i0 += U) {
-            float4 x[U];
-            float d[U];
+            float x[U][8], d[U];
 #pragma unroll
             for (int j = 0; j < U; ++j) {
-                const int i = i0 + j;
-                if (i >= hi) continue;
-                x[j] = *reinterpret_cast<const float4*>(cp.loc + ((size_t)(i - cp.c0) * p.h + h) * size + e);
+                const int i = min(i0 + j, hi - 1);
+                const float* src = cp.loc + ((size_t)(i - cp.c0) * p.h + h) * size + e;
+                *reinterpret_cast<float4*>(x[j]) = *reinterpret_cast<const float4*>(src);
+                *reinterpret_cast<float4*>(x[j] + 4) = *reinterpret_cast<const float4*>(src + 4);
                 if (KIND == KIND_GLA) {
                     const int* ch = cp.chunks + (size_t)i * 4;
-                    d[j] = expf(cp.b[(size_t)(ch[1] + ch[2] - 1) * (p.h * dk) + h * dk + c]);
+                    d[j] = cp.b[(size_t)(ch[1] + ch[2] - 1) * (p.h * dk) + h * dk + c];
                 }
             }
 #pragma unroll
             for (int j = 0; j < U; ++j) {
                 const int i = i0 + j;
-                if (i >= hi) continue;
-                float add = 1.f, keep = d[j];
+                if (i >= hi) break;
+                float add = 1.f, keep = KIND == KIND_GLA ? exp2f(d[j]) : 1.f;
                 if (KIND == KIND_MLSTM) {
                     const float* sc = cp.scal + ((size_t)(i - cp.c0) * p.h + h) * 4;
                     const float top = fmaxf(m, sc[1]);
@@ -239,14 +257,18 @@ __global__ void __launch_bounds__(256) chunk_scan_kernel(GatedChunkParams cp) {
                     add = expf(sc[1] - top);
                     m = sc[0] + top;
                 }
-                uint4 w;
-                w.x = pack_split(S.x); w.y = pack_split(S.y); w.z = pack_split(S.z); w.w = pack_split(S.w);
-                *reinterpret_cast<uint4*>(cp.loc + ((size_t)(i - cp.c0) * p.h + h) * size + e) = w;
-                S.x = keep * S.x + add * x[j].x; S.y = keep * S.y + add * x[j].y;
-                S.z = keep * S.z + add * x[j].z; S.w = keep * S.w + add * x[j].w;
+                uint4 wh, wl;
+                split_bf162(S[0], S[1], wh.x, wl.x); split_bf162(S[2], S[3], wh.y, wl.y);
+                split_bf162(S[4], S[5], wh.z, wl.z); split_bf162(S[6], S[7], wh.w, wl.w);
+                uint4* dst = reinterpret_cast<uint4*>(cp.loc + ((size_t)(i - cp.c0) * p.h + h) * size + e);
+                dst[0] = wh;
+                dst[1] = wl;
+#pragma unroll
+                for (int y = 0; y < 8; ++y) S[y] = keep * S[y] + add * x[j][y];
             }
         }
-        *reinterpret_cast<float4*>(p.S + slot * size + e) = S;
+        *reinterpret_cast<float4*>(p.S + slot * size + e) = *reinterpret_cast<const float4*>(S);
+        *reinterpret_cast<float4*>(p.S + slot * size + e + 4) = *reinterpret_cast<const float4*>(S + 4);
     }
     if (KIND == KIND_MLSTM && blockIdx.x == 0) {
         // normaliser and running maximum; m itself is stored by the output kernel (other blocks of this grid still read it)
@@ -279,13 +301,14 @@ constexpr int OUT_THREADS = 512;             // 16 warps: 4 row tiles of 16 toke
 constexpr int LDA = CT + 8;
 constexpr int SLAB = 64;                     // state rows in shared memory at a time
 
-template <int KIND>
-size_t output_smem(int dk, int dv) {
+size_t output_smem(int kind, int dk, int dv, int slab_bufs) {
     const int dkp = (dk + 15) / 16 * 16;
-    size_t b = (size_t)CT * (dkp + 8) * 2 * 2 + (size_t)CT * (dv + 8) * 2 + (size_t)2 * SLAB * (dv + 8) * 2 + (size_t)2 * CT * LDA * 2;
-    b += KIND == KIND_GLA ? (size_t)CT * (dkp + 4) * 4 : 0;
+    size_t b = (size_t)CT * (dkp + 8) * 2 * 2 + (size_t)CT * (dv + 8) * 2 + (size_t)slab_bufs * 2 * SLAB * (dv + 8) * 2 + (size_t)2 * CT * LDA * 2;
+    b += kind == KIND_GLA ? (size_t)CT * (dkp + 4) * 4 : 0;
     return b + (size_t)CT * 12 * 4;
 }
+constexpr size_t SMEM_MAX = 220 * 1024;
+int slab_buffers(int kind, int dk, int dv) { return dk > SLAB && output_smem(kind, dk, dv, 2) <= SMEM_MAX ? 2 : 1; }
 
 // grid (chunks of the pass, h).  NT: 8-wide value tiles per column quarter (dv <= 32 * NT).
 template <int KIND, int NT>
@@ -301,9 +324,8 @@ __global__ void __launch_bounds__(OUT_THREADS) chunk_output_kernel(GatedChunkPar
     bf16* qs = reinterpret_cast<bf16*>(smraw);           // [CT][ldk]
     bf16* ks = qs + CT * ldk;
     bf16* vs = ks + CT * ldk;                            // [CT][ldv]
-    bf16* sh = vs + CT * ldv;                            // [SLAB][ldv] state rows, high and low terms
-    bf16* sl = sh + SLAB * ldv;
-    bf16* ah = sl + SLAB * ldv;                          // [CT][LDA] scores
+    bf16* slabs = vs + CT * ldv;                         // state rows [SLAB][ldv], high and low terms, one or two slabs
+    bf16* ah = slabs + cp.slab_bufs * 2 * SLAB * ldv;        // [CT][LDA] scores
     bf16* al = ah + CT * LDA;
     float* fs = reinterpret_cast<float*>(al + CT * LDA);
     float* bs = fs;                                      // GLA: [CT][ldb]
@@ -311,18 +333,40 @@ __global__ void __launch_bounds__(OUT_THREADS) chunk_output_kernel(GatedChunkPar
     float *ga = rows, *gb = rows + CT, *gx = rows + 2 * CT, *qn = rows + 3 * CT, *nq = rows + 4 * CT, *ssq = rows + 8 * CT;
     const float qscale = rsqrtf((float)dk);
     const size_t base = (size_t)ci * p.h + h;
+    const bf16* sin = reinterpret_cast<const bf16*>(cp.loc + base * dk * dv);
+    auto load_slab = [&](int k0) {
+        bf16* sh = slabs + (k0 / SLAB) % cp.slab_bufs * 2 * SLAB * ldv;
+        const int per = dv / 8, rowsn = min(SLAB, dkp - k0);
+        for (int i = tid; i < rowsn * per; i += OUT_THREADS) {
+            const int r = i / per, c = i % per;
+            bf16* dst = sh + r * ldv + c * 8;
+            if (k0 + r < dk) {
+                const bf16* src = sin + ((size_t)(k0 + r) * dv + c * 8) * 2;
+                cp_async16(dst, src);
+                cp_async16(dst + SLAB * ldv, src + 8);
+            } else {
+                *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<uint4*>(dst + SLAB * ldv) = make_uint4(0, 0, 0, 0);
+            }
+        }
+    };
     load_rows(qs, ldk, (const bf16*)p.q + (size_t)t0 * p.ld + h * dk, p.ld, n, dk, dkp);
     load_rows(ks, ldk, (const bf16*)p.k + (size_t)t0 * p.ld + h * dk, p.ld, n, dk, dkp);
-    load_rows(vs, ldv, (const bf16*)p.v + (size_t)t0 * p.ld + h * dv, p.ld, n, dv, dv);
-    const float m_in = KIND == KIND_MLSTM ? cp.scal[base * 4 + 2] : 0.f;
     if (KIND == KIND_GLA) {
-        for (int i = tid; i < CT * dkp; i += OUT_THREADS) {
-            const int s = i / dkp, c = i % dkp;
-            bs[s * ldb + c] = (s < n && c < dk) ? cp.b[(size_t)(t0 + s) * (p.h * dk) + h * dk + c] : 0.f;
+        const int per = dkp / 4;
+        for (int i = tid; i < CT * per; i += OUT_THREADS) {
+            const int s = i / per, c = (i % per) * 4;
+            if (s < n && c < dk) cp_async16(bs + s * ldb + c, cp.b + (size_t)(t0 + s) * (p.h * dk) + h * dk + c);
+            else *reinterpret_cast<float4*>(bs + s * ldb + c) = make_float4(0.f, 0.f, 0.f, 0.f);
         }
-    } else if (warp == 0) {
-        mlstm_gates(p, t0, n, h, ga, gb, gx);
     }
+    cp_async_commit();
+    load_rows(vs, ldv, (const bf16*)p.v + (size_t)t0 * p.ld + h * dv, p.ld, n, dv, dv);
+    load_slab(0);
+    if (cp.slab_bufs > 1) load_slab(SLAB);
+    cp_async_commit();
+    const float m_in = KIND == KIND_MLSTM ? cp.scal[base * 4 + 2] : 0.f;
+    if (KIND == KIND_MLSTM && warp == 0) mlstm_gates(p, t0, n, h, ga, gb, gx);
+    cp_async_wait<1>();
     __syncthreads();
     if (KIND == KIND_MLSTM) {
         if (tid < CT) gx[tid] = fmaxf(gx[tid], m_in);
@@ -352,7 +396,7 @@ __global__ void __launch_bounds__(OUT_THREADS) chunk_output_kernel(GatedChunkPar
                         const float2 x = bf162_to_f2(*reinterpret_cast<const uint32_t*>(qs + r * ldk + c));
                         const float2 b = *reinterpret_cast<const float2*>(bs + r * ldb + c);
                         const float2 an = *reinterpret_cast<const float2*>(bs + (rt * 16 - 1) * ldb + c);
-                        split_bf162(x.x * __expf(fminf(b.x - an.x, 0.f)), x.y * __expf(fminf(b.y - an.y, 0.f)), a[i], a2[i]);
+                        split_bf162(x.x * exp2_fast(fminf(b.x - an.x, 0.f)), x.y * exp2_fast(fminf(b.y - an.y, 0.f)), a[i], a2[i]);
                     }
                 }
 #pragma unroll
@@ -370,7 +414,7 @@ __global__ void __launch_bounds__(OUT_THREADS) chunk_output_kernel(GatedChunkPar
                             const float2 x = bf162_to_f2(*reinterpret_cast<const uint32_t*>(ks + (s + g) * ldk + c));
                             const float2 b = *reinterpret_cast<const float2*>(bs + (s + g) * ldb + c);
                             const float2 an = *reinterpret_cast<const float2*>(bs + (rt * 16 - 1) * ldb + c);
-                            split_bf162(x.x * __expf(fminf(an.x - b.x, 0.f)), x.y * __expf(fminf(an.y - b.y, 0.f)), bh[i], bl[i]);
+                            split_bf162(x.x * exp2_fast(fminf(an.x - b.x, 0.f)), x.y * exp2_fast(fminf(an.y - b.y, 0.f)), bh[i], bl[i]);
                         }
                         mma_bf16_16816(sc[t], a, bh[0], bh[1]);
                         mma_bf16_16816(sc[t], a, bl[0], bl[1]);
@@ -410,14 +454,22 @@ __global__ void __launch_bounds__(OUT_THREADS) chunk_output_kernel(GatedChunkPar
         }
     }
     if (KIND == KIND_GLA) {
-        // diagonal blocks: a quad of lanes per (t, s) pair, channels interleaved over the quad
-        for (int it = tid >> 2; it < 4 * 256; it += OUT_THREADS / 4) {
-            const int r = (it >> 8) * 16 + ((it >> 4) & 15), s = (it >> 8) * 16 + (it & 15);
-            float a = 0.f;
-            if (s <= r && r < n) {
-                for (int c = tid & 3; c < dk; c += 4)
-                    a += __bfloat162float(qs[r * ldk + c]) * __bfloat162float(ks[s * ldk + c]) * __expf(bs[r * ldb + c] - bs[s * ldb + c]);
+        // diagonal blocks: the 136 pairs s <= r of each, a quad of lanes per pair, channel pairs interleaved over the quad
+        for (int it = tid >> 2; it < 4 * 136; it += OUT_THREADS / 4) {
+            const int blk = it / 136, x = it % 136, i = x / 17, j = x % 17;          // rows i and 15 - i together have 17 pairs
+            const int r = blk * 16 + (j <= i ? i : 15 - i), s = blk * 16 + (j <= i ? j : j - i - 1);
+            float a0 = 0.f, a1 = 0.f;
+            if (r < n) {
+#pragma unroll 4
+                for (int c = (tid & 3) * 2; c < dk; c += 8) {
+                    const float2 qv = bf162_to_f2(*reinterpret_cast<const uint32_t*>(qs + r * ldk + c));
+                    const float2 kv = bf162_to_f2(*reinterpret_cast<const uint32_t*>(ks + s * ldk + c));
+                    const float2 br = *reinterpret_cast<const float2*>(bs + r * ldb + c), b2 = *reinterpret_cast<const float2*>(bs + s * ldb + c);
+                    a0 += qv.x * kv.x * exp2_fast(br.x - b2.x);
+                    a1 += qv.y * kv.y * exp2_fast(br.y - b2.y);
+                }
             }
+            float a = a0 + a1;
             a += __shfl_xor_sync(0xffffffffu, a, 1);
             a += __shfl_xor_sync(0xffffffffu, a, 2);
             if ((tid & 3) == 0) {
@@ -425,6 +477,7 @@ __global__ void __launch_bounds__(OUT_THREADS) chunk_output_kernel(GatedChunkPar
                 const bf16 hi = __float2bfloat16(a);
                 ah[r * LDA + s] = hi;
                 al[r * LDA + s] = __float2bfloat16(a - __bfloat162float(hi));
+                if (s != r) ah[s * LDA + r] = al[s * LDA + r] = __float2bfloat16(0.f);
             }
         }
     }
@@ -434,18 +487,16 @@ __global__ void __launch_bounds__(OUT_THREADS) chunk_output_kernel(GatedChunkPar
     float acc[NT][4];
 #pragma unroll
     for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-    const uint32_t* sin = reinterpret_cast<const uint32_t*>(cp.loc) + base * dk * dv;
+    cp_async_wait<0>();
+    __syncthreads();
     for (int k0 = 0; k0 < dkp; k0 += SLAB) {
         const int rowsn = min(SLAB, dkp - k0);
-        __syncthreads();
-        for (int i = tid; i < rowsn * (dv / 4); i += OUT_THREADS) {
-            const int r = i / (dv / 4), c = (i % (dv / 4)) * 4;
-            uint4 w = make_uint4(0, 0, 0, 0);
-            if (k0 + r < dk) w = *reinterpret_cast<const uint4*>(sin + (size_t)(k0 + r) * dv + c);
-            *reinterpret_cast<uint2*>(sh + r * ldv + c) = make_uint2(__byte_perm(w.x, w.y, 0x5410), __byte_perm(w.z, w.w, 0x5410));
-            *reinterpret_cast<uint2*>(sl + r * ldv + c) = make_uint2(__byte_perm(w.x, w.y, 0x7632), __byte_perm(w.z, w.w, 0x7632));
+        const bf16* sh = slabs + (k0 / SLAB) % cp.slab_bufs * 2 * SLAB * ldv;
+        const bf16* sl = sh + SLAB * ldv;
+        if (k0 >= cp.slab_bufs * SLAB) {                             // further slabs take the buffers in turn
+            cp_async_wait<0>();
+            __syncthreads();
         }
-        __syncthreads();
         for (int kk = 0; kk < rowsn; kk += 16) {
             uint32_t a[4], a2[4];
             if (KIND == KIND_MLSTM) {
@@ -456,7 +507,7 @@ __global__ void __launch_bounds__(OUT_THREADS) chunk_output_kernel(GatedChunkPar
                     const int r = (i & 1) ? r1 : r0, c = k0 + kk + c4 * 2 + (i >> 1) * 8;
                     const float2 x = bf162_to_f2(*reinterpret_cast<const uint32_t*>(qs + r * ldk + c));
                     const float2 b = *reinterpret_cast<const float2*>(bs + r * ldb + c);
-                    split_bf162(x.x * qscale * __expf(b.x), x.y * qscale * __expf(b.y), a[i], a2[i]);
+                    split_bf162(x.x * qscale * exp2_fast(b.x), x.y * qscale * exp2_fast(b.y), a[i], a2[i]);
                 }
             }
 #pragma unroll
@@ -469,6 +520,11 @@ __global__ void __launch_bounds__(OUT_THREADS) chunk_output_kernel(GatedChunkPar
                 mma_bf16_16816(acc[i], a, l0, l1);
                 if (KIND == KIND_GLA) mma_bf16_16816(acc[i], a2, b0, b1);
             }
+        }
+        if (k0 + cp.slab_bufs * SLAB < dkp) {
+            __syncthreads();
+            load_slab(k0 + cp.slab_bufs * SLAB);
+            cp_async_commit();
         }
     }
     float e0 = 1.f, e1 = 1.f;
@@ -534,17 +590,20 @@ __global__ void __launch_bounds__(OUT_THREADS) chunk_output_kernel(GatedChunkPar
 
 size_t state_smem(int kind, int dk, int dv, int rank) {
     const int dkp = (dk + 15) / 16 * 16;
-    return (size_t)CT * (dkp + 8) * 4 + (size_t)CT * (dv + 8) * 2 + (kind == KIND_GLA ? (size_t)CT * (dk + rank) * 4 : (size_t)3 * CT * 4);
+    return (size_t)CT * (dkp + 8) * 4 + (size_t)CT * (dv + 8) * 2 + (kind == KIND_GLA ? (size_t)CT * (dk + rank) * 4 + (size_t)dk * rank * 2 : (size_t)3 * CT * 4);
 }
 
 template <int KIND>
-int run_chunks(const GatedChunkParams* p, int B, cudaStream_t s) {
+int run_chunks(const GatedChunkParams* args, int B, cudaStream_t s) {
+    GatedChunkParams params = *args;
+    params.slab_bufs = slab_buffers(KIND, args->s.dk, args->s.dv);
+    const GatedChunkParams* p = &params;
     const int dk = p->s.dk, dv = p->s.dv, h = p->s.h, nc = p->c1 - p->c0;
-    const size_t s1 = state_smem(KIND, dk, dv, p->s.rank), s3 = output_smem<KIND>(dk, dv);
+    const size_t s1 = state_smem(KIND, dk, dv, p->s.rank), s3 = output_smem(KIND, dk, dv, p->slab_bufs);
     auto k1 = chunk_state_kernel<KIND>;
     if (s1 > 48 * 1024) cudaFuncSetAttribute(k1, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1);
     sl_launch(k1, dim3(nc, h), 256, s1, s, *p);
-    sl_launch(chunk_scan_kernel<KIND>, dim3((dk * dv + 1023) / 1024, h, B), 256, 0, s, *p);
+    sl_launch(chunk_scan_kernel<KIND>, dim3((dk * dv + 2047) / 2048, h, B), 256, 0, s, *p);
     if (dv <= 128) {
         auto k3 = chunk_output_kernel<KIND, 4>;
         cudaFuncSetAttribute(k3, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s3);
@@ -562,8 +621,7 @@ int run_chunks(const GatedChunkParams* p, int B, cudaStream_t s) {
 // 1 when the chunked kernels take these sizes (head rows of whole 16-byte pieces, tiles that fit in shared memory).
 SL_API int sl_gated_chunk_ok(int kind, int dk, int dv, int rank) {
     if (dk < 8 || dv < 8 || dk % 8 != 0 || dv % 8 != 0 || dv > 256) return 0;
-    const size_t s3 = kind == KIND_GLA ? output_smem<KIND_GLA>(dk, dv) : output_smem<KIND_MLSTM>(dk, dv);
-    return state_smem(kind, dk, dv, rank) <= 220 * 1024 && s3 <= 220 * 1024;
+    return state_smem(kind, dk, dv, rank) <= SMEM_MAX && output_smem(kind, dk, dv, slab_buffers(kind, dk, dv)) <= SMEM_MAX;
 }
 
 // One pass over the chunks [c0, c1) of B sequences (bf16 rows in and out).  Passes of one step run in order on one stream.
