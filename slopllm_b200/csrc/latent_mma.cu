@@ -3,7 +3,7 @@
 //  * latent_gather_kernel: the cache rows that a step's portions can see, copied out of the pages in order.
 //  * latent_prefill_kernel: expanded form for portions of prompts.  Keys and values of the visible rows were materialised per
 //    head by two GEMMs; FlashAttention-2 style over 128 queries x 1 head per CTA, the shared rotated key part is read beside
-//    the head's own, K/V tiles of 64 keys are double-buffered with cp.async.
+//    the head's own, tiles of 64 keys come through a three-stage cp.async ring filled by a warp of its own.
 //  * latent_decode_kernel: absorbed form, one query token per page-table row.  A CTA takes 16 heads x a range of keys: all
 //    heads share the key rows, whose first `rank` values are the value rows as well, so a tile is read once for both products.
 //    Key splits leave (o, log-sum-exp) partials for `sl_combine_vexpand` / `sl_mla_combine`; the sink belongs to split 0.
@@ -11,6 +11,7 @@
 // Scores and softmax are fp32; the weights enter the second product as two bf16 terms (hi + lo), so they keep fp32-like accuracy.
 #include "common.cuh"
 #include "mma_sync.cuh"
+#include "tcgen05.cuh"
 
 namespace {
 
@@ -49,32 +50,55 @@ struct LatentPrefillParams {
     float scale;
     const float* sink;                    // [heads] or null
     bf16* out;                            // [T, heads * vdim]
+    int* err;                             // status word: set when a wait inside the kernel expired
+    int stages;                           // set by the launcher: key tiles in shared memory
 };
 
-constexpr int BQ = 128, BK = 64;
+constexpr int BQ = 128, BK = 64, MAX_STAGES = 3;
+constexpr int CONSUMERS = BQ / 16, PT = (CONSUMERS + 1) * 32;      // a warp per 16 queries, one warp that fetches
 
-// grid (heads of the group, tiles), block 256 (8 warps x 16 queries).  NT: 8-wide value tiles (vdim <= 8 * NT).
+// 16 bytes global -> shared, or zeros
+__device__ __forceinline__ void cp_async16_or_zero(void* dst, const void* src, bool valid) {
+    const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(valid ? 16 : 0) : "memory");
+}
+// arrive on `bar` when all copies this thread has issued so far have landed (the barrier counts one arrival per thread)
+__device__ __forceinline__ void cp_async_arrive(uint64_t* bar) {
+    asm volatile("cp.async.mbarrier.arrive.noinc.shared.b64 [%0];" ::"r"(tc::smem_u32(bar)) : "memory");
+}
+
+__device__ __forceinline__ float exp2_fast(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+// grid (heads of the group, tiles).  NT: 8-wide value tiles (vdim <= 8 * NT).  The fetching warp runs ahead of the consumers by
+// up to `stages` key tiles; consumer warps do not wait for one another.
 template <int NT>
-__global__ void __launch_bounds__(256) latent_prefill_kernel(LatentPrefillParams p) {
+__global__ void __launch_bounds__(PT, 1) latent_prefill_kernel(LatentPrefillParams p) {
     pdl_grid_sync();
     extern __shared__ __align__(16) unsigned char smraw[];
     const int hg = blockIdx.x, h = p.h0 + hg, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, c4 = lane & 3;
-    const int* tl = p.tiles + blockIdx.y * 4;
+    const int* tl = p.tiles + (gridDim.y - 1 - blockIdx.y) * 4;      // late positions see most keys: start them first
     const int q0 = tl[0], nq = tl[1], pos0 = tl[2], koff = tl[3];
     const int dq = p.dim + p.rot_dim, dqp = (dq + 15) / 16 * 16, ld = dqp + 8, ldv = NT * 8 + 8;
     bf16* qs = reinterpret_cast<bf16*>(smraw);            // [BQ][ld]
-    bf16* ks = qs + BQ * ld;                              // 2 x [BK][ld]
-    bf16* vs = ks + 2 * BK * ld;                          // 2 x [BK][ldv]
+    const int stages = p.stages;
+    bf16* ks = qs + BQ * ld;                              // stages x [BK][ld]
+    bf16* vs = ks + stages * BK * ld;                     // stages x [BK][ldv]
+    __shared__ uint64_t full[MAX_STAGES], empty[MAX_STAGES];
+    __shared__ int gave_up;
     const int nd = p.dim / 8, nr = p.rot_dim / 8, nv = p.vdim / 8;
     const int last = pos0 + nq - 1;
     const int first = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
     const int ntiles = (last - first) / BK + 1;
 
     // columns that no copy writes: the query / key padding to 16 and the value padding
-    for (int i = tid; i < (BQ + 2 * BK) * (dqp - dq); i += 256) qs[(i / (dqp - dq)) * ld + dq + i % (dqp - dq)] = __float2bfloat16(0.f);
+    for (int i = tid; i < (BQ + stages * BK) * (dqp - dq); i += PT) qs[(i / (dqp - dq)) * ld + dq + i % (dqp - dq)] = __float2bfloat16(0.f);
     const int vpad = NT * 8 - p.vdim;
-    for (int i = tid; i < 2 * BK * vpad; i += 256) vs[(i / vpad) * ldv + p.vdim + i % vpad] = __float2bfloat16(0.f);
-    for (int i = tid; i < BQ * (nd + nr); i += 256) {
+    for (int i = tid; i < stages * BK * vpad; i += PT) vs[(i / vpad) * ldv + p.vdim + i % vpad] = __float2bfloat16(0.f);
+    for (int i = tid; i < BQ * (nd + nr); i += PT) {
         const int r = i / (nd + nr), c = i % (nd + nr);
         uint4 x = make_uint4(0, 0, 0, 0);
         if (r < nq)
@@ -82,27 +106,53 @@ __global__ void __launch_bounds__(256) latent_prefill_kernel(LatentPrefillParams
                        : *reinterpret_cast<const uint4*>(p.q_rot + ((size_t)(q0 + r) * p.heads + h) * p.rot_dim + (c - nd) * 8);
         *reinterpret_cast<uint4*>(qs + r * ld + c * 8) = x;
     }
-    auto load_tile = [&](int j) {
-        bf16* kd = ks + (j & 1) * BK * ld;
-        bf16* vd = vs + (j & 1) * BK * ldv;
-        const int k0 = first + j * BK;
-        const int per = nd + nr + nv;
-        for (int i = tid; i < BK * per; i += 256) {
-            const int r = i / per, c = i % per, kp = k0 + r;
-            bf16* dst = c < nd + nr ? kd + r * ld + c * 8 : vd + r * ldv + (c - nd - nr) * 8;
-            if (kp <= last) {
-                const size_t row = (size_t)(kp + koff);
-                const bf16* src = c < nd ? p.k + row * p.ldk + hg * p.dim + c * 8
-                                : c < nd + nr ? p.rows + row * p.row + p.rank + (c - nd) * 8
-                                              : p.v + row * p.ldv + hg * p.vdim + (c - nd - nr) * 8;
-                cp_async16(dst, src);
-            } else {
-                *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
-            }
+    if (tid == 0) {
+        gave_up = 0;
+        for (int i = 0; i < stages; ++i) {
+            tc::mbar_init(&full[i], 32);
+            tc::mbar_init(&empty[i], CONSUMERS);
         }
-        cp_async_commit();
+        tc::mbar_fence_init();
+    }
+    __syncthreads();
+    volatile int* dead = &gave_up;                        // a wait expired somewhere in the block: nobody waits any longer
+    auto wait = [&](uint64_t* bar, int parity) {
+        if (tc::mbar_wait(bar, parity) || *dead) return;
+        *dead = 1;
+        if (p.err != nullptr) atomicCAS(p.err, 0, 41);
     };
-    load_tile(0);
+    if (warp == CONSUMERS) {
+        // a lane copies the same 16-byte column of every (32 / pieces)-th row of a part (a row has at most 32 pieces)
+        struct Part { int row, step; bool on; };
+        auto part = [&](int pieces) { Part x; x.step = 32 / pieces; x.row = lane / pieces; x.on = x.row < x.step; return x; };
+        const Part pk = part(nd), pr = part(nr), pv = part(nv);
+        const bf16* kcol = p.k + hg * p.dim + lane % nd * 8;
+        const bf16* rcol = p.rows + p.rank + lane % nr * 8;
+        const bf16* vcol = p.v + hg * p.vdim + lane % nv * 8;
+        auto copy = [&](const Part& x, bf16* dst, int dld, const bf16* col, size_t sld, int k0) {
+            if (!x.on) return;
+            const bf16* src = col + (size_t)(k0 + x.row + koff) * sld;
+            dst += x.row * dld;
+            const int n = min(BK, last + 1 - k0), dstep = x.step * dld;
+            const size_t sstep = (size_t)x.step * sld;
+            int r = x.row;
+#pragma unroll 4
+            for (; r < n; r += x.step, src += sstep, dst += dstep) cp_async16(dst, src);
+            for (; r < BK; r += x.step, dst += dstep) cp_async16_or_zero(dst, col, false);
+        };
+        for (int j = 0; j < ntiles && !*dead; ++j) {
+            const int st = j % stages, k0 = first + j * BK;
+            if (j >= stages) wait(&empty[st], (j / stages - 1) & 1);
+            bf16* kd = ks + st * BK * ld;
+            bf16* vd = vs + st * BK * ldv;
+            copy(pk, kd + lane % nd * 8, ld, kcol, p.ldk, k0);
+            copy(pr, kd + p.dim + lane % nr * 8, ld, rcol, p.row, k0);
+            copy(pv, vd + lane % nv * 8, ldv, vcol, p.ldv, k0);
+            cp_async_arrive(&full[st]);
+        }
+        cp_async_wait_all();
+        return;
+    }
 
     const int r0 = warp * 16 + g, r1 = r0 + 8, p0 = pos0 + r0, p1 = pos0 + r1;
     const int lo0 = p.window > 0 ? p0 - p.window + 1 : 0, lo1 = p.window > 0 ? p1 - p.window + 1 : 0;
@@ -115,15 +165,11 @@ __global__ void __launch_bounds__(256) latent_prefill_kernel(LatentPrefillParams
     const int wq0 = pos0 + warp * 16, wlo = p.window > 0 ? wq0 - p.window + 1 : 0;      // range of the warp's rows
 
     for (int j = 0; j < ntiles; ++j) {
-        if (j + 1 < ntiles) {
-            load_tile(j + 1);
-            cp_async_wait<1>();
-        } else {
-            cp_async_wait<0>();
-        }
-        __syncthreads();
-        const bf16* kt = ks + (j & 1) * BK * ld;
-        const bf16* vt = vs + (j & 1) * BK * ldv;
+        const int st = j % stages;
+        wait(&full[st], (j / stages) & 1);
+        if (*dead) break;
+        const bf16* kt = ks + st * BK * ld;
+        const bf16* vt = vs + st * BK * ldv;
         const int k0 = first + j * BK;
         if (k0 <= wq0 + 15 && k0 + BK - 1 >= wlo && warp * 16 < nq) {                    // the tile meets the warp's range
             float s[BK / 8][4];
@@ -142,14 +188,25 @@ __global__ void __launch_bounds__(256) latent_prefill_kernel(LatentPrefillParams
             }
             const bool whole = k0 + BK - 1 <= wq0 && k0 >= wlo + 15;
             float x0 = m0, x1 = m1;
+            if (whole) {
+#pragma unroll
+                for (int n = 0; n < BK / 8; ++n) {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) s[n][i] *= scale_log2;
+                }
+            } else {
+#pragma unroll
+                for (int n = 0; n < BK / 8; ++n) {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        const int key = k0 + n * 8 + 2 * c4 + (i & 1);
+                        const bool in = i < 2 ? (key <= p0 && key >= lo0) : (key <= p1 && key >= lo1);
+                        s[n][i] = in ? s[n][i] * scale_log2 : -INFINITY;
+                    }
+                }
+            }
 #pragma unroll
             for (int n = 0; n < BK / 8; ++n) {
-#pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    const int key = k0 + n * 8 + 2 * c4 + (i & 1);
-                    const bool in = whole || (i < 2 ? (key <= p0 && key >= lo0) : (key <= p1 && key >= lo1));
-                    s[n][i] = in ? s[n][i] * scale_log2 : -INFINITY;
-                }
                 x0 = fmaxf(x0, fmaxf(s[n][0], s[n][1]));
                 x1 = fmaxf(x1, fmaxf(s[n][2], s[n][3]));
             }
@@ -167,7 +224,7 @@ __global__ void __launch_bounds__(256) latent_prefill_kernel(LatentPrefillParams
 #pragma unroll
                 for (int u = 0; u < 2; ++u) {
                     float* sn = s[2 * n + u];
-                    const float e0 = exp2f(sn[0] - z0), e1 = exp2f(sn[1] - z0), e2 = exp2f(sn[2] - z1), e3 = exp2f(sn[3] - z1);
+                    const float e0 = exp2_fast(sn[0] - z0), e1 = exp2_fast(sn[1] - z0), e2 = exp2_fast(sn[2] - z1), e3 = exp2_fast(sn[3] - z1);
                     sum0 += e0 + e1;
                     sum1 += e2 + e3;
                     split_bf162(e0, e1, ph[u * 2], pl[u * 2]);
@@ -188,7 +245,8 @@ __global__ void __launch_bounds__(256) latent_prefill_kernel(LatentPrefillParams
             l0 = l0 * f0 + sum0;
             l1 = l1 * f1 + sum1;
         }
-        __syncthreads();                                   // the next iteration refills the buffer just read
+        __syncwarp();
+        if (lane == 0) tc::mbar_arrive(&empty[st]);
     }
     const float i0 = l0 > 0.f ? 1.f / l0 : 0.f, i1 = l1 > 0.f ? 1.f / l1 : 0.f;
 #pragma unroll
@@ -200,11 +258,15 @@ __global__ void __launch_bounds__(256) latent_prefill_kernel(LatentPrefillParams
     }
 }
 
-template <int NT>
-size_t prefill_smem(int dq) {
+int value_tiles(int vdim) { return vdim <= 32 ? 4 : vdim <= 64 ? 8 : vdim <= 128 ? 16 : 32; }
+size_t prefill_smem(int dq, int nt, int stages) {
     const int ld = (dq + 15) / 16 * 16 + 8;
-    return ((size_t)(BQ + 2 * BK) * ld + (size_t)2 * BK * (NT * 8 + 8)) * sizeof(bf16);
+    return ((size_t)(BQ + stages * BK) * ld + (size_t)stages * BK * (nt * 8 + 8)) * sizeof(bf16);
 }
+constexpr size_t SMEM_MAX = 224 * 1024;
+int prefill_stages(int dq, int nt) { return prefill_smem(dq, nt, MAX_STAGES) <= SMEM_MAX ? MAX_STAGES : 2; }
+
+constexpr int DK_T = 64;                  // keys per tile of the decode kernel
 
 struct LatentDecodeParams {
     const bf16* q_abs;                    // [T, heads, rank]
@@ -229,14 +291,14 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(LatentDecodeParams p
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, c4 = lane & 3;
     const int row = p.rank + p.rot_dim, dqp = (row + 15) / 16 * 16, ld = dqp + 8;
     bf16* qs = reinterpret_cast<bf16*>(smraw);            // [16][ld]
-    bf16* ks = qs + 16 * ld;                              // [BK][ld]
-    float* sc = reinterpret_cast<float*>(ks + BK * ld);   // [16][BK + 4]
-    bf16* ph = reinterpret_cast<bf16*>(sc + 16 * (BK + 4));      // [16][BK + 8]
-    bf16* pl = ph + 16 * (BK + 8);
-    float* fac = reinterpret_cast<float*>(pl + 16 * (BK + 8));   // [16] rescale of the tile, then 1 / l
+    bf16* ks = qs + 16 * ld;                              // [DK_T][ld]
+    float* sc = reinterpret_cast<float*>(ks + DK_T * ld);   // [16][DK_T + 4]
+    bf16* ph = reinterpret_cast<bf16*>(sc + 16 * (DK_T + 4));      // [16][DK_T + 8]
+    bf16* pl = ph + 16 * (DK_T + 8);
+    float* fac = reinterpret_cast<float*>(pl + 16 * (DK_T + 8));   // [16] rescale of the tile, then 1 / l
     const int pos = p.positions[t];
     const int first = p.window > 0 ? max(0, pos - p.window + 1) : 0;
-    const int tiles = (pos - first) / BK + 1, per = (tiles + p.splits - 1) / p.splits;
+    const int tiles = (pos - first) / DK_T + 1, per = (tiles + p.splits - 1) / p.splits;
     const int tb = min(tiles, split * per), te = min(tiles, tb + per);
     const int* pt = p.page_table + (size_t)p.batch_idx[t] * p.pt_stride;
     for (int i = tid; i < 16 * (dqp / 8); i += 256) {
@@ -247,7 +309,7 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(LatentDecodeParams p
                            : *reinterpret_cast<const uint4*>(p.q_rot + ((size_t)t * p.heads + h0 + r) * p.rot_dim + c - p.rank);
         *reinterpret_cast<uint4*>(qs + r * ld + c) = x;
     }
-    if (dqp > row && tid < BK) *reinterpret_cast<uint4*>(ks + tid * ld + row) = make_uint4(0, 0, 0, 0);     // (row % 8 == 0)
+    if (dqp > row && tid < DK_T) *reinterpret_cast<uint4*>(ks + tid * ld + row) = make_uint4(0, 0, 0, 0);     // (row % 8 == 0)
     float m[2], l[2];                                     // softmax state of rows 2 * warp, 2 * warp + 1
 #pragma unroll
     for (int u = 0; u < 2; ++u) {
@@ -262,7 +324,7 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(LatentDecodeParams p
     for (int i = 0; i < NTW; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
     const float scale_log2 = p.scale * LOG2E;
     for (int j = tb; j < te; ++j) {
-        const int k0 = first + j * BK, nk = min(BK, pos + 1 - k0);
+        const int k0 = first + j * DK_T, nk = min(DK_T, pos + 1 - k0);
         __syncthreads();
         long long slot = -1;                              // lanes 0-7: the warp's eight rows
         if (lane < 8 && warp * 8 + lane < nk) {
@@ -292,16 +354,16 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(LatentDecodeParams p
         }
         {
             const int kc = warp * 8 + c4 * 2;
-            sc[g * (BK + 4) + kc] = kc < nk ? s4[0] * scale_log2 : -INFINITY;
-            sc[g * (BK + 4) + kc + 1] = kc + 1 < nk ? s4[1] * scale_log2 : -INFINITY;
-            sc[(g + 8) * (BK + 4) + kc] = kc < nk ? s4[2] * scale_log2 : -INFINITY;
-            sc[(g + 8) * (BK + 4) + kc + 1] = kc + 1 < nk ? s4[3] * scale_log2 : -INFINITY;
+            sc[g * (DK_T + 4) + kc] = kc < nk ? s4[0] * scale_log2 : -INFINITY;
+            sc[g * (DK_T + 4) + kc + 1] = kc + 1 < nk ? s4[1] * scale_log2 : -INFINITY;
+            sc[(g + 8) * (DK_T + 4) + kc] = kc < nk ? s4[2] * scale_log2 : -INFINITY;
+            sc[(g + 8) * (DK_T + 4) + kc + 1] = kc + 1 < nk ? s4[3] * scale_log2 : -INFINITY;
         }
         __syncthreads();
 #pragma unroll
         for (int u = 0; u < 2; ++u) {
             const int r = warp * 2 + u;
-            const float2 v = *reinterpret_cast<const float2*>(sc + r * (BK + 4) + lane * 2);
+            const float2 v = *reinterpret_cast<const float2*>(sc + r * (DK_T + 4) + lane * 2);
             const float x = fmaxf(m[u], warp_max(fmaxf(v.x, v.y)));
             const float f = m[u] == -INFINITY ? 0.f : exp2f(m[u] - x);
             const float e0 = exp2f(v.x - x), e1 = exp2f(v.y - x);
@@ -309,8 +371,8 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(LatentDecodeParams p
             m[u] = x;
             uint32_t hi, lo;
             split_bf162(e0, e1, hi, lo);
-            *reinterpret_cast<uint32_t*>(ph + r * (BK + 8) + lane * 2) = hi;
-            *reinterpret_cast<uint32_t*>(pl + r * (BK + 8) + lane * 2) = lo;
+            *reinterpret_cast<uint32_t*>(ph + r * (DK_T + 8) + lane * 2) = hi;
+            *reinterpret_cast<uint32_t*>(pl + r * (DK_T + 8) + lane * 2) = lo;
             if (lane == 0) fac[r] = f;
         }
         __syncthreads();
@@ -318,10 +380,10 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(LatentDecodeParams p
 #pragma unroll
         for (int i = 0; i < NTW; ++i) { acc[i][0] *= f0; acc[i][1] *= f0; acc[i][2] *= f1; acc[i][3] *= f1; }
 #pragma unroll
-        for (int kk = 0; kk < BK; kk += 16) {
+        for (int kk = 0; kk < DK_T; kk += 16) {
             uint32_t a[4], a2[4];
-            ldsm_x4(a, ph + (lane & 15) * (BK + 8) + kk + (lane >> 4) * 8);
-            ldsm_x4(a2, pl + (lane & 15) * (BK + 8) + kk + (lane >> 4) * 8);
+            ldsm_x4(a, ph + (lane & 15) * (DK_T + 8) + kk + (lane >> 4) * 8);
+            ldsm_x4(a2, pl + (lane & 15) * (DK_T + 8) + kk + (lane >> 4) * 8);
 #pragma unroll
             for (int i = 0; i < NTW; ++i) {
                 if (i >= nn) break;
@@ -361,7 +423,7 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(LatentDecodeParams p
 
 size_t decode_smem(int row) {
     const int ld = (row + 15) / 16 * 16 + 8;
-    return (size_t)(16 + BK) * ld * 2 + (size_t)16 * (BK + 4) * 4 + (size_t)2 * 16 * (BK + 8) * 2 + 64;
+    return (size_t)(16 + DK_T) * ld * 2 + (size_t)16 * (DK_T + 4) * 4 + (size_t)2 * 16 * (DK_T + 8) * 2 + 64;
 }
 
 }  // namespace
@@ -375,23 +437,29 @@ SL_API int sl_latent_gather(const LatentGatherParams* p, int B, int longest, cud
 
 // 1 when the tensor-core kernels take these sizes.
 SL_API int sl_latent_mma_ok(int dim, int rot_dim, int vdim, int rank) {
-    if (dim % 8 != 0 || rot_dim % 8 != 0 || vdim % 8 != 0 || rank % 8 != 0 || vdim > 256 || dim + rot_dim > 256) return 0;
-    return rank <= 1024 && decode_smem(rank + rot_dim) <= 220 * 1024;
+    if (dim < 8 || rot_dim < 8 || dim % 8 != 0 || rot_dim % 8 != 0 || vdim % 8 != 0 || rank % 8 != 0 || vdim > 256 || dim + rot_dim > 256) return 0;
+    if (prefill_smem(dim + rot_dim, value_tiles(vdim), 2) > SMEM_MAX) return 0;
+    return rank <= 1024 && decode_smem(rank + rot_dim) <= SMEM_MAX;
 }
 
 // `heads` of the launch are h0 .. h0 + group - 1.
-SL_API int sl_latent_prefill(const LatentPrefillParams* p, int group, int tiles, cudaStream_t s) {
+SL_API int sl_latent_prefill(const LatentPrefillParams* args, int group, int tiles, cudaStream_t s) {
+    LatentPrefillParams params = *args;
+    LatentPrefillParams* p = &params;
     if (group == 0 || tiles == 0) return 0;
     if (!sl_latent_mma_ok(p->dim, p->rot_dim, p->vdim, p->rank) || tiles > 65535) return -1;
+    if (((uintptr_t)p->k | (uintptr_t)p->v | (uintptr_t)p->rows | (uintptr_t)p->q | (uintptr_t)p->q_rot) % 16 != 0) return -1;
     if (p->ldq % 8 != 0 || p->q_head % 8 != 0 || p->ldk % 8 != 0 || p->ldv % 8 != 0 || p->row % 8 != 0) return -1;
+    const int nt = value_tiles(p->vdim), dq = p->dim + p->rot_dim;
+    p->stages = prefill_stages(dq, nt);
+    const size_t smem = prefill_smem(dq, nt, p->stages);
 #define SL_LP(NT)                                                                                                       \
     {                                                                                                                   \
-        const size_t smem = prefill_smem<NT>(p->dim + p->rot_dim);                                                      \
         auto kern = latent_prefill_kernel<NT>;                                                                          \
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                             \
-        sl_launch(kern, dim3(group, tiles), 256, smem, s, *p);                                                          \
+        sl_launch(kern, dim3(group, tiles), PT, smem, s, *p);                                                          \
     }
-    if (p->vdim <= 32) SL_LP(4) else if (p->vdim <= 64) SL_LP(8) else if (p->vdim <= 128) SL_LP(16) else SL_LP(32)
+    if (nt == 4) SL_LP(4) else if (nt == 8) SL_LP(8) else if (nt == 16) SL_LP(16) else SL_LP(32)
 #undef SL_LP
     return SL_LAUNCH_CHECK();
 }
@@ -401,7 +469,7 @@ SL_API int sl_latent_decode(const LatentDecodeParams* p, int T, cudaStream_t s) 
     if (p->rank % 8 != 0 || p->rot_dim % 8 != 0 || p->rank > 1024 || p->splits < 1 || T > 65535) return -1;
     if (p->o_final != nullptr && p->splits != 1) return -1;
     const size_t smem = decode_smem(p->rank + p->rot_dim);
-    if (smem > 220 * 1024) return -1;
+    if (smem > SMEM_MAX) return -1;
     const dim3 grid(p->splits, (p->heads + 15) / 16, T);
 #define SL_LD(NTW)                                                                                                      \
     {                                                                                                                   \

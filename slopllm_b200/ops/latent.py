@@ -45,7 +45,7 @@ class LatentPrefillParams(C.Structure):
     _fields_ = [("q", C.c_void_p), ("ldq", C.c_int), ("q_head", C.c_int), ("q_rot", C.c_void_p), ("k", C.c_void_p), ("ldk", C.c_int),
                 ("v", C.c_void_p), ("ldv", C.c_int), ("rows", C.c_void_p), ("row", C.c_int), ("rank", C.c_int), ("tiles", C.c_void_p),
                 ("heads", C.c_int), ("h0", C.c_int), ("dim", C.c_int), ("rot_dim", C.c_int), ("vdim", C.c_int), ("window", C.c_int),
-                ("scale", C.c_float), ("sink", C.c_void_p), ("out", C.c_void_p)]
+                ("scale", C.c_float), ("sink", C.c_void_p), ("out", C.c_void_p), ("err", C.c_void_p), ("stages", C.c_int)]
 
 
 class LatentDecodeParams(C.Structure):
@@ -208,10 +208,11 @@ def latent_prefill(qd, q_rot, s: LatentShape, w: LatentWeights, st, cache, ops) 
 def latent_prefill_kernel(qd, q_rot, s: LatentShape, w: LatentWeights, rows, k, v, plan: PortionPlan, h0: int, heads: int, out) -> None:
     """Attention of heads h0 .. h0 + heads - 1 over their expanded keys k [rows, heads * dim] and values v [rows, heads * vdim]."""
     N = _native()
+    from . import tcgen05
     p = LatentPrefillParams(q=qd.data_ptr(), ldq=qd.stride(0), q_head=s.dim + s.rot_dim, q_rot=q_rot.data_ptr(), k=k.data_ptr(),
                             ldk=k.stride(0), v=v.data_ptr(), ldv=v.stride(0), rows=rows.data_ptr(), row=s.row, rank=s.rank,
                             tiles=plan.tiles.data_ptr(), heads=s.heads, h0=h0, dim=s.dim, rot_dim=s.rot_dim, vdim=s.vdim,
-                            window=s.window, scale=s.scale, sink=N.ptr(w.sink), out=out.data_ptr())
+                            window=s.window, scale=s.scale, sink=N.ptr(w.sink), out=out.data_ptr(), err=tcgen05.error_flag(out.device).data_ptr())
     N.call("sl_latent_prefill", C.byref(p), heads, plan.tile_count, N.stream())
 
 
