@@ -33,7 +33,7 @@ struct GatedChunkParams {
                                              // then their eight low terms, in the place of every eight values
     float* nloc;                             // mLSTM: [chunks of the pass, h, dk], then n_in
     float* scal;                             // mLSTM: [chunks of the pass, h, 4]: b_C, M_C, m_in, m after the chunk
-    int slab_bufs;                           // set by the launcher: state slabs in shared memory at a time (1 or 2)
+    int slab, slab_bufs;                     // set by the launcher: state rows per slab, slabs in shared memory at a time (1 or 2)
 };
 
 // rows [n][dim] (bf16, 16-byte pieces) -> shared [CT][ld] with cp.async, zero beyond n rows and beyond dim columns up to `padded`
@@ -233,14 +233,17 @@ __global__ void __launch_bounds__(256) chunk_scan_kernel(GatedChunkParams cp) {
         float m = m0;
         constexpr int U = 4;                              // chunks whose contributions are in flight
         for (int i0 = lo; i0 < hi; i0 += U) {
-            float x[U][8], d[U];
+            float x[U][8], d[U], bc[U];                   // (mLSTM: d = M_C, bc = b_C)
 #pragma unroll
             for (int j = 0; j < U; ++j) {
                 const int i = min(i0 + j, hi - 1);
                 const float* src = cp.loc + ((size_t)(i - cp.c0) * p.h + h) * size + e;
                 *reinterpret_cast<float4*>(x[j]) = *reinterpret_cast<const float4*>(src);
                 *reinterpret_cast<float4*>(x[j] + 4) = *reinterpret_cast<const float4*>(src + 4);
-                if (KIND == KIND_GLA) {
+                if (KIND == KIND_MLSTM) {
+                    bc[j] = cp.scal[((size_t)(i - cp.c0) * p.h + h) * 4];
+                    d[j] = cp.scal[((size_t)(i - cp.c0) * p.h + h) * 4 + 1];
+                } else {
                     const int* ch = cp.chunks + (size_t)i * 4;
                     d[j] = cp.b[(size_t)(ch[1] + ch[2] - 1) * (p.h * dk) + h * dk + c];
                 }
@@ -251,11 +254,10 @@ __global__ void __launch_bounds__(256) chunk_scan_kernel(GatedChunkParams cp) {
                 if (i >= hi) break;
                 float add = 1.f, keep = KIND == KIND_GLA ? exp2f(d[j]) : 1.f;
                 if (KIND == KIND_MLSTM) {
-                    const float* sc = cp.scal + ((size_t)(i - cp.c0) * p.h + h) * 4;
-                    const float top = fmaxf(m, sc[1]);
+                    const float top = fmaxf(m, d[j]);
                     keep = expf(m - top);
-                    add = expf(sc[1] - top);
-                    m = sc[0] + top;
+                    add = expf(d[j] - top);
+                    m = bc[j] + top;
                 }
                 uint4 wh, wl;
                 split_bf162(S[0], S[1], wh.x, wl.x); split_bf162(S[2], S[3], wh.y, wl.y);
@@ -274,24 +276,29 @@ __global__ void __launch_bounds__(256) chunk_scan_kernel(GatedChunkParams cp) {
         // normaliser and running maximum; m itself is stored by the output kernel (other blocks of this grid still read it)
         for (int c = threadIdx.x; c < dk; c += 256) {
             float nn = p.n[slot * dk + c], m = m0;
-            for (int i = lo; i < hi; ++i) {
-                const size_t at = (size_t)(i - cp.c0) * p.h + h;
-                const float* sc = cp.scal + at * 4;
-                const float top = fmaxf(m, sc[1]), x = cp.nloc[at * dk + c];
-                cp.nloc[at * dk + c] = nn;
-                nn = expf(m - top) * nn + expf(sc[1] - top) * x;
-                m = sc[0] + top;
+            constexpr int U = 8;
+            for (int i0 = lo; i0 < hi; i0 += U) {
+                float x[U], bc[U], mc[U];
+#pragma unroll
+                for (int j = 0; j < U; ++j) {
+                    const size_t at = (size_t)(min(i0 + j, hi - 1) - cp.c0) * p.h + h;
+                    x[j] = cp.nloc[at * dk + c];
+                    bc[j] = cp.scal[at * 4];
+                    mc[j] = cp.scal[at * 4 + 1];
+                }
+#pragma unroll
+                for (int j = 0; j < U; ++j) {
+                    if (i0 + j >= hi) break;
+                    const size_t at = (size_t)(i0 + j - cp.c0) * p.h + h;
+                    const float top = fmaxf(m, mc[j]);
+                    cp.nloc[at * dk + c] = nn;
+                    nn = expf(m - top) * nn + expf(mc[j] - top) * x[j];
+                    if (c == 0) cp.scal[at * 4 + 2] = m;
+                    m = bc[j] + top;
+                    if (c == 0) cp.scal[at * 4 + 3] = m;
+                }
             }
             p.n[slot * dk + c] = nn;
-        }
-        if (threadIdx.x == 0) {
-            float m = m0;
-            for (int i = lo; i < hi; ++i) {
-                float* sc = cp.scal + ((size_t)(i - cp.c0) * p.h + h) * 4;
-                sc[2] = m;
-                m = sc[0] + fmaxf(m, sc[1]);
-                sc[3] = m;
-            }
         }
     }
 }
@@ -299,20 +306,32 @@ __global__ void __launch_bounds__(256) chunk_scan_kernel(GatedChunkParams cp) {
 // ---- 3: outputs --------------------------------------------------------------------------------------------------------------
 constexpr int OUT_THREADS = 512;             // 16 warps: 4 row tiles of 16 tokens x 4 column quarters
 constexpr int LDA = CT + 8;
-constexpr int SLAB = 64;                     // state rows in shared memory at a time
 
-size_t output_smem(int kind, int dk, int dv, int slab_bufs) {
+size_t output_smem(int kind, int dk, int dv, int slab, int bufs) {
     const int dkp = (dk + 15) / 16 * 16;
-    size_t b = (size_t)CT * (dkp + 8) * 2 * 2 + (size_t)CT * (dv + 8) * 2 + (size_t)slab_bufs * 2 * SLAB * (dv + 8) * 2 + (size_t)2 * CT * LDA * 2;
+    const size_t slabs = (size_t)bufs * 2 * slab * (dv + 8) * 2, scores = (size_t)2 * CT * LDA * 2;
+    size_t b = (size_t)CT * (dkp + 8) * 2 * 2 + (size_t)CT * (dv + 8) * 2 + (slabs > scores ? slabs : scores);
     b += kind == KIND_GLA ? (size_t)CT * (dkp + 4) * 4 : 0;
     return b + (size_t)CT * 12 * 4;
 }
-constexpr size_t SMEM_MAX = 220 * 1024;
-int slab_buffers(int kind, int dk, int dv) { return dk > SLAB && output_smem(kind, dk, dv, 2) <= SMEM_MAX ? 2 : 1; }
+constexpr size_t SMEM_MAX = 220 * 1024, SMEM_TWO = 112 * 1024;       // one block per SM, two
+
+// Slabs that let two blocks share an SM where possible, then as much of the state as fits.  Returns the bytes.
+size_t plan_output(int kind, int dk, int dv, int& slab, int& bufs) {
+    const int plans[][2] = {{64, 2}, {64, 1}, {32, 2}, {32, 1}, {16, 1}};
+    for (size_t limit : {SMEM_TWO, SMEM_MAX})
+        for (auto& pl : plans) {
+            slab = pl[0];
+            bufs = pl[1];
+            const size_t b = output_smem(kind, dk, dv, slab, bufs);
+            if (b <= limit && (bufs == 1 || dk > slab)) return b;
+        }
+    return SMEM_MAX + 1;
+}
 
 // grid (chunks of the pass, h).  NT: 8-wide value tiles per column quarter (dv <= 32 * NT).
 template <int KIND, int NT>
-__global__ void __launch_bounds__(OUT_THREADS) chunk_output_kernel(GatedChunkParams cp) {
+__global__ void __launch_bounds__(OUT_THREADS, NT <= 4 ? 2 : 1) chunk_output_kernel(GatedChunkParams cp) {
     pdl_grid_sync();
     extern __shared__ __align__(16) unsigned char smraw[];
     const GatedScanParams& p = cp.s;
@@ -324,10 +343,11 @@ __global__ void __launch_bounds__(OUT_THREADS) chunk_output_kernel(GatedChunkPar
     bf16* qs = reinterpret_cast<bf16*>(smraw);           // [CT][ldk]
     bf16* ks = qs + CT * ldk;
     bf16* vs = ks + CT * ldk;                            // [CT][ldv]
-    bf16* slabs = vs + CT * ldv;                         // state rows [SLAB][ldv], high and low terms, one or two slabs
-    bf16* ah = slabs + cp.slab_bufs * 2 * SLAB * ldv;        // [CT][LDA] scores
+    bf16* slabs = vs + CT * ldv;                         // state rows [slab][ldv], high and low terms, one or two slabs; then
+    bf16* ah = slabs;                                    // [CT][LDA] scores, high and low terms
     bf16* al = ah + CT * LDA;
-    float* fs = reinterpret_cast<float*>(al + CT * LDA);
+    const int slab = cp.slab, region = max(cp.slab_bufs * 2 * slab * ldv, 2 * CT * LDA);
+    float* fs = reinterpret_cast<float*>(slabs + region);
     float* bs = fs;                                      // GLA: [CT][ldb]
     float* rows = fs + (KIND == KIND_GLA ? CT * ldb : 0);
     float *ga = rows, *gb = rows + CT, *gx = rows + 2 * CT, *qn = rows + 3 * CT, *nq = rows + 4 * CT, *ssq = rows + 8 * CT;
@@ -335,22 +355,21 @@ __global__ void __launch_bounds__(OUT_THREADS) chunk_output_kernel(GatedChunkPar
     const size_t base = (size_t)ci * p.h + h;
     const bf16* sin = reinterpret_cast<const bf16*>(cp.loc + base * dk * dv);
     auto load_slab = [&](int k0) {
-        bf16* sh = slabs + (k0 / SLAB) % cp.slab_bufs * 2 * SLAB * ldv;
-        const int per = dv / 8, rowsn = min(SLAB, dkp - k0);
+        bf16* sh = slabs + (k0 / slab) % cp.slab_bufs * 2 * slab * ldv;
+        const int per = dv / 8, rowsn = min(slab, dkp - k0);
         for (int i = tid; i < rowsn * per; i += OUT_THREADS) {
             const int r = i / per, c = i % per;
             bf16* dst = sh + r * ldv + c * 8;
             if (k0 + r < dk) {
                 const bf16* src = sin + ((size_t)(k0 + r) * dv + c * 8) * 2;
                 cp_async16(dst, src);
-                cp_async16(dst + SLAB * ldv, src + 8);
+                cp_async16(dst + slab * ldv, src + 8);
             } else {
-                *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<uint4*>(dst + SLAB * ldv) = make_uint4(0, 0, 0, 0);
+                *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<uint4*>(dst + slab * ldv) = make_uint4(0, 0, 0, 0);
             }
         }
     };
     load_rows(qs, ldk, (const bf16*)p.q + (size_t)t0 * p.ld + h * dk, p.ld, n, dk, dkp);
-    load_rows(ks, ldk, (const bf16*)p.k + (size_t)t0 * p.ld + h * dk, p.ld, n, dk, dkp);
     if (KIND == KIND_GLA) {
         const int per = dkp / 4;
         for (int i = tid; i < CT * per; i += OUT_THREADS) {
@@ -359,10 +378,11 @@ __global__ void __launch_bounds__(OUT_THREADS) chunk_output_kernel(GatedChunkPar
             else *reinterpret_cast<float4*>(bs + s * ldb + c) = make_float4(0.f, 0.f, 0.f, 0.f);
         }
     }
-    cp_async_commit();
-    load_rows(vs, ldv, (const bf16*)p.v + (size_t)t0 * p.ld + h * dv, p.ld, n, dv, dv);
     load_slab(0);
-    if (cp.slab_bufs > 1) load_slab(SLAB);
+    if (cp.slab_bufs > 1) load_slab(slab);
+    cp_async_commit();
+    load_rows(ks, ldk, (const bf16*)p.k + (size_t)t0 * p.ld + h * dk, p.ld, n, dk, dkp);
+    load_rows(vs, ldv, (const bf16*)p.v + (size_t)t0 * p.ld + h * dv, p.ld, n, dv, dv);
     cp_async_commit();
     const float m_in = KIND == KIND_MLSTM ? cp.scal[base * 4 + 2] : 0.f;
     if (KIND == KIND_MLSTM && warp == 0) mlstm_gates(p, t0, n, h, ga, gb, gx);
@@ -380,6 +400,59 @@ __global__ void __launch_bounds__(OUT_THREADS) chunk_output_kernel(GatedChunkPar
         if ((tid & 7) == 0) qn[r] = a;
         __syncthreads();
     }
+    // ---- S_in part: rows of the state in slabs ----
+    const int ntiles = dv / 8, tq = (ntiles + 3) / 4, nt0 = quarter * tq, ntn = max(0, min(tq, ntiles - nt0));
+    const int r0 = rt * 16 + g, r1 = r0 + 8;
+    float acc[NT][4];
+#pragma unroll
+    for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    for (int k0 = 0; k0 < dkp; k0 += slab) {
+        const int rowsn = min(slab, dkp - k0);
+        const bf16* sh = slabs + (k0 / slab) % cp.slab_bufs * 2 * slab * ldv;
+        const bf16* sl = sh + slab * ldv;
+        if (k0 >= cp.slab_bufs * slab) {                             // further slabs take the buffers in turn
+            cp_async_wait<0>();
+            __syncthreads();
+        }
+        for (int kk = 0; kk < rowsn; kk += 16) {
+            uint32_t a[4], a2[4];
+            if (KIND == KIND_MLSTM) {
+                ldsm_x4(a, qs + (rt * 16 + (lane & 15)) * ldk + k0 + kk + (lane >> 4) * 8);
+            } else {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const int r = (i & 1) ? r1 : r0, c = k0 + kk + c4 * 2 + (i >> 1) * 8;
+                    const float2 x = bf162_to_f2(*reinterpret_cast<const uint32_t*>(qs + r * ldk + c));
+                    const float2 b = *reinterpret_cast<const float2*>(bs + r * ldb + c);
+                    split_bf162(x.x * qscale * exp2_fast(b.x), x.y * qscale * exp2_fast(b.y), a[i], a2[i]);
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < NT; ++i) {
+                if (i >= ntn) break;
+                uint32_t b0, b1, l0, l1;
+                ldsm_x2_trans(b0, b1, sh + (kk + (lane & 15)) * ldv + (nt0 + i) * 8);
+                ldsm_x2_trans(l0, l1, sl + (kk + (lane & 15)) * ldv + (nt0 + i) * 8);
+                mma_bf16_16816(acc[i], a, b0, b1);
+                mma_bf16_16816(acc[i], a, l0, l1);
+                if (KIND == KIND_GLA) mma_bf16_16816(acc[i], a2, b0, b1);
+            }
+        }
+        if (k0 + cp.slab_bufs * slab < dkp) {
+            __syncthreads();
+            load_slab(k0 + cp.slab_bufs * slab);
+            cp_async_commit();
+        }
+    }
+    float e0 = 1.f, e1 = 1.f;
+    if (KIND == KIND_MLSTM) {
+        e0 = __expf(m_in - gx[r0]) * qscale;
+        e1 = __expf(m_in - gx[r1]) * qscale;
+#pragma unroll
+        for (int i = 0; i < NT; ++i) { acc[i][0] *= e0; acc[i][1] *= e0; acc[i][2] *= e1; acc[i][3] *= e1; }
+    }
+    cp_async_wait<0>();
+    __syncthreads();                                     // (the scores take the place of the state slabs)
     // ---- scores of (row tile rt, key tile J = quarter) ----
     {
         const int J = quarter, r0 = rt * 16 + g, r1 = r0 + 8;
@@ -481,59 +554,7 @@ __global__ void __launch_bounds__(OUT_THREADS) chunk_output_kernel(GatedChunkPar
             }
         }
     }
-    // ---- S_in part: rows of the state in slabs ----
-    const int ntiles = dv / 8, tq = (ntiles + 3) / 4, nt0 = quarter * tq, ntn = max(0, min(tq, ntiles - nt0));
-    const int r0 = rt * 16 + g, r1 = r0 + 8;
-    float acc[NT][4];
-#pragma unroll
-    for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-    cp_async_wait<0>();
     __syncthreads();
-    for (int k0 = 0; k0 < dkp; k0 += SLAB) {
-        const int rowsn = min(SLAB, dkp - k0);
-        const bf16* sh = slabs + (k0 / SLAB) % cp.slab_bufs * 2 * SLAB * ldv;
-        const bf16* sl = sh + SLAB * ldv;
-        if (k0 >= cp.slab_bufs * SLAB) {                             // further slabs take the buffers in turn
-            cp_async_wait<0>();
-            __syncthreads();
-        }
-        for (int kk = 0; kk < rowsn; kk += 16) {
-            uint32_t a[4], a2[4];
-            if (KIND == KIND_MLSTM) {
-                ldsm_x4(a, qs + (rt * 16 + (lane & 15)) * ldk + k0 + kk + (lane >> 4) * 8);
-            } else {
-#pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    const int r = (i & 1) ? r1 : r0, c = k0 + kk + c4 * 2 + (i >> 1) * 8;
-                    const float2 x = bf162_to_f2(*reinterpret_cast<const uint32_t*>(qs + r * ldk + c));
-                    const float2 b = *reinterpret_cast<const float2*>(bs + r * ldb + c);
-                    split_bf162(x.x * qscale * exp2_fast(b.x), x.y * qscale * exp2_fast(b.y), a[i], a2[i]);
-                }
-            }
-#pragma unroll
-            for (int i = 0; i < NT; ++i) {
-                if (i >= ntn) break;
-                uint32_t b0, b1, l0, l1;
-                ldsm_x2_trans(b0, b1, sh + (kk + (lane & 15)) * ldv + (nt0 + i) * 8);
-                ldsm_x2_trans(l0, l1, sl + (kk + (lane & 15)) * ldv + (nt0 + i) * 8);
-                mma_bf16_16816(acc[i], a, b0, b1);
-                mma_bf16_16816(acc[i], a, l0, l1);
-                if (KIND == KIND_GLA) mma_bf16_16816(acc[i], a2, b0, b1);
-            }
-        }
-        if (k0 + cp.slab_bufs * SLAB < dkp) {
-            __syncthreads();
-            load_slab(k0 + cp.slab_bufs * SLAB);
-            cp_async_commit();
-        }
-    }
-    float e0 = 1.f, e1 = 1.f;
-    if (KIND == KIND_MLSTM) {
-        e0 = __expf(m_in - gx[r0]) * qscale;
-        e1 = __expf(m_in - gx[r1]) * qscale;
-#pragma unroll
-        for (int i = 0; i < NT; ++i) { acc[i][0] *= e0; acc[i][1] *= e0; acc[i][2] *= e1; acc[i][3] *= e1; }
-    }
     // ---- intra-chunk part ----
     for (int kk = 0; kk <= rt * 16; kk += 16) {
         uint32_t a[4], a2[4];
@@ -596,10 +617,10 @@ size_t state_smem(int kind, int dk, int dv, int rank) {
 template <int KIND>
 int run_chunks(const GatedChunkParams* args, int B, cudaStream_t s) {
     GatedChunkParams params = *args;
-    params.slab_bufs = slab_buffers(KIND, args->s.dk, args->s.dv);
+    const size_t s3 = plan_output(KIND, args->s.dk, args->s.dv, params.slab, params.slab_bufs);
     const GatedChunkParams* p = &params;
     const int dk = p->s.dk, dv = p->s.dv, h = p->s.h, nc = p->c1 - p->c0;
-    const size_t s1 = state_smem(KIND, dk, dv, p->s.rank), s3 = output_smem(KIND, dk, dv, p->slab_bufs);
+    const size_t s1 = state_smem(KIND, dk, dv, p->s.rank);
     auto k1 = chunk_state_kernel<KIND>;
     if (s1 > 48 * 1024) cudaFuncSetAttribute(k1, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1);
     sl_launch(k1, dim3(nc, h), 256, s1, s, *p);
@@ -621,7 +642,8 @@ int run_chunks(const GatedChunkParams* args, int B, cudaStream_t s) {
 // 1 when the chunked kernels take these sizes (head rows of whole 16-byte pieces, tiles that fit in shared memory).
 SL_API int sl_gated_chunk_ok(int kind, int dk, int dv, int rank) {
     if (dk < 8 || dv < 8 || dk % 8 != 0 || dv % 8 != 0 || dv > 256) return 0;
-    return state_smem(kind, dk, dv, rank) <= SMEM_MAX && output_smem(kind, dk, dv, slab_buffers(kind, dk, dv)) <= SMEM_MAX;
+    int slab, bufs;
+    return state_smem(kind, dk, dv, rank) <= SMEM_MAX && plan_output(kind, dk, dv, slab, bufs) <= SMEM_MAX;
 }
 
 // One pass over the chunks [c0, c1) of B sequences (bf16 rows in and out).  Passes of one step run in order on one stream.

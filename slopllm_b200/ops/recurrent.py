@@ -111,7 +111,7 @@ CHUNK_SCRATCH_BYTES = 96 << 20      # chunk states of one pass (they stay in L2)
 
 class GatedChunkParams(C.Structure):
     _fields_ = [("s", GatedScanParams), ("chunks", C.c_void_p), ("seq_chunks", C.c_void_p), ("c0", C.c_int), ("c1", C.c_int),
-                ("b", C.c_void_p), ("loc", C.c_void_p), ("nloc", C.c_void_p), ("scal", C.c_void_p), ("slab_bufs", C.c_int)]
+                ("b", C.c_void_p), ("loc", C.c_void_p), ("nloc", C.c_void_p), ("scal", C.c_void_p), ("slab", C.c_int), ("slab_bufs", C.c_int)]
 
 
 class ChunkPlan:
