@@ -128,8 +128,13 @@ def main():
         return 0
 
     if args.hybrid:
-        from slopllm_b200.cli.hybrid_bench import main as hybrid_main
-        return hybrid_main(["--sizes", args.hybrid, "--iters", str(args.steps)])
+        from slopllm_b200.cli import hybrid_bench
+        sampler = ClockSampler(0)
+        sampler.start()
+        out = hybrid_bench.run(["--sizes", args.hybrid, "--iters", str(args.steps)])
+        out["clocks"] = sampler.stop()
+        print(json.dumps(out), flush=True)
+        return 0
 
     # the contract is ONE line on stdout: libraries that print there (NCCL's version banner) are sent to stderr for the
     # whole run, the JSON line goes to the saved descriptor at the end

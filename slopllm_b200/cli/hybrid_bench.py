@@ -130,7 +130,7 @@ def _params(model) -> int:
     return total
 
 
-def main(argv=None) -> int:
+def run(argv=None) -> dict:
     ap = argparse.ArgumentParser(prog="slopllm_b200.cli.hybrid_bench", description=__doc__.split("\n")[0])
     ap.add_argument("--sizes", default="small,medium,large")
     ap.add_argument("--batches", default="1,8,64")
@@ -146,9 +146,13 @@ def main(argv=None) -> int:
             rows.append(run_arm(family, size, [int(b) for b in args.batches.split(",")], args.prompt, args.iters, flush))
             gc.collect()
             torch.cuda.empty_cache()
-    print(json.dumps({"metric": "hybrid_families_prefill_decode", "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic",
-                      "config": {"vocab": VOCAB, "window": WINDOW, "sizes": {k: dict(zip(("width", "ff", "heads"), v)) for k, v in SIZES.items()},
-                                 "l2": "256 MB written before every timed run"}, "rows": rows}), flush=True)
+    return {"metric": "hybrid_families_prefill_decode", "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic",
+            "config": {"vocab": VOCAB, "window": WINDOW, "sizes": {k: dict(zip(("width", "ff", "heads"), v)) for k, v in SIZES.items()},
+                       "l2": "256 MB written before every timed run"}, "rows": rows}
+
+
+def main(argv=None) -> int:
+    print(json.dumps(run(argv)), flush=True)
     return 0
 
 

@@ -151,6 +151,10 @@ def mixer_rows(emit, tokens, iters: int, flush, peaks, dev, h: int = 16, dk: int
         full = T * (T + 1) / 2 if prompt else T * kv
         emit(roofline_row("paged_attention (full context)", T, us, 2.0 * (T if prompt else T * kv) * n_kv * 256 + 4.0 * T * h * 128,
                           4.0 * full * h * 128, peaks))
+        qk = bf(T, (h + 2 * n_kv) * 128)
+        us = time_op(lambda: D.qk_norm_rope_cache(qk[:, :h * 128], qk[:, h * 128:(h + n_kv) * 128], qk[:, (h + n_kv) * 128:], None, None, st.positions,
+                                                  st.batch_idx, pt, 64, kc, vc, h, n_kv, 128, 64, 1e6, 1e-6), iters, flush)
+        emit(roofline_row("qk_norm_rope_cache", T, us, 4 * T * (h + 2 * n_kv) * 128, 0.0, peaks))
         # norms
         H = h * 128
         y, res, wf, wb = rnd(T, H), rnd(T, H), rnd(H), bf(H)

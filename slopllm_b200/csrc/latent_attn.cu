@@ -27,8 +27,11 @@ struct LatentPreParams {
     int* guard;
 };
 
+constexpr int PRE_Q = 1024;              // rotated query values per block
+
+// grid (T, 1 + ceil(heads * rot_dim / PRE_Q)), block 256: block y = 0 makes the cache row, the others rotate query parts
 template <typename T>
-__global__ void __launch_bounds__(128) latent_pre_kernel(LatentPreParams p) {
+__global__ void __launch_bounds__(256) latent_pre_kernel(LatentPreParams p) {
     pdl_grid_sync();
     extern __shared__ float sm[];
     __shared__ float scratch[33];
@@ -36,43 +39,47 @@ __global__ void __launch_bounds__(128) latent_pre_kernel(LatentPreParams p) {
     float* cs = sm;
     float* sn = sm + half;
     const int pos = p.positions[t];
-    const int page = p.page_table[(size_t)p.batch_idx[t] * p.pt_stride + pos / p.page_size];
-    const long long slot = (long long)page * p.page_size + pos % p.page_size;
-    for (int i = tid; i < half; i += blockDim.x) {
+    const T* row = (const T*)p.qd + (size_t)t * p.ld;
+    const int qs = p.dim + p.rot_dim;
+    for (int i = tid; i < half; i += 256) {
         float a, b;
         sincosf((float)pos * p.freq[i], &a, &b);
         sn[i] = a * p.rot_gain;
         cs[i] = b * p.rot_gain;
     }
-    const T* row = (const T*)p.qd + (size_t)t * p.ld;
-    const int qs = p.dim + p.rot_dim;
+    // value i of a rotated part that starts at x
+    auto rotated = [&](const T* x, int i) {
+        const float v = to_f(x[i]);
+        if (i < half) return v * cs[i] - to_f(x[i + half]) * sn[i];
+        if (i < p.rot_dims) return v * cs[i - half] + to_f(x[i - half]) * sn[i - half];
+        return v;
+    };
+    if (blockIdx.y > 0) {
+        __syncthreads();
+        T* qo = (T*)p.q_rot + (size_t)t * p.heads * p.rot_dim;
+        const int j0 = (blockIdx.y - 1) * PRE_Q, total = p.heads * p.rot_dim;
+#pragma unroll
+        for (int u = 0; u < PRE_Q / 256; ++u) {
+            const int j = j0 + u * 256 + tid;
+            if (j < total) put(qo + j, rotated(row + (size_t)(j / p.rot_dim) * qs + p.dim, j % p.rot_dim));
+        }
+        return;
+    }
+    const int page = p.page_table[(size_t)p.batch_idx[t] * p.pt_stride + pos / p.page_size];
+    const long long slot = (long long)page * p.page_size + pos % p.page_size;
     const T* lat = row + (size_t)p.heads * qs;
     float ss = 0.f;
-    for (int i = tid; i < p.rank; i += blockDim.x) {
+#pragma unroll 4
+    for (int i = tid; i < p.rank; i += 256) {
         const float v = to_f(lat[i]);
         ss += v * v;
     }
     const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)p.rank + p.eps);      // (also orders the cos / sin table)
-    if (guard_ok(p.guard, 21, slot, p.num_slots)) {
-        T* dst = (T*)p.cache + (size_t)slot * (p.rank + p.rot_dim);
-        for (int i = tid; i < p.rank; i += blockDim.x) put(dst + i, to_f(lat[i]) * inv * p.norm_w[i]);
-        const T* kr = lat + p.rank;
-        for (int i = tid; i < p.rot_dim; i += blockDim.x) {
-            float v = to_f(kr[i]);
-            if (i < half) v = v * cs[i] - to_f(kr[i + half]) * sn[i];
-            else if (i < p.rot_dims) v = v * cs[i - half] + to_f(kr[i - half]) * sn[i - half];
-            put(dst + p.rank + i, v);
-        }
-    }
-    T* qo = (T*)p.q_rot + (size_t)t * p.heads * p.rot_dim;
-    for (int j = tid; j < p.heads * p.rot_dim; j += blockDim.x) {
-        const int h = j / p.rot_dim, i = j % p.rot_dim;
-        const T* q = row + (size_t)h * qs + p.dim;
-        float v = to_f(q[i]);
-        if (i < half) v = v * cs[i] - to_f(q[i + half]) * sn[i];
-        else if (i < p.rot_dims) v = v * cs[i - half] + to_f(q[i - half]) * sn[i - half];
-        put(qo + j, v);
-    }
+    if (!guard_ok(p.guard, 21, slot, p.num_slots)) return;
+    T* dst = (T*)p.cache + (size_t)slot * (p.rank + p.rot_dim);
+#pragma unroll 4
+    for (int i = tid; i < p.rank; i += 256) put(dst + i, to_f(lat[i]) * inv * p.norm_w[i]);
+    for (int i = tid; i < p.rot_dim; i += 256) put(dst + p.rank + i, rotated(lat + p.rank, i));
 }
 
 struct LatentRowsParams {
@@ -160,8 +167,9 @@ SL_API int sl_latent_pre(const LatentPreParams* p, int T, int f32, cudaStream_t 
     if (T == 0) return 0;
     if (p->rot_dims > p->rot_dim || p->rot_dims % 2 != 0) return -1;
     const size_t smem = (size_t)p->rot_dims * sizeof(float);
-    if (f32) sl_launch(latent_pre_kernel<float>, T, 128, smem, s, *p);
-    else sl_launch(latent_pre_kernel<bf16>, T, 128, smem, s, *p);
+    const dim3 grid(T, 1 + (p->heads * p->rot_dim + PRE_Q - 1) / PRE_Q);
+    if (f32) sl_launch(latent_pre_kernel<float>, grid, 256, smem, s, *p);
+    else sl_launch(latent_pre_kernel<bf16>, grid, 256, smem, s, *p);
     return SL_LAUNCH_CHECK();
 }
 
