@@ -238,7 +238,7 @@ class Glm5NextModel:
                           norm=get("o_norm.weight"), out=get("o_proj.weight"), a_log=get("A_log").to(torch.float32),
                           dt_bias=get("dt_bias").to(torch.float32))
 
-    def allocate_cache(self, num_pages: int):
+    def allocate_cache(self, num_pages: int, max_states: int = 64):
         raise NotImplementedError("the glm5_next hybrid chat cache is not implemented")
 
     def forward_hidden(self, st, cache):
