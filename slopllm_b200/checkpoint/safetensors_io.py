@@ -187,3 +187,13 @@ def iter_dir(model_dir: str) -> Iterable[str]:
                 seen.append(fn)
         return [os.path.join(model_dir, s) for s in seen]
     return sorted(os.path.join(model_dir, f) for f in os.listdir(model_dir) if f.endswith(".safetensors"))
+
+
+def load_dir(model_dir: str) -> Dict[str, torch.Tensor]:
+    """Every tensor of a checkpoint directory (CPU tensors backed by the mappings: do not write to them)."""
+    out: Dict[str, torch.Tensor] = {}
+    for path in iter_dir(model_dir):
+        sf = SafetensorsFile(path)
+        for name in sf.names():
+            out[name] = sf.tensor(name)
+    return out

@@ -133,12 +133,14 @@ def mixer_rows(emit, tokens, iters: int, flush, peaks, dev, h: int = 16, dk: int
         q_rot = L.latent_pre(qd, sh, w, rt, st, cache)
         pairs = sum(min(start + i + 1, window) for i in range(T)) if prompt else T * min(kv, window)
         if prompt:
-            us = time_op(lambda: L.latent_prefill(qd, q_rot, sh, w, st, cache, ops), iters, flush)
+            out = bf(T, h * dv)
+            us = time_op(lambda: L.latent_prefill(qd, q_rot, sh, w, st, cache, ops, out), iters, flush)
             fl = 2.0 * pairs * h * (dk + rot + dv) + 2.0 * T * rank * h * (dk + dv)
             emit(roofline_row("latent_prefill (gather, expand, attend)", T, us, 2.0 * T * (sh.row + h * (dk + rot + dv)), fl, peaks))
             rows, k, v = bf(T, sh.row), bf(T, h * dk), bf(T, h * dv)
-            out, pp = bf(T, h * dv), L.PortionPlan.of(st, window)
-            us = time_op(lambda: L.latent_prefill_kernel(qd, q_rot, sh, w, rows, k, v, pp, 0, h, out), iters, flush)
+            pp = L.PortionPlan.of(st, window)
+            us = time_op(lambda: L.portion_attention(qd, dk + rot, q_rot, k, v, pp, out, heads=h, h0=0, group=h, dim=dk, vdim=dv, window=window,
+                                                     scale=sh.scale, sink=w.sink, rot_dim=rot, rows=rows, rank=rank), iters, flush)
             emit(roofline_row("latent_prefill kernel", T, us, 2.0 * T * h * (2 * (dk + dv) + rot), 2.0 * pairs * h * (dk + rot + dv), peaks))
         else:
             us = time_op(lambda: L.latent_attention(qd, q_rot, sh, w, st, cache, ops), iters, flush)

@@ -1,0 +1,223 @@
+// Gated delta rule with one decay per key channel, token by token (definition in ops/delta.py):
+//
+//   S = diag(g) S;  u = beta (v - S^T k);  S = S + k u^T;  o = S^T q;  out = rms(o) * w * sigmoid(g2 low_g)
+//
+// One block per (sequence, head).  The state stays in registers over the sequence's tokens (a thread holds four columns of every
+// rg-th row), or in global memory for sizes that do not fit.  A decode step is one launch from the projections to the output
+// projection's input: convolutions, unit norms, low-rank decay and gate, state update, head norm.  State, gates, norms and sums
+// are fp32.
+#include "common.cuh"
+
+namespace {
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void put(float* p, float v) { *p = v; }
+__device__ __forceinline__ void put(bf16* p, float v) { *p = __float2bfloat16(v); }
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+
+struct DeltaStepParams {
+    void* out; int ldo;                      // [T, ldo]: head h at h * dv
+    const void *q, *k, *v; int ld;           // token-major rows; query / key head i at i * dk, value head i at i * dv
+    const float* low; int ld_low, ra, rg;    // [T, ra (decay) | rg (gate)]
+    const float* b;                          // [T, h] with the stride of `low`
+    const void *a2, *g2;                     // [h * dk, ra], [h * dv, rg]
+    const float *dt_bias, *A_log, *norm_w;   // [h * dk], [h], [dv]
+    float eps, unit_eps;
+    float* S;                                // [slots, h, dk, dv]
+    const float* conv_w; float* conv; int taps;      // [taps, C], [slots, taps, C]; conv null: rows are convolved already
+    const int* positions; const int* qo_indptr; const int* state_idx;
+    int h, hk, dk, dv;
+};
+
+// MAXR > 0: dv % 4 == 0 and at most MAXR state rows per thread, in registers.  MAXR == 0: state in global memory.
+template <int MAXR, typename TI, typename TO>
+__global__ void __launch_bounds__(256) delta_step_kernel(DeltaStepParams p) {
+    pdl_grid_sync();
+    extern __shared__ float sm[];
+    __shared__ float scratch[33], ss_q, ss_k;
+    const int seq = blockIdx.x / p.h, h = blockIdx.x % p.h, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int t_begin = p.qo_indptr[seq], t_end = p.qo_indptr[seq + 1];
+    if (t_begin >= t_end) return;
+    const int dk = p.dk, dv = p.dv, group = p.h / p.hk, hk = h / group;
+    constexpr int VW = MAXR > 0 ? 4 : 1, NR = MAXR > 0 ? MAXR : 1;
+    const int nc = dv / VW, rg = nc >= 256 ? 1 : 256 / nc;          // column groups, row groups that share a column
+    const int dkp = (dk + 3) / 4 * 4, dvp = (dv + 3) / 4 * 4;
+    float *sq = sm, *sk = sq + dkp, *sa = sk + dkp, *sv = sa + dkp, *sg = sv + dvp, *slow = sg + dvp;
+    float* part = slow + (p.ra + p.rg + 3) / 4 * 4;                 // [rg][dv]
+    const int slot = p.state_idx[seq];
+    float* S = p.S + ((size_t)slot * p.h + h) * dk * dv;
+    const int c = tid % nc, r = tid / nc;
+    const bool on = MAXR > 0 && r < rg;
+    float4 st[NR];
+    if (MAXR > 0) {
+#pragma unroll
+        for (int i = 0; i < NR; ++i) {
+            const int row = r + i * rg;
+            st[i] = on && row < dk ? *reinterpret_cast<const float4*>(S + (size_t)row * dv + c * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    }
+    const float rate = expf(p.A_log[h]), qscale = 1.f / sqrtf((float)dk);
+    for (int t = t_begin; t < t_end; ++t) {
+        const TI* q = (const TI*)p.q + (size_t)t * p.ld + hk * dk;
+        const TI* k = (const TI*)p.k + (size_t)t * p.ld + hk * dk;
+        const TI* v = (const TI*)p.v + (size_t)t * p.ld + h * dv;
+        const float* low = p.low + (size_t)t * p.ld_low;
+        __syncthreads();
+        for (int i = tid; i < p.ra + p.rg; i += 256) slow[i] = low[i];
+        const int pos = p.positions[t];
+        for (int i = tid; i < 2 * dk + dv; i += 256) {
+            const TI* src = i < dk ? q + i : i < 2 * dk ? k + i - dk : v + i - 2 * dk;
+            float x = to_f(*src);
+            if (p.conv != nullptr) {
+                const int C = 2 * p.hk * dk + p.h * dv;
+                const int ch = i < dk ? hk * dk + i : i < 2 * dk ? (p.hk + hk) * dk + i - dk : 2 * p.hk * dk + h * dv + i - 2 * dk;
+                float* ring = p.conv + (size_t)slot * p.taps * C + ch;
+                float a = p.conv_w[(size_t)(p.taps - 1) * C + ch] * x;
+                for (int j = 1; j < p.taps && j <= pos; ++j)
+                    a += p.conv_w[(size_t)(p.taps - 1 - j) * C + ch] * ring[(size_t)((pos - j) % p.taps) * C];
+                // (nobody reads this row of the ring in this launch, so the heads that share the channel need no order)
+                if (i >= 2 * dk || h % group == 0) ring[(size_t)(pos % p.taps) * C] = x;
+                x = a * sigmoid_f(a);
+            }
+            (i < dk ? sq[i] : i < 2 * dk ? sk[i - dk] : sv[i - 2 * dk]) = x;
+        }
+        const float beta = sigmoid_f(p.b[(size_t)t * p.ld_low + h]);
+        __syncthreads();
+        if (warp < 2) {
+            const float* x = warp == 0 ? sq : sk;
+            float ss = 0.f;
+            for (int i = lane; i < dk; i += 32) ss += x[i] * x[i];
+            ss = warp_sum(ss);
+            if (lane == 0) (warp == 0 ? ss_q : ss_k) = ss;
+        }
+        for (int i = warp; i < dk + dv; i += 8) {
+            const bool dec = i < dk;
+            const int rank = dec ? p.ra : p.rg;
+            const TO* w = dec ? (const TO*)p.a2 + (size_t)(h * dk + i) * rank : (const TO*)p.g2 + (size_t)(h * dv + i - dk) * rank;
+            const float* x = dec ? slow : slow + p.ra;
+            float z = 0.f;
+            for (int j = lane; j < rank; j += 32) z += to_f(w[j]) * x[j];
+            z = warp_sum(z);
+            if (lane == 0) {
+                if (dec) sa[i] = expf(-rate * softplus_f(z + p.dt_bias[h * dk + i]));
+                else sg[i - dk] = sigmoid_f(z);
+            }
+        }
+        __syncthreads();
+        const float qs = qscale / sqrtf(ss_q + p.unit_eps), ks = 1.f / sqrtf(ss_k + p.unit_eps);
+        if (MAXR > 0) {
+            float4 kv = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int i = 0; i < NR; ++i) {
+                const int row = r + i * rg;
+                if (row >= dk) break;
+                const float a = sa[row], kk = sk[row];
+                st[i].x *= a; st[i].y *= a; st[i].z *= a; st[i].w *= a;
+                kv.x += st[i].x * kk; kv.y += st[i].y * kk; kv.z += st[i].z * kk; kv.w += st[i].w * kk;
+            }
+            if (on) *reinterpret_cast<float4*>(part + r * dv + c * 4) = kv;
+            __syncthreads();
+            float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
+            for (int i = 0; i < rg; ++i) {
+                const float4 x = *reinterpret_cast<const float4*>(part + i * dv + c * 4);
+                sum.x += x.x; sum.y += x.y; sum.z += x.z; sum.w += x.w;
+            }
+            const float4 vv = *reinterpret_cast<const float4*>(sv + c * 4);
+            const float4 u = make_float4(beta * (vv.x - sum.x * ks) * ks, beta * (vv.y - sum.y * ks) * ks, beta * (vv.z - sum.z * ks) * ks,
+                                         beta * (vv.w - sum.w * ks) * ks);
+            __syncthreads();
+            float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int i = 0; i < NR; ++i) {
+                const int row = r + i * rg;
+                if (row >= dk) break;
+                const float kk = sk[row], qq = sq[row];
+                st[i].x += kk * u.x; st[i].y += kk * u.y; st[i].z += kk * u.z; st[i].w += kk * u.w;
+                o.x += st[i].x * qq; o.y += st[i].y * qq; o.z += st[i].z * qq; o.w += st[i].w * qq;
+            }
+            if (on) *reinterpret_cast<float4*>(part + r * dv + c * 4) = o;
+        } else {
+            for (int pass = 0; pass < 2; ++pass) {
+                for (int c0 = 0; c0 < nc; c0 += 256) {
+                    const int cc = nc >= 256 ? c0 + tid : c, rr = nc >= 256 ? 0 : r;
+                    if (cc >= nc || rr >= rg) continue;
+                    float acc = 0.f, u = 0.f;
+                    if (pass == 1) u = sv[cc];                      // (the update, left there by the first pass)
+                    for (int row = rr; row < dk; row += rg) {
+                        float* x = S + (size_t)row * dv + cc;
+                        const float s = pass == 0 ? *x * sa[row] : *x + sk[row] * u;
+                        *x = s;
+                        acc += s * (pass == 0 ? sk[row] : sq[row]);
+                    }
+                    part[rr * dv + cc] = acc;
+                }
+                __syncthreads();
+                if (pass == 0) {
+                    for (int j = tid; j < dv; j += 256) {
+                        float sum = 0.f;
+                        for (int i = 0; i < rg; ++i) sum += part[i * dv + j];
+                        sv[j] = beta * (sv[j] - sum * ks) * ks;
+                    }
+                    __syncthreads();
+                }
+            }
+        }
+        __syncthreads();
+        float ss = 0.f;
+        for (int j = tid; j < dv; j += 256) {
+            float o = 0.f;
+            for (int i = 0; i < rg; ++i) o += part[i * dv + j];
+            o *= qs;
+            part[j] = o;                                            // (column j of every group was read by this thread alone)
+            ss += o * o;
+        }
+        const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)dv + p.eps);
+        TO* out = (TO*)p.out + (size_t)t * p.ldo + (size_t)h * dv;
+        for (int j = tid; j < dv; j += 256) put(out + j, part[j] * inv * p.norm_w[j] * sg[j]);
+    }
+    if (MAXR > 0 && on) {
+#pragma unroll
+        for (int i = 0; i < NR; ++i) {
+            const int row = r + i * rg;
+            if (row < dk) *reinterpret_cast<float4*>(S + (size_t)row * dv + c * 4) = st[i];
+        }
+    }
+}
+
+}  // namespace
+
+// in_f32: q, k, v rows are fp32 (else bf16); out_f32: `out`, a2 and g2 are fp32 (needs in_f32).  With `conv` every range has at
+// most one token.
+SL_API int sl_delta_step(const DeltaStepParams* p, int B, int in_f32, int out_f32, cudaStream_t s) {
+    if (B == 0) return 0;
+    if ((out_f32 && !in_f32) || p->dk < 1 || p->dv < 1 || p->hk < 1 || p->h % p->hk != 0 || (p->conv != nullptr && p->taps < 1)) return -1;
+    const bool v4 = p->dv % 4 == 0 && p->dv <= 1024;
+    int nc = v4 ? p->dv / 4 : p->dv, rg = nc >= 256 ? 1 : 256 / nc;
+    const int rows = (p->dk + rg - 1) / rg;
+    const int maxr = !v4 ? 0 : rows <= 4 ? 4 : rows <= 8 ? 8 : rows <= 16 ? 16 : 0;
+    if (maxr == 0) {
+        nc = p->dv;
+        rg = nc >= 256 ? 1 : 256 / nc;
+    }
+    const int low = (p->ra + p->rg + 3) / 4 * 4;
+    const size_t smem = (size_t)(3 * ((p->dk + 3) / 4 * 4) + 2 * ((p->dv + 3) / 4 * 4) + low + rg * p->dv) * sizeof(float);
+    if (smem > 200 * 1024) return -1;
+#define SL_DS(R, TI, TO)                                                                                           \
+    {                                                                                                              \
+        auto kern = delta_step_kernel<R, TI, TO>;                                                                  \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);  \
+        sl_launch(kern, B * p->h, 256, smem, s, *p);                                                               \
+    }
+#define SL_DS_T(R)                                  \
+    {                                               \
+        if (out_f32) SL_DS(R, float, float)         \
+        else if (in_f32) SL_DS(R, float, bf16)      \
+        else SL_DS(R, bf16, bf16)                   \
+    }
+    if (maxr == 4) SL_DS_T(4) else if (maxr == 8) SL_DS_T(8) else if (maxr == 16) SL_DS_T(16) else SL_DS_T(0)
+#undef SL_DS_T
+#undef SL_DS
+    return SL_LAUNCH_CHECK();
+}

@@ -349,7 +349,7 @@ SL_API int sl_q_post(const QPostParams* p, int T, cudaStream_t s) {
 // result is also written as f16 in the fragment order of the NVFP4 streaming kernels (rows up to `tpad`).
 template <int TT, typename Stage>
 __device__ __forceinline__ void bmv_core(bf16* __restrict__ y, uint4* __restrict__ xp, const bf16* __restrict__ M, int T,
-                                         int Hh, int K, int N, int h, int n0, int t0, Stage stage) {
+                                         int Hh, int K, int N, int ldy, int h, int n0, int t0, Stage stage) {
     extern __shared__ float xs[];            // [TT][K], then red[8][TT][32]
     float* red = xs + TT * K;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -406,7 +406,7 @@ __device__ __forceinline__ void bmv_core(bf16* __restrict__ y, uint4* __restrict
             float v = 0.f;
 #pragma unroll
             for (int w = 0; w < 8; ++w) v += red[(w * TT + tt) * 32 + c];
-            y[((size_t)(t0 + tt) * Hh + h) * N + n0 + c] = __float2bfloat16(v);
+            y[(size_t)(t0 + tt) * ldy + (size_t)h * N + n0 + c] = __float2bfloat16(v);
             red[tt * 32 + c] = v;            // warp 0's slot (only this thread reads or writes column c of row tt)
         }
     }
@@ -437,7 +437,7 @@ template <int TT>
 __device__ __forceinline__ void bmv_body(bf16* __restrict__ y, const void* __restrict__ x, const bf16* __restrict__ M, int T,
                                          int Hh, int K, int N, int xs_t, int xs_h, int n_slabs, long long slab_stride, int h,
                                          int n0, int t0) {
-    bmv_core<TT>(y, nullptr, M, T, Hh, K, N, h, n0, t0, [&](float* xs) {
+    bmv_core<TT>(y, nullptr, M, T, Hh, K, N, Hh * N, h, n0, t0, [&](float* xs) {
         for (int i = threadIdx.x; i < TT * K; i += blockDim.x) {
             const int tt = i / K, kk = i % K;
             xs[i] = (t0 + tt < T) ? load_act(x, n_slabs, slab_stride, (size_t)(t0 + tt) * xs_t + (size_t)h * xs_h + kk) : 0.f;
@@ -455,6 +455,7 @@ struct CombineExpandParams {
     bf16* y;                  // [T, Hh * N]
     uint4* xp;                // fragment-ordered f16 copy [tpad, Hh * N], or null
     int T, tpad, Hh, K, N, np;
+    int ldy;                  // row stride of y (0: Hh * N)
 };
 
 template <int TT>
@@ -480,7 +481,7 @@ __global__ void __launch_bounds__(256) combine_vexpand_kernel(CombineExpandParam
         if (lane == 0) s_inv[warp] = den > 0.f ? 1.f / den : 0.f;
     }
     __syncthreads();
-    bmv_core<TT>(p.y, p.xp, p.w_v, p.T, p.Hh, p.K, p.N, h, n0, t0, [&](float* xs) {
+    bmv_core<TT>(p.y, p.xp, p.w_v, p.T, p.Hh, p.K, p.N, p.ldy > 0 ? p.ldy : p.Hh * p.N, h, n0, t0, [&](float* xs) {
         const int k4 = p.K / 4;
         for (int i = tid; i < TT * k4; i += 256) {
             const int tt = i / k4, d = (i % k4) * 4, t = t0 + tt;

@@ -1,0 +1,413 @@
+// Grouped-query attention over a paged cache: query / key norm, rotary table, sliding window with kept first tokens, softmax
+// sink, values of their own or the key projections themselves.  (Portions of prompts attend in latent_mma.cu.)
+//
+//  * grouped_pre_kernel: per-head RMS norm and rotate-half of queries and keys; keys and values go into their cache slots.
+//  * grouped_rows_kernel: independent token rows on the CUDA cores, any sizes, bf16 or fp32.
+//  * grouped_decode_kernel: one query token per page-table row on the tensor cores: a CTA takes the query heads of one key head
+//    (16 at a time) x a range of the visible keys, which come through two cp.async stages.  grouped_merge_kernel joins the key
+//    splits; the sink belongs to split 0, so it counts once.
+//
+// The keys that a row sees are numbered 0 .. n-1: first the kept ones before the window, then the window.
+#include "common.cuh"
+#include "mma_sync.cuh"
+
+namespace {
+
+constexpr float LOG2E = 1.4426950408889634f;
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void put(float* p, float v) { *p = v; }
+__device__ __forceinline__ void put(bf16* p, float v) { *p = __float2bfloat16(v); }
+
+struct GroupedPreParams {
+    const void *q, *k, *v; int ld;       // token-major projection rows (v may be k)
+    int heads, kv_heads, dim, vdim, rot_dims;
+    const float *q_norm, *k_norm;        // [dim] or null
+    const float* freq; float rot_gain, eps;
+    const int* positions; const int* batch_idx; const int* page_table;
+    int pt_stride, page_size;
+    void *k_cache, *v_cache; int num_slots;      // [slots, kv_heads, dim], [slots, kv_heads, vdim]
+    void* q_out;                         // [T, heads, dim]
+    int* guard;
+};
+
+// grid (T, ceil((heads + kv_heads) / 8)), block 256: a warp per head
+template <typename TI, typename TO>
+__global__ void __launch_bounds__(256) grouped_pre_kernel(GroupedPreParams p) {
+    pdl_grid_sync();
+    extern __shared__ float sm[];
+    const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, half = p.rot_dims / 2;
+    float *cs = sm, *sn = cs + half, *x = sn + half + warp * p.dim;
+    const int pos = p.positions[t];
+    for (int i = tid; i < half; i += 256) {
+        float a, b;
+        sincosf((float)pos * p.freq[i], &a, &b);
+        sn[i] = a * p.rot_gain;
+        cs[i] = b * p.rot_gain;
+    }
+    const int hh = blockIdx.y * 8 + warp;
+    const bool is_q = hh < p.heads, on = hh < p.heads + p.kv_heads;
+    const int h = is_q ? hh : hh - p.heads;
+    const float* w = is_q ? p.q_norm : p.k_norm;
+    float inv = 1.f;
+    if (on) {
+        const TI* src = (const TI*)(is_q ? p.q : p.k) + (size_t)t * p.ld + (size_t)h * p.dim;
+        float ss = 0.f;
+        for (int i = lane; i < p.dim; i += 32) {
+            const float v = to_f(src[i]);
+            x[i] = v;
+            ss += v * v;
+        }
+        if (w != nullptr) inv = 1.f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);
+        __syncwarp();
+        if (w != nullptr)
+            for (int i = lane; i < p.dim; i += 32) x[i] = x[i] * inv * w[i];
+    }
+    __syncthreads();
+    if (!on) return;
+    TO* dst;
+    if (is_q) {
+        dst = (TO*)p.q_out + ((size_t)t * p.heads + h) * p.dim;
+    } else {
+        const int page = p.page_table[(size_t)p.batch_idx[t] * p.pt_stride + pos / p.page_size];
+        const long long slot = (long long)page * p.page_size + pos % p.page_size;
+        if (!guard_ok(p.guard, 25, slot, p.num_slots)) return;
+        dst = (TO*)p.k_cache + ((size_t)slot * p.kv_heads + h) * p.dim;
+        const TI* vs = (const TI*)p.v + (size_t)t * p.ld + (size_t)h * p.vdim;
+        TO* vd = (TO*)p.v_cache + ((size_t)slot * p.kv_heads + h) * p.vdim;
+        for (int i = lane; i < p.vdim; i += 32) put(vd + i, to_f(vs[i]));
+    }
+    for (int i = lane; i < p.dim; i += 32) {
+        float v = x[i];
+        if (i < half) v = v * cs[i] - x[i + half] * sn[i];
+        else if (i < p.rot_dims) v = v * cs[i - half] + x[i - half] * sn[i - half];
+        put(dst + i, v);
+    }
+}
+
+struct GroupedAttnParams {
+    const void* q;                       // [T, heads, dim]
+    const void *k_cache, *v_cache; int num_slots;
+    const int* positions; const int* batch_idx; const int* page_table;
+    int pt_stride, page_size;
+    int heads, kv_heads, dim, vdim, window, keep_first, splits;
+    float scale;
+    const float* sink;                   // [heads] or null
+    void* out; int ldo;                  // [T, ldo]: head h at h * vdim
+    float *o_part, *lse_part;            // [T, heads, splits, vdim], [T, heads, splits] (decode with more than one split)
+    int* guard;
+};
+
+// The keys a position sees: n of them, number i is position at(i).
+struct Visible {
+    int kept, first, n;
+    __device__ __forceinline__ Visible(const GroupedAttnParams& p, int pos) {
+        first = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+        kept = min(p.keep_first, first);
+        n = kept + pos + 1 - first;
+    }
+    __device__ __forceinline__ int at(int i) const { return i < kept ? i : first + i - kept; }
+};
+
+constexpr int ROWS_KT = 64, ROWS_MAXV = 4;      // keys per tile; values per thread (vdim <= 512)
+
+// grid (heads, T), block 128
+template <typename T>
+__global__ void __launch_bounds__(128) grouped_rows_kernel(GroupedAttnParams p) {
+    pdl_grid_sync();
+    extern __shared__ float q[];
+    __shared__ float sc[ROWS_KT];
+    __shared__ long long slots[ROWS_KT];
+    __shared__ float scratch[33];
+    const int h = blockIdx.x, t = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int hkv = h / (p.heads / p.kv_heads);
+    for (int i = tid; i < p.dim; i += 128) q[i] = to_f(((const T*)p.q)[((size_t)t * p.heads + h) * p.dim + i]);
+    const Visible vis(p, p.positions[t]);
+    const int* pt = p.page_table + (size_t)p.batch_idx[t] * p.pt_stride;
+    const T *kc = (const T*)p.k_cache + (size_t)hkv * p.dim, *vc = (const T*)p.v_cache + (size_t)hkv * p.vdim;
+    const size_t krow = (size_t)p.kv_heads * p.dim, vrow = (size_t)p.kv_heads * p.vdim;
+    float m = p.sink != nullptr ? p.sink[h] : -INFINITY, l = p.sink != nullptr ? 1.f : 0.f;
+    float o[ROWS_MAXV];
+#pragma unroll
+    for (int i = 0; i < ROWS_MAXV; ++i) o[i] = 0.f;
+    for (int k0 = 0; k0 < vis.n; k0 += ROWS_KT) {
+        const int nk = min(ROWS_KT, vis.n - k0);
+        __syncthreads();
+        if (tid < nk) {
+            const int kp = vis.at(k0 + tid);
+            const long long s = (long long)pt[kp / p.page_size] * p.page_size + kp % p.page_size;
+            slots[tid] = guard_ok(p.guard, 26, s, p.num_slots) ? s : 0;
+        }
+        __syncthreads();
+        for (int k = warp; k < nk; k += 4) {
+            const T* row = kc + (size_t)slots[k] * krow;
+            float a = 0.f;
+            for (int i = lane; i < p.dim; i += 32) a += q[i] * to_f(row[i]);
+            a = warp_sum(a);
+            if (lane == 0) sc[k] = a * p.scale;
+        }
+        __syncthreads();
+        const float top = fmaxf(m, block_max(tid < nk ? sc[tid] : -FLT_MAX, scratch));
+        const float e = tid < nk ? expf(sc[tid] - top) : 0.f;
+        const float f = m == -INFINITY ? 0.f : expf(m - top);
+        const float sum = block_sum(e, scratch);
+        if (tid < nk) sc[tid] = e;
+        l = l * f + sum;
+        m = top;
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < ROWS_MAXV; ++i) {
+            const int d = tid + i * 128;
+            if (d >= p.vdim) break;
+            float a = o[i] * f;
+            for (int k = 0; k < nk; ++k) a += sc[k] * to_f(vc[(size_t)slots[k] * vrow + d]);
+            o[i] = a;
+        }
+    }
+    const float inv = 1.f / l;
+#pragma unroll
+    for (int i = 0; i < ROWS_MAXV; ++i) {
+        const int d = tid + i * 128;
+        if (d < p.vdim) put((T*)p.out + (size_t)t * p.ldo + (size_t)h * p.vdim + d, o[i] * inv);
+    }
+}
+
+constexpr int KT = 64, STAGES = 2, DT = 128;     // keys per tile, threads of the decode kernel
+
+// grid (splits, kv_heads * head groups of 16, T), block 128.  NTW: 8-wide value tiles per warp (vdim <= 32 * NTW).
+template <int NTW>
+__global__ void __launch_bounds__(DT) grouped_decode_kernel(GroupedAttnParams p) {
+    pdl_grid_sync();
+    extern __shared__ __align__(16) unsigned char smraw[];
+    const int group = p.heads / p.kv_heads, hg = (group + 15) / 16;
+    const int split = blockIdx.x, hkv = blockIdx.y / hg, t = blockIdx.z;
+    const int r_lo = blockIdx.y % hg * 16, nr = min(16, group - r_lo), h0 = hkv * group + r_lo;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, c4 = lane & 3;
+    const int dqp = (p.dim + 15) / 16 * 16, ld = dqp + 8, ldv = p.vdim + 8;
+    bf16* qs = reinterpret_cast<bf16*>(smraw);                      // [16][ld]
+    bf16* ks = qs + 16 * ld;                                        // STAGES x [KT][ld]
+    bf16* vs = ks + STAGES * KT * ld;                               // STAGES x [KT][ldv]
+    float* sc = reinterpret_cast<float*>(vs + STAGES * KT * ldv);   // [16][KT + 4]
+    bf16* ph = reinterpret_cast<bf16*>(sc + 16 * (KT + 4));         // [16][KT + 8]
+    bf16* pl = ph + 16 * (KT + 8);
+    float* fac = reinterpret_cast<float*>(pl + 16 * (KT + 8));      // [16]
+    const Visible vis(p, p.positions[t]);
+    const int tiles = (vis.n + KT - 1) / KT, per = (tiles + p.splits - 1) / p.splits;
+    const int tb = min(tiles, split * per), te = min(tiles, tb + per);
+    const int* pt = p.page_table + (size_t)p.batch_idx[t] * p.pt_stride;
+    const bf16 *kc = (const bf16*)p.k_cache + (size_t)hkv * p.dim, *vc = (const bf16*)p.v_cache + (size_t)hkv * p.vdim;
+    const size_t krow = (size_t)p.kv_heads * p.dim, vrow = (size_t)p.kv_heads * p.vdim;
+    const int kpc = p.dim / 8, vpc = p.vdim / 8;
+    // a warp fetches 16 rows of a tile
+    auto fetch = [&](int j) {
+        if (j < te) {
+            const int k0 = j * KT, nk = min(KT, vis.n - k0), st = (j - tb) % STAGES;
+            long long slot = -1;
+            if (lane < 16 && warp * 16 + lane < nk) {
+                const int kp = vis.at(k0 + warp * 16 + lane);
+                const long long s = (long long)pt[kp / p.page_size] * p.page_size + kp % p.page_size;
+                slot = guard_ok(p.guard, 27, s, p.num_slots) ? s : -1;
+            }
+            bf16 *kd = ks + (st * KT + warp * 16) * ld, *vd = vs + (st * KT + warp * 16) * ldv;
+            for (int i = lane; i < 16 * kpc; i += 32) {
+                const int r = i / kpc, c = i % kpc * 8;
+                const long long s = __shfl_sync(__activemask(), slot, r);
+                if (s >= 0) cp_async16(kd + r * ld + c, kc + (size_t)s * krow + c);
+                else *reinterpret_cast<uint4*>(kd + r * ld + c) = make_uint4(0, 0, 0, 0);
+            }
+            for (int i = lane; i < 16 * vpc; i += 32) {
+                const int r = i / vpc, c = i % vpc * 8;
+                const long long s = __shfl_sync(__activemask(), slot, r);
+                if (s >= 0) cp_async16(vd + r * ldv + c, vc + (size_t)s * vrow + c);
+                else *reinterpret_cast<uint4*>(vd + r * ldv + c) = make_uint4(0, 0, 0, 0);
+            }
+        }
+        cp_async_commit();
+    };
+    for (int i = tid; i < 16 * (dqp / 8); i += DT) {
+        const int r = i / (dqp / 8), c = i % (dqp / 8) * 8;
+        uint4 x = make_uint4(0, 0, 0, 0);
+        if (r < nr && c < p.dim) x = *reinterpret_cast<const uint4*>((const bf16*)p.q + ((size_t)t * p.heads + h0 + r) * p.dim + c);
+        *reinterpret_cast<uint4*>(qs + r * ld + c) = x;
+    }
+    if (dqp > p.dim)                                                // (dim % 8 == 0: one column piece of padding)
+        for (int r = tid; r < STAGES * KT; r += DT) *reinterpret_cast<uint4*>(ks + r * ld + p.dim) = make_uint4(0, 0, 0, 0);
+    float m[4], l[4];                                               // softmax state of rows 4 * warp ..
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+        const int r = warp * 4 + u;
+        const bool s = split == 0 && p.sink != nullptr && r < nr;
+        m[u] = s ? p.sink[h0 + r] * LOG2E : -INFINITY;
+        l[u] = s ? 1.f : 0.f;
+    }
+    const int nt = p.vdim / 8, tw = (nt + 3) / 4, n0 = warp * tw, nn = max(0, min(tw, nt - n0));
+    float acc[NTW][4];
+#pragma unroll
+    for (int i = 0; i < NTW; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    const float scale_log2 = p.scale * LOG2E;
+    fetch(tb);
+    for (int j = tb; j < te; ++j) {
+        fetch(j + 1);
+        cp_async_wait<1>();
+        __syncthreads();
+        const int nk = min(KT, vis.n - j * KT), st = (j - tb) % STAGES;
+        const bf16 *kt = ks + st * KT * ld, *vt = vs + st * KT * ldv;
+        float s4[2][4] = {};                                        // 16 heads x the warp's 16 keys
+        for (int kk = 0; kk < dqp; kk += 16) {
+            uint32_t a[4], b[4];
+            ldsm_x4(a, qs + (lane & 15) * ld + kk + (lane >> 4) * 8);
+            ldsm_x4(b, kt + (warp * 16 + (lane & 7) + (lane >> 4) * 8) * ld + kk + ((lane >> 3) & 1) * 8);
+            mma_bf16_16816(s4[0], a, b[0], b[1]);
+            mma_bf16_16816(s4[1], a, b[2], b[3]);
+        }
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+            const int kcol = warp * 16 + u * 8 + c4 * 2;
+            sc[g * (KT + 4) + kcol] = kcol < nk ? s4[u][0] * scale_log2 : -INFINITY;
+            sc[g * (KT + 4) + kcol + 1] = kcol + 1 < nk ? s4[u][1] * scale_log2 : -INFINITY;
+            sc[(g + 8) * (KT + 4) + kcol] = kcol < nk ? s4[u][2] * scale_log2 : -INFINITY;
+            sc[(g + 8) * (KT + 4) + kcol + 1] = kcol + 1 < nk ? s4[u][3] * scale_log2 : -INFINITY;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            const int r = warp * 4 + u;
+            const float2 v = *reinterpret_cast<const float2*>(sc + r * (KT + 4) + lane * 2);
+            const float x = fmaxf(m[u], warp_max(fmaxf(v.x, v.y)));
+            const float f = m[u] == -INFINITY ? 0.f : exp2f(m[u] - x);
+            const float e0 = exp2f(v.x - x), e1 = exp2f(v.y - x);
+            l[u] = l[u] * f + warp_sum(e0 + e1);
+            m[u] = x;
+            uint32_t hi, lo;
+            split_bf162(e0, e1, hi, lo);
+            *reinterpret_cast<uint32_t*>(ph + r * (KT + 8) + lane * 2) = hi;
+            *reinterpret_cast<uint32_t*>(pl + r * (KT + 8) + lane * 2) = lo;
+            if (lane == 0) fac[r] = f;
+        }
+        __syncthreads();
+        const float f0 = fac[g], f1 = fac[g + 8];
+#pragma unroll
+        for (int i = 0; i < NTW; ++i) { acc[i][0] *= f0; acc[i][1] *= f0; acc[i][2] *= f1; acc[i][3] *= f1; }
+#pragma unroll
+        for (int kk = 0; kk < KT; kk += 16) {
+            uint32_t a[4], a2[4];
+            ldsm_x4(a, ph + (lane & 15) * (KT + 8) + kk + (lane >> 4) * 8);
+            ldsm_x4(a2, pl + (lane & 15) * (KT + 8) + kk + (lane >> 4) * 8);
+#pragma unroll
+            for (int i = 0; i < NTW; ++i) {
+                if (i >= nn) break;
+                uint32_t b0, b1;
+                ldsm_x2_trans(b0, b1, vt + (kk + (lane & 15)) * ldv + (n0 + i) * 8);
+                mma_bf16_16816(acc[i], a, b0, b1);
+                mma_bf16_16816(acc[i], a2, b0, b1);
+            }
+        }
+        __syncthreads();                                            // (the stage is filled again by the next fetch)
+    }
+    cp_async_wait_all();
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+        const int r = warp * 4 + u;
+        if (lane == 0) {
+            fac[r] = l[u] > 0.f ? 1.f / l[u] : 0.f;
+            if (r < nr && p.splits > 1)
+                p.lse_part[((size_t)t * p.heads + h0 + r) * p.splits + split] = l[u] > 0.f ? (m[u] + log2f(l[u])) / LOG2E : -INFINITY;
+        }
+    }
+    __syncthreads();
+    const float i0 = fac[g], i1 = fac[g + 8];
+#pragma unroll
+    for (int i = 0; i < NTW; ++i) {
+        if (i >= nn) break;
+        const int d = (n0 + i) * 8 + c4 * 2;
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+            const int r = g + u * 8;
+            if (r >= nr) continue;
+            const float inv = u ? i1 : i0, x = acc[i][u * 2] * inv, y = acc[i][u * 2 + 1] * inv;
+            if (p.splits == 1) *reinterpret_cast<uint32_t*>((bf16*)p.out + (size_t)t * p.ldo + (size_t)(h0 + r) * p.vdim + d) = f2_to_bf162(x, y);
+            else *reinterpret_cast<float2*>(p.o_part + (((size_t)t * p.heads + h0 + r) * p.splits + split) * p.vdim + d) = make_float2(x, y);
+        }
+    }
+}
+
+// grid (heads, T), block 64: two values per thread and pass
+__global__ void __launch_bounds__(64) grouped_merge_kernel(GroupedAttnParams p) {
+    pdl_grid_sync();
+    __shared__ float w[64];
+    const int h = blockIdx.x, t = blockIdx.y, tid = threadIdx.x, lane = tid & 31;
+    const size_t row = (size_t)t * p.heads + h;
+    const float a = lane < p.splits ? p.lse_part[row * p.splits + lane] : -INFINITY;
+    const float b = lane + 32 < p.splits ? p.lse_part[row * p.splits + lane + 32] : -INFINITY;
+    const float top = warp_max(fmaxf(a, b));
+    const float ea = a == -INFINITY ? 0.f : expf(a - top), eb = b == -INFINITY ? 0.f : expf(b - top);
+    const float den = warp_sum(ea + eb), inv = den > 0.f ? 1.f / den : 0.f;
+    if (tid < 32) {
+        w[lane] = ea * inv;
+        w[lane + 32] = eb * inv;
+    }
+    __syncthreads();
+    for (int d = tid * 2; d < p.vdim; d += 128) {
+        float x = 0.f, y = 0.f;
+#pragma unroll 8
+        for (int i = 0; i < p.splits; ++i) {
+            const float2 v = *reinterpret_cast<const float2*>(p.o_part + (row * p.splits + i) * p.vdim + d);
+            x += w[i] * v.x;
+            y += w[i] * v.y;
+        }
+        *reinterpret_cast<uint32_t*>((bf16*)p.out + (size_t)t * p.ldo + (size_t)h * p.vdim + d) = f2_to_bf162(x, y);
+    }
+}
+
+size_t decode_smem(int dim, int vdim) {
+    const int ld = (dim + 15) / 16 * 16 + 8;
+    return (size_t)16 * ld * 2 + (size_t)STAGES * KT * (ld + vdim + 8) * 2 + (size_t)16 * (KT + 4) * 4 + (size_t)2 * 16 * (KT + 8) * 2 + 64;
+}
+
+}  // namespace
+
+SL_API int sl_grouped_pre(const GroupedPreParams* p, int T, int in_f32, int out_f32, cudaStream_t s) {
+    if (T == 0) return 0;
+    if (p->rot_dims > p->dim || p->rot_dims % 2 != 0 || (out_f32 && !in_f32)) return -1;
+    const size_t smem = (size_t)(p->rot_dims + 8 * p->dim) * sizeof(float);
+    if (smem > 48 * 1024) return -1;
+    const dim3 grid(T, (p->heads + p->kv_heads + 7) / 8);
+    if (out_f32) sl_launch(grouped_pre_kernel<float, float>, grid, 256, smem, s, *p);
+    else if (in_f32) sl_launch(grouped_pre_kernel<float, bf16>, grid, 256, smem, s, *p);
+    else sl_launch(grouped_pre_kernel<bf16, bf16>, grid, 256, smem, s, *p);
+    return SL_LAUNCH_CHECK();
+}
+
+SL_API int sl_grouped_rows(const GroupedAttnParams* p, int T, int f32, cudaStream_t s) {
+    if (T == 0) return 0;
+    if (p->vdim > 128 * ROWS_MAXV || T > 65535 || p->heads % p->kv_heads != 0) return -1;
+    const size_t smem = (size_t)p->dim * sizeof(float);
+    if (smem > 40 * 1024) return -1;
+    if (f32) sl_launch(grouped_rows_kernel<float>, dim3(p->heads, T), 128, smem, s, *p);
+    else sl_launch(grouped_rows_kernel<bf16>, dim3(p->heads, T), 128, smem, s, *p);
+    return SL_LAUNCH_CHECK();
+}
+
+// 1 when the tensor-core decode kernel takes these sizes.
+SL_API int sl_grouped_decode_ok(int dim, int vdim) {
+    return dim >= 8 && vdim >= 8 && dim % 8 == 0 && vdim % 8 == 0 && dim <= 256 && vdim <= 256 && decode_smem(dim, vdim) <= 200 * 1024;
+}
+
+SL_API int sl_grouped_decode(const GroupedAttnParams* p, int T, cudaStream_t s) {
+    if (T == 0) return 0;
+    if (!sl_grouped_decode_ok(p->dim, p->vdim) || p->splits < 1 || p->splits > 64 || T > 65535 || p->heads % p->kv_heads != 0) return -1;
+    if (p->ldo % 2 != 0 || (p->splits > 1 && (p->o_part == nullptr || p->lse_part == nullptr))) return -1;
+    const size_t smem = decode_smem(p->dim, p->vdim);
+    const dim3 grid(p->splits, p->kv_heads * ((p->heads / p->kv_heads + 15) / 16), T);
+#define SL_GD(NTW)                                                                                                      \
+    {                                                                                                                   \
+        auto kern = grouped_decode_kernel<NTW>;                                                                         \
+        cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                             \
+        sl_launch(kern, grid, DT, smem, s, *p);                                                                         \
+    }
+    if (p->vdim <= 64) SL_GD(2) else if (p->vdim <= 128) SL_GD(4) else SL_GD(8)
+#undef SL_GD
+    if (p->splits > 1) sl_launch(grouped_merge_kernel, dim3(p->heads, T), 64, 0, s, *p);
+    return SL_LAUNCH_CHECK();
+}

@@ -1,9 +1,11 @@
 // Tensor-core kernels of latent attention (bf16 cache rows [latent | rotated key part], sliding window, softmax sink).
 //
 //  * latent_gather_kernel: the cache rows that a step's portions can see, copied out of the pages in order.
-//  * latent_prefill_kernel: expanded form for portions of prompts.  Keys and values of the visible rows were materialised per
-//    head by two GEMMs; FlashAttention-2 style over 128 queries x 1 head per CTA, the shared rotated key part is read beside
-//    the head's own, tiles of 64 keys come through a three-stage cp.async ring filled by a warp of its own.
+//  * portion_attn_kernel: attention of portions of prompts over gathered rows, also used by grouped-query attention.  In latent
+//    attention it is the expanded form: keys and values of the visible rows were materialised per head by two GEMMs, and a
+//    shared rotated key part may be read beside the head's own.  FlashAttention-2 style over 128 queries x 1 head per CTA, tiles
+//    of 64 keys come through a three-stage cp.async ring filled by a warp of its own.  A sliding window may keep the sequence's
+//    first tokens visible: their tiles come before the window's.
 //  * latent_decode_kernel: absorbed form, one query token per page-table row.  A CTA takes 16 heads x a range of keys: all
 //    heads share the key rows, whose first `rank` values are the value rows as well, so a tile is read once for both products.
 //    Key splits leave (o, log-sum-exp) partials for `sl_combine_vexpand` / `sl_mla_combine`; the sink belongs to split 0.
@@ -39,17 +41,18 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(LatentGatherParams p
     for (int c = lane; c < p.row / 8; c += 32) dst[c] = src[c];
 }
 
-struct LatentPrefillParams {
-    const bf16* q; int ldq, q_head;       // unrotated query of head i at i * q_head
-    const bf16* q_rot;                    // [T, heads, rot_dim]
-    const bf16* k; int ldk;               // expanded keys [rows, ldk], head h0 + i at i * dim
-    const bf16* v; int ldv;               // expanded values, head h0 + i at i * vdim
+struct PortionAttnParams {
+    const bf16* q; int ldq, q_head;       // (unrotated) query of head i at i * q_head
+    const bf16* q_rot;                    // [T, heads, rot_dim] (rot_dim 0: none)
+    const bf16* k; int ldk;               // keys [rows, ldk], key head of h0 + i at (i / kv_group) * dim
+    const bf16* v; int ldv;               // values, likewise at (i / kv_group) * vdim
     const bf16* rows; int row, rank;      // gathered cache rows: rotated key part at `rank`
-    const int* tiles;                     // [tiles][4]: first token, tokens, position of the first token, (key row - key position)
-    int heads, h0, dim, rot_dim, vdim, window;
+    const int* tiles;                     // [tiles][5]: first token, tokens, position of the first token, (key row - key position)
+                                          // of the window's keys and of the kept first ones
+    int heads, h0, dim, rot_dim, vdim, kv_group, window, keep_first;
     float scale;
     const float* sink;                    // [heads] or null
-    bf16* out;                            // [T, heads * vdim]
+    bf16* out; int ldo;                   // [T, ldo]: head i at i * vdim
     int* err;                             // status word: set when a wait inside the kernel expired
     int stages;                           // set by the launcher: key tiles in shared memory
 };
@@ -76,12 +79,12 @@ __device__ __forceinline__ float exp2_fast(float x) {
 // grid (heads of the group, tiles).  NT: 8-wide value tiles (vdim <= 8 * NT).  The fetching warp runs ahead of the consumers by
 // up to `stages` key tiles; consumer warps do not wait for one another.
 template <int NT>
-__global__ void __launch_bounds__(PT, 1) latent_prefill_kernel(LatentPrefillParams p) {
+__global__ void __launch_bounds__(PT, 1) portion_attn_kernel(PortionAttnParams p) {
     pdl_grid_sync();
     extern __shared__ __align__(16) unsigned char smraw[];
     const int hg = blockIdx.x, h = p.h0 + hg, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, c4 = lane & 3;
-    const int* tl = p.tiles + (gridDim.y - 1 - blockIdx.y) * 4;      // late positions see most keys: start them first
-    const int q0 = tl[0], nq = tl[1], pos0 = tl[2], koff = tl[3];
+    const int* tl = p.tiles + (gridDim.y - 1 - blockIdx.y) * 5;      // late positions see most keys: start them first
+    const int q0 = tl[0], nq = tl[1], pos0 = tl[2], koff = tl[3], koff_kept = tl[4], hk = hg / p.kv_group;
     const int dq = p.dim + p.rot_dim, dqp = (dq + 15) / 16 * 16, ld = dqp + 8, ldv = NT * 8 + 8;
     bf16* qs = reinterpret_cast<bf16*>(smraw);            // [BQ][ld]
     const int stages = p.stages;
@@ -92,7 +95,9 @@ __global__ void __launch_bounds__(PT, 1) latent_prefill_kernel(LatentPrefillPara
     const int nd = p.dim / 8, nr = p.rot_dim / 8, nv = p.vdim / 8;
     const int last = pos0 + nq - 1;
     const int first = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
-    const int ntiles = (last - first) / BK + 1;
+    const int kept = min(p.keep_first, first), kept_tiles = (kept + BK - 1) / BK;      // kept keys in front of the tile's window
+    const int ntiles = kept_tiles + (last - first) / BK + 1;
+    auto tile_start = [&](int j) { return j < kept_tiles ? j * BK : first + (j - kept_tiles) * BK; };
 
     // columns that no copy writes: the query / key padding to 16 and the value padding
     for (int i = tid; i < (BQ + stages * BK) * (dqp - dq); i += PT) qs[(i / (dqp - dq)) * ld + dq + i % (dqp - dq)] = __float2bfloat16(0.f);
@@ -124,16 +129,22 @@ __global__ void __launch_bounds__(PT, 1) latent_prefill_kernel(LatentPrefillPara
     if (warp == CONSUMERS) {
         // a lane copies the same 16-byte column of every (32 / pieces)-th row of a part (a row has at most 32 pieces)
         struct Part { int row, step; bool on; };
-        auto part = [&](int pieces) { Part x; x.step = 32 / pieces; x.row = lane / pieces; x.on = x.row < x.step; return x; };
+        auto part = [&](int pieces) {
+            Part x;
+            x.step = pieces > 0 ? 32 / pieces : 1;
+            x.row = pieces > 0 ? lane / pieces : 0;
+            x.on = pieces > 0 && x.row < x.step;
+            return x;
+        };
         const Part pk = part(nd), pr = part(nr), pv = part(nv);
-        const bf16* kcol = p.k + hg * p.dim + lane % nd * 8;
-        const bf16* rcol = p.rows + p.rank + lane % nr * 8;
-        const bf16* vcol = p.v + hg * p.vdim + lane % nv * 8;
-        auto copy = [&](const Part& x, bf16* dst, int dld, const bf16* col, size_t sld, int k0) {
+        const bf16* kcol = p.k + hk * p.dim + lane % nd * 8;
+        const bf16* rcol = nr > 0 ? p.rows + p.rank + lane % nr * 8 : nullptr;
+        const bf16* vcol = p.v + hk * p.vdim + lane % nv * 8;
+        auto copy = [&](const Part& x, bf16* dst, int dld, const bf16* col, size_t sld, int k0, int n, int off) {
             if (!x.on) return;
-            const bf16* src = col + (size_t)(k0 + x.row + koff) * sld;
+            const bf16* src = col + (ptrdiff_t)(k0 + x.row + off) * (ptrdiff_t)sld;
             dst += x.row * dld;
-            const int n = min(BK, last + 1 - k0), dstep = x.step * dld;
+            const int dstep = x.step * dld;
             const size_t sstep = (size_t)x.step * sld;
             int r = x.row;
 #pragma unroll 4
@@ -141,13 +152,14 @@ __global__ void __launch_bounds__(PT, 1) latent_prefill_kernel(LatentPrefillPara
             for (; r < BK; r += x.step, dst += dstep) cp_async16_or_zero(dst, col, false);
         };
         for (int j = 0; j < ntiles && !*dead; ++j) {
-            const int st = j % stages, k0 = first + j * BK;
+            const int st = j % stages, k0 = tile_start(j), n = min(BK, (j < kept_tiles ? kept : last + 1) - k0);
+            const int off = j < kept_tiles ? koff_kept : koff;
             if (j >= stages) wait(&empty[st], (j / stages - 1) & 1);
             bf16* kd = ks + st * BK * ld;
             bf16* vd = vs + st * BK * ldv;
-            copy(pk, kd + lane % nd * 8, ld, kcol, p.ldk, k0);
-            copy(pr, kd + p.dim + lane % nr * 8, ld, rcol, p.row, k0);
-            copy(pv, vd + lane % nv * 8, ldv, vcol, p.ldv, k0);
+            copy(pk, kd + lane % nd * 8, ld, kcol, p.ldk, k0, n, off);
+            if (nr > 0) copy(pr, kd + p.dim + lane % nr * 8, ld, rcol, p.row, k0, n, off);
+            copy(pv, vd + lane % nv * 8, ldv, vcol, p.ldv, k0, n, off);
             cp_async_arrive(&full[st]);
         }
         cp_async_wait_all();
@@ -170,8 +182,8 @@ __global__ void __launch_bounds__(PT, 1) latent_prefill_kernel(LatentPrefillPara
         if (*dead) break;
         const bf16* kt = ks + st * BK * ld;
         const bf16* vt = vs + st * BK * ldv;
-        const int k0 = first + j * BK;
-        if (k0 <= wq0 + 15 && k0 + BK - 1 >= wlo && warp * 16 < nq) {                    // the tile meets the warp's range
+        const int k0 = tile_start(j), ke = j < kept_tiles ? kept : last + 1;
+        if (warp * 16 < nq && (j < kept_tiles || (k0 <= wq0 + 15 && (k0 + BK - 1 >= wlo || k0 < p.keep_first)))) {      // it meets the warp's rows
             float s[BK / 8][4];
 #pragma unroll
             for (int n = 0; n < BK / 8; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
@@ -186,7 +198,8 @@ __global__ void __launch_bounds__(PT, 1) latent_prefill_kernel(LatentPrefillPara
                     mma_bf16_16816(s[2 * n + 1], a, b[2], b[3]);
                 }
             }
-            const bool whole = k0 + BK - 1 <= wq0 && k0 >= wlo + 15;
+            const int kl = k0 + BK - 1;                    // every row of the warp sees every key of the tile
+            const bool whole = kl < ke && kl <= wq0 && (k0 >= wlo + 15 || kl < p.keep_first);
             float x0 = m0, x1 = m1;
             if (whole) {
 #pragma unroll
@@ -195,12 +208,14 @@ __global__ void __launch_bounds__(PT, 1) latent_prefill_kernel(LatentPrefillPara
                     for (int i = 0; i < 4; ++i) s[n][i] *= scale_log2;
                 }
             } else {
+                const int hi0 = min(p0, ke - 1), hi1 = min(p1, ke - 1);
 #pragma unroll
                 for (int n = 0; n < BK / 8; ++n) {
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
                         const int key = k0 + n * 8 + 2 * c4 + (i & 1);
-                        const bool in = i < 2 ? (key <= p0 && key >= lo0) : (key <= p1 && key >= lo1);
+                        const bool in = i < 2 ? (key <= hi0 && (key >= lo0 || key < p.keep_first))
+                                              : (key <= hi1 && (key >= lo1 || key < p.keep_first));
                         s[n][i] = in ? s[n][i] * scale_log2 : -INFINITY;
                     }
                 }
@@ -253,8 +268,8 @@ __global__ void __launch_bounds__(PT, 1) latent_prefill_kernel(LatentPrefillPara
     for (int i = 0; i < NT; ++i) {
         const int d = i * 8 + 2 * c4;
         if (d >= p.vdim) break;
-        if (r0 < nq) *reinterpret_cast<uint32_t*>(p.out + ((size_t)(q0 + r0) * p.heads + h) * p.vdim + d) = f2_to_bf162(acc[i][0] * i0, acc[i][1] * i0);
-        if (r1 < nq) *reinterpret_cast<uint32_t*>(p.out + ((size_t)(q0 + r1) * p.heads + h) * p.vdim + d) = f2_to_bf162(acc[i][2] * i1, acc[i][3] * i1);
+        if (r0 < nq) *reinterpret_cast<uint32_t*>(p.out + (size_t)(q0 + r0) * p.ldo + (size_t)h * p.vdim + d) = f2_to_bf162(acc[i][0] * i0, acc[i][1] * i0);
+        if (r1 < nq) *reinterpret_cast<uint32_t*>(p.out + (size_t)(q0 + r1) * p.ldo + (size_t)h * p.vdim + d) = f2_to_bf162(acc[i][2] * i1, acc[i][3] * i1);
     }
 }
 
@@ -435,27 +450,32 @@ SL_API int sl_latent_gather(const LatentGatherParams* p, int B, int longest, cud
     return SL_LAUNCH_CHECK();
 }
 
-// 1 when the tensor-core kernels take these sizes.
+// 1 when portion_attn_kernel takes these sizes.
+SL_API int sl_portion_attn_ok(int dim, int rot_dim, int vdim) {
+    if (dim < 8 || rot_dim < 0 || vdim < 8 || dim % 8 != 0 || rot_dim % 8 != 0 || vdim % 8 != 0 || vdim > 256 || dim + rot_dim > 256) return 0;
+    return prefill_smem(dim + rot_dim, value_tiles(vdim), 2) <= SMEM_MAX;
+}
+
+// 1 when the tensor-core kernels of latent attention take these sizes.
 SL_API int sl_latent_mma_ok(int dim, int rot_dim, int vdim, int rank) {
-    if (dim < 8 || rot_dim < 8 || dim % 8 != 0 || rot_dim % 8 != 0 || vdim % 8 != 0 || rank % 8 != 0 || vdim > 256 || dim + rot_dim > 256) return 0;
-    if (prefill_smem(dim + rot_dim, value_tiles(vdim), 2) > SMEM_MAX) return 0;
-    return rank <= 1024 && decode_smem(rank + rot_dim) <= SMEM_MAX;
+    return sl_portion_attn_ok(dim, rot_dim, vdim) && rank >= 8 && rank % 8 == 0 && rank <= 1024 && decode_smem(rank + rot_dim) <= SMEM_MAX;
 }
 
 // `heads` of the launch are h0 .. h0 + group - 1.
-SL_API int sl_latent_prefill(const LatentPrefillParams* args, int group, int tiles, cudaStream_t s) {
-    LatentPrefillParams params = *args;
-    LatentPrefillParams* p = &params;
+SL_API int sl_portion_attn(const PortionAttnParams* args, int group, int tiles, cudaStream_t s) {
+    PortionAttnParams params = *args;
+    PortionAttnParams* p = &params;
     if (group == 0 || tiles == 0) return 0;
-    if (!sl_latent_mma_ok(p->dim, p->rot_dim, p->vdim, p->rank) || tiles > 65535) return -1;
-    if (((uintptr_t)p->k | (uintptr_t)p->v | (uintptr_t)p->rows | (uintptr_t)p->q | (uintptr_t)p->q_rot) % 16 != 0) return -1;
-    if (p->ldq % 8 != 0 || p->q_head % 8 != 0 || p->ldk % 8 != 0 || p->ldv % 8 != 0 || p->row % 8 != 0) return -1;
+    if (!sl_portion_attn_ok(p->dim, p->rot_dim, p->vdim) || tiles > 65535 || p->kv_group < 1) return -1;
+    if (((uintptr_t)p->k | (uintptr_t)p->v | (uintptr_t)p->q) % 16 != 0 || ((uintptr_t)p->out | (uintptr_t)(p->ldo * 2)) % 4 != 0) return -1;
+    if (p->rot_dim > 0 && (((uintptr_t)p->rows | (uintptr_t)p->q_rot) % 16 != 0 || p->row % 8 != 0 || p->rank % 8 != 0)) return -1;
+    if (p->ldq % 8 != 0 || p->q_head % 8 != 0 || p->ldk % 8 != 0 || p->ldv % 8 != 0) return -1;
     const int nt = value_tiles(p->vdim), dq = p->dim + p->rot_dim;
     p->stages = prefill_stages(dq, nt);
     const size_t smem = prefill_smem(dq, nt, p->stages);
 #define SL_LP(NT)                                                                                                       \
     {                                                                                                                   \
-        auto kern = latent_prefill_kernel<NT>;                                                                          \
+        auto kern = portion_attn_kernel<NT>;                                                                          \
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                             \
         sl_launch(kern, dim3(group, tiles), PT, smem, s, *p);                                                          \
     }

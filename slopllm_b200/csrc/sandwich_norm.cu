@@ -1,6 +1,7 @@
 // Residual stream of decoders that normalise a sublayer's output before it is added ("sandwich" norms):
 //
-//   residual' = residual + rms(y) * w_post          (y: the sublayer's output, fp32; absent in front of the first sublayer)
+//   residual' = residual + rms(y) * w_post          (y: the sublayer's output, fp32; absent in front of the first sublayer;
+//                                                    without w_post it is added as it is)
 //   out       = rms(residual') * w_next             (input of the next sublayer, or of the output head)
 //
 // in one pass over the token's row, which stays in registers between the two reductions.  The first call of a step gathers
@@ -13,7 +14,7 @@ struct PostNormParams {
     void* out; int out_f32;          // [T, H]
     float* res_out;                  // [T, H]
     const float* y; int ldy;         // [T, ldy] or null
-    const float* w_post;             // [H] (with y)
+    const float* w_post;             // [H] or null (with y)
     const float* res_in;             // [T, H] or null: gathered from `table`
     const long long* ids; const void* table; int table_f32, vocab;
     const float* w_next;             // [H]
@@ -89,10 +90,15 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(PostNormParams p) {
         wn[i] = ld<VW>(p.w_next + c, in);
         if (p.y != nullptr) {
             y[i] = ld<VW>(p.y + (size_t)t * p.ldy + c, in);
-            wp[i] = ld<VW>(p.w_post + c, in);
+            if (p.w_post != nullptr) wp[i] = ld<VW>(p.w_post + c, in);
         }
     }
-    if (p.y != nullptr) {
+    if (p.y != nullptr && p.w_post == nullptr) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+#pragma unroll
+            for (int j = 0; j < VW; ++j) r[i].v[j] += y[i].v[j];
+    } else if (p.y != nullptr) {
         float ss = 0.f;
 #pragma unroll
         for (int i = 0; i < NV; ++i)

@@ -1,0 +1,85 @@
+// Depthwise causal convolution over time with silu, parallel over tokens:
+//
+//   y[t, c] = silu(sum_j w[j, c] x[t - (taps-1) + j, c])
+//
+// Inputs before the token range of a sequence come from its ring, state[slot][p % taps][c] = input of position p (zeros before
+// the start).  The block of a range's first tokens also stores the range's last inputs: a thread reads what it needs of its
+// channel before it overwrites it, and no other block touches the ring, so one launch suffices.
+#include "common.cuh"
+
+namespace {
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void put(float* p, float v) { *p = v; }
+__device__ __forceinline__ void put(bf16* p, float v) { *p = __float2bfloat16(v); }
+
+constexpr int CHUNK = 32;        // tokens per block
+
+// grid (ceil(C / 128), ceil(longest / CHUNK), B), block 128: a thread per channel.  taps <= MAXT.
+template <int MAXT, typename TI, typename TO>
+__global__ void __launch_bounds__(128) short_conv_kernel(TO* __restrict__ y, const TI* __restrict__ x, int ldx, const float* __restrict__ w,
+                                                         float* __restrict__ state, const int* __restrict__ positions,
+                                                         const int* __restrict__ qo_indptr, const int* __restrict__ state_idx, int C, int taps) {
+    pdl_grid_sync();
+    const int c = blockIdx.x * 128 + threadIdx.x, seq = blockIdx.z;
+    const int lo = qo_indptr[seq], hi = qo_indptr[seq + 1], t0 = lo + blockIdx.y * CHUNK, t1 = min(hi, t0 + CHUNK);
+    if (c >= C || t0 >= t1) return;
+    float* ring = state + (size_t)state_idx[seq] * taps * C + c;
+    const int start = positions[lo];
+    float win[MAXT], wt[MAXT];
+#pragma unroll
+    for (int j = 0; j < MAXT; ++j) {
+        wt[j] = j < taps ? w[(size_t)j * C + c] : 0.f;
+        win[j] = 0.f;
+        const int t = t0 - (taps - 1) + j;                         // win[j] is the input of token t
+        if (j < taps - 1) {
+            const int p = start + t - lo;
+            if (t >= lo) win[j] = to_f(x[(size_t)t * ldx + c]);
+            else if (p >= 0) win[j] = ring[(size_t)(p % taps) * C];
+        }
+    }
+    for (int t = t0; t < t1; t += 8) {
+        float in[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) in[i] = t + i < t1 ? to_f(x[(size_t)(t + i) * ldx + c]) : 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            if (t + i >= t1) break;
+            float a = 0.f;
+#pragma unroll
+            for (int j = 0; j < MAXT; ++j) {
+                if (j == taps - 1) win[j] = in[i];
+                a += wt[j] * win[j];
+            }
+            put(y + (size_t)(t + i) * C + c, a / (1.f + expf(-a)));
+#pragma unroll
+            for (int j = 0; j + 1 < MAXT; ++j) win[j] = win[j + 1];
+        }
+    }
+    if (blockIdx.y == 0)
+        for (int t = max(lo, hi - taps); t < hi; ++t) ring[(size_t)((start + t - lo) % taps) * C] = to_f(x[(size_t)t * ldx + c]);
+}
+
+}  // namespace
+
+// y [T, C], x [T, ldx], w fp32 [taps, C], state fp32 [slots, taps, C].
+SL_API int sl_short_conv(void* y, const void* x, int ldx, const void* w, void* state, const void* positions, const void* qo_indptr,
+                         const void* state_idx, int B, int longest, int C, int taps, int in_f32, int out_f32, cudaStream_t s) {
+    if (B == 0 || longest == 0 || C == 0) return 0;
+    if (taps < 1 || taps > 16 || B > 65535 || (longest + CHUNK - 1) / CHUNK > 65535 || (out_f32 && !in_f32)) return -1;
+    const dim3 grid((C + 127) / 128, (longest + CHUNK - 1) / CHUNK, B);
+#define SL_CONV(M, TI, TO)                                                                                                            \
+    sl_launch(short_conv_kernel<M, TI, TO>, grid, 128, 0, s, (TO*)y, (const TI*)x, ldx, (const float*)w, (float*)state, (const int*)positions, \
+              (const int*)qo_indptr, (const int*)state_idx, C, taps)
+#define SL_CONV_T(M)                                \
+    {                                               \
+        if (out_f32) SL_CONV(M, float, float);      \
+        else if (in_f32) SL_CONV(M, float, bf16);   \
+        else SL_CONV(M, bf16, bf16);                \
+    }
+    if (taps <= 4) SL_CONV_T(4) else if (taps <= 8) SL_CONV_T(8) else SL_CONV_T(16)
+#undef SL_CONV_T
+#undef SL_CONV
+    return SL_LAUNCH_CHECK();
+}

@@ -232,12 +232,7 @@ class GidisunModel(DecoderStack):
 
 def load_gidisun_model(model_dir: str, ctx: Optional[ParallelContext] = None, dtype=torch.bfloat16):
     """(cfg, model) from a directory of config.json and safetensors shards."""
-    from ..checkpoint.safetensors_io import SafetensorsFile, iter_dir
+    from ..checkpoint.safetensors_io import load_dir
     with open(os.path.join(model_dir, "config.json")) as f:
         cfg = GidisunConfig.from_dict(json.load(f))
-    tensors: Dict[str, torch.Tensor] = {}
-    for path in iter_dir(model_dir):
-        sf = SafetensorsFile(path)
-        for name in sf.names():
-            tensors[name] = sf.tensor(name)
-    return cfg, GidisunModel.from_tensors(cfg, tensors, ctx, dtype)
+    return cfg, GidisunModel.from_tensors(cfg, load_dir(model_dir), ctx, dtype)

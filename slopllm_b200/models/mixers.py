@@ -5,15 +5,19 @@ projection completes in the caller's all-reduce).  Every size and constant is a 
 from __future__ import annotations
 
 from dataclasses import dataclass
+from typing import Optional, Union
 
 import torch
 
 from ..kv.hybrid import CacheSpec
+from ..ops import delta as DL
+from ..ops import experts as EX
+from ..ops import grouped as G
 from ..ops import latent as L
 from ..ops import recurrent as RC
 from ..ops.rotary import RotaryTable
 from ..utils.tracing import traced
-from .weights import LinearWeight
+from .weights import ExpertWeights, LinearWeight
 
 SMALL_T = 32         # up to this many rows a layer's input projections are one fp32-output product (weight streaming)
 
@@ -33,13 +37,17 @@ class LatentAttention:
     def spec(self) -> CacheSpec:
         return CacheSpec(rows={"latent": (self.shape.row,)})
 
+    fp32_rows = False                # `mix` takes the projection in the activation type only
+
+    def mix(self, model, qd, fine, st, cache, out=None):
+        """Up to the output projection, from the rows of `w_in`."""
+        rows = cache.rows[self.index]["latent"]
+        q_rot = L.latent_pre(qd, self.shape, self.w, self.rot, st, rows)
+        return L.latent_attention(qd, q_rot, self.shape, self.w, st, rows, model.ops, out)
+
     @traced(lambda self, *a, **k: f"layer{self.index}.latent_attention")
     def __call__(self, model, x, st, cache):
-        rows = cache.rows[self.index]["latent"]
-        qd = model.ops.linear(x, self.w_in)
-        q_rot = L.latent_pre(qd, self.shape, self.w, self.rot, st, rows)
-        o = L.latent_attention(qd, q_rot, self.shape, self.w, st, rows, model.ops)
-        return model.ops.linear(o, self.o_proj, out_f32=True)
+        return model.ops.linear(self.mix(model, model.ops.linear(x, self.w_in), None, st, cache), self.o_proj, out_f32=True)
 
 
 class _GatedRecurrence:
@@ -112,3 +120,104 @@ class MLstm(_GatedRecurrence):
         o = RC.mlstm_mix(proj, gates, self.i_b, self.f_b, self.cap, self.norm, self.eps, (s["S"], s["n"], s["m"]), qo, sidx,
                          self.heads, self.dk, self.dv, x.dtype, RC.ChunkPlan.of(st))
         return model.ops.linear(o, self.o_proj, out_f32=True)
+
+
+@dataclass
+class GroupedAttention:
+    """Grouped-query attention with query / key norm, rotation, sliding window with kept first tokens and sink
+    (`ops/grouped.py`).  Projection rows: q | k (| v)."""
+
+    index: int
+    shape: G.GroupedShape
+    rot: RotaryTable
+    w: G.GroupedWeights
+
+    fp32_rows = True
+
+    @property
+    def spec(self) -> CacheSpec:
+        s = self.shape
+        return CacheSpec(rows={"k": (s.kv_heads, s.dim), "v": (s.kv_heads, s.vdim)})
+
+    def mix(self, model, main, fine, st, cache, out):
+        rows = cache.rows[self.index]
+        q = G.grouped_pre(main, self.shape, self.w, self.rot, st, rows["k"], rows["v"], out.dtype)
+        G.grouped_attention(q, self.shape, self.w, st, rows["k"], rows["v"], out)
+
+
+@dataclass
+class ChannelDelta:
+    """Gated delta rule with a decay per key channel behind short convolutions (`ops/delta.py`).  Projection rows: q | k | v, and
+    with fp32 results low-rank decay input | low-rank gate input | beta."""
+
+    index: int
+    shape: DL.DeltaShape
+    w: DL.DeltaWeights
+
+    fp32_rows = True
+
+    @property
+    def spec(self) -> CacheSpec:
+        s = self.shape
+        return CacheSpec(state={"S": (s.heads, s.dk, s.dv), "conv": (s.taps, s.channels)})
+
+    def mix(self, model, main, fine, st, cache, out):
+        state = cache.state[self.index]
+        qo, sidx = model.scan_ranges(st)
+        DL.channel_delta_mix(main, fine, self.shape, self.w, state["S"], state["conv"], st, qo, sidx, out, model.ops, RC.ChunkPlan.of(st))
+
+
+@dataclass
+class Experts:
+    """Softmax-routed SwiGLU experts (`ops/experts.py`); the router's logits come from the caller's projection."""
+
+    w: ExpertWeights
+    top: int
+    groups: int = 1
+    keep: int = 1
+
+    def add(self, model, x, logits, out):
+        ids, wts = EX.route_softmax(logits, self.top, self.groups, self.keep)
+        EX.add_experts(x, self.w, ids, wts, out, model.ops)
+
+
+@dataclass
+class ParallelBlock:
+    """A mixer and a feed-forward that read the same normed input and whose outputs are added: one input product makes the rows of
+    both, one output product takes the mixer's result and the activation side by side; routed experts add to its result.
+
+    `w_in` rows: mixer | gate | up (dense feed-forward) and then, with fp32 results, the mixer's fine rows | router."""
+
+    index: int
+    kind: str
+    mixer: Union[LatentAttention, GroupedAttention, ChannelDelta]
+    w_in: LinearWeight
+    w_out: LinearWeight
+    main: int                        # mixer rows
+    out: int                         # values the mixer hands to `w_out`
+    ff: int = 0                      # width of the dense feed-forward
+    fine: int = 0                    # the mixer's fine rows
+    experts: Optional[Experts] = None
+
+    @property
+    def spec(self) -> CacheSpec:
+        return self.mixer.spec
+
+    @traced(lambda self, *a, **k: f"layer{self.index}.{self.kind}")
+    def __call__(self, model, x, st, cache):
+        ops, T, m, w = model.ops, x.shape[0], self.main + 2 * self.ff, self.w_in.weight
+        if w.shape[0] == m:
+            main, fine = ops.linear(x, self.w_in), None
+        elif w.dtype == torch.float32 or (T <= SMALL_T and self.mixer.fp32_rows):
+            y = ops.linear(x, self.w_in, out_f32=True)
+            main, fine = y[:, :m], y[:, m:]
+        else:
+            main, fine = ops.linear(x, LinearWeight(w[:m])), ops.linear(x, LinearWeight(w[m:]), out_f32=True)
+        both = torch.empty(T, self.out + self.ff, dtype=x.dtype, device=x.device)
+        self.mixer.mix(model, main[:, :self.main], fine, st, cache, both[:, :self.out])
+        if self.ff:
+            ops.silu_mul(main[:, self.main:], both[:, self.out:])
+        y = ops.linear(both, self.w_out, out_f32=True)
+        if self.experts is not None:
+            self.experts.add(model, x, fine[:, self.fine:], y)
+        return y

@@ -1,5 +1,5 @@
 """The decoder loop and the engine hooks shared by the model families whose layers are mixer + feed-forward sublayers over a
-:class:`~slopllm_b200.kv.hybrid.HybridCache`: Qwen3 / Qwen3.5 (`models/dense.py`) and Gidisun (`models/gidisun.py`).
+:class:`~slopllm_b200.kv.hybrid.HybridCache`: Qwen3 / Qwen3.5 (`models/dense.py`), Gidisun (`models/gidisun.py`) and Zemezen (`models/zemezen.py`).
 
 A family builds a flat list of :class:`Sublayer`; the loop runs  x -> run(norm(x)) -> [post norm] -> residual add -> next norm
 with the residual in fp32, and completes the tensor-parallel partial sums in between.
@@ -40,6 +40,7 @@ class DecoderStack:
 
     sublayers: List[Sublayer]
     specs: List[CacheSpec]
+    fp32_norms = False        # norm weights are fp32 although no sublayer has a post norm
 
     def _init_stack(self, ctx: ParallelContext, ops, comm: Optional[Comm], cache_dtype) -> None:
         self.ctx, self.ops, self.comm = ctx, ops, comm or Comm(ctx)
@@ -77,13 +78,13 @@ class DecoderStack:
 
     def _enter(self, st, norm):
         ops, eps = self.ops, self.cfg.rms_norm_eps
-        if self.sublayers[0].post_norm is not None:
+        if self.fp32_norms or self.sublayers[0].post_norm is not None:
             return ops.embed_norm(st.input_ids, self.w.embed, norm, eps)
         return ops.add_rmsnorm(ops.embed(st.input_ids, self.w.embed), None, norm, eps)
 
     def _join(self, y, residual, sub: Sublayer, norm):
         ops, eps = self.ops, self.cfg.rms_norm_eps
-        if sub.post_norm is not None:
+        if self.fp32_norms or sub.post_norm is not None:
             return ops.post_norm(self.comm.all_reduce(y), residual, sub.post_norm, norm, eps)
         return self.comm.allreduce_add_rmsnorm(ops, y, residual, norm, eps)
 

@@ -44,7 +44,7 @@ class RefOps:
         return R.rmsnorm(r, w_next, eps), r
 
     def post_norm(self, y, residual, w_post, w_next, eps):
-        r = residual + R.rmsnorm(y, w_post, eps)
+        r = residual + (y if w_post is None else R.rmsnorm(y, w_post, eps))
         return R.rmsnorm(r, w_next, eps), r
 
     def linear(self, x, w, out_f32: bool = False, sink=None, defer_reduce: bool = False):
@@ -118,6 +118,9 @@ class RefOps:
     # -- MLP ------------------------------------------------------------------------------------
     def dense_mlp(self, x, lw, sink=None):
         return R.linear(R.silu_mul(R.linear(x, lw.mlp_w13)), lw.mlp_w2)
+
+    def silu_mul(self, gate_up, out):
+        out.copy_(R.silu_mul(gate_up))
 
     def route(self, x, lw):
         c = self.cfg

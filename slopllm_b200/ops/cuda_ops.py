@@ -109,11 +109,12 @@ class CudaOps:
                                table_f32=int(table.dtype == torch.float32), vocab=table.shape[0])
 
     def post_norm(self, y, residual, w_post, w_next, eps):
-        """residual' = residual + rms(y) * w_post; returns (rms(residual') * w_next, residual').  fp32 weights and sums."""
+        """residual' = residual + rms(y) * w_post (w_post None: + y); returns (rms(residual') * w_next, residual').  fp32 weights
+        and sums."""
         if y.dtype != torch.float32 or y.stride(-1) != 1:
             y = y.to(torch.float32).contiguous()
         T, H = y.shape
-        return self._post_norm(T, H, w_next, eps, y.device, y=y.data_ptr(), ldy=y.stride(0), w_post=w_post.data_ptr(),
+        return self._post_norm(T, H, w_next, eps, y.device, y=y.data_ptr(), ldy=y.stride(0), w_post=N.ptr(w_post),
                                res_in=residual.data_ptr())
 
     @staticmethod
@@ -467,7 +468,7 @@ class CudaOps:
             out._sl_perm = perm
         return out
 
-    def _head_batched_gemm(self, a, a_stride: int, K: int, owner, w):
+    def _head_batched_gemm(self, a, a_stride: int, K: int, owner, w, out=None):
         """out[t, h * n + j] = sum_k a[t, h * a_stride + k] * W[h, k, j] on the persistent tcgen05 GEMM (`W` [heads, K, n];
         its output-major copy [heads * n, K] is made once and kept on the tensor's owner).  None when the shape is not one
         the tile walk takes.  Replaces the library bmm of the absorb and value-expansion steps of a prefill chunk
@@ -489,9 +490,10 @@ class CudaOps:
             else:
                 w._sl_out_major = wt
         T = a.shape[0]
-        out = torch.empty(T, heads * n, dtype=torch.bfloat16, device=a.device)
+        if out is None:
+            out = torch.empty(T, heads * n, dtype=torch.bfloat16, device=a.device)
         N.call("sl_gemm_bf16_tcgen05_batched", a.data_ptr(), wt.data_ptr(), out.data_ptr(), T, heads, n, K, a.stride(0), a_stride,
-               K, heads * n, 0, tcgen05.error_flag(a.device).data_ptr(), N.stream())
+               K, out.stride(0), 0, tcgen05.error_flag(a.device).data_ptr(), N.stream())
         return out
 
     def v_expand(self, o, w_v):
@@ -517,6 +519,12 @@ class CudaOps:
         act = torch.empty(T, I2 // 2, dtype=gu.dtype, device=x.device)
         N.call("sl_silu_mul_f32" if gu.dtype == torch.float32 else "sl_silu_mul", act.data_ptr(), gu.data_ptr(), T, I2 // 2, N.stream())
         return self.linear(act, lw.mlp_w2, out_f32=True, sink=sink)
+
+    def silu_mul(self, gate_up, out):
+        """out = silu(gate) * up for gate_up [T, 2I] = gate | up and out [T, I], rows of any stride."""
+        T, I = out.shape
+        N.call("sl_silu_mul_rows", out.data_ptr(), out.stride(0), gate_up.data_ptr(), gate_up.stride(0), T, I,
+               int(gate_up.dtype == torch.float32), int(out.dtype == torch.float32), N.stream())
 
     def route(self, x, lw):
         c = self.cfg

@@ -159,11 +159,11 @@ def experts_fp4(experts, xq3, plan, out_kind: int = OUT_BF16) -> torch.Tensor:
     return fp4.grouped_gemm_fp4(experts.w2, sf2, experts.g2, aq, sfa, ga, plan, experts.hidden, False, out_kind)
 
 
-def moe_large(ops, x, experts, shared, ids, wts) -> torch.Tensor:
+def moe_large(ops, x, experts, shared, ids, wts, out=None) -> torch.Tensor:
     """Expert MLP for many tokens: routes sorted by expert on the device, gate/up and down as grouped GEMMs over
     the sorted rows (NVFP4 experts: weights expanded inside the GEMM; otherwise bf16 weights, expanded in groups
     that bound the transient copy), SiLU·mul in between, weighted un-sort into the shared expert's result.
-    Returns fp32 [T, H] (this rank's partial sum)."""
+    Returns fp32 [T, H] (this rank's partial sum); `out` (fp32 [T, H], contiguous): what the experts are added to."""
     T, H = x.shape
     k = ids.shape[1]
     E, I = experts.num_experts, experts.inter
@@ -182,7 +182,9 @@ def moe_large(ops, x, experts, shared, ids, wts) -> torch.Tensor:
     wts = wts.to(torch.float32).contiguous()
     use_fp4 = fp4_moe_ok(experts, H) and xb.stride(-1) == 1
     # the shared expert writes the fp32 result first, the routed experts accumulate into it
-    out = _shared_expert_large(xb, shared, use_fp4) if shared is not None else None
+    if shared is not None:
+        base, out = out, _shared_expert_large(xb, shared, use_fp4)
+        out = out if base is None else out + base
     if out is not None and (out.stride(0) != H or out.dtype != torch.float32):
         out = out.to(torch.float32).contiguous()
     acc = 0 if out is None else 1

@@ -41,11 +41,12 @@ class LatentGatherParams(C.Structure):
                 ("page_table", C.c_void_p), ("pt_stride", C.c_int), ("page_size", C.c_int), ("guard", C.c_void_p)]
 
 
-class LatentPrefillParams(C.Structure):
+class PortionAttnParams(C.Structure):
     _fields_ = [("q", C.c_void_p), ("ldq", C.c_int), ("q_head", C.c_int), ("q_rot", C.c_void_p), ("k", C.c_void_p), ("ldk", C.c_int),
                 ("v", C.c_void_p), ("ldv", C.c_int), ("rows", C.c_void_p), ("row", C.c_int), ("rank", C.c_int), ("tiles", C.c_void_p),
-                ("heads", C.c_int), ("h0", C.c_int), ("dim", C.c_int), ("rot_dim", C.c_int), ("vdim", C.c_int), ("window", C.c_int),
-                ("scale", C.c_float), ("sink", C.c_void_p), ("out", C.c_void_p), ("err", C.c_void_p), ("stages", C.c_int)]
+                ("heads", C.c_int), ("h0", C.c_int), ("dim", C.c_int), ("rot_dim", C.c_int), ("vdim", C.c_int), ("kv_group", C.c_int),
+                ("window", C.c_int), ("keep_first", C.c_int), ("scale", C.c_float), ("sink", C.c_void_p), ("out", C.c_void_p),
+                ("ldo", C.c_int), ("err", C.c_void_p), ("stages", C.c_int)]
 
 
 class LatentDecodeParams(C.Structure):
@@ -107,41 +108,45 @@ def latent_pre(qd: torch.Tensor, s: LatentShape, w: LatentWeights, rot: RotaryTa
     return rot.apply(qd[:, :s.heads * qs].reshape(T, s.heads, qs)[..., s.dim:], st.positions).to(qd.dtype)
 
 
-def head_product(x: torch.Tensor, x_head: int, w: torch.Tensor, ops) -> torch.Tensor:
-    """out[t, h * n + j] = sum_k x[t, h * x_head + k] w[h, k, j] for every head (w [heads, K, n])."""
+def head_product(x: torch.Tensor, x_head: int, w: torch.Tensor, ops, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out[t, h * n + j] = sum_k x[t, h * x_head + k] w[h, k, j] for every head (w [heads, K, n]); `out`: rows of any stride."""
     N = _native()
     T, (h, K, n) = x.shape[0], w.shape
-    if w.dtype == torch.bfloat16 and x.stride(0) % 8 == 0 and n % 8 == 0 and x_head % 8 == 0:
+    if w.dtype == torch.bfloat16 and x.stride(0) % 8 == 0 and n % 8 == 0 and x_head % 8 == 0 and (out is None or out.stride(0) % 8 == 0):
         if T > 32:
-            out = ops._head_batched_gemm(x, x_head, K, None, w)
-            if out is not None:
-                return out
-        out = torch.empty(T, h * n, dtype=torch.bfloat16, device=x.device)
-        N.call("sl_bmv", out.data_ptr(), x.data_ptr(), w.data_ptr(), T, h, K, n, x.stride(0), x_head, 0, 0, N.stream())
-        return out
-    out = torch.empty(T, h * n, dtype=w.dtype, device=x.device)
-    p = N.SimtLinearParams(y=out.data_ptr(), x=x.data_ptr(), w=w.data_ptr(), T=T, N=n, K=K, batch=h, y_t=h * n, y_b=n, x_t=x.stride(0),
+            o = ops._head_batched_gemm(x, x_head, K, None, w, out)
+            if o is not None:
+                return o
+        if out is None or out.is_contiguous():
+            out = torch.empty(T, h * n, dtype=torch.bfloat16, device=x.device) if out is None else out
+            N.call("sl_bmv", out.data_ptr(), x.data_ptr(), w.data_ptr(), T, h, K, n, x.stride(0), x_head, 0, 0, N.stream())
+            return out
+    out = torch.empty(T, h * n, dtype=w.dtype, device=x.device) if out is None else out
+    p = N.SimtLinearParams(y=out.data_ptr(), x=x.data_ptr(), w=w.data_ptr(), T=T, N=n, K=K, batch=h, y_t=out.stride(0), y_b=n, x_t=x.stride(0),
                            x_b=x_head, w_n=1, w_k=n, w_b=K * n)
     N.call("sl_linear_simt", C.byref(p), int(w.dtype == torch.float32), int(w.dtype == torch.float32), N.stream())
     return out
 
 
-def latent_attention(qd: torch.Tensor, q_rot: torch.Tensor, s: LatentShape, w: LatentWeights, st, cache: torch.Tensor, ops=None) -> torch.Tensor:
+def latent_attention(qd: torch.Tensor, q_rot: torch.Tensor, s: LatentShape, w: LatentWeights, st, cache: torch.Tensor, ops=None,
+                     out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of every token row over the cached rows of its sequence that its window shows.  The unrotated queries are
-    read from the projection rows `qd`.  Returns [T, heads * vdim]."""
+    read from the projection rows `qd`.  Returns [T, heads * vdim] (`out`, rows of any stride, when given)."""
     T, qs = qd.shape[0], s.dim + s.rot_dim
+    if out is None:
+        out = torch.empty(T, s.heads * s.vdim, dtype=qd.dtype, device=qd.device)
     if qd.is_cuda:
         N = _native()
-        mma = qd.dtype == torch.bfloat16 and qd.stride(0) % 8 == 0 and N.fn("sl_latent_mma_ok")(s.dim, s.rot_dim, s.vdim, s.rank)
+        mma = (qd.dtype == torch.bfloat16 and qd.stride(0) % 8 == 0 and qd.data_ptr() % 16 == 0 and out.stride(0) % 8 == 0
+               and N.fn("sl_latent_mma_ok")(s.dim, s.rot_dim, s.vdim, s.rank))
         if mma and "spans" in st.extra:
-            return latent_prefill(qd, q_rot, s, w, st, cache, ops)
+            return latent_prefill(qd, q_rot, s, w, st, cache, ops, out)
         q_abs = head_product(qd, qs, w.uk, ops)
         if mma:
-            return latent_decode(q_abs, q_rot, s, w, st, cache, ops)
+            return latent_decode(q_abs, q_rot, s, w, st, cache, ops, out)
         o = latent_rows(q_abs, q_rot, s, w, st, cache)
-        return head_product(o.view(T, s.heads * s.rank), s.rank, w.uv_t, ops)
+        return head_product(o.view(T, s.heads * s.rank), s.rank, w.uv_t, ops, out)
     q = qd[:, :s.heads * qs].reshape(T, s.heads, qs)[..., :s.dim].to(torch.float32)
-    out = torch.empty(T, s.heads, s.vdim, dtype=torch.float32)
     for t in range(T):
         pos = int(st.positions[t])
         kp = torch.arange(max(0, pos - s.window + 1) if s.window else 0, pos + 1)
@@ -152,48 +157,71 @@ def latent_attention(qd: torch.Tensor, q_rot: torch.Tensor, s: LatentShape, w: L
         if w.sink is not None:
             sc = torch.cat([sc, w.sink.view(-1, 1)], -1)
         p = torch.softmax(sc, -1)[:, :kp.numel()]
-        out[t] = torch.einsum("hvr,hr->hv", w.uv.to(torch.float32), p @ c)
-    return out.reshape(T, s.heads * s.vdim).to(qd.dtype)
+        out[t] = torch.einsum("hvr,hr->hv", w.uv.to(torch.float32), p @ c).reshape(-1).to(out.dtype)
+    return out
 
 
 class PortionPlan:
-    """Key ranges and query tiles of a step's portions for one window size, on the device."""
+    """Key ranges and query tiles of a step's portions for one window size and number of kept first tokens, on the device.  A
+    sequence's visible rows are gathered as its kept rows (those in front of the window) followed by the window's."""
 
-    def __init__(self, spans, window: int, device):
+    def __init__(self, spans, window: int, keep_first: int, device):
         ranges, tiles = [], []
         row = tok = 0
         for b, (start, n) in enumerate(spans):
             lo = max(0, start - window + 1) if window else 0
-            ranges.append((b, lo, start + n - lo, row))
-            tiles += [(tok + o, min(QUERY_TILE, n - o), start + o, row - lo) for o in range(0, n, QUERY_TILE)]
-            row += start + n - lo
+            kept = min(keep_first, lo)
+            if kept:
+                ranges.append((b, 0, kept, row))
+            ranges.append((b, lo, start + n - lo, row + kept))
+            tiles += [(tok + o, min(QUERY_TILE, n - o), start + o, row + kept - lo, row) for o in range(0, n, QUERY_TILE)]
+            row += kept + start + n - lo
             tok += n
-        self.batch, self.tile_count, self.rows, self.longest = len(ranges), len(tiles), row, max(r[2] for r in ranges)
+        self.range_count, self.tile_count, self.rows, self.longest = len(ranges), len(tiles), row, max(r[2] for r in ranges)
         t = torch.tensor([x for r in ranges + tiles for x in r], dtype=torch.int32, device=device)
-        self.ranges, self.tiles = t[:4 * self.batch], t[4 * self.batch:]
+        self.ranges, self.tiles = t[:4 * len(ranges)], t[4 * len(ranges):]
 
     @staticmethod
-    def of(st, window: int) -> "PortionPlan":
+    def of(st, window: int, keep_first: int = 0) -> "PortionPlan":
         plans = st.extra.setdefault("portion_plans", {})
-        if window not in plans:
-            plans[window] = PortionPlan(st.extra["spans"], window, st.input_ids.device)
-        return plans[window]
+        key = (window, keep_first)
+        if key not in plans:
+            plans[key] = PortionPlan(st.extra["spans"], window, keep_first, st.input_ids.device)
+        return plans[key]
 
 
-def latent_prefill(qd, q_rot, s: LatentShape, w: LatentWeights, st, cache, ops) -> torch.Tensor:
+def gather_rows(cache: torch.Tensor, plan: PortionPlan, st) -> torch.Tensor:
+    """The bf16 cache rows [slots, row] that a step's portions can see, copied out of the pages in the plan's order."""
+    N = _native()
+    from . import tcgen05
+    rows = torch.empty(plan.rows, cache.shape[1], dtype=torch.bfloat16, device=cache.device)
+    gp = LatentGatherParams(out=rows.data_ptr(), cache=cache.data_ptr(), num_slots=cache.shape[0], row=cache.shape[1], ranges=plan.ranges.data_ptr(),
+                            page_table=st.page_table.data_ptr(), pt_stride=st.page_table.stride(0), page_size=st.page_size,
+                            guard=tcgen05.error_flag(cache.device).data_ptr() + 16)
+    N.call("sl_latent_gather", C.byref(gp), plan.range_count, plan.longest, N.stream())
+    return rows
+
+
+def portion_attention(q, q_head: int, q_rot, k, v, plan: PortionPlan, out, *, heads: int, h0: int, group: int, dim: int, vdim: int,
+                      scale: float, sink=None, kv_group: int = 1, window: int = 0, keep_first: int = 0, rot_dim: int = 0, rows=None,
+                      rank: int = 0) -> None:
+    """Attention of heads h0 .. h0 + group - 1 over gathered keys k and values v [rows, ...], into `out` (rows of any stride)."""
+    N = _native()
+    from . import tcgen05
+    p = PortionAttnParams(q=q.data_ptr(), ldq=q.stride(0), q_head=q_head, q_rot=N.ptr(q_rot), k=k.data_ptr(), ldk=k.stride(0),
+                          v=v.data_ptr(), ldv=v.stride(0), rows=N.ptr(rows), row=0 if rows is None else rows.shape[1], rank=rank,
+                          tiles=plan.tiles.data_ptr(), heads=heads, h0=h0, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_group=kv_group,
+                          window=window, keep_first=keep_first, scale=scale, sink=N.ptr(sink), out=out.data_ptr(), ldo=out.stride(0),
+                          err=tcgen05.error_flag(out.device).data_ptr())
+    N.call("sl_portion_attn", C.byref(p), group, plan.tile_count, N.stream())
+
+
+def latent_prefill(qd, q_rot, s: LatentShape, w: LatentWeights, st, cache, ops, out) -> torch.Tensor:
     """Expanded attention of a step's portions: the visible cache rows are copied out of the pages, two GEMMs make the heads'
     keys and values, one kernel attends."""
     from ..models.weights import LinearWeight
-    N = _native()
-    from . import tcgen05
-    T, dev = qd.shape[0], qd.device
     plan = PortionPlan.of(st, s.window)
-    rows = torch.empty(plan.rows, s.row, dtype=torch.bfloat16, device=dev)
-    gp = LatentGatherParams(out=rows.data_ptr(), cache=cache.data_ptr(), num_slots=cache.shape[0], row=s.row, ranges=plan.ranges.data_ptr(),
-                            page_table=st.page_table.data_ptr(), pt_stride=st.page_table.stride(0), page_size=st.page_size,
-                            guard=tcgen05.error_flag(dev).data_ptr() + 16)
-    N.call("sl_latent_gather", C.byref(gp), plan.batch, plan.longest, N.stream())
-    out = torch.empty(T, s.heads * s.vdim, dtype=torch.bfloat16, device=dev)
+    rows = gather_rows(cache, plan, st)
     group = max(1, min(s.heads, EXPAND_BUDGET_BYTES // (plan.rows * (s.dim + s.vdim) * 2)))
     lat = rows[:, :s.rank]
     uk, uv = w.uk.view(s.heads * s.dim, s.rank), w.uv.view(s.heads * s.vdim, s.rank)
@@ -201,19 +229,9 @@ def latent_prefill(qd, q_rot, s: LatentShape, w: LatentWeights, st, cache, ops) 
         hn = min(group, s.heads - h0)
         k = ops.linear(lat, LinearWeight(uk[h0 * s.dim:(h0 + hn) * s.dim]))
         v = ops.linear(lat, LinearWeight(uv[h0 * s.vdim:(h0 + hn) * s.vdim]))
-        latent_prefill_kernel(qd, q_rot, s, w, rows, k, v, plan, h0, hn, out)
+        portion_attention(qd, s.dim + s.rot_dim, q_rot, k, v, plan, out, heads=s.heads, h0=h0, group=hn, dim=s.dim, vdim=s.vdim,
+                          window=s.window, scale=s.scale, sink=w.sink, rot_dim=s.rot_dim, rows=rows, rank=s.rank)
     return out
-
-
-def latent_prefill_kernel(qd, q_rot, s: LatentShape, w: LatentWeights, rows, k, v, plan: PortionPlan, h0: int, heads: int, out) -> None:
-    """Attention of heads h0 .. h0 + heads - 1 over their expanded keys k [rows, heads * dim] and values v [rows, heads * vdim]."""
-    N = _native()
-    from . import tcgen05
-    p = LatentPrefillParams(q=qd.data_ptr(), ldq=qd.stride(0), q_head=s.dim + s.rot_dim, q_rot=q_rot.data_ptr(), k=k.data_ptr(),
-                            ldk=k.stride(0), v=v.data_ptr(), ldv=v.stride(0), rows=rows.data_ptr(), row=s.row, rank=s.rank,
-                            tiles=plan.tiles.data_ptr(), heads=s.heads, h0=h0, dim=s.dim, rot_dim=s.rot_dim, vdim=s.vdim,
-                            window=s.window, scale=s.scale, sink=N.ptr(w.sink), out=out.data_ptr(), err=tcgen05.error_flag(out.device).data_ptr())
-    N.call("sl_latent_prefill", C.byref(p), heads, plan.tile_count, N.stream())
 
 
 def decode_splits(T: int, heads: int, keys: int) -> int:
@@ -222,7 +240,7 @@ def decode_splits(T: int, heads: int, keys: int) -> int:
     return max(1, min(-(-296 // ctas), -(-keys // KEY_TILE), 64))
 
 
-def latent_decode(q_abs, q_rot, s: LatentShape, w: LatentWeights, st, cache, ops) -> torch.Tensor:
+def latent_decode(q_abs, q_rot, s: LatentShape, w: LatentWeights, st, cache, ops, out) -> torch.Tensor:
     """Absorbed attention of one query token per page-table row and the value expansion -> [T, heads * vdim]."""
     N = _native()
     from . import tcgen05
@@ -238,19 +256,18 @@ def latent_decode(q_abs, q_rot, s: LatentShape, w: LatentWeights, st, cache, ops
         o = torch.empty(T, s.heads, s.rank, dtype=torch.bfloat16, device=dev)
         p.o_final = o.data_ptr()
         N.call("sl_latent_decode", C.byref(p), T, N.stream())
-        return head_product(o.view(T, s.heads * s.rank), s.rank, w.uv_t, ops)
+        return head_product(o.view(T, s.heads * s.rank), s.rank, w.uv_t, ops, out)
     o_part = torch.empty(T, s.heads, splits, s.rank, dtype=torch.float32, device=dev)
     lse = torch.empty(T, s.heads, splits, dtype=torch.float32, device=dev)
     p.o_part, p.lse_part = o_part.data_ptr(), lse.data_ptr()
     N.call("sl_latent_decode", C.byref(p), T, N.stream())
     if fused:
-        out = torch.empty(T, s.heads * s.vdim, dtype=torch.bfloat16, device=dev)
         cp = N.CombineExpandParams(o_part=o_part.data_ptr(), lse_part=lse.data_ptr(), w_v=w.uv_t.data_ptr(), y=out.data_ptr(), T=T,
-                                   tpad=T, Hh=s.heads, K=s.rank, N=s.vdim, np=splits)
+                                   tpad=T, Hh=s.heads, K=s.rank, N=s.vdim, np=splits, ldy=out.stride(0))
         N.call("sl_combine_vexpand", C.byref(cp), N.stream())
         return out
     o, _ = ops.combine([o_part], [lse], want_lse=False)
-    return head_product(o.view(T, s.heads * s.rank), s.rank, w.uv_t, ops)
+    return head_product(o.view(T, s.heads * s.rank), s.rank, w.uv_t, ops, out)
 
 
 def latent_rows(q_abs, q_rot, s: LatentShape, w: LatentWeights, st, cache) -> torch.Tensor:

@@ -147,7 +147,7 @@ class CombineParams(C.Structure):
 
 class CombineExpandParams(C.Structure):
     _fields_ = [("o_part", vp), ("lse_part", vp), ("w_v", vp), ("y", vp), ("xp", vp), ("T", i32), ("tpad", i32), ("Hh", i32),
-                ("K", i32), ("N", i32), ("np", i32)]
+                ("K", i32), ("N", i32), ("np", i32), ("ldy", i32)]
 
 
 class MoeGateUpParams(C.Structure):
@@ -216,7 +216,17 @@ _SIGS = {
     "sl_gated_step": [vp, i32, i32, i32, i32, vp],
     "sl_latent_gather": [vp, i32, i32, vp],
     "sl_latent_mma_ok": [i32, i32, i32, i32],
-    "sl_latent_prefill": [vp, i32, i32, vp],
+    "sl_portion_attn_ok": [i32, i32, i32],
+    "sl_portion_attn": [vp, i32, i32, vp],
+    "sl_grouped_pre": [vp, i32, i32, i32, vp],
+    "sl_grouped_rows": [vp, i32, i32, vp],
+    "sl_grouped_decode_ok": [i32, i32],
+    "sl_grouped_decode": [vp, i32, vp],
+    "sl_silu_mul_rows": [vp, i32, vp, i32, i32, i32, i32, i32, vp],
+    "sl_short_conv": [vp, vp, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp],
+    "sl_delta_step": [vp, i32, i32, i32, vp],
+    "sl_route_softmax": [vp, vp, vp, i32, i32, i32, i32, i32, i32, vp],
+    "sl_expert_stream": [vp, i32, vp],
     "sl_latent_decode": [vp, i32, vp],
     "sl_gated_chunk_ok": [i32, i32, i32, i32],
     "sl_gated_chunks": [vp, i32, i32, vp],
