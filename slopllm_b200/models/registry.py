@@ -66,7 +66,7 @@ MODEL_REGISTRY: Dict[str, ModelRegistration] = {
                                  kernel_sources=("elementwise", "gated_chunk", "gated_scan", "gemm_tcgen05", "gemv", "latent_attn", "latent_mma", "linear_simt",
                                                  "sampling", "sandwich_norm", "sparse_mla")),
     "zemezen": ModelRegistration(False, False, False, False, _load_zemezen, float32=True,
-                                 kernel_sources=("delta_step", "elementwise", "gemm_tcgen05", "gemv", "grouped_attn", "latent_attn", "latent_mma",
+                                 kernel_sources=("delta_chunk", "delta_step", "elementwise", "gemm_tcgen05", "gemv", "grouped_attn", "latent_attn", "latent_mma",
                                                  "linear_simt", "moe_sort", "moe_stream", "parallel_block", "sampling", "sandwich_norm",
                                                  "short_conv", "sparse_mla")),
 }

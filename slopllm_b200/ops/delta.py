@@ -102,7 +102,7 @@ def channel_delta_mix(main: torch.Tensor, fine: torch.Tensor, s: DeltaShape, w: 
         portions = "spans" in st.extra
         longest = st.extra.get("max_q", 1)
         x = short_conv(main, w.conv, conv, st.positions, qo_indptr, state_idx, longest, out.dtype) if portions else main
-        if portions and DC.usable(s, plan, out):
+        if portions and DC.usable(s, plan, x, out):
             DC.run(x, fine, s, w, S, qo_indptr, state_idx, out, ops, plan)
             return
         _step(x, fine, s, w, S, None if portions else conv, st, qo_indptr, state_idx, out)

@@ -225,6 +225,8 @@ _SIGS = {
     "sl_silu_mul_rows": [vp, i32, vp, i32, i32, i32, i32, i32, vp],
     "sl_short_conv": [vp, vp, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp],
     "sl_delta_step": [vp, i32, i32, i32, vp],
+    "sl_delta_chunk_ok": [i32, i32],
+    "sl_delta_chunks": [vp, i32, vp],
     "sl_route_softmax": [vp, vp, vp, i32, i32, i32, i32, i32, i32, vp],
     "sl_expert_stream": [vp, i32, vp],
     "sl_latent_decode": [vp, i32, vp],

@@ -100,7 +100,8 @@ class GatedScanParams(C.Structure):
                 ("gates", C.c_void_p), ("ld_gates", C.c_int), ("a2", C.c_void_p), ("a2_b", C.c_void_p), ("rank", C.c_int),
                 ("inv_tau", C.c_float), ("i_b", C.c_void_p), ("f_b", C.c_void_p), ("cap", C.c_float), ("norm_w", C.c_void_p),
                 ("eps", C.c_float), ("S", C.c_void_p), ("n", C.c_void_p), ("m", C.c_void_p), ("qo_indptr", C.c_void_p),
-                ("state_idx", C.c_void_p), ("h", C.c_int), ("dk", C.c_int), ("dv", C.c_int)]
+                ("state_idx", C.c_void_p), ("h", C.c_int), ("dk", C.c_int), ("dv", C.c_int), ("ldg", C.c_int), ("ldo", C.c_int),
+                ("group", C.c_int)]
 
 
 KIND_GLA, KIND_MLSTM = 0, 1
@@ -111,7 +112,8 @@ CHUNK_SCRATCH_BYTES = 96 << 20      # chunk states of one pass (they stay in L2)
 
 class GatedChunkParams(C.Structure):
     _fields_ = [("s", GatedScanParams), ("chunks", C.c_void_p), ("seq_chunks", C.c_void_p), ("c0", C.c_int), ("c1", C.c_int),
-                ("b", C.c_void_p), ("loc", C.c_void_p), ("nloc", C.c_void_p), ("scal", C.c_void_p), ("slab", C.c_int), ("slab_bufs", C.c_int)]
+                ("b", C.c_void_p), ("loc", C.c_void_p), ("nloc", C.c_void_p), ("scal", C.c_void_p), ("u", C.c_void_p),
+                ("unit", C.c_void_p), ("slab", C.c_int), ("slab_bufs", C.c_int)]
 
 
 class ChunkPlan:
@@ -146,7 +148,8 @@ def _gated_params(p_in, h, dk, dv, out, norm_w, eps, qo_indptr, state_idx) -> Ga
     base = p_in.data_ptr()
     return GatedScanParams(out=out.data_ptr(), q=base, k=base + h * dk * esz, v=base + 2 * h * dk * esz,
                            g=base + (2 * h * dk + h * dv) * esz, ld=p_in.stride(0), norm_w=norm_w.data_ptr(), eps=float(eps),
-                           qo_indptr=qo_indptr.data_ptr(), state_idx=state_idx.data_ptr(), h=h, dk=dk, dv=dv)
+                           qo_indptr=qo_indptr.data_ptr(), state_idx=state_idx.data_ptr(), h=h, dk=dk, dv=dv, ldg=p_in.stride(0),
+                           ldo=h * dv, group=1)
 
 
 def _run_gated(kind: int, p: GatedScanParams, proj, out, qo_indptr, plan=None) -> torch.Tensor:

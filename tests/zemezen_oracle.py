@@ -168,3 +168,86 @@ def forward(raw, t, ids, dtype=torch.float32, trace=None):
         if trace is not None:
             trace.append(x)
     return matmul(norm(x, t["final.norm"], eps), t["head"])
+
+
+# ---- small random models --------------------------------------------------------------------------------------------
+
+def _layer(kind, mixer, mlp):
+    return {"type": kind, "mixer": mixer, "mlp": mlp}
+
+
+def dense(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe(count, top, ff, groups=None, keep=None):
+    r = {"experts": count, "top": top}
+    if groups:
+        r["groups"] = {"count": groups, "keep": keep}
+    return {"kind": "moe", "expert": {"ff": ff}, "router": r}
+
+
+def attention_layer(heads=4, kv_heads=2, dim=16, dims=None, base=10000.0, window=9, keep=2, scale=None, mlp=None):
+    return _layer("attention", {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "rot": {"base": base, "dims": dims or dim},
+                                "mask": {"size": window, "keep_first": keep} if window else None,
+                                "scale": scale if scale is not None else dim ** -0.5}, mlp)
+
+
+def latent_layer(heads=3, dim=16, vdim=24, kv_rank=40, scale=None, mlp=None):
+    return _layer("latent_attention", {"heads": heads, "dim": dim, "vdim": vdim, "kv_rank": kv_rank,
+                                       "scale": scale if scale is not None else dim ** -0.5}, mlp)
+
+
+def delta_layer(heads=4, kv_heads=2, dim=16, vdim=24, conv=4, mlp=None):
+    return _layer("channel_delta", {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}, mlp)
+
+
+def config(layers, width=48, vocab=97, eps=1e-5):
+    """A layer given as a number uses that layer's weights."""
+    out = [dict(layers[l], weights_of=l) if isinstance(l, int) else l for l in layers]
+    return {"architecture": "Zemezen", "layers": out, "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
+def random_tensors(raw, seed=0, ranks=(6, 5)):
+    """bf16 checkpoint tensors of a configuration; `ranks`: widths of the low-rank decay and gate.  Norm weights, biases and sinks
+    are spread so that leaving one out or mixing two up shows in the logits."""
+    g = torch.Generator().manual_seed(seed)
+    W, V = raw["width"], raw["vocab"]
+
+    def mat(n, k, gain=1.0):
+        return (torch.randn(n, k, generator=g) * gain * k ** -0.5).to(torch.bfloat16)
+
+    def vec(n, spread, shift=0.0):
+        return (torch.randn(n, generator=g) * spread + shift).to(torch.bfloat16)
+
+    t = {"embed": torch.randn(V, W, generator=g).to(torch.bfloat16), "final.norm": vec(W, 0.3, 1.0), "head": mat(V, W)}
+
+    def feed(p, ff):
+        t[p + "gate"], t[p + "up"], t[p + "down"] = mat(ff, W), mat(ff, W), mat(W, ff)
+
+    for i, layer in enumerate(raw["layers"]):
+        if "weights_of" in layer:
+            continue
+        p, c, mlp = f"l{i}.", layer["mixer"], layer.get("mlp")
+        t[p + "norm1"] = vec(W, 0.3, 1.0)
+        if mlp and mlp["kind"] == "dense":
+            feed(p + "mlp.", mlp["ff"])
+        elif mlp:
+            for e in range(mlp["router"]["experts"]):
+                feed(f"{p}mlp.e{e}.", mlp["expert"]["ff"])
+            t[p + "mlp.router"] = mat(mlp["router"]["experts"], W, 3.0)
+        p, H, D = p + "mix.", c["heads"], c["dim"]
+        if layer["type"] == "attention":
+            t[p + "q"], t[p + "k"], t[p + "o"] = mat(H * D, W), mat(c["kv_heads"] * D, W), mat(W, H * D)
+            t[p + "q.norm"], t[p + "k.norm"], t[p + "sink"] = vec(D, 0.4, 1.5), vec(D, 0.4, 1.5), vec(H, 1.0, 1.0)
+        elif layer["type"] == "latent_attention":
+            R = c["kv_rank"]
+            t[p + "q"], t[p + "dkv"], t[p + "dkv.norm"] = mat(H * D, W, 2.0), mat(R, W), vec(R, 0.3, 1.0)
+            t[p + "uk"], t[p + "uv"], t[p + "o"] = mat(H * D, R), mat(H * c["vdim"], R), mat(W, H * c["vdim"])
+        else:
+            for n, rows in (("q", c["kv_heads"] * D), ("k", c["kv_heads"] * D), ("v", H * c["vdim"])):
+                t[p + n], t[p + n + ".conv"] = mat(rows, W), mat(rows, c["conv"], 1.5)
+            t[p + "b"], t[p + "A_log"], t[p + "norm"] = mat(H, W), vec(H, 0.7, 0.5), vec(c["vdim"], 0.3, 1.0)
+            t[p + "a1"], t[p + "a2"], t[p + "dt_bias"] = mat(ranks[0], W), mat(H * D, ranks[0]), vec(H * D, 1.5, -3.0)
+            t[p + "g1"], t[p + "g2"], t[p + "o"] = mat(ranks[1], W), mat(H * c["vdim"], ranks[1], 2.0), mat(W, H * c["vdim"])
+    return t
