@@ -1,9 +1,11 @@
-"""Prefill and decode throughput of the hybrid families side by side: Gidisun and Qwen3.5 at equal width, heads, head sizes and
-feed-forward, random weights, layers of a real model's size.
+"""Prefill and decode throughput of the hybrid families side by side: Zemezen, Gidisun and Qwen3.5 at equal width, heads, head sizes
+and feed-forward, random weights, layers of a real model's size.
 
     python -m slopllm_b200.cli.hybrid_bench [--sizes small,medium,large] [--batches 1,8,64] [--prompt 4096]
 
-Both stacks have four layers (three recurrent mixers and one attention layer, a feed-forward each).  Every number is device
+Every stack has four layers with a feed-forward each: three recurrent mixers and one attention layer; Zemezen two of its recurrent
+mixers, one windowed and one latent attention layer.  `zemezen_moe` has 32 experts of a quarter of the feed-forward's width in
+every layer, of which a token uses four.  Every number is device
 time (CUDA events, three warm-up runs, a 256 MB write in front of every timed run so that nothing is served from L2); decode is
 a replay of the captured step.  Prints one JSON line; `python bench.py --hybrid [sizes]` prints the same.
 """
@@ -43,7 +45,24 @@ def qwen35_config(size: str):
                        eos_token_ids=[])
 
 
+def zemezen_config(size: str, moe: bool = False):
+    from ..models.zemezen import ZemezenConfig, ZemezenExperts, ZemezenLayer
+    H, ff, h = SIZES[size]
+    attn = {"heads": h, "kv_heads": max(1, h // 8), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "rot": {"base": 1e6, "dims": 128},
+            "mask": {"size": WINDOW, "keep_first": 4}}
+    delta = {"heads": h, "kv_heads": h, "dim": 128, "vdim": 128, "conv": 4}
+    latent = {"heads": h, "dim": 128, "vdim": 128, "kv_rank": 512, "scale": 128 ** -0.5}
+    mlp = (0, ZemezenExperts(32, 4, ff // 4, 4, 2)) if moe else (ff, None)
+    return ZemezenConfig(hidden_size=H, vocab_size=VOCAB, rms_norm_eps=1e-6,
+                         layers=[ZemezenLayer("channel_delta", delta, *mlp), ZemezenLayer("channel_delta", delta, *mlp),
+                                 ZemezenLayer("attention", attn, *mlp), ZemezenLayer("latent_attention", latent, *mlp)])
+
+
 def build(family: str, size: str, ctx):
+    if family in ("zemezen", "zemezen_moe"):
+        from ..models.zemezen import ZemezenModel, random_zemezen_tensors
+        cfg = zemezen_config(size, family == "zemezen_moe")
+        return cfg, ZemezenModel.from_tensors(cfg, random_zemezen_tensors(cfg, 0, 128, device=ctx.device), ctx)
     if family == "gidisun":
         from ..models.gidisun import GidisunModel, random_gidisun_tensors
         cfg = gidisun_config(size)
@@ -86,7 +105,8 @@ def run_arm(family: str, size: str, batches, prompt: int, iters: int, flush) -> 
     st, _, _ = eng._pack([s], [ids])
 
     def prefill():
-        st.extra.pop("chunk_plan", None)
+        for name in ("chunk_plan", "portion_plans"):
+            st.extra.pop(name, None)
         return model.forward_hidden(st, eng.cache)
 
     ms = median_ms(prefill, iters, flush)
@@ -136,7 +156,7 @@ def run(argv=None) -> dict:
     ap.add_argument("--batches", default="1,8,64")
     ap.add_argument("--prompt", type=int, default=4096)
     ap.add_argument("--iters", type=int, default=10)
-    ap.add_argument("--families", default="gidisun,qwen3_5")
+    ap.add_argument("--families", default="zemezen,zemezen_moe,gidisun,qwen3_5")
     args = ap.parse_args(argv)
     torch.cuda.set_device(0)
     flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")

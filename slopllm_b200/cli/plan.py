@@ -29,8 +29,11 @@ def _config(args) -> GlmMoeDsaConfig:
         if model_type == "gidisun":
             from ..models.gidisun import GidisunConfig
             return GidisunConfig.from_dict(raw)
+        if model_type == "zemezen":
+            from ..models.zemezen import ZemezenConfig
+            return ZemezenConfig.from_dict(raw)
         if model_type != "glm_moe_dsa":
-            raise SystemExit(f"plan: the sizing arithmetic covers glm_moe_dsa, qwen3, qwen3_5 and gidisun; {args.model} is {model_type}")
+            raise SystemExit(f"plan: the sizing arithmetic covers glm_moe_dsa, qwen3, qwen3_5, gidisun and zemezen; {args.model} is {model_type}")
         return load_config(model_dir)
     spec = args.random_init or "glm5"
     if spec.startswith("qwen"):
@@ -39,6 +42,9 @@ def _config(args) -> GlmMoeDsaConfig:
     if spec.startswith("gidisun"):
         from ..models.gidisun import GidisunConfig
         return GidisunConfig.tiny()
+    if spec.startswith("zemezen"):
+        from ..models.zemezen import ZemezenConfig
+        return ZemezenConfig.tiny()
     if spec.startswith("glm5"):
         return GlmMoeDsaConfig.glm5(num_layers=int(spec.split(":")[1]) if ":" in spec else 78)
     return GlmMoeDsaConfig.tiny()
@@ -47,7 +53,7 @@ def _config(args) -> GlmMoeDsaConfig:
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="slopllm_b200.cli.plan", description=__doc__.split("\n")[0])
     ap.add_argument("--model", default="", help="checkpoint directory or hub id (only config.json is read)")
-    ap.add_argument("--random-init", default="", help="glm5[:layers], tiny, qwen3, qwen35 or gidisun instead of a checkpoint")
+    ap.add_argument("--random-init", default="", help="glm5[:layers], tiny, qwen3, qwen35, gidisun or zemezen instead of a checkpoint")
     ap.add_argument("--world", type=int, default=1, help="GPUs of one replica")
     ap.add_argument("--cp", action="store_true")
     ap.add_argument("--ep", action="store_true")
@@ -61,8 +67,8 @@ def main(argv=None) -> int:
     args = ap.parse_args(argv)
     cfg = _config(args)
     if not isinstance(cfg, GlmMoeDsaConfig):
-        from ..utils.sizing import plan_dense, plan_gidisun
-        planner = plan_gidisun if cfg.model_type == "gidisun" else plan_dense
+        from ..utils.sizing import plan_dense, plan_gidisun, plan_zemezen
+        planner = {"gidisun": plan_gidisun, "zemezen": plan_zemezen}.get(cfg.model_type, plan_dense)
         p = planner(cfg, world=args.world, batch_size=args.batch_size, chunk_size=args.chunk_size, max_pages=args.max_pages,
                        arena_gb=args.arena, device_gb=args.device_gb)
     else:

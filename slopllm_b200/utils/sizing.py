@@ -227,15 +227,71 @@ def gidisun_cache_bytes(cfg, tp: int = 1, elem: int = 2):
 
 def plan_gidisun(cfg, world: int = 1, batch_size: int = 8, chunk_size: int = 8192, max_pages: int = 0, arena_gb: float = 0.0,
                  device_gb: float = 180.0, elem: int = 2, reserve_gb: float = 4.0) -> MemoryPlan:
-    """`plan_memory` for Gidisun (tensor parallel only).  The workspace estimate is the widest layer's rows of one chunk, the
-    recurrent state of every slot, and the transient keys, values and chunk states of a prefill."""
-    weights = gidisun_weight_bytes(cfg, world, elem)
-    page, state = gidisun_cache_bytes(cfg, world, elem)
-    requested = max_pages if max_pages > 0 else batch_size * -(-chunk_size // PAGE_SIZE)
+    """`plan_memory` for Gidisun (tensor parallel only)."""
     row = max(max(3 * l.ff, 6 * l.mixer["heads"] * (l.mixer["dim"] + l.mixer["vdim"])) for l in cfg.layers) // world
+    return _plan_hybrid(cfg, gidisun_weight_bytes(cfg, world, elem), *gidisun_cache_bytes(cfg, world, elem), row, world, batch_size, chunk_size,
+                        max_pages, arena_gb, device_gb, elem, reserve_gb)
+
+
+def _plan_hybrid(cfg, weights: int, page: int, state: int, row: int, world: int, batch_size: int, chunk_size: int, max_pages: int, arena_gb: float,
+                 device_gb: float, elem: int, reserve_gb: float) -> MemoryPlan:
+    """Plan of a model with paged rows and per-sequence states.  The workspace estimate is the widest layer's rows of one chunk
+    (`row` values a token), the recurrent state of every slot, and the transient keys, values and chunk states of a prefill."""
+    requested = max_pages if max_pages > 0 else batch_size * -(-chunk_size // PAGE_SIZE)
     work = chunk_size * (cfg.hidden_size * 12 + row * elem) + state * max(64, batch_size) + (1 << 30)
     budget = int(((arena_gb if arena_gb > 0 else device_gb) - reserve_gb) * GIB)
     fit = max(0, (budget - weights - work) // max(1, page))
     return MemoryPlan(tp=world, cp=1, ep=False, weights_bytes=weights, page_bytes=page, tokens_per_page=PAGE_SIZE,
                       workspace_bytes=work, budget_bytes=budget, max_pages=int(fit), max_tokens=int(fit) * PAGE_SIZE,
                       requested_pages=requested, requested_fits=requested <= fit)
+
+
+# ---- Zemezen --------------------------------------------------------------------------------------------------------------
+
+def zemezen_weight_bytes(cfg, tp: int = 1, elem: int = 2, low_rank: int = 16) -> int:
+    """Per-rank weight bytes, as :func:`gidisun_weight_bytes`; experts are sharded like a feed-forward, a layer that uses another's
+    weights has none.  `low_rank`: width of the decay and gate projections (tensor shapes, not in the configuration)."""
+    H = cfg.hidden_size
+    b = cfg.vocab_size * H * elem + (cfg.vocab_size // tp) * H * elem + 4 * H
+    for l in cfg.layers:
+        if l.weights_of is not None:
+            continue
+        c, h, dk = l.mixer, l.mixer["heads"] // tp, l.mixer["dim"]
+        kv, dv = c.get("kv_heads", c["heads"]) // tp, c.get("vdim", dk)
+        b += 4 * H + h * dv * H * elem + 3 * (l.ff // tp) * H * elem
+        if l.experts is not None:
+            b += l.experts.count * (3 * (l.experts.ff // tp) + 1) * H * elem
+        if l.type == "attention":
+            b += (h + kv) * dk * H * elem + 4 * (2 * dk + h)
+        elif l.type == "latent_attention":
+            R = c["kv_rank"]
+            b += (h * dk + R) * H * elem + h * (dk + 2 * dv) * R * elem + 4 * R                       # (values in two layouts)
+        else:
+            rows = 2 * kv * dk + h * dv
+            b += (rows + 2 * low_rank + h) * H * elem + h * (dk + dv) * low_rank * elem + 4 * (rows * c["conv"] + h * dk + h + dv)
+    return b
+
+
+def zemezen_cache_bytes(cfg, tp: int = 1, elem: int = 2):
+    """(bytes of one 64-token page, bytes of one sequence's recurrent state) on one rank."""
+    page = state = 0
+    for l in cfg.layers:
+        c = l.mixer
+        if l.type == "attention":
+            page += 2 * (c["kv_heads"] // tp) * c["dim"] * elem * PAGE_SIZE
+        elif l.type == "latent_attention":
+            page += c["kv_rank"] * elem * PAGE_SIZE
+        else:
+            h, kv = c["heads"] // tp, c["kv_heads"] // tp
+            state += 4 * (h * c["dim"] * c["vdim"] + c["conv"] * (2 * kv * c["dim"] + h * c["vdim"]))
+    return page, state
+
+
+def plan_zemezen(cfg, world: int = 1, batch_size: int = 8, chunk_size: int = 8192, max_pages: int = 0, arena_gb: float = 0.0,
+                 device_gb: float = 180.0, elem: int = 2, reserve_gb: float = 4.0) -> MemoryPlan:
+    """`plan_memory` for Zemezen (tensor parallel only)."""
+    def width(l):
+        experts = 0 if l.experts is None else l.experts.top * (3 * l.experts.ff + 2 * cfg.hidden_size * world)
+        return max(3 * l.ff, experts) + 8 * l.mixer["heads"] * (l.mixer["dim"] + l.mixer.get("vdim", l.mixer["dim"]))
+    return _plan_hybrid(cfg, zemezen_weight_bytes(cfg, world, elem), *zemezen_cache_bytes(cfg, world, elem), max(width(l) for l in cfg.layers) // world,
+                        world, batch_size, chunk_size, max_pages, arena_gb, device_gb, elem, reserve_gb)
