@@ -82,11 +82,11 @@ def time_op(fn: Callable[[], object], iters: int, flush: torch.Tensor) -> float:
 
 def mixer_rows(emit, tokens, iters: int, flush, peaks, dev, h: int = 16, dk: int = 128, dv: int = 128, rank: int = 512, rot: int = 64,
                window: int = 1024, context: int = 2048, n_kv: int = 4) -> None:
-    """Token mixers of the hybrid families at 16 heads of 128: GLA, mLSTM and latent attention beside Gated DeltaNet and paged
-    grouped-query attention.  More than 64 tokens: one prompt; fewer: that many sequences of `context` tokens decode one each."""
+    """Token mixers of the hybrid families at 16 heads of 128: channel-wise delta rule, windowed grouped-query attention, GLA, mLSTM and
+    latent attention beside Gated DeltaNet and paged grouped-query attention.  More than 64 tokens: one prompt; fewer: that many sequences of `context` tokens decode one each."""
     import types
     from ..models.glm_moe_dsa import StepState
-    from ..ops import dense as D, get_ops, latent as L, recurrent as RC
+    from ..ops import delta as DL, dense as D, get_ops, grouped as G, latent as L, recurrent as RC
     from ..ops.rotary import rotary_table
     ops = get_ops(types.SimpleNamespace(rms_norm_eps=1e-6), dev)
     g = torch.Generator(device=dev).manual_seed(3)
@@ -122,6 +122,33 @@ def mixer_rows(emit, tokens, iters: int, flush, peaks, dev, h: int = 16, dk: int
         qkv, ab = bf(T, h * (2 * dk + dv)), bf(T, h)
         us = time_op(lambda: RC.gdn_scan(qkv, ab, ab, ib, fb, S, qo, sidx, h, dk, dv), iters, flush)
         emit(roofline_row("gdn (scan alone)", T, us, T * h * (2 * dk + 2 * dv) * 2 + 2 * B * h * dk * dv * 4, flops, peaks))
+        # gated delta rule with a decay per key channel (low ranks of 128, four taps)
+        ds = DL.DeltaShape(h, h, dk, dv, 4, 1e-6)
+        dw = DL.DeltaWeights(rnd(4, ds.channels), bf(h * dk, 128, k=0.09), bf(h * dv, 128, k=0.09), rnd(h * dk) - 3, rnd(h) * 0.5, nw)
+        dmain, fine, ring = (bf if prompt else rnd)(T, ds.channels), rnd(T, 256 + h), torch.zeros(B, 4, ds.channels, device=dev)
+        dout = bf(T, h * dv)
+        us = time_op(lambda: DL.channel_delta_mix(dmain, fine, ds, dw, S, ring, st, qo, sidx, dout, ops, plan), iters, flush)
+        low = 2.0 * T * 128 * h * (dk + dv)
+        emit(roofline_row("channel_delta (convolutions, low-rank gates, recurrence)", T, us,
+                          T * ds.channels * (2 if prompt else 4) + T * (256 + h) * 4 + T * h * dv * 2 + 2 * B * h * dk * dv * 4 + h * (dk + dv) * 256
+                          + (0 if prompt else 2 * B * ds.channels * 16), 3 * flops / 2 + low, peaks))
+        if prompt:
+            us = time_op(lambda: DL.short_conv(dmain, dw.conv, ring, st.positions, qo, sidx, T, torch.bfloat16), iters, flush)
+            emit(roofline_row("short_conv", T, us, 4.0 * T * ds.channels, 0.0, peaks))
+            cw, cs = bf(ds.channels, 4), torch.zeros(B, ds.channels, 3, device=dev)
+            us = time_op(lambda: RC.causal_conv1d(dmain, cw, None, cs, qo, sidx), iters, flush)
+            emit(roofline_row("causal_conv1d (sequential)", T, us, 4.0 * T * ds.channels, 0.0, peaks))
+        # windowed grouped-query attention whose values are its keys
+        gs = G.GroupedShape(h, n_kv, 128, 128, 128 ** -0.5, window, 4, 1e-6, own_values=False)
+        gw = G.GroupedWeights(rnd(128), rnd(128), rnd(h))
+        gproj, gk, gv, gout = (bf if prompt else rnd)(T, (h + n_kv) * 128), bf(B * width * 64, n_kv, 128), bf(B * width * 64, n_kv, 128), bf(T, h * 128)
+        table = rotary_table(128, 1e6).to(dev)
+        us = time_op(lambda: G.grouped_pre(gproj, gs, gw, table, st, gk, gv, torch.bfloat16), iters, flush)
+        emit(roofline_row("grouped_pre", T, us, T * 128 * ((h + n_kv) * (2 if prompt else 4) + 2 * (h + 2 * n_kv)), 0.0, peaks))
+        gq = G.grouped_pre(gproj, gs, gw, table, st, gk, gv, torch.bfloat16)
+        us = time_op(lambda: G.grouped_attention(gq, gs, gw, st, gk, gv, gout), iters, flush)
+        seen = sum(min(start + i + 1, window + 4) for i in range(T)) if prompt else T * min(kv, window + 4)
+        emit(roofline_row("grouped_attention (window)", T, us, 2.0 * (T if prompt else seen) * n_kv * 256 + 4.0 * T * h * 128, 4.0 * seen * h * 128, peaks))
         # attention
         sh = L.LatentShape(h, dk, rot, dv, rank, (dk + rot) ** -0.5, window)
         uv = bf(h, dv, rank, k=rank ** -0.5)
@@ -239,6 +266,24 @@ def main(argv=None) -> int:
             del w, q
     if "mixers" in cases:
         mixer_rows(emit, tokens, args.iters, flush, peaks, dev)
+    if "experts" in cases:
+        # small bf16 experts (softmax routing) of a 2048-wide model, 32 of 2048 and 128 of 768 with 4 and 8 a token
+        from ..models.weights import ExpertWeights
+        from ..ops import experts as EX
+        for E, top, I, Hh in ((32, 4, 2048, 2048), (128, 8, 768, 2048)):
+            r = lambda *s: (torch.randn(*s, device=dev, generator=g) * s[-1] ** -0.5).to(torch.bfloat16)
+            ex = ExpertWeights(r(E, 2 * I, Hh), r(E, Hh, I))
+            for T in tokens:
+                x, z, out = r(T, Hh) * Hh ** 0.5, torch.randn(T, E, device=dev, generator=g), torch.zeros(T, Hh, device=dev)
+                ids, wts = EX.route_softmax(z, top, 4, 2)
+                us = time_op(lambda: EX.route_softmax(z, top, 4, 2), args.iters, flush)
+                emit(roofline_row(f"route_softmax_{E}", T, us, 4.0 * T * E, 0.0, peaks))
+                us = time_op(lambda: EX.add_experts(x, ex, ids, wts, out, ops), args.iters, flush)
+                uniq = int(torch.unique(ids).numel())
+                row = roofline_row(f"experts_{E}x{I}", T, us, uniq * 3 * I * Hh * 2 + T * Hh * 10, 6.0 * T * top * I * Hh, peaks)
+                row["experts_touched"] = uniq
+                emit(row)
+            del ex
     H = cfg.hidden_size
     if "mlp" in cases:
         lw = random_layer(cfg, 0, 0, dev, torch.bfloat16, 0, args.tp_shape, exact=False)

@@ -58,6 +58,8 @@ __global__ void __launch_bounds__(256) delta_step_kernel(DeltaStepParams p) {
             st[i] = on && row < dk ? *reinterpret_cast<const float4*>(S + (size_t)row * dv + c * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
     }
+    // rows of a2 and g2 as 16-byte pieces
+    const bool wide_low = sizeof(TO) == 2 && p.ra % 8 == 0 && p.rg % 8 == 0 && ((uintptr_t)p.a2 | (uintptr_t)p.g2) % 16 == 0;
     const float rate = expf(p.A_log[h]), qscale = 1.f / sqrtf((float)dk);
     for (int t = t_begin; t < t_end; ++t) {
         const TI* q = (const TI*)p.q + (size_t)t * p.ld + hk * dk;
@@ -75,7 +77,10 @@ __global__ void __launch_bounds__(256) delta_step_kernel(DeltaStepParams p) {
                 const int ch = i < dk ? hk * dk + i : i < 2 * dk ? (p.hk + hk) * dk + i - dk : 2 * p.hk * dk + h * dv + i - 2 * dk;
                 float* ring = p.conv + (size_t)slot * p.taps * C + ch;
                 float a = p.conv_w[(size_t)(p.taps - 1) * C + ch] * x;
-                for (int j = 1; j < p.taps && j <= pos; ++j)
+#pragma unroll
+                for (int j = 1; j < 4; ++j)
+                    if (j < p.taps && j <= pos) a += p.conv_w[(size_t)(p.taps - 1 - j) * C + ch] * ring[(size_t)((pos - j) % p.taps) * C];
+                for (int j = 4; j < p.taps && j <= pos; ++j)
                     a += p.conv_w[(size_t)(p.taps - 1 - j) * C + ch] * ring[(size_t)((pos - j) % p.taps) * C];
                 // (nobody reads this row of the ring in this launch, so the heads that share the channel need no order)
                 if (i >= 2 * dk || h % group == 0) ring[(size_t)(pos % p.taps) * C] = x;
@@ -92,15 +97,28 @@ __global__ void __launch_bounds__(256) delta_step_kernel(DeltaStepParams p) {
             ss = warp_sum(ss);
             if (lane == 0) (warp == 0 ? ss_q : ss_k) = ss;
         }
-        for (int i = warp; i < dk + dv; i += 8) {
-            const bool dec = i < dk;
-            const int rank = dec ? p.ra : p.rg;
+        // low-rank decay and gate: four lanes per row
+        for (int i0 = warp * 8; i0 < dk + dv; i0 += 64) {
+            const int i = i0 + (lane >> 2), c4 = lane & 3;
+            const bool dec = i < dk, in = i < dk + dv;
+            const int rank = !in ? 0 : dec ? p.ra : p.rg;
             const TO* w = dec ? (const TO*)p.a2 + (size_t)(h * dk + i) * rank : (const TO*)p.g2 + (size_t)(h * dv + i - dk) * rank;
             const float* x = dec ? slow : slow + p.ra;
             float z = 0.f;
-            for (int j = lane; j < rank; j += 32) z += to_f(w[j]) * x[j];
-            z = warp_sum(z);
-            if (lane == 0) {
+            if (wide_low) {
+#pragma unroll 4
+                for (int j = c4 * 8; j < rank; j += 32) {
+                    const uint4 v = *reinterpret_cast<const uint4*>(w + j);
+                    const float2 a = bf162_to_f2(v.x), b = bf162_to_f2(v.y), c = bf162_to_f2(v.z), d = bf162_to_f2(v.w);
+                    const float4 x0 = *reinterpret_cast<const float4*>(x + j), x1 = *reinterpret_cast<const float4*>(x + j + 4);
+                    z += a.x * x0.x + a.y * x0.y + b.x * x0.z + b.y * x0.w + c.x * x1.x + c.y * x1.y + d.x * x1.z + d.y * x1.w;
+                }
+            } else {
+                for (int j = c4; j < rank; j += 4) z += to_f(w[j]) * x[j];
+            }
+            z += __shfl_xor_sync(0xffffffffu, z, 1);
+            z += __shfl_xor_sync(0xffffffffu, z, 2);
+            if (c4 == 0 && in) {
                 if (dec) sa[i] = expf(-rate * softplus_f(z + p.dt_bias[h * dk + i]));
                 else sg[i - dk] = sigmoid_f(z);
             }

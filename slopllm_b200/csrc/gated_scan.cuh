@@ -12,7 +12,7 @@ __device__ __forceinline__ void put(bf16* p, float v) { *p = __float2bfloat16(v)
 __device__ __forceinline__ float logsigmoid_f(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 
-enum { KIND_GLA = 0, KIND_MLSTM = 1, KIND_DELTA = 2 };
+enum { KIND_GLA = 0, KIND_MLSTM = 1 };
 
 struct GatedScanParams {
     void* out;                            // [T, h * dv]
@@ -25,7 +25,7 @@ struct GatedScanParams {
     float *S, *n, *m;                     // state
     const int* qo_indptr; const int* state_idx;
     int h, dk, dv;
-    int ldg, ldo, group;                  // chunked kernels: row strides of g and out, heads that share a q / k head
+    int ldg, ldo, group;                  // delta rule: row strides of g and out, heads that share a q / k head
 };
 
 }  // namespace

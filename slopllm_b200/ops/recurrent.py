@@ -112,8 +112,7 @@ CHUNK_SCRATCH_BYTES = 96 << 20      # chunk states of one pass (they stay in L2)
 
 class GatedChunkParams(C.Structure):
     _fields_ = [("s", GatedScanParams), ("chunks", C.c_void_p), ("seq_chunks", C.c_void_p), ("c0", C.c_int), ("c1", C.c_int),
-                ("b", C.c_void_p), ("loc", C.c_void_p), ("nloc", C.c_void_p), ("scal", C.c_void_p), ("u", C.c_void_p),
-                ("unit", C.c_void_p), ("slab", C.c_int), ("slab_bufs", C.c_int)]
+                ("b", C.c_void_p), ("loc", C.c_void_p), ("nloc", C.c_void_p), ("scal", C.c_void_p), ("slab", C.c_int), ("slab_bufs", C.c_int)]
 
 
 class ChunkPlan:
@@ -148,8 +147,7 @@ def _gated_params(p_in, h, dk, dv, out, norm_w, eps, qo_indptr, state_idx) -> Ga
     base = p_in.data_ptr()
     return GatedScanParams(out=out.data_ptr(), q=base, k=base + h * dk * esz, v=base + 2 * h * dk * esz,
                            g=base + (2 * h * dk + h * dv) * esz, ld=p_in.stride(0), norm_w=norm_w.data_ptr(), eps=float(eps),
-                           qo_indptr=qo_indptr.data_ptr(), state_idx=state_idx.data_ptr(), h=h, dk=dk, dv=dv, ldg=p_in.stride(0),
-                           ldo=h * dv, group=1)
+                           qo_indptr=qo_indptr.data_ptr(), state_idx=state_idx.data_ptr(), h=h, dk=dk, dv=dv)
 
 
 def _run_gated(kind: int, p: GatedScanParams, proj, out, qo_indptr, plan=None) -> torch.Tensor:
