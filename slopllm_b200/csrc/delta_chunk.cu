@@ -16,8 +16,8 @@
 //   2 delta_scan_kernel     (value columns, head, sequence): carries the fp32 state over the chunks; leaves S_in and U of each
 //   3 delta_output_kernel   (chunk, head): the two products of o, head norm, output gate
 //
-// No exponent is ever positive: e^{b_t - b_s} is taken directly inside 16-token diagonal blocks and through an anchor between the
-// blocks elsewhere (token 31 between the halves, tokens 15 and 47 inside them).  The inverse is fp32: 16 x 16 diagonal blocks by
+// No exponent is ever positive: e^{b_t - b_s} is taken directly inside 8-token diagonal blocks and through an anchor between the
+// blocks elsewhere (token 31 between the halves, tokens 15 and 47 between the quarters, 7, 23, 39 and 55 inside those).  The inverse is fp32: 16 x 16 diagonal blocks by
 // substitution, the others from products of blocks.  Every fp32 operand of a tensor-core product is split into two bf16 terms.
 #include "gated_chunk.cuh"
 
@@ -40,7 +40,12 @@ struct DeltaChunkParams {
     int stages;                              // set by the launcher: chunks of W and keys in shared memory
 };
 
-__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+// max(x, 0) + log(1 + e^-|x|); the series keeps the relative accuracy of small values
+__device__ __forceinline__ float softplus_f(float x) {
+    const float t = __expf(-fabsf(x));
+    const float series = t * (1.f - t * (0.5f - t * (0.33333333f - t * 0.25f)));
+    return fmaxf(x, 0.f) + (t < 0.04f ? series : __logf(1.f + t));
+}
 
 constexpr int LDI = CT + 4, LDP = CT + 8;    // fp32 rows of A and of the inverse, bf16 rows of T and the scores
 
@@ -57,7 +62,7 @@ template <int NP>
 __global__ void __launch_bounds__(256, NP <= 16 ? 2 : 1) delta_prepare_kernel(DeltaChunkParams dp) {
     pdl_grid_sync();
     extern __shared__ __align__(16) unsigned char smraw[];
-    __shared__ int next_pairs;
+    __shared__ int next_work;
     const GatedScanParams& p = dp.s;
     const int ci = blockIdx.x, h = blockIdx.y, hq = h / p.group, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, c4 = lane & 3;
     const int* ch = dp.chunks + (size_t)(dp.c0 + ci) * 4;
@@ -85,7 +90,7 @@ __global__ void __launch_bounds__(256, NP <= 16 ? 2 : 1) delta_prepare_kernel(De
         *reinterpret_cast<float4*>(bs + s * ldb + c) = x;
     }
     if (tid < CT) beta[tid] = tid < n ? sigmoid_f(dp.beta[(size_t)(t0 + tid) * dp.ld_beta + h]) : 0.f;
-    if (tid == 0) next_pairs = 0;
+    if (tid == 0) next_work = 0;
     __syncthreads();
     // running sums: 16 tokens of a channel at a time, then what came before each
     for (int i = tid; i < 4 * dkp; i += 256) {
@@ -136,7 +141,7 @@ __global__ void __launch_bounds__(256, NP <= 16 ? 2 : 1) delta_prepare_kernel(De
     __syncthreads();
     bf16 *ph = dp.pm + base * 2 * CT * CT, *pl = ph + CT * CT;
     if (tid < dk) dp.decay[base * dk + tid] = exp2f(bs[(n - 1) * ldb + tid]);
-    // ---- A and the scores outside the diagonal blocks: 16 x 16 blocks, one per warp ----
+    // ---- A and the scores outside the 16 x 16 diagonal blocks: a block per warp ----
     if (warp < 6) {
         const int bi = warp < 4 ? 2 + (warp >> 1) : warp == 4 ? 1 : 3, bj = warp < 4 ? (warp & 1) : warp == 4 ? 0 : 2;
         const int r0 = bi * 16 + g, r1 = r0 + 8;
@@ -184,14 +189,51 @@ __global__ void __launch_bounds__(256, NP <= 16 ? 2 : 1) delta_prepare_kernel(De
                 *reinterpret_cast<uint32_t*>(pl + r * CT + s) = lo;
             }
     }
-    // ---- diagonal blocks: the 136 pairs s <= r of each, a quad of lanes per pair, eight pairs at a time to whoever is free ----
+    // ---- the rest, to whoever is free: the lower left 8 x 8 quarters of the four diagonal blocks (rows 8 - 15 of a tile), then the
+    //      pairs s <= r of eight 8 x 8 blocks, a quad of lanes per pair ----
     for (;;) {
         int it = 0;
-        if (lane == 0) it = atomicAdd(&next_pairs, 8);
-        it = __shfl_sync(0xffffffffu, it, 0) + g;
-        if (it >= 4 * 136) break;                        // (4 * 136 is a multiple of 8: the same for the whole warp)
-        const int blk = it / 136, x = it % 136, i = x / 17, j = x % 17;              // rows i and 15 - i together have 17 pairs
-        const int r = blk * 16 + (j <= i ? i : 15 - i), s = blk * 16 + (j <= i ? j : j - i - 1);
+        if (lane == 0) it = atomicAdd(&next_work, 1);
+        it = __shfl_sync(0xffffffffu, it, 0);
+        if (it >= 4 + 8 * 36 / 8) break;
+        if (it < 4) {
+            const int r = it * 16 + 8 + g;
+            const float* an = bs + (it * 16 + 7) * ldb;
+            float aa[4] = {}, pp[4] = {};
+            for (int kk = 0; kk < dkp; kk += 16) {
+                uint32_t a[4] = {}, a2[4] = {}, q[4] = {}, q2[4] = {}, bh[2], bl[2];
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    const int s = it * 16 + g, c = kk + c4 * 2 + i * 8;
+                    const float2 o = *reinterpret_cast<const float2*>(an + c);
+                    const float2 b = *reinterpret_cast<const float2*>(bs + r * ldb + c), e = *reinterpret_cast<const float2*>(bs + s * ldb + c);
+                    const float ex = exp2_fast(b.x - o.x), ey = exp2_fast(b.y - o.y);
+                    const float2 x = bf162_to_f2(*reinterpret_cast<const uint32_t*>(ks + r * ldk + c)), y = bf162_to_f2(*reinterpret_cast<const uint32_t*>(qs + r * ldk + c));
+                    split_bf162(x.x * ex, x.y * ey, a[i * 2 + 1], a2[i * 2 + 1]);
+                    split_bf162(y.x * ex, y.y * ey, q[i * 2 + 1], q2[i * 2 + 1]);
+                    const float2 z = bf162_to_f2(*reinterpret_cast<const uint32_t*>(ks + s * ldk + c));
+                    split_bf162(z.x * exp2_fast(o.x - e.x), z.y * exp2_fast(o.y - e.y), bh[i], bl[i]);
+                }
+                mma_bf16_16816(aa, a, bh[0], bh[1]);
+                mma_bf16_16816(pp, q, bh[0], bh[1]);
+                mma_bf16_16816(aa, a, bl[0], bl[1]);
+                mma_bf16_16816(pp, q, bl[0], bl[1]);
+                mma_bf16_16816(aa, a2, bh[0], bh[1]);
+                mma_bf16_16816(pp, q2, bh[0], bh[1]);
+            }
+            const int s = it * 16 + c4 * 2;
+            const float k0 = rk[s], k1 = rk[s + 1], fa = beta[r] * rk[r], fp = rq[r];
+            *reinterpret_cast<float2*>(A + r * LDI + s) = make_float2(aa[2] * fa * k0, aa[3] * fa * k1);
+            uint32_t hi, lo;
+            split_bf162(pp[2] * fp * k0, pp[3] * fp * k1, hi, lo);
+            *reinterpret_cast<uint32_t*>(ph + r * CT + s) = hi;
+            *reinterpret_cast<uint32_t*>(pl + r * CT + s) = lo;
+            *reinterpret_cast<uint32_t*>(ph + (r - 8) * CT + s + 8) = 0;             // (above the diagonal)
+            *reinterpret_cast<uint32_t*>(pl + (r - 8) * CT + s + 8) = 0;
+            continue;
+        }
+        const int y = (it - 4) * 8 + g, blk = y / 36, x = y % 36, i = x / 9, j = x % 9;      // rows i and 7 - i together have 9 pairs
+        const int r = blk * 8 + (j <= i ? i : 7 - i), s = blk * 8 + (j <= i ? j : j - i - 1);
         float a0 = 0.f, a1 = 0.f, p0 = 0.f, p1 = 0.f;
         if (r < n) {
             const bf16 *kr = ks + r * ldk, *qr = qs + r * ldk, *k2 = ks + s * ldk;

@@ -31,9 +31,9 @@ struct DeltaStepParams {
     int h, hk, dk, dv;
 };
 
-// MAXR > 0: dv % 4 == 0 and at most MAXR state rows per thread, in registers.  MAXR == 0: state in global memory.
-template <int MAXR, typename TI, typename TO>
-__global__ void __launch_bounds__(256) delta_step_kernel(DeltaStepParams p) {
+// NT threads.  MAXR > 0: dv % 4 == 0 and at most MAXR state rows per thread, in registers.  MAXR == 0: state in global memory.
+template <int NT, int MAXR, typename TI, typename TO>
+__global__ void __launch_bounds__(NT) delta_step_kernel(DeltaStepParams p) {
     pdl_grid_sync();
     extern __shared__ float sm[];
     __shared__ float scratch[33], ss_q, ss_k;
@@ -42,7 +42,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(DeltaStepParams p) {
     if (t_begin >= t_end) return;
     const int dk = p.dk, dv = p.dv, group = p.h / p.hk, hk = h / group;
     constexpr int VW = MAXR > 0 ? 4 : 1, NR = MAXR > 0 ? MAXR : 1;
-    const int nc = dv / VW, rg = nc >= 256 ? 1 : 256 / nc;          // column groups, row groups that share a column
+    const int nc = dv / VW, rg = nc >= NT ? 1 : NT / nc;          // column groups, row groups that share a column
     const int dkp = (dk + 3) / 4 * 4, dvp = (dv + 3) / 4 * 4;
     float *sq = sm, *sk = sq + dkp, *sa = sk + dkp, *sv = sa + dkp, *sg = sv + dvp, *slow = sg + dvp;
     float* part = slow + (p.ra + p.rg + 3) / 4 * 4;                 // [rg][dv]
@@ -67,9 +67,9 @@ __global__ void __launch_bounds__(256) delta_step_kernel(DeltaStepParams p) {
         const TI* v = (const TI*)p.v + (size_t)t * p.ld + h * dv;
         const float* low = p.low + (size_t)t * p.ld_low;
         __syncthreads();
-        for (int i = tid; i < p.ra + p.rg; i += 256) slow[i] = low[i];
+        for (int i = tid; i < p.ra + p.rg; i += NT) slow[i] = low[i];
         const int pos = p.positions[t];
-        for (int i = tid; i < 2 * dk + dv; i += 256) {
+        for (int i = tid; i < 2 * dk + dv; i += NT) {
             const TI* src = i < dk ? q + i : i < 2 * dk ? k + i - dk : v + i - 2 * dk;
             float x = to_f(*src);
             if (p.conv != nullptr) {
@@ -98,7 +98,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(DeltaStepParams p) {
             if (lane == 0) (warp == 0 ? ss_q : ss_k) = ss;
         }
         // low-rank decay and gate: four lanes per row
-        for (int i0 = warp * 8; i0 < dk + dv; i0 += 64) {
+        for (int i0 = warp * 8; i0 < dk + dv; i0 += NT / 4) {
             const int i = i0 + (lane >> 2), c4 = lane & 3;
             const bool dec = i < dk, in = i < dk + dv;
             const int rank = !in ? 0 : dec ? p.ra : p.rg;
@@ -158,8 +158,8 @@ __global__ void __launch_bounds__(256) delta_step_kernel(DeltaStepParams p) {
             if (on) *reinterpret_cast<float4*>(part + r * dv + c * 4) = o;
         } else {
             for (int pass = 0; pass < 2; ++pass) {
-                for (int c0 = 0; c0 < nc; c0 += 256) {
-                    const int cc = nc >= 256 ? c0 + tid : c, rr = nc >= 256 ? 0 : r;
+                for (int c0 = 0; c0 < nc; c0 += NT) {
+                    const int cc = nc >= NT ? c0 + tid : c, rr = nc >= NT ? 0 : r;
                     if (cc >= nc || rr >= rg) continue;
                     float acc = 0.f, u = 0.f;
                     if (pass == 1) u = sv[cc];                      // (the update, left there by the first pass)
@@ -173,7 +173,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(DeltaStepParams p) {
                 }
                 __syncthreads();
                 if (pass == 0) {
-                    for (int j = tid; j < dv; j += 256) {
+                    for (int j = tid; j < dv; j += NT) {
                         float sum = 0.f;
                         for (int i = 0; i < rg; ++i) sum += part[i * dv + j];
                         sv[j] = beta * (sv[j] - sum * ks) * ks;
@@ -184,7 +184,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(DeltaStepParams p) {
         }
         __syncthreads();
         float ss = 0.f;
-        for (int j = tid; j < dv; j += 256) {
+        for (int j = tid; j < dv; j += NT) {
             float o = 0.f;
             for (int i = 0; i < rg; ++i) o += part[i * dv + j];
             o *= qs;
@@ -193,7 +193,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(DeltaStepParams p) {
         }
         const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)dv + p.eps);
         TO* out = (TO*)p.out + (size_t)t * p.ldo + (size_t)h * dv;
-        for (int j = tid; j < dv; j += 256) put(out + j, part[j] * inv * p.norm_w[j] * sg[j]);
+        for (int j = tid; j < dv; j += NT) put(out + j, part[j] * inv * p.norm_w[j] * sg[j]);
     }
     if (MAXR > 0 && on) {
 #pragma unroll
@@ -212,29 +212,31 @@ SL_API int sl_delta_step(const DeltaStepParams* p, int B, int in_f32, int out_f3
     if (B == 0) return 0;
     if ((out_f32 && !in_f32) || p->dk < 1 || p->dv < 1 || p->hk < 1 || p->h % p->hk != 0 || (p->conv != nullptr && p->taps < 1)) return -1;
     const bool v4 = p->dv % 4 == 0 && p->dv <= 1024;
-    int nc = v4 ? p->dv / 4 : p->dv, rg = nc >= 256 ? 1 : 256 / nc;
-    const int rows = (p->dk + rg - 1) / rg;
-    const int maxr = !v4 ? 0 : rows <= 4 ? 4 : rows <= 8 ? 8 : rows <= 16 ? 16 : 0;
-    if (maxr == 0) {
-        nc = p->dv;
-        rg = nc >= 256 ? 1 : 256 / nc;
-    }
+    auto rows = [&](int threads) { const int nc = p->dv / 4, rg = nc >= threads ? 1 : threads / nc; return (p->dk + rg - 1) / rg; };
+    // as few state rows per thread as two blocks of 512 threads on an SM leave registers for
+    const int threads = v4 && rows(256) > 8 ? 512 : 256, per = v4 ? rows(threads) : 0;
+    const int maxr = !v4 ? 0 : per <= 4 ? 4 : per <= 8 ? 8 : per <= 16 ? 16 : 0;
+    const int nc = maxr > 0 ? p->dv / 4 : p->dv, rg = nc >= threads ? 1 : threads / nc;
     const int low = (p->ra + p->rg + 3) / 4 * 4;
     const size_t smem = (size_t)(3 * ((p->dk + 3) / 4 * 4) + 2 * ((p->dv + 3) / 4 * 4) + low + rg * p->dv) * sizeof(float);
     if (smem > 200 * 1024) return -1;
-#define SL_DS(R, TI, TO)                                                                                           \
+#define SL_DS(N, R, TI, TO)                                                                                        \
     {                                                                                                              \
-        auto kern = delta_step_kernel<R, TI, TO>;                                                                  \
+        auto kern = delta_step_kernel<N, R, TI, TO>;                                                               \
         if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);  \
-        sl_launch(kern, B * p->h, 256, smem, s, *p);                                                               \
+        sl_launch(kern, B * p->h, N, smem, s, *p);                                                                 \
     }
-#define SL_DS_T(R)                                  \
-    {                                               \
-        if (out_f32) SL_DS(R, float, float)         \
-        else if (in_f32) SL_DS(R, float, bf16)      \
-        else SL_DS(R, bf16, bf16)                   \
+#define SL_DS_T(N, R)                                  \
+    {                                                  \
+        if (out_f32) SL_DS(N, R, float, float)         \
+        else if (in_f32) SL_DS(N, R, float, bf16)      \
+        else SL_DS(N, R, bf16, bf16)                   \
     }
-    if (maxr == 4) SL_DS_T(4) else if (maxr == 8) SL_DS_T(8) else if (maxr == 16) SL_DS_T(16) else SL_DS_T(0)
+    if (threads == 512) {
+        if (maxr == 8 || maxr == 4) SL_DS_T(512, 8) else if (maxr == 16) SL_DS_T(512, 16) else SL_DS_T(512, 0)
+    } else {
+        if (maxr == 4) SL_DS_T(256, 4) else if (maxr == 8) SL_DS_T(256, 8) else SL_DS_T(256, 0)
+    }
 #undef SL_DS_T
 #undef SL_DS
     return SL_LAUNCH_CHECK();

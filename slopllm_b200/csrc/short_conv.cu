@@ -78,7 +78,7 @@ __global__ void __launch_bounds__(128) short_conv_kernel(TO* __restrict__ y, con
                 for (int u = 0; u < V; ++u) a.v[u] += wt[j].v[u] * win[j].v[u];
             }
 #pragma unroll
-            for (int u = 0; u < V; ++u) a.v[u] = a.v[u] / (1.f + expf(-a.v[u]));
+            for (int u = 0; u < V; ++u) a.v[u] = sizeof(TO) == 2 ? __fdividef(a.v[u], 1.f + __expf(-a.v[u])) : a.v[u] / (1.f + expf(-a.v[u]));
             store<V>(y + (size_t)(t + i) * C + c, a);
 #pragma unroll
             for (int j = 0; j + 1 < MAXT; ++j) win[j] = win[j + 1];

@@ -7,7 +7,7 @@ import torch
 
 from .recurrent import CHUNK, CHUNK_MIN_Q, GatedScanParams
 
-SCRATCH_BYTES = 192 << 20           # operands and states of the chunks of one pass; longer steps run in several passes
+SCRATCH_BYTES = 256 << 20           # operands and states of the chunks of one pass; longer steps run in several passes
 
 
 class DeltaChunkParams(C.Structure):

@@ -347,7 +347,7 @@ def test_chunk_passes_carry_the_state(monkeypatch):
     from slopllm_b200.ops import delta_chunk as DC
     args, _, _ = delta_case([300, 90], 2, 1, 32, 40, 4, torch.bfloat16, seed=5)
     out = []
-    for budget in (192 << 20, 2 * 2 * DC.scratch_bytes(32, 40)):
+    for budget in (256 << 20, 2 * 2 * DC.scratch_bytes(32, 40)):
         monkeypatch.setattr(DC, "SCRATCH_BYTES", budget)
         out.append(run_delta(args, torch.bfloat16, RC.ChunkPlan([300, 90], "cuda")))
     for a, b in zip(*out):
