@@ -26,14 +26,14 @@ struct DeltaStepParams {
     const float *dt_bias, *A_log, *norm_w;   // [h * dk], [h], [dv]
     float eps, unit_eps;
     float* S;                                // [slots, h, dk, dv]
-    const float* conv_w; float* conv; int taps;      // [taps, C], [slots, taps, C]; conv null: rows are convolved already
+    const float* conv_w; float* conv; int taps;      // [taps, C], [slots, taps, C] (one token per sequence)
     const int* positions; const int* qo_indptr; const int* state_idx;
     int h, hk, dk, dv;
 };
 
-// NT threads.  MAXR > 0: dv % 4 == 0 and at most MAXR state rows per thread, in registers.  MAXR == 0: state in global memory.
-template <int NT, int MAXR, typename TI, typename TO>
-__global__ void __launch_bounds__(NT) delta_step_kernel(DeltaStepParams p) {
+// NT threads.  ONE: one token per sequence, convolutions included (without it rows are convolved already).  MAXR > 0: dv % 4 == 0 and at most MAXR state rows per thread, in registers.  MAXR == 0: state in global memory.
+template <int NT, int MAXR, bool ONE, typename TI, typename TO>
+__global__ void __launch_bounds__(NT, ONE && NT == 512 && MAXR <= 8 ? 2 : 1) delta_step_kernel(DeltaStepParams p) {
     pdl_grid_sync();
     extern __shared__ float sm[];
     __shared__ float scratch[33], ss_q, ss_k;
@@ -51,17 +51,13 @@ __global__ void __launch_bounds__(NT) delta_step_kernel(DeltaStepParams p) {
     const int c = tid % nc, r = tid / nc;
     const bool on = MAXR > 0 && r < rg;
     float4 st[NR];
-    if (MAXR > 0) {
-#pragma unroll
-        for (int i = 0; i < NR; ++i) {
-            const int row = r + i * rg;
-            st[i] = on && row < dk ? *reinterpret_cast<const float4*>(S + (size_t)row * dv + c * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
-        }
-    }
+    // the state is read when the first token's gates are done; until then it travels to L2 and takes no registers
+    if (MAXR > 0)
+        for (int i = tid * 32; i < dk * dv; i += NT * 32) prefetch_l2_line(S + i);
     // rows of a2 and g2 as 16-byte pieces
     const bool wide_low = sizeof(TO) == 2 && p.ra % 8 == 0 && p.rg % 8 == 0 && ((uintptr_t)p.a2 | (uintptr_t)p.g2) % 16 == 0;
     const float rate = expf(p.A_log[h]), qscale = 1.f / sqrtf((float)dk);
-    for (int t = t_begin; t < t_end; ++t) {
+    for (int t = t_begin; ONE ? t == t_begin : t < t_end; ++t) {
         const TI* q = (const TI*)p.q + (size_t)t * p.ld + hk * dk;
         const TI* k = (const TI*)p.k + (size_t)t * p.ld + hk * dk;
         const TI* v = (const TI*)p.v + (size_t)t * p.ld + h * dv;
@@ -72,7 +68,7 @@ __global__ void __launch_bounds__(NT) delta_step_kernel(DeltaStepParams p) {
         for (int i = tid; i < 2 * dk + dv; i += NT) {
             const TI* src = i < dk ? q + i : i < 2 * dk ? k + i - dk : v + i - 2 * dk;
             float x = to_f(*src);
-            if (p.conv != nullptr) {
+            if (ONE) {
                 const int C = 2 * p.hk * dk + p.h * dv;
                 const int ch = i < dk ? hk * dk + i : i < 2 * dk ? (p.hk + hk) * dk + i - dk : 2 * p.hk * dk + h * dv + i - 2 * dk;
                 float* ring = p.conv + (size_t)slot * p.taps * C + ch;
@@ -121,6 +117,13 @@ __global__ void __launch_bounds__(NT) delta_step_kernel(DeltaStepParams p) {
             if (c4 == 0 && in) {
                 if (dec) sa[i] = expf(-rate * softplus_f(z + p.dt_bias[h * dk + i]));
                 else sg[i - dk] = sigmoid_f(z);
+            }
+        }
+        if (MAXR > 0 && t == t_begin) {
+#pragma unroll
+            for (int i = 0; i < NR; ++i) {
+                const int row = r + i * rg;
+                st[i] = on && row < dk ? *reinterpret_cast<const float4*>(S + (size_t)row * dv + c * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
             }
         }
         __syncthreads();
@@ -222,7 +225,7 @@ SL_API int sl_delta_step(const DeltaStepParams* p, int B, int in_f32, int out_f3
     if (smem > 200 * 1024) return -1;
 #define SL_DS(N, R, TI, TO)                                                                                        \
     {                                                                                                              \
-        auto kern = delta_step_kernel<N, R, TI, TO>;                                                               \
+        auto kern = p->conv != nullptr ? delta_step_kernel<N, R, true, TI, TO> : delta_step_kernel<N, R, false, TI, TO>; \
         if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);  \
         sl_launch(kern, B * p->h, N, smem, s, *p);                                                                 \
     }
