@@ -86,7 +86,7 @@ def mixer_rows(emit, tokens, iters: int, flush, peaks, dev, h: int = 16, dk: int
     latent attention beside Gated DeltaNet and paged grouped-query attention.  More than 64 tokens: one prompt; fewer: that many sequences of `context` tokens decode one each."""
     import types
     from ..models.glm_moe_dsa import StepState
-    from ..ops import delta as DL, dense as D, get_ops, grouped as G, latent as L, recurrent as RC
+    from ..ops import delta as DL, delta_chunk as DC, dense as D, get_ops, grouped as G, latent as L, recurrent as RC
     from ..ops.rotary import rotary_table
     ops = get_ops(types.SimpleNamespace(rms_norm_eps=1e-6), dev)
     g = torch.Generator(device=dev).manual_seed(3)
@@ -133,6 +133,10 @@ def mixer_rows(emit, tokens, iters: int, flush, peaks, dev, h: int = 16, dk: int
                           T * ds.channels * (2 if prompt else 4) + T * (256 + h) * 4 + T * h * dv * 2 + 2 * B * h * dk * dv * 4 + h * (dk + dv) * 256
                           + (0 if prompt else 2 * B * ds.channels * 16), 3 * flops / 2 + low, peaks))
         if prompt:
+            zf, gt = rnd(T, h * dk), bf(T, h * dv)
+            us = time_op(lambda: DC.run_chunks(dmain, zf, gt, fine[:, 256:], ds, dw, S, qo, sidx, dout, plan), iters, flush)
+            emit(roofline_row("channel_delta recurrence (3 launches)", T, us, T * (ds.channels * 2 + h * (dk * 4 + dv * 4)) + 2 * h * dk * dv * 4,
+                              3 * flops / 2, peaks))
             us = time_op(lambda: DL.short_conv(dmain, dw.conv, ring, st.positions, qo, sidx, T, torch.bfloat16), iters, flush)
             emit(roofline_row("short_conv", T, us, 4.0 * T * ds.channels, 0.0, peaks))
             cw, cs = bf(ds.channels, 4), torch.zeros(B, ds.channels, 3, device=dev)

@@ -36,13 +36,18 @@ def usable(s, plan, x, out) -> bool:
 def run(x, fine, s, w, S, qo_indptr, state_idx, out, ops, plan) -> None:
     """x bf16 [T, q | k | v channels] behind the convolutions, fine fp32 [T, decay rank | gate rank | heads (beta)]."""
     from ..models.weights import LinearWeight
-    from . import native as N
-    from .delta import UNIT_EPS
-    T, h, dk, dv, dev = x.shape[0], s.heads, s.dk, s.dv, x.device
-    ra, rg, qk = w.a2.shape[1], w.g2.shape[1], s.kv_heads * dk
+    ra, rg = w.a2.shape[1], w.g2.shape[1]
     low = fine[:, :ra + rg].to(torch.bfloat16)
     z = ops.linear(low[:, :ra], LinearWeight(w.a2), out_f32=True)
     gate = ops.linear(low[:, ra:], LinearWeight(w.g2))
+    run_chunks(x, z, gate, fine[:, ra + rg:], s, w, S, qo_indptr, state_idx, out, plan)
+
+
+def run_chunks(x, z, gate, beta, s, w, S, qo_indptr, state_idx, out, plan) -> None:
+    """The recurrence itself: z fp32 [T, heads * dk] (decay input without bias), gate bf16 [T, heads * dv], beta fp32 [T, heads]."""
+    from . import native as N
+    from .delta import UNIT_EPS
+    h, dk, dv, qk = s.heads, s.dk, s.dv, s.kv_heads * s.dk
     if z.stride(0) != h * dk:
         z = z.contiguous()
     per_pass = min(plan.count, max(1, SCRATCH_BYTES // (h * scratch_bytes(dk, dv))))
@@ -50,13 +55,13 @@ def run(x, fine, s, w, S, qo_indptr, state_idx, out, ops, plan) -> None:
     for name, nbytes in scratch_parts(dk, dv).items():
         at_byte[name] = off
         off += per_pass * h * nbytes
-    scratch = torch.empty(off, dtype=torch.uint8, device=dev)
+    scratch = torch.empty(off, dtype=torch.uint8, device=x.device)
     at = lambda i: x.data_ptr() + 2 * i
     sp = GatedScanParams(out=out.data_ptr(), q=at(0), k=at(qk), v=at(2 * qk), g=gate.data_ptr(), ld=x.stride(0), norm_w=w.norm.data_ptr(),
                          eps=s.eps, S=S.data_ptr(), qo_indptr=qo_indptr.data_ptr(), state_idx=state_idx.data_ptr(), h=h, dk=dk, dv=dv,
                          ldg=gate.stride(0), ldo=out.stride(0), group=h // s.kv_heads)
     p = DeltaChunkParams(s=sp, chunks=plan.table.data_ptr(), seq_chunks=plan.seq_chunks.data_ptr(), z=z.data_ptr(), dt_bias=w.dt_bias.data_ptr(),
-                         A_log=w.A_log.data_ptr(), beta=fine.data_ptr() + 4 * (ra + rg), ld_beta=fine.stride(0), unit_eps=UNIT_EPS,
+                         A_log=w.A_log.data_ptr(), beta=beta.data_ptr(), ld_beta=beta.stride(0), unit_eps=UNIT_EPS,
                          **{name: scratch.data_ptr() + o for name, o in at_byte.items()})
     for c0 in range(0, plan.count, per_pass):
         p.c0, p.c1 = c0, min(plan.count, c0 + per_pass)
