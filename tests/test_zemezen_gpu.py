@@ -186,7 +186,7 @@ def test_decode_key_splits():
 
 # ---- latent attention without positions ---------------------------------------------------------------------------------
 
-@pytest.mark.parametrize("heads,dim,vdim,rank", [(3, 16, 24, 40), (2, 128, 128, 512), (5, 32, 80, 64), (2, 24, 136, 264), (3, 12, 20, 36), (17, 64, 32, 128)])
+@pytest.mark.parametrize("heads,dim,vdim,rank", [(3, 16, 24, 40), (2, 128, 128, 512), (5, 40, 88, 64), (2, 24, 136, 264), (3, 12, 20, 36), (17, 64, 32, 128)])
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_latent_attention(heads, dim, vdim, rank, dtype):
     for spans in SPANS + [[(1500, 1), (64, 1)]]:
@@ -376,7 +376,7 @@ def test_a_lost_term_shows():
 
 # ---- routed experts -----------------------------------------------------------------------------------------------------
 
-@pytest.mark.parametrize("E,top,groups,keep", [(12, 3, 3, 2), (1, 1, 1, 1), (40, 6, 8, 3), (9, 4, 3, 2), (64, 8, 1, 1), (256, 8, 8, 4), (300, 5, 100, 2), (1000, 16, 10, 10)])
+@pytest.mark.parametrize("E,top,groups,keep", [(15, 4, 5, 3), (1, 1, 1, 1), (40, 6, 8, 3), (9, 4, 3, 2), (64, 8, 1, 1), (256, 8, 8, 4), (300, 5, 100, 2), (1000, 16, 10, 10)])
 def test_routing(E, top, groups, keep):
     g = gen(E)
     z = torch.randn(37, E + 3, generator=g) * 2
@@ -392,7 +392,7 @@ def test_routing(E, top, groups, keep):
 
 
 @pytest.mark.parametrize("T", [1, 2, 9, 32, 33, 200])
-@pytest.mark.parametrize("E,top,H,I", [(12, 3, 64, 32), (4, 2, 256, 64), (5, 5, 44, 12), (40, 6, 128, 48), (16, 4, 1024, 256)])
+@pytest.mark.parametrize("E,top,H,I", [(11, 3, 64, 32), (4, 2, 256, 64), (5, 5, 44, 12), (40, 6, 128, 48), (16, 4, 1024, 256)])
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_experts(T, E, top, H, I, dtype):
     g = gen(T + E)
