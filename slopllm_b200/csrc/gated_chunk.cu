@@ -8,6 +8,10 @@
 //          S_t^T q_t = e^{m_in - x_t} S_in^T q_t + sum_{s<=t} e^{a_s - x_t} (q_t . k_s) v_s   (n_t . q_t likewise without v)
 //          S_out = e^{m_in - x_C} S_in + e^{M_C - x_C} sum_s (k_s e^{a_s - M_C}) v_s^T
 //
+//   retention  with t, s the places inside the chunk, gamma the head's decay, q and k turned by their positions:
+//          o_t = gamma^{t+1} q_t . S_in + sum_{s<=t} gamma^{t-s} (q_t . k_s) v_s
+//          S_out = gamma^C S_in + sum_s (k_s gamma^{C-1-s}) v_s^T
+//
 // in three launches:
 //   1 chunk_state_kernel   (chunk, head): decays, the chunk's own state contribution
 //   2 chunk_scan_kernel    (elements, head, sequence): carries the fp32 state over the chunks and leaves each chunk's S_in
@@ -15,7 +19,7 @@
 //
 // No exponent is ever positive: the products e^{b_t - b_s} of GLA are taken directly inside 16-token diagonal blocks and
 // through an anchor between the blocks otherwise.  q, k, v come as bf16; every other operand of a tensor-core product (decayed
-// keys and queries, scores, the state) is split into two bf16 terms, so the results keep fp32-like accuracy.
+// keys and queries, turned ones, scores, the state) is split into two bf16 terms, so the results keep fp32-like accuracy.
 #include "gated_chunk.cuh"
 
 namespace {
@@ -129,23 +133,26 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(GatedChunkParams cp) {
             const int s = i / (dk / 4), c = (i % (dk / 4)) * 4;
             *reinterpret_cast<float4*>(cp.b + (size_t)(t0 + s) * (p.h * dk) + h * dk + c) = *reinterpret_cast<const float4*>(fs + s * dk + c);
         }
-    } else if (warp == 0) {
+    } else if (KIND == KIND_MLSTM && warp == 0) {
         mlstm_gates(p, t0, n, h, fs, fs + CT, fs + 2 * CT);
     }
     cp_async_wait<0>();
     __syncthreads();
-    const float top = KIND == KIND_MLSTM ? fs[2 * CT + n - 1] : 0.f;
+    const float top = KIND == KIND_MLSTM ? fs[2 * CT + n - 1] : 0.f, rate = KIND == KIND_RETENTION ? p.decay[p.h + h] : 0.f;
     for (int i = tid; i < CT * (dkp / 2); i += 256) {
         const int s = i / (dkp / 2), c = (i % (dkp / 2)) * 2;
         uint32_t hi = 0, lo = 0;
         if (s < n && c < dk) {
-            const float2 k = bf162_to_f2(*reinterpret_cast<const uint32_t*>(kh + s * ldk + c));
+            float2 k = bf162_to_f2(*reinterpret_cast<const uint32_t*>(kh + s * ldk + c));
+            if (KIND == KIND_RETENTION) k = turned(p, t0 + s, c, k);
             float w0, w1;
             if (KIND == KIND_GLA) {
                 w0 = exp2_fast(fs[(n - 1) * dk + c] - fs[s * dk + c]);
                 w1 = exp2_fast(fs[(n - 1) * dk + c + 1] - fs[s * dk + c + 1]);
-            } else {
+            } else if (KIND == KIND_MLSTM) {
                 w0 = w1 = __expf(fs[s] - top);
+            } else {
+                w0 = w1 = exp2f((float)(n - 1 - s) * rate);
             }
             split_bf162(k.x * w0, k.y * w1, hi, lo);
         }
@@ -225,14 +232,14 @@ __global__ void __launch_bounds__(256) chunk_scan_kernel(GatedChunkParams cp) {
                     d[j] = cp.scal[((size_t)(i - cp.c0) * p.h + h) * 4 + 1];
                 } else {
                     const int* ch = cp.chunks + (size_t)i * 4;
-                    d[j] = cp.b[(size_t)(ch[1] + ch[2] - 1) * (p.h * dk) + h * dk + c];
+                    d[j] = KIND == KIND_RETENTION ? (float)ch[2] * p.decay[p.h + h] : cp.b[(size_t)(ch[1] + ch[2] - 1) * (p.h * dk) + h * dk + c];
                 }
             }
 #pragma unroll
             for (int j = 0; j < U; ++j) {
                 const int i = i0 + j;
                 if (i >= hi) break;
-                float add = 1.f, keep = KIND == KIND_GLA ? exp2f(d[j]) : 1.f;
+                float add = 1.f, keep = KIND == KIND_MLSTM ? 1.f : exp2f(d[j]);
                 if (KIND == KIND_MLSTM) {
                     const float top = fmaxf(m, d[j]);
                     keep = expf(m - top);
@@ -291,7 +298,7 @@ size_t output_smem(int kind, int dk, int dv, int slab, int bufs) {
     const int dkp = (dk + 15) / 16 * 16;
     const size_t slabs = (size_t)bufs * 2 * slab * (dv + 8) * 2, scores = (size_t)2 * CT * LDA * 2;
     size_t b = (size_t)CT * (dkp + 8) * 2 * 2 + (size_t)CT * (dv + 8) * 2 + (slabs > scores ? slabs : scores);
-    b += kind == KIND_GLA ? (size_t)CT * (dkp + 4) * 4 : 0;
+    b += kind == KIND_GLA ? (size_t)CT * (dkp + 4) * 4 : kind == KIND_RETENTION ? (size_t)CT * (dkp + 8) * 2 * 2 : 0;
     return b + (size_t)CT * 12 * 4;
 }
 
@@ -328,7 +335,9 @@ __global__ void __launch_bounds__(OUT_THREADS, NT <= 4 ? 2 : 1) chunk_output_ker
     const int slab = cp.slab, region = max(cp.slab_bufs * 2 * slab * ldv, 2 * CT * LDA);
     float* fs = reinterpret_cast<float*>(slabs + region);
     float* bs = fs;                                      // GLA: [CT][ldb]
-    float* rows = fs + (KIND == KIND_GLA ? CT * ldb : 0);
+    bf16* ql = reinterpret_cast<bf16*>(fs);              // retention: [CT][ldk] low terms of the turned queries and keys
+    bf16* kl = ql + CT * ldk;
+    float* rows = fs + (KIND == KIND_GLA ? CT * ldb : KIND == KIND_RETENTION ? CT * ldk : 0);
     float *ga = rows, *gb = rows + CT, *gx = rows + 2 * CT, *qn = rows + 3 * CT, *nq = rows + 4 * CT, *ssq = rows + 8 * CT;
     const float qscale = rsqrtf((float)dk);
     const size_t base = (size_t)ci * p.h + h;
@@ -363,6 +372,21 @@ __global__ void __launch_bounds__(OUT_THREADS, NT <= 4 ? 2 : 1) chunk_output_ker
     load_rows(ks, ldk, (const bf16*)p.k + (size_t)t0 * p.ld + h * dk, p.ld, n, dk, dkp);
     load_rows(vs, ldv, (const bf16*)p.v + (size_t)t0 * p.ld + h * dv, p.ld, n, dv, dv);
     cp_async_commit();
+    // a token's row, as it was loaded -> turned by its position, high and low terms
+    auto turn_rows = [&](bf16* hi, bf16* lo) {
+        const int per = dkp / 2;
+        for (int i = tid; i < CT * per; i += OUT_THREADS) {
+            const int r = i / per, c = i % per * 2;
+            uint32_t a = 0, b = 0;
+            if (r < n && c < dk) {
+                const float2 x = turned(p, t0 + r, c, bf162_to_f2(*reinterpret_cast<const uint32_t*>(hi + r * ldk + c)));
+                split_bf162(x.x, x.y, a, b);
+            }
+            *reinterpret_cast<uint32_t*>(hi + r * ldk + c) = a;
+            *reinterpret_cast<uint32_t*>(lo + r * ldk + c) = b;
+        }
+    };
+    const float rate = KIND == KIND_RETENTION ? p.decay[p.h + h] : 0.f;
     const float m_in = KIND == KIND_MLSTM ? cp.scal[base * 4 + 2] : 0.f;
     if (KIND == KIND_MLSTM && warp == 0) mlstm_gates(p, t0, n, h, ga, gb, gx);
     cp_async_wait<1>();
@@ -377,6 +401,10 @@ __global__ void __launch_bounds__(OUT_THREADS, NT <= 4 ? 2 : 1) chunk_output_ker
 #pragma unroll
         for (int o = 1; o < 8; o <<= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
         if ((tid & 7) == 0) qn[r] = a;
+        __syncthreads();
+    }
+    if (KIND == KIND_RETENTION) {
+        turn_rows(qs, ql);
         __syncthreads();
     }
     // ---- S_in part: rows of the state in slabs ----
@@ -395,8 +423,9 @@ __global__ void __launch_bounds__(OUT_THREADS, NT <= 4 ? 2 : 1) chunk_output_ker
         }
         for (int kk = 0; kk < rowsn; kk += 16) {
             uint32_t a[4], a2[4];
-            if (KIND == KIND_MLSTM) {
+            if (KIND != KIND_GLA) {
                 ldsm_x4(a, qs + (rt * 16 + (lane & 15)) * ldk + k0 + kk + (lane >> 4) * 8);
+                if (KIND == KIND_RETENTION) ldsm_x4(a2, ql + (rt * 16 + (lane & 15)) * ldk + k0 + kk + (lane >> 4) * 8);
             } else {
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
@@ -414,7 +443,7 @@ __global__ void __launch_bounds__(OUT_THREADS, NT <= 4 ? 2 : 1) chunk_output_ker
                 ldsm_x2_trans(l0, l1, sl + (kk + (lane & 15)) * ldv + (nt0 + i) * 8);
                 mma_bf16_16816(acc[i], a, b0, b1);
                 mma_bf16_16816(acc[i], a, l0, l1);
-                if (KIND == KIND_GLA) mma_bf16_16816(acc[i], a2, b0, b1);
+                if (KIND != KIND_MLSTM) mma_bf16_16816(acc[i], a2, b0, b1);
             }
         }
         if (k0 + cp.slab_bufs * slab < dkp) {
@@ -424,23 +453,28 @@ __global__ void __launch_bounds__(OUT_THREADS, NT <= 4 ? 2 : 1) chunk_output_ker
         }
     }
     float e0 = 1.f, e1 = 1.f;
-    if (KIND == KIND_MLSTM) {
-        e0 = __expf(m_in - gx[r0]) * qscale;
-        e1 = __expf(m_in - gx[r1]) * qscale;
+    if (KIND != KIND_GLA) {
+        e0 = (KIND == KIND_MLSTM ? __expf(m_in - gx[r0]) : exp2f((float)(r0 + 1) * rate)) * qscale;
+        e1 = (KIND == KIND_MLSTM ? __expf(m_in - gx[r1]) : exp2f((float)(r1 + 1) * rate)) * qscale;
 #pragma unroll
         for (int i = 0; i < NT; ++i) { acc[i][0] *= e0; acc[i][1] *= e0; acc[i][2] *= e1; acc[i][3] *= e1; }
     }
     cp_async_wait<0>();
     __syncthreads();                                     // (the scores take the place of the state slabs)
+    if (KIND == KIND_RETENTION) {
+        turn_rows(ks, kl);
+        __syncthreads();
+    }
     // ---- scores of (row tile rt, key tile J = quarter) ----
     {
         const int J = quarter, r0 = rt * 16 + g, r1 = r0 + 8;
         float sc[2][4] = {};
-        if (KIND == KIND_MLSTM ? J <= rt : J < rt) {
+        if (KIND != KIND_GLA ? J <= rt : J < rt) {
             for (int kk = 0; kk < dkp; kk += 16) {
                 uint32_t a[4], a2[4];
-                if (KIND == KIND_MLSTM) {
+                if (KIND != KIND_GLA) {
                     ldsm_x4(a, qs + (rt * 16 + (lane & 15)) * ldk + kk + (lane >> 4) * 8);
+                    if (KIND == KIND_RETENTION) ldsm_x4(a2, ql + (rt * 16 + (lane & 15)) * ldk + kk + (lane >> 4) * 8);
                 } else {
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
@@ -454,10 +488,15 @@ __global__ void __launch_bounds__(OUT_THREADS, NT <= 4 ? 2 : 1) chunk_output_ker
 #pragma unroll
                 for (int t = 0; t < 2; ++t) {
                     const int s = J * 16 + t * 8;
-                    if (KIND == KIND_MLSTM) {
+                    if (KIND != KIND_GLA) {
                         uint32_t b0, b1;
                         ldsm_x2(b0, b1, ks + (s + (lane & 7)) * ldk + kk + ((lane >> 3) & 1) * 8);
                         mma_bf16_16816(sc[t], a, b0, b1);
+                        if (KIND == KIND_RETENTION) {
+                            mma_bf16_16816(sc[t], a2, b0, b1);
+                            ldsm_x2(b0, b1, kl + (s + (lane & 7)) * ldk + kk + ((lane >> 3) & 1) * 8);
+                            mma_bf16_16816(sc[t], a, b0, b1);
+                        }
                     } else {
                         uint32_t bh[2], bl[2];
 #pragma unroll
@@ -475,7 +514,7 @@ __global__ void __launch_bounds__(OUT_THREADS, NT <= 4 ? 2 : 1) chunk_output_ker
                 }
             }
         }
-        if (KIND == KIND_MLSTM || J != rt) {
+        if (KIND != KIND_GLA || J != rt) {
             float sum0 = 0.f, sum1 = 0.f;
 #pragma unroll
             for (int t = 0; t < 2; ++t) {
@@ -485,6 +524,7 @@ __global__ void __launch_bounds__(OUT_THREADS, NT <= 4 ? 2 : 1) chunk_output_ker
                     const int r = i < 2 ? r0 : r1, s = J * 16 + t * 8 + c4 * 2 + (i & 1);
                     float w = qscale;
                     if (KIND == KIND_MLSTM) w *= s < n ? __expf(ga[s] - gx[r]) : 0.f;
+                    if (KIND == KIND_RETENTION) w *= exp2f((float)max(r - s, 0) * rate);
                     v[i] = s <= r ? sc[t][i] * w : 0.f;
                 }
                 sum0 += v[0] + v[1];
@@ -573,7 +613,7 @@ __global__ void __launch_bounds__(OUT_THREADS, NT <= 4 ? 2 : 1) chunk_output_ker
     for (int i = 0; i < NT; ++i) {
         if (i >= ntn) break;
         const int j = (nt0 + i) * 8 + c4 * 2;
-        const float2 w = make_float2(nw[j], nw[j + 1]);
+        const float2 w = KIND == KIND_RETENTION ? make_float2(p.out_scale, p.out_scale) : make_float2(nw[j], nw[j + 1]);
 #pragma unroll
         for (int u = 0; u < 2; ++u) {
             const int r = u ? r1 : r0;
@@ -581,8 +621,8 @@ __global__ void __launch_bounds__(OUT_THREADS, NT <= 4 ? 2 : 1) chunk_output_ker
             const float inv = u ? i1 : i0;
             const float2 gt = bf162_to_f2(*reinterpret_cast<const uint32_t*>((const bf16*)p.g + (size_t)(t0 + r) * p.ld + h * dv + j));
             const float x = 1.f / (1.f + __expf(-gt.x)), y = 1.f / (1.f + __expf(-gt.y));
-            const float gx0 = KIND == KIND_GLA ? gt.x * x : x, gy0 = KIND == KIND_GLA ? gt.y * y : y;
-            *reinterpret_cast<uint32_t*>((bf16*)p.out + ((size_t)(t0 + r) * p.h + h) * dv + j) =
+            const float gx0 = KIND == KIND_MLSTM ? x : gt.x * x, gy0 = KIND == KIND_MLSTM ? y : gt.y * y;
+            *reinterpret_cast<uint32_t*>((bf16*)p.out + (size_t)(t0 + r) * p.ldo + h * dv + j) =
                 f2_to_bf162(acc[i][u * 2] * inv * w.x * gx0, acc[i][u * 2 + 1] * inv * w.y * gy0);
         }
     }
@@ -629,5 +669,7 @@ SL_API int sl_gated_chunk_ok(int kind, int dk, int dv, int rank) {
 SL_API int sl_gated_chunks(const GatedChunkParams* p, int B, int kind, cudaStream_t s) {
     if (B == 0 || p->c1 <= p->c0) return 0;
     if (!sl_gated_chunk_ok(kind, p->s.dk, p->s.dv, p->s.rank) || p->s.ld % 8 != 0 || B > 65535 || p->s.h > 65535) return -1;
+    if (p->s.ldo % 2 != 0 || (uintptr_t)p->s.out % 4 != 0) return -1;
+    if (kind == KIND_RETENTION) return p->s.rot_dims <= p->s.dk && p->s.rot_dims % 2 == 0 ? run_chunks<KIND_RETENTION>(p, B, s) : -1;
     return kind == KIND_GLA ? run_chunks<KIND_GLA>(p, B, s) : kind == KIND_MLSTM ? run_chunks<KIND_MLSTM>(p, B, s) : -1;
 }

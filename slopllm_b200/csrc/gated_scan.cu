@@ -6,8 +6,10 @@
 //          S_t = e^(f_t + m_{t-1} - m_t) S_{t-1} + e^(i_t - m_t) k_t v_t^T,  n_t likewise with k alone
 //          o_t = S_t^T q_t / (max(|n_t . q_t|, e^(-m_t)) + 1e-6)
 //          i = cap tanh((i_raw + b) / cap), f = logsigmoid(cap tanh((f_raw + b) / cap)), one each per head
+//   retention  S_t = gamma S_{t-1} + k_t v_t^T,                o_t = S_t^T q_t
+//          one fixed decay per head; queries and keys turn with their position (adjacent pairs, angles from a table)
 //
-// followed by the head's RMS norm, its weight and an output gate (silu for GLA, sigmoid for mLSTM).  State [slot, h, dk, dv]
+// followed by the head's RMS norm, its weight (none for retention) and an output gate (silu, sigmoid for mLSTM).  State [slot, h, dk, dv]
 // (and n [slot, h, dk], m [slot, h]), gates and accumulation are fp32; q is scaled by dk^-0.5.
 //
 //  * gated_step_kernel: one block per (sequence, head) walks the sequence's tokens with the state in global memory: the decode
@@ -42,7 +44,7 @@ __global__ void __launch_bounds__(256) gated_step_kernel(GatedScanParams p) {
         const TI* k = (const TI*)p.k + (size_t)t * p.ld + h * dk;
         const TI* v = (const TI*)p.v + (size_t)t * p.ld + h * dv;
         const TI* g = (const TI*)p.g + (size_t)t * p.ld + h * dv;
-        float keep = 1.f, add = 1.f;
+        float keep = KIND == KIND_RETENTION ? p.decay[h] : 1.f, add = 1.f;
         if (KIND == KIND_MLSTM) {
             const float* gr = p.gates + (size_t)t * p.ld_gates;
             const float gi = p.cap * tanhf((gr[h] + p.i_b[h]) / p.cap);
@@ -54,6 +56,18 @@ __global__ void __launch_bounds__(256) gated_step_kernel(GatedScanParams p) {
         }
         __syncthreads();
         for (int i = tid; i < dk; i += 256) {
+            if (KIND == KIND_RETENTION) {
+                float2 a = make_float2(to_f(q[i]), 0.f), b = make_float2(to_f(k[i]), 0.f);
+                if (i < p.rot_dims) {
+                    const int e = i & ~1;
+                    a = turned(p, t, e, make_float2(to_f(q[e]), to_f(q[e + 1])));
+                    b = turned(p, t, e, make_float2(to_f(k[e]), to_f(k[e + 1])));
+                    if (i & 1) { a.x = a.y; b.x = b.y; }
+                }
+                sq[i] = a.x * qscale;
+                sk[i] = b.x;
+                continue;
+            }
             sq[i] = to_f(q[i]) * qscale;
             sk[i] = to_f(k[i]);
             if (KIND == KIND_GLA) {
@@ -111,10 +125,10 @@ __global__ void __launch_bounds__(256) gated_step_kernel(GatedScanParams p) {
             ss += o * o;
         }
         const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)dv + p.eps);
-        TO* out = (TO*)p.out + ((size_t)t * p.h + h) * dv;
+        TO* out = (TO*)p.out + (size_t)t * p.ldo + h * dv;
         for (int j = tid; j < dv; j += 256) {
-            const float gg = to_f(g[j]), act = KIND == KIND_GLA ? gg * sigmoid_f(gg) : sigmoid_f(gg);
-            put(out + j, part[j] * inv * nw[j] * act);
+            const float gg = to_f(g[j]), act = KIND == KIND_MLSTM ? sigmoid_f(gg) : gg * sigmoid_f(gg);
+            put(out + j, part[j] * inv * (KIND == KIND_RETENTION ? p.out_scale : nw[j]) * act);
         }
     }
     if (KIND == KIND_MLSTM && tid == 0) p.m[sh] = m;
@@ -137,7 +151,7 @@ int launch_step(const GatedScanParams* p, int B, int in_f32, int out_f32, size_t
 
 }  // namespace
 
-// kind 0: GLA, 1: mLSTM.  in_f32: q, k, v, g rows are fp32 (else bf16); out_f32: `out` and `a2` are fp32 (needs in_f32).
+// kind 0: GLA, 1: mLSTM, 2: retention.  in_f32: q, k, v, g rows are fp32 (else bf16); out_f32: `out` and `a2` are fp32 (needs in_f32).
 SL_API int sl_gated_step(const GatedScanParams* p, int B, int kind, int in_f32, int out_f32, cudaStream_t s) {
     if (B == 0) return 0;
     if ((out_f32 && !in_f32) || p->dk < 1 || p->dv < 1) return -1;
@@ -147,5 +161,7 @@ SL_API int sl_gated_step(const GatedScanParams* p, int B, int kind, int in_f32, 
     if (smem > 200 * 1024) return -1;
     if (kind == KIND_GLA) return v4 ? launch_step<KIND_GLA, 4>(p, B, in_f32, out_f32, smem, s) : launch_step<KIND_GLA, 1>(p, B, in_f32, out_f32, smem, s);
     if (kind == KIND_MLSTM) return v4 ? launch_step<KIND_MLSTM, 4>(p, B, in_f32, out_f32, smem, s) : launch_step<KIND_MLSTM, 1>(p, B, in_f32, out_f32, smem, s);
+    if (kind == KIND_RETENTION && p->rot_dims <= p->dk && p->rot_dims % 2 == 0)
+        return v4 ? launch_step<KIND_RETENTION, 4>(p, B, in_f32, out_f32, smem, s) : launch_step<KIND_RETENTION, 1>(p, B, in_f32, out_f32, smem, s);
     return -1;
 }

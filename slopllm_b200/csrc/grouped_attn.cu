@@ -2,10 +2,15 @@
 // sink, values of their own or the key projections themselves.  (Portions of prompts attend in latent_mma.cu.)
 //
 //  * grouped_pre_kernel: per-head RMS norm and rotate-half of queries and keys; keys and values go into their cache slots.
+//  * grouped_row_pre_kernel: the same step for norms over the whole query / key rows: biases, norms, rotation of adjacent pairs from
+//    a table of angles, a factor per query head, and values that turn with their position.
 //  * grouped_rows_kernel: independent token rows on the CUDA cores, any sizes, bf16 or fp32.
 //  * grouped_decode_kernel: one query token per page-table row on the tensor cores: a CTA takes the query heads of one key head
 //    (16 at a time) x a range of the visible keys, which come through two cp.async stages.  grouped_merge_kernel joins the key
 //    splits; the sink belongs to split 0, so it counts once.
+//
+// Values that were turned by their position are turned back by the query's when a row's sum is complete (`turn`): every kernel
+// holds the adjacent values of a pair in one thread (or two neighbouring lanes) then.
 //
 // The keys that a row sees are numbered 0 .. n-1: first the kept ones before the window, then the window.
 #include "common.cuh"
@@ -86,6 +91,134 @@ __global__ void __launch_bounds__(256) grouped_pre_kernel(GroupedPreParams p) {
     }
 }
 
+struct GroupedRowPreParams {
+    const void *q, *k, *v; int ld;       // token-major projection rows
+    int heads, kv_heads, dim, vdim, rot_dims;
+    const float *q_bias, *k_bias, *v_bias;       // per projection row, or null
+    const float *q_norm, *k_norm;        // [heads * dim], [kv_heads * dim]
+    const float* sums;                   // [T, 2] sums of squares of the whole rows, or null: this launch's own rows are whole
+    float q_count, k_count, eps;         // values of a whole row
+    const float* gain;                   // [heads] factor on a head's queries, or null
+    const float2 *qk_turn, *v_turn; int ldt;     // (cos, sin) of pair m of token t at t * ldt + m (v_turn null: values do not turn)
+    const int* positions; const int* batch_idx; const int* page_table;
+    int pt_stride, page_size;
+    void *k_cache, *v_cache; int num_slots;      // [slots, kv_heads, dim], [slots, kv_heads, vdim]
+    void* q_out;                         // [T, heads, dim]
+    int* guard;
+};
+
+template <int VW, typename T>
+__device__ __forceinline__ float2 load_pair(const T* p) {
+    if (VW == 1) return make_float2(to_f(p[0]), 0.f);
+    if (sizeof(T) == 4) return *reinterpret_cast<const float2*>(p);
+    return bf162_to_f2(*reinterpret_cast<const uint32_t*>(p));
+}
+template <int VW, typename T>
+__device__ __forceinline__ void store_pair(T* p, float2 x) {
+    if (VW == 1) put(p, x.x);
+    else if (sizeof(T) == 4) *reinterpret_cast<float2*>(p) = x;
+    else *reinterpret_cast<uint32_t*>(p) = f2_to_bf162(x.x, x.y);
+}
+__device__ __forceinline__ float2 turned(float2 x, float2 cs) { return make_float2(x.x * cs.x - x.y * cs.y, x.y * cs.x + x.x * cs.y); }
+__device__ __forceinline__ float2 turned_back(float2 x, float2 cs) { return make_float2(x.x * cs.x + x.y * cs.y, x.y * cs.x - x.x * cs.y); }
+
+// A block per token.  VW 2: a thread takes pairs (even sizes and strides); 1: single values, whose partner it looks up.
+template <int VW, typename TI, typename TO>
+__global__ void __launch_bounds__(256) grouped_row_pre_kernel(GroupedRowPreParams p) {
+    pdl_grid_sync();
+    extern __shared__ __align__(8) float row[];          // [heads * dim | kv_heads * dim] with biases
+    __shared__ float part[2][8];
+    const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int nq = p.heads * p.dim, nk = p.kv_heads * p.dim, nv = p.kv_heads * p.vdim, pos = p.positions[t];
+    const TI *q = (const TI*)p.q + (size_t)t * p.ld, *k = (const TI*)p.k + (size_t)t * p.ld, *v = (const TI*)p.v + (size_t)t * p.ld;
+    float sq = 0.f, sk = 0.f;
+    for (int i = tid * VW; i < nq + nk; i += 256 * VW) {
+        const bool is_q = i < nq;
+        const int j = is_q ? i : i - nq;
+        const float* b = is_q ? p.q_bias : p.k_bias;
+        float2 x = load_pair<VW>((is_q ? q : k) + j);
+        if (b != nullptr) {
+            x.x += b[j];
+            if (VW == 2) x.y += b[j + 1];
+        }
+        row[i] = x.x;
+        if (VW == 2) row[i + 1] = x.y;
+        (is_q ? sq : sk) += x.x * x.x + (VW == 2 ? x.y * x.y : 0.f);
+    }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if (lane == 0) { part[0][warp] = sq; part[1][warp] = sk; }
+    __syncthreads();
+    sq = sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) { sq += part[0][i]; sk += part[1][i]; }
+    if (p.sums != nullptr) { sq = p.sums[t * 2]; sk = p.sums[t * 2 + 1]; }
+    const float iq = 1.f / sqrtf(sq / p.q_count + p.eps), ik = 1.f / sqrtf(sk / p.k_count + p.eps);
+    const int page = p.page_table[(size_t)p.batch_idx[t] * p.pt_stride + pos / p.page_size];
+    const long long slot = (long long)page * p.page_size + pos % p.page_size;
+    const bool cached = guard_ok(p.guard, 28, slot, p.num_slots);
+    TO *kd = (TO*)p.k_cache + (cached ? (size_t)slot * nk : 0), *vd = (TO*)p.v_cache + (cached ? (size_t)slot * nv : 0);
+    TO* qd = (TO*)p.q_out + (size_t)t * nq;
+    const float2* qk_turn = p.qk_turn + (size_t)t * p.ldt;
+    for (int i = tid * VW; i < nq + nk; i += 256 * VW) {
+        const bool is_q = i < nq;
+        if (!is_q && !cached) break;
+        const int j = is_q ? i : i - nq, d = j % p.dim;
+        const float* w = is_q ? p.q_norm : p.k_norm;
+        const float inv = (is_q ? iq : ik) * (is_q && p.gain != nullptr ? p.gain[j / p.dim] : 1.f);
+        float2 x = make_float2(row[i] * inv * w[j], VW == 2 ? row[i + 1] * inv * w[j + 1] : 0.f);
+        if (d < p.rot_dims) {
+            const float2 cs = qk_turn[d >> 1];
+            if (VW == 2) {
+                x = turned(x, cs);
+            } else {
+                const int o = d & 1 ? -1 : 1;
+                const float y = row[i + o] * inv * w[j + o];
+                x.x = x.x * cs.x + (d & 1 ? y : -y) * cs.y;
+            }
+        }
+        store_pair<VW>((is_q ? qd : kd) + j, x);
+    }
+    if (!cached) return;
+    const float2* v_turn = p.v_turn != nullptr ? p.v_turn + (size_t)t * p.ldt : nullptr;
+    auto value = [&](int i) { return to_f(v[i]) + (p.v_bias != nullptr ? p.v_bias[i] : 0.f); };
+    for (int i = tid * VW; i < nv; i += 256 * VW) {
+        const int d = i % p.vdim;
+        float2 x = make_float2(value(i), VW == 2 ? value(i + 1) : 0.f);
+        if (v_turn != nullptr) {
+            const float2 cs = v_turn[d >> 1];
+            if (VW == 2) {
+                x = turned(x, cs);
+            } else {
+                const float y = value(i + (d & 1 ? -1 : 1));
+                x.x = x.x * cs.x + (d & 1 ? y : -y) * cs.y;
+            }
+        }
+        store_pair<VW>(vd + i, x);
+    }
+}
+
+// out[t] = sums of squares of the query and key rows with their biases: what a rank that holds some of the heads adds to the norms.
+// grid T, block 256
+template <typename TI>
+__global__ void __launch_bounds__(256) row_sums_kernel(float* __restrict__ out, GroupedRowPreParams p) {
+    pdl_grid_sync();
+    __shared__ float scratch[33];
+    const int t = blockIdx.x, nq = p.heads * p.dim, nk = p.kv_heads * p.dim;
+    const TI *q = (const TI*)p.q + (size_t)t * p.ld, *k = (const TI*)p.k + (size_t)t * p.ld;
+    float sq = 0.f, sk = 0.f;
+    for (int i = threadIdx.x; i < nq + nk; i += 256) {
+        const bool is_q = i < nq;
+        const int j = is_q ? i : i - nq;
+        const float* b = is_q ? p.q_bias : p.k_bias;
+        const float x = to_f(is_q ? q[j] : k[j]) + (b != nullptr ? b[j] : 0.f);
+        (is_q ? sq : sk) += x * x;
+    }
+    sq = block_sum(sq, scratch);
+    sk = block_sum(sk, scratch);
+    if (threadIdx.x == 0) { out[t * 2] = sq; out[t * 2 + 1] = sk; }
+}
+
 struct GroupedAttnParams {
     const void* q;                       // [T, heads, dim]
     const void *k_cache, *v_cache; int num_slots;
@@ -97,7 +230,13 @@ struct GroupedAttnParams {
     void* out; int ldo;                  // [T, ldo]: head h at h * vdim
     float *o_part, *lse_part;            // [T, heads, splits, vdim], [T, heads, splits] (decode with more than one split)
     int* guard;
+    const float2* turn; int ldt;         // (cos, sin) by which pair m of token t's values is turned back, at t * ldt + m (or null)
+    float out_scale;                     // factor on the output
 };
+
+__device__ __forceinline__ float2 finished(const GroupedAttnParams& p, int t, int d, float x, float y) {
+    return p.turn == nullptr ? make_float2(x, y) : turned_back(make_float2(x, y), p.turn[(size_t)t * p.ldt + (d >> 1)]);
+}
 
 // The keys a position sees: n of them, number i is position at(i).
 struct Visible {
@@ -165,11 +304,14 @@ __global__ void __launch_bounds__(128) grouped_rows_kernel(GroupedAttnParams p) 
             o[i] = a;
         }
     }
-    const float inv = 1.f / l;
+    const float inv = p.out_scale / l;
 #pragma unroll
     for (int i = 0; i < ROWS_MAXV; ++i) {
         const int d = tid + i * 128;
-        if (d < p.vdim) put((T*)p.out + (size_t)t * p.ldo + (size_t)h * p.vdim + d, o[i] * inv);
+        const float x = o[i] * inv, y = __shfl_xor_sync(0xffffffffu, x, 1);
+        if (d >= p.vdim) continue;
+        const float2 f = d & 1 ? finished(p, t, d, y, x) : finished(p, t, d, x, y);
+        put((T*)p.out + (size_t)t * p.ldo + (size_t)h * p.vdim + d, d & 1 ? f.y : f.x);
     }
 }
 
@@ -310,7 +452,7 @@ __global__ void __launch_bounds__(DT) grouped_decode_kernel(GroupedAttnParams p)
     for (int u = 0; u < 4; ++u) {
         const int r = warp * 4 + u;
         if (lane == 0) {
-            fac[r] = l[u] > 0.f ? 1.f / l[u] : 0.f;
+            fac[r] = l[u] > 0.f ? (p.splits == 1 ? p.out_scale : 1.f) / l[u] : 0.f;
             if (r < nr && p.splits > 1)
                 p.lse_part[((size_t)t * p.heads + h0 + r) * p.splits + split] = l[u] > 0.f ? (m[u] + log2f(l[u])) / LOG2E : -INFINITY;
         }
@@ -326,8 +468,10 @@ __global__ void __launch_bounds__(DT) grouped_decode_kernel(GroupedAttnParams p)
             const int r = g + u * 8;
             if (r >= nr) continue;
             const float inv = u ? i1 : i0, x = acc[i][u * 2] * inv, y = acc[i][u * 2 + 1] * inv;
-            if (p.splits == 1) *reinterpret_cast<uint32_t*>((bf16*)p.out + (size_t)t * p.ldo + (size_t)(h0 + r) * p.vdim + d) = f2_to_bf162(x, y);
-            else *reinterpret_cast<float2*>(p.o_part + (((size_t)t * p.heads + h0 + r) * p.splits + split) * p.vdim + d) = make_float2(x, y);
+            if (p.splits == 1) {
+                const float2 f = finished(p, t, d, x, y);
+                *reinterpret_cast<uint32_t*>((bf16*)p.out + (size_t)t * p.ldo + (size_t)(h0 + r) * p.vdim + d) = f2_to_bf162(f.x, f.y);
+            } else *reinterpret_cast<float2*>(p.o_part + (((size_t)t * p.heads + h0 + r) * p.splits + split) * p.vdim + d) = make_float2(x, y);
         }
     }
 }
@@ -342,7 +486,7 @@ __global__ void __launch_bounds__(64) grouped_merge_kernel(GroupedAttnParams p) 
     const float b = lane + 32 < p.splits ? p.lse_part[row * p.splits + lane + 32] : -INFINITY;
     const float top = warp_max(fmaxf(a, b));
     const float ea = a == -INFINITY ? 0.f : expf(a - top), eb = b == -INFINITY ? 0.f : expf(b - top);
-    const float den = warp_sum(ea + eb), inv = den > 0.f ? 1.f / den : 0.f;
+    const float den = warp_sum(ea + eb), inv = den > 0.f ? p.out_scale / den : 0.f;
     if (tid < 32) {
         w[lane] = ea * inv;
         w[lane + 32] = eb * inv;
@@ -356,7 +500,8 @@ __global__ void __launch_bounds__(64) grouped_merge_kernel(GroupedAttnParams p) 
             x += w[i] * v.x;
             y += w[i] * v.y;
         }
-        *reinterpret_cast<uint32_t*>((bf16*)p.out + (size_t)t * p.ldo + (size_t)h * p.vdim + d) = f2_to_bf162(x, y);
+        const float2 f = finished(p, t, d, x, y);
+        *reinterpret_cast<uint32_t*>((bf16*)p.out + (size_t)t * p.ldo + (size_t)h * p.vdim + d) = f2_to_bf162(f.x, f.y);
     }
 }
 
@@ -379,9 +524,41 @@ SL_API int sl_grouped_pre(const GroupedPreParams* p, int T, int in_f32, int out_
     return SL_LAUNCH_CHECK();
 }
 
+SL_API int sl_grouped_row_pre(const GroupedRowPreParams* p, int T, int in_f32, int out_f32, cudaStream_t s) {
+    if (T == 0) return 0;
+    if (p->rot_dims > p->dim || p->rot_dims % 2 != 0 || (out_f32 && !in_f32) || (p->v_turn != nullptr && p->vdim % 2 != 0)) return -1;
+    const size_t smem = (size_t)(p->heads + p->kv_heads) * p->dim * sizeof(float);
+    if (smem > 200 * 1024) return -1;
+    const uintptr_t at = (uintptr_t)p->q | (uintptr_t)p->k | (uintptr_t)p->v;
+    const bool pairs = p->dim % 2 == 0 && p->vdim % 2 == 0 && p->ld % 2 == 0 && at % (in_f32 ? 8 : 4) == 0;
+#define SL_RP(VW, TI, TO)                                                                                              \
+    {                                                                                                                  \
+        auto kern = grouped_row_pre_kernel<VW, TI, TO>;                                                                \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);      \
+        sl_launch(kern, T, 256, smem, s, *p);                                                                          \
+    }
+    if (out_f32) {
+        if (pairs) SL_RP(2, float, float) else SL_RP(1, float, float)
+    } else if (in_f32) {
+        if (pairs) SL_RP(2, float, bf16) else SL_RP(1, float, bf16)
+    } else {
+        if (pairs) SL_RP(2, bf16, bf16) else SL_RP(1, bf16, bf16)
+    }
+#undef SL_RP
+    return SL_LAUNCH_CHECK();
+}
+
+// out [T, 2]: see row_sums_kernel (the norms, angles, caches and q_out of `p` are not read)
+SL_API int sl_grouped_row_sums(const GroupedRowPreParams* p, float* out, int T, int in_f32, cudaStream_t s) {
+    if (T == 0) return 0;
+    if (in_f32) sl_launch(row_sums_kernel<float>, T, 256, 0, s, out, *p);
+    else sl_launch(row_sums_kernel<bf16>, T, 256, 0, s, out, *p);
+    return SL_LAUNCH_CHECK();
+}
+
 SL_API int sl_grouped_rows(const GroupedAttnParams* p, int T, int f32, cudaStream_t s) {
     if (T == 0) return 0;
-    if (p->vdim > 128 * ROWS_MAXV || T > 65535 || p->heads % p->kv_heads != 0) return -1;
+    if (p->vdim > 128 * ROWS_MAXV || (p->turn != nullptr && p->vdim % 2 != 0) || T > 65535 || p->heads % p->kv_heads != 0) return -1;
     const size_t smem = (size_t)p->dim * sizeof(float);
     if (smem > 40 * 1024) return -1;
     if (f32) sl_launch(grouped_rows_kernel<float>, dim3(p->heads, T), 128, smem, s, *p);

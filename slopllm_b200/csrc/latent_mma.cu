@@ -55,6 +55,9 @@ struct PortionAttnParams {
     bf16* out; int ldo;                   // [T, ldo]: head i at i * vdim
     int* err;                             // status word: set when a wait inside the kernel expired
     int stages;                           // set by the launcher: key tiles in shared memory
+    const float2* turn; int ldt;          // values that turned with their position: (cos, sin) by which the adjacent pair m of token
+                                          // t's output is turned back, at t * ldt + m (or null)
+    float out_scale;                      // factor on the output
 };
 
 constexpr int BQ = 128, BK = 64, MAX_STAGES = 3;
@@ -263,13 +266,23 @@ __global__ void __launch_bounds__(PT, 1) portion_attn_kernel(PortionAttnParams p
         __syncwarp();
         if (lane == 0) tc::mbar_arrive(&empty[st]);
     }
-    const float i0 = l0 > 0.f ? 1.f / l0 : 0.f, i1 = l1 > 0.f ? 1.f / l1 : 0.f;
+    const float i0 = l0 > 0.f ? p.out_scale / l0 : 0.f, i1 = l1 > 0.f ? p.out_scale / l1 : 0.f;
+    auto store = [&](int r, int d, float x, float y) {
+        if (r >= nq) return;
+        if (p.turn != nullptr) {
+            const float2 cs = p.turn[(size_t)(q0 + r) * p.ldt + (d >> 1)];
+            const float a = x * cs.x + y * cs.y;
+            y = y * cs.x - x * cs.y;
+            x = a;
+        }
+        *reinterpret_cast<uint32_t*>(p.out + (size_t)(q0 + r) * p.ldo + (size_t)h * p.vdim + d) = f2_to_bf162(x, y);
+    };
 #pragma unroll
     for (int i = 0; i < NT; ++i) {
         const int d = i * 8 + 2 * c4;
         if (d >= p.vdim) break;
-        if (r0 < nq) *reinterpret_cast<uint32_t*>(p.out + (size_t)(q0 + r0) * p.ldo + (size_t)h * p.vdim + d) = f2_to_bf162(acc[i][0] * i0, acc[i][1] * i0);
-        if (r1 < nq) *reinterpret_cast<uint32_t*>(p.out + (size_t)(q0 + r1) * p.ldo + (size_t)h * p.vdim + d) = f2_to_bf162(acc[i][2] * i1, acc[i][3] * i1);
+        store(r0, d, acc[i][0] * i0, acc[i][1] * i0);
+        store(r1, d, acc[i][2] * i1, acc[i][3] * i1);
     }
 }
 

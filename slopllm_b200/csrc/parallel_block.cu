@@ -1,10 +1,17 @@
-// Activation of a feed-forward that runs beside a mixer: silu(gate) * up from columns of a wider projection into columns of a
-// wider operand, so that both sublayers share one input and one output product.
+// Activation of a gated feed-forward: act(gate + bias) * (up + bias) from columns of a projection into columns of an operand.  Either
+// may be part of wider rows: a feed-forward that runs beside a mixer shares its input and output product.
 #include "common.cuh"
 
 namespace {
 
-__device__ __forceinline__ float silu_f(float g) { return g / (1.f + expf(-g)); }
+enum { ACT_SILU = 0, ACT_GELU_TANH = 1 };
+
+template <int ACT>
+__device__ __forceinline__ float act_f(float g) {
+    if (ACT == ACT_SILU) return g / (1.f + expf(-g));
+    // 0.5 g (1 + tanh(x)) = g sigmoid(2x), x = sqrt(2 / pi) (g + 0.044715 g^3)
+    return g / (1.f + expf(-1.5957691216057308f * (g + 0.044715f * g * g * g)));
+}
 
 template <typename T>
 struct Four;
@@ -29,35 +36,49 @@ struct Four<bf16> {
     static __device__ __forceinline__ void put(bf16* p, float v) { *p = __float2bfloat16(v); }
 };
 
-// grid (ceil(I / (256 * VW)), T)
-template <int VW, typename TI, typename TO>
-__global__ void __launch_bounds__(256) silu_mul_rows_kernel(TO* __restrict__ out, int ldo, const TI* __restrict__ gu, int ld, int I) {
+// grid (ceil(I / (256 * VW)), T); bias [2 I] (gate | up) or null
+template <int ACT, int VW, typename TI, typename TO>
+__global__ void __launch_bounds__(256) gated_act_rows_kernel(TO* __restrict__ out, int ldo, const TI* __restrict__ gu, int ld, const float* __restrict__ bias, int I) {
     pdl_grid_sync();
     const int i = (blockIdx.x * 256 + threadIdx.x) * VW, t = blockIdx.y;
     if (i >= I) return;
     const TI* g = gu + (size_t)t * ld + i;
     TO* o = out + (size_t)t * ldo + i;
     if (VW == 4) {
-        const float4 a = Four<TI>::load(g), b = Four<TI>::load(g + I);
-        Four<TO>::store(o, make_float4(silu_f(a.x) * b.x, silu_f(a.y) * b.y, silu_f(a.z) * b.z, silu_f(a.w) * b.w));
+        float4 a = Four<TI>::load(g), b = Four<TI>::load(g + I);
+        if (bias != nullptr) {
+            const float4 x = Four<float>::load(bias + i), y = Four<float>::load(bias + I + i);
+            a.x += x.x; a.y += x.y; a.z += x.z; a.w += x.w;
+            b.x += y.x; b.y += y.y; b.z += y.z; b.w += y.w;
+        }
+        Four<TO>::store(o, make_float4(act_f<ACT>(a.x) * b.x, act_f<ACT>(a.y) * b.y, act_f<ACT>(a.z) * b.z, act_f<ACT>(a.w) * b.w));
     } else {
-        Four<TO>::put(o, silu_f(Four<TI>::one(g)) * Four<TI>::one(g + I));
+        float a = Four<TI>::one(g), b = Four<TI>::one(g + I);
+        if (bias != nullptr) { a += bias[i]; b += bias[I + i]; }
+        Four<TO>::put(o, act_f<ACT>(a) * b);
     }
 }
 
-template <typename TI, typename TO>
-int run(void* out, int ldo, const void* gu, int ld, int T, int I, cudaStream_t s) {
+template <int ACT, typename TI, typename TO>
+int run(void* out, int ldo, const void* gu, int ld, const float* bias, int T, int I, cudaStream_t s) {
     const bool v4 = I % 4 == 0 && ldo % 4 == 0 && ld % 4 == 0 && (uintptr_t)out % (4 * sizeof(TO)) == 0 && (uintptr_t)gu % (4 * sizeof(TI)) == 0;
-    if (v4) sl_launch(silu_mul_rows_kernel<4, TI, TO>, dim3((I / 4 + 255) / 256, T), 256, 0, s, (TO*)out, ldo, (const TI*)gu, ld, I);
-    else sl_launch(silu_mul_rows_kernel<1, TI, TO>, dim3((I + 255) / 256, T), 256, 0, s, (TO*)out, ldo, (const TI*)gu, ld, I);
+    if (v4) sl_launch(gated_act_rows_kernel<ACT, 4, TI, TO>, dim3((I / 4 + 255) / 256, T), 256, 0, s, (TO*)out, ldo, (const TI*)gu, ld, bias, I);
+    else sl_launch(gated_act_rows_kernel<ACT, 1, TI, TO>, dim3((I + 255) / 256, T), 256, 0, s, (TO*)out, ldo, (const TI*)gu, ld, bias, I);
     return SL_LAUNCH_CHECK();
+}
+
+template <int ACT>
+int run_types(void* out, int ldo, const void* gu, int ld, const float* bias, int T, int I, int in_f32, int out_f32, cudaStream_t s) {
+    if (out_f32) return run<ACT, float, float>(out, ldo, gu, ld, bias, T, I, s);
+    return in_f32 ? run<ACT, float, bf16>(out, ldo, gu, ld, bias, T, I, s) : run<ACT, bf16, bf16>(out, ldo, gu, ld, bias, T, I, s);
 }
 
 }  // namespace
 
-SL_API int sl_silu_mul_rows(void* out, int ldo, const void* gu, int ld, int T, int I, int in_f32, int out_f32, cudaStream_t s) {
+// act 0: silu, 1: the tanh form of gelu
+SL_API int sl_gated_act_rows(void* out, int ldo, const void* gu, int ld, const float* bias, int T, int I, int act, int in_f32, int out_f32, cudaStream_t s) {
     if (T == 0 || I == 0) return 0;
     if (T > 65535 || (out_f32 && !in_f32)) return -1;
-    if (out_f32) return run<float, float>(out, ldo, gu, ld, T, I, s);
-    return in_f32 ? run<float, bf16>(out, ldo, gu, ld, T, I, s) : run<bf16, bf16>(out, ldo, gu, ld, T, I, s);
+    if (act == ACT_SILU) return run_types<ACT_SILU>(out, ldo, gu, ld, bias, T, I, in_f32, out_f32, s);
+    return act == ACT_GELU_TANH ? run_types<ACT_GELU_TANH>(out, ldo, gu, ld, bias, T, I, in_f32, out_f32, s) : -1;
 }

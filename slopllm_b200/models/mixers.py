@@ -5,7 +5,7 @@ projection completes in the caller's all-reduce).  Every size and constant is a 
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Optional, Union
+from typing import List, Optional, Union
 
 import torch
 
@@ -15,7 +15,7 @@ from ..ops import experts as EX
 from ..ops import grouped as G
 from ..ops import latent as L
 from ..ops import recurrent as RC
-from ..ops.rotary import RotaryTable
+from ..ops.rotary import RotaryTable, Turn
 from ..utils.tracing import traced
 from .weights import ExpertWeights, LinearWeight
 
@@ -143,6 +143,122 @@ class GroupedAttention:
         rows = cache.rows[self.index]
         q = G.grouped_pre(main, self.shape, self.w, self.rot, st, rows["k"], rows["v"], out.dtype)
         G.grouped_attention(q, self.shape, self.w, st, rows["k"], rows["v"], out)
+
+
+@dataclass
+class RowNormAttention:
+    """Grouped-query attention with one norm over all heads' queries (and keys), biases, a factor per head on the scores and values
+    that turn with their position (`ops/grouped.py`).  Projection rows: q | k | v, each head's in adjacent order."""
+
+    index: int
+    shape: G.GroupedShape
+    turn: Turn
+    v_turn: Optional[Turn]
+    w: G.RowNormWeights
+    scale: float = 1.0               # on the output
+
+    @property
+    def spec(self) -> CacheSpec:
+        s = self.shape
+        return CacheSpec(rows={"k": (s.kv_heads, s.dim), "v": (s.kv_heads, s.vdim)})
+
+    def mix(self, model, main, fine, st, cache, out):
+        rows, angles = cache.rows[self.index], model.angles.of(st)
+        q = G.grouped_row_pre(main, self.shape, self.w, self.turn, self.v_turn, angles, st, rows["k"], rows["v"], out.dtype, model.comm)
+        G.grouped_attention(q, self.shape, self.w, st, rows["k"], rows["v"], out, G.Finish(self.v_turn, angles, self.scale))
+
+
+@dataclass
+class Retention:
+    """Linear attention with a fixed decay per head and rotated queries and keys (`ops/recurrent.py: retention_mix`).  Projection
+    rows: q | k (each head's in adjacent order) | v | output gate."""
+
+    index: int
+    heads: int
+    dk: int
+    dv: int
+    eps: float
+    turn: Turn
+    decay: torch.Tensor              # fp32 [2, heads], `recurrent.retention_decays`
+    scale: float = 1.0               # on the output
+
+    @property
+    def spec(self) -> CacheSpec:
+        return CacheSpec(state={"S": (self.heads, self.dk, self.dv)})
+
+    def mix(self, model, main, fine, st, cache, out):
+        qo, sidx = model.scan_ranges(st)
+        RC.retention_mix(main, self.decay, self.turn, model.angles.of(st), self.eps, cache.state[self.index]["S"], qo, sidx, self.heads, self.dk,
+                         self.dv, out, self.scale, RC.ChunkPlan.of(st))
+
+
+@dataclass
+class SideBySide:
+    """Mixers that read the same input and whose outputs are added: one input product makes the rows of all, one output product takes
+    their results side by side."""
+
+    index: int
+    kind: str
+    parts: list                      # mixers with `mix`
+    rows: List[int]                  # projection rows of each
+    outs: List[int]                  # values that each hands to `w_out`
+    w_in: LinearWeight
+    w_out: LinearWeight
+
+    @property
+    def spec(self) -> CacheSpec:
+        return CacheSpec(rows={n: x for m in self.parts for n, x in m.spec.rows.items()},
+                         state={n: x for m in self.parts for n, x in m.spec.state.items()})
+
+    @traced(lambda self, *a, **k: f"layer{self.index}.{self.kind}")
+    def __call__(self, model, x, st, cache):
+        main = model.ops.linear(x, self.w_in, out_f32=x.shape[0] <= SMALL_T)
+        both = torch.empty(x.shape[0], sum(self.outs), dtype=x.dtype, device=x.device)
+        r = o = 0
+        for m, nr, no in zip(self.parts, self.rows, self.outs):
+            m.mix(model, main[:, r:r + nr], None, st, cache, both[:, o:o + no])
+            r, o = r + nr, o + no
+        return model.ops.linear(both, self.w_out, out_f32=True)
+
+
+@dataclass
+class MinGru:
+    """Element-wise gated recurrence with an output gate (`ops/recurrent.py: min_gru_mix`)."""
+
+    index: int
+    width: int
+    w_in: LinearWeight               # z | candidate | output gate
+    bias: torch.Tensor               # fp32 [z | candidate]
+    o_proj: LinearWeight
+
+    @property
+    def spec(self) -> CacheSpec:
+        return CacheSpec(state={"S": (self.width,)})
+
+    @traced(lambda self, *a, **k: f"layer{self.index}.mingru")
+    def __call__(self, model, x, st, cache):
+        proj = model.ops.linear(x, self.w_in, out_f32=x.shape[0] <= SMALL_T)
+        qo, sidx = model.scan_ranges(st)
+        y = RC.min_gru_mix(proj, self.bias, cache.state[self.index]["S"], qo, sidx, self.width, x.dtype, RC.ChunkPlan.of(st))
+        return model.ops.linear(y, self.o_proj, out_f32=True)
+
+
+@dataclass
+class GatedFeedForward:
+    """act(gate x + b) * (up x + b'), projected down; the down projection's bias belongs to the caller's join."""
+
+    index: int
+    w_in: LinearWeight               # gate | up
+    bias: Optional[torch.Tensor]     # fp32 [gate | up]
+    w_out: LinearWeight
+    act: str = "silu"
+
+    @traced(lambda self, *a, **k: f"layer{self.index}.mlp")
+    def __call__(self, model, x, st, cache):
+        gu = model.ops.linear(x, self.w_in)
+        act = torch.empty(x.shape[0], gu.shape[1] // 2, dtype=x.dtype, device=x.device)
+        model.ops.gated_act(gu, act, self.act, self.bias)
+        return model.ops.linear(act, self.w_out, out_f32=True)
 
 
 @dataclass

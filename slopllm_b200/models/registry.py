@@ -57,6 +57,13 @@ def _load_zemezen(model_dir: str, ctx: ParallelContext, mtp: int = 0, dtype=None
     return load_zemezen_model(model_dir, ctx, dtype)
 
 
+def _load_vononex(model_dir: str, ctx: ParallelContext, mtp: int = 0, dtype=None):
+    from .vononex import load_vononex_model
+    if dtype is None:
+        dtype = torch.bfloat16 if ctx.device.type == "cuda" else torch.float32
+    return load_vononex_model(model_dir, ctx, dtype)
+
+
 MODEL_REGISTRY: Dict[str, ModelRegistration] = {
     "glm_moe_dsa": ModelRegistration(True, True, True, True, _load_glm_moe_dsa),
     "glm5_next": ModelRegistration(False, False, False, True, _load_glm5_next),
@@ -69,6 +76,9 @@ MODEL_REGISTRY: Dict[str, ModelRegistration] = {
                                  kernel_sources=("delta_chunk", "delta_step", "elementwise", "gemm_tcgen05", "gemv", "grouped_attn", "latent_attn", "latent_mma",
                                                  "linear_simt", "moe_sort", "moe_stream", "parallel_block", "sampling", "sandwich_norm",
                                                  "short_conv", "sparse_mla")),
+    "vononex": ModelRegistration(False, False, False, False, _load_vononex, float32=True,
+                                 kernel_sources=("elementwise", "gated_chunk", "gated_scan", "gemm_tcgen05", "gemv", "grouped_attn", "latent_mma", "linear_simt",
+                                                 "min_gru", "parallel_block", "rotary", "sampling", "sandwich_norm")),
 }
 
 

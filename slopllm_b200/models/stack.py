@@ -1,8 +1,10 @@
 """The decoder loop and the engine hooks shared by the model families whose layers are mixer + feed-forward sublayers over a
-:class:`~slopllm_b200.kv.hybrid.HybridCache`: Qwen3 / Qwen3.5 (`models/dense.py`), Gidisun (`models/gidisun.py`) and Zemezen (`models/zemezen.py`).
+:class:`~slopllm_b200.kv.hybrid.HybridCache`: Qwen3 / Qwen3.5 (`models/dense.py`), Gidisun (`models/gidisun.py`), Zemezen
+(`models/zemezen.py`) and Vononex (`models/vononex.py`).
 
-A family builds a flat list of :class:`Sublayer`; the loop runs  x -> run(norm(x)) -> [post norm] -> residual add -> next norm
-with the residual in fp32, and completes the tensor-parallel partial sums in between.
+A family builds a flat list of :class:`Sublayer`; the loop runs  x -> run(norm(x)) -> [post norm] -> residual add -> next norm,
+or, in families that normalise the sum,  x -> norm(alpha x + run(x) + bias),  with the residual in fp32, and completes the
+tensor-parallel partial sums in between.
 """
 from __future__ import annotations
 
@@ -18,8 +20,11 @@ from ..parallel.dist import Comm, ParallelContext
 @dataclass
 class Sublayer:
     run: Callable                              # (x, st, cache) -> this rank's partial sum [T, H]
-    norm: torch.Tensor                         # weight of the RMS norm in front
-    post_norm: Optional[torch.Tensor] = None   # fp32 weight of the RMS norm on the output (None: the output is added as it is)
+    norm: Optional[torch.Tensor]               # weight of the RMS norm in front (None: `run` reads the residual itself)
+    post_norm: Optional[torch.Tensor] = None   # fp32 weight of the RMS norm on the output (None: the output is added as it is),
+                                               # with `alpha` on the sum
+    alpha: Optional[float] = None              # factor on the residual of a sublayer whose sum is normalised
+    bias: Optional[torch.Tensor] = None        # fp32 [H], added to the complete output (sums that are normalised)
 
 
 def token_ranges(st):
@@ -78,12 +83,16 @@ class DecoderStack:
 
     def _enter(self, st, norm):
         ops, eps = self.ops, self.cfg.rms_norm_eps
+        if norm is None:
+            return ops.embed_rows(st.input_ids, self.w.embed)
         if self.fp32_norms or self.sublayers[0].post_norm is not None:
             return ops.embed_norm(st.input_ids, self.w.embed, norm, eps)
         return ops.add_rmsnorm(ops.embed(st.input_ids, self.w.embed), None, norm, eps)
 
     def _join(self, y, residual, sub: Sublayer, norm):
         ops, eps = self.ops, self.cfg.rms_norm_eps
+        if sub.alpha is not None:
+            return ops.sum_norm(self.comm.all_reduce(y), residual, sub.alpha, sub.bias, sub.post_norm, norm, eps)
         if self.fp32_norms or sub.post_norm is not None:
             return ops.post_norm(self.comm.all_reduce(y), residual, sub.post_norm, norm, eps)
         return self.comm.allreduce_add_rmsnorm(ops, y, residual, norm, eps)

@@ -47,6 +47,14 @@ class RefOps:
         r = residual + (y if w_post is None else R.rmsnorm(y, w_post, eps))
         return R.rmsnorm(r, w_next, eps), r
 
+    def embed_rows(self, ids, table):
+        r = self.embed(ids, table)
+        return r, r
+
+    def sum_norm(self, y, residual, alpha, bias, w, w_next, eps):
+        r = R.rmsnorm(alpha * residual + (y if bias is None else y + bias), w, eps)
+        return (r if w_next is None else R.rmsnorm(r, w_next, eps)), r
+
     def linear(self, x, w, out_f32: bool = False, sink=None, defer_reduce: bool = False):
         return R.linear(x, w)
 
@@ -119,8 +127,11 @@ class RefOps:
     def dense_mlp(self, x, lw, sink=None):
         return R.linear(R.silu_mul(R.linear(x, lw.mlp_w13)), lw.mlp_w2)
 
+    def gated_act(self, gate_up, out, act: str = "silu", bias=None):
+        out.copy_(R.gated_act(gate_up if bias is None else gate_up + bias, act))
+
     def silu_mul(self, gate_up, out):
-        out.copy_(R.silu_mul(gate_up))
+        self.gated_act(gate_up, out)
 
     def route(self, x, lw):
         c = self.cfg

@@ -117,6 +117,29 @@ class CudaOps:
         return self._post_norm(T, H, w_next, eps, y.device, y=y.data_ptr(), ldy=y.stride(0), w_post=N.ptr(w_post),
                                res_in=residual.data_ptr())
 
+    def _sum_norm(self, T: int, H: int, w_next, eps, dev, **src):
+        out = torch.empty(T, H, dtype=self.act_dtype, device=dev)
+        res = torch.empty(T, H, dtype=torch.float32, device=dev)
+        p = N.SumNormParams(out=out.data_ptr(), out_f32=int(self.act_dtype == torch.float32), res_out=res.data_ptr(), w_next=N.ptr(w_next),
+                            H=H, eps=float(eps), **src)
+        N.call("sl_sum_norm", C.byref(p), T, N.stream())
+        return out, res
+
+    def embed_rows(self, ids, table):
+        """Rows of the embedding table as (input of the first sublayer, fp32 residual)."""
+        ids = ids.to(torch.int64).contiguous()
+        return self._sum_norm(ids.shape[0], table.shape[1], None, 0.0, table.device, ids=ids.data_ptr(), table=table.data_ptr(),
+                              table_f32=int(table.dtype == torch.float32), vocab=table.shape[0])
+
+    def sum_norm(self, y, residual, alpha: float, bias, w, w_next, eps):
+        """residual' = rms(alpha * residual + y + bias) * w; returns (residual', or rms(residual') * w_next, and residual').  fp32
+        weights and sums; bias and w_next may be None."""
+        if y.dtype != torch.float32 or y.stride(-1) != 1:
+            y = y.to(torch.float32).contiguous()
+        T, H = y.shape
+        return self._sum_norm(T, H, w_next, eps, y.device, y=y.data_ptr(), ldy=y.stride(0), bias=N.ptr(bias), alpha=float(alpha), w=w.data_ptr(),
+                              res_in=residual.data_ptr())
+
     @staticmethod
     def _perm_of(x, T: int, K: int):
         """The permuted f16 copy that x's producer left with it, if it has the shape this consumer needs."""
@@ -520,11 +543,16 @@ class CudaOps:
         N.call("sl_silu_mul_f32" if gu.dtype == torch.float32 else "sl_silu_mul", act.data_ptr(), gu.data_ptr(), T, I2 // 2, N.stream())
         return self.linear(act, lw.mlp_w2, out_f32=True, sink=sink)
 
+    def gated_act(self, gate_up, out, act: str = "silu", bias=None):
+        """out = act(gate + b) * (up + b') for gate_up [T, 2I] = gate | up, bias fp32 [2I] = b | b' (None: 0) and out [T, I], rows of
+        any stride.  act: "silu" or "gelu_tanh"."""
+        T, I = out.shape
+        N.call("sl_gated_act_rows", out.data_ptr(), out.stride(0), gate_up.data_ptr(), gate_up.stride(0), N.ptr(bias), T, I,
+               {"silu": 0, "gelu_tanh": 1}[act], int(gate_up.dtype == torch.float32), int(out.dtype == torch.float32), N.stream())
+
     def silu_mul(self, gate_up, out):
         """out = silu(gate) * up for gate_up [T, 2I] = gate | up and out [T, I], rows of any stride."""
-        T, I = out.shape
-        N.call("sl_silu_mul_rows", out.data_ptr(), out.stride(0), gate_up.data_ptr(), gate_up.stride(0), T, I,
-               int(gate_up.dtype == torch.float32), int(out.dtype == torch.float32), N.stream())
+        self.gated_act(gate_up, out)
 
     def route(self, x, lw):
         c = self.cfg

@@ -46,7 +46,7 @@ class PortionAttnParams(C.Structure):
                 ("v", C.c_void_p), ("ldv", C.c_int), ("rows", C.c_void_p), ("row", C.c_int), ("rank", C.c_int), ("tiles", C.c_void_p),
                 ("heads", C.c_int), ("h0", C.c_int), ("dim", C.c_int), ("rot_dim", C.c_int), ("vdim", C.c_int), ("kv_group", C.c_int),
                 ("window", C.c_int), ("keep_first", C.c_int), ("scale", C.c_float), ("sink", C.c_void_p), ("out", C.c_void_p),
-                ("ldo", C.c_int), ("err", C.c_void_p), ("stages", C.c_int)]
+                ("ldo", C.c_int), ("err", C.c_void_p), ("stages", C.c_int), ("turn", C.c_void_p), ("ldt", C.c_int), ("out_scale", C.c_float)]
 
 
 class LatentDecodeParams(C.Structure):
@@ -204,15 +204,16 @@ def gather_rows(cache: torch.Tensor, plan: PortionPlan, st) -> torch.Tensor:
 
 def portion_attention(q, q_head: int, q_rot, k, v, plan: PortionPlan, out, *, heads: int, h0: int, group: int, dim: int, vdim: int,
                       scale: float, sink=None, kv_group: int = 1, window: int = 0, keep_first: int = 0, rot_dim: int = 0, rows=None,
-                      rank: int = 0) -> None:
-    """Attention of heads h0 .. h0 + group - 1 over gathered keys k and values v [rows, ...], into `out` (rows of any stride)."""
+                      rank: int = 0, finish: Optional[dict] = None) -> None:
+    """Attention of heads h0 .. h0 + group - 1 over gathered keys k and values v [rows, ...], into `out` (rows of any stride).
+    `finish`: kernel arguments of a rotation and factor on the output (`ops/grouped.py: Finish`)."""
     N = _native()
     from . import tcgen05
     p = PortionAttnParams(q=q.data_ptr(), ldq=q.stride(0), q_head=q_head, q_rot=N.ptr(q_rot), k=k.data_ptr(), ldk=k.stride(0),
                           v=v.data_ptr(), ldv=v.stride(0), rows=N.ptr(rows), row=0 if rows is None else rows.shape[1], rank=rank,
                           tiles=plan.tiles.data_ptr(), heads=heads, h0=h0, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_group=kv_group,
                           window=window, keep_first=keep_first, scale=scale, sink=N.ptr(sink), out=out.data_ptr(), ldo=out.stride(0),
-                          err=tcgen05.error_flag(out.device).data_ptr())
+                          err=tcgen05.error_flag(out.device).data_ptr(), **(finish or dict(out_scale=1.0)))
     N.call("sl_portion_attn", C.byref(p), group, plan.tile_count, N.stream())
 
 

@@ -205,12 +205,21 @@ class PostNormParams(C.Structure):
                 ("table", vp), ("table_f32", i32), ("vocab", i32), ("w_next", vp), ("H", i32), ("eps", f32)]
 
 
+class SumNormParams(C.Structure):
+    _fields_ = [("out", vp), ("out_f32", i32), ("res_out", vp), ("y", vp), ("ldy", i32), ("bias", vp), ("alpha", f32), ("w", vp),
+                ("res_in", vp), ("ids", vp), ("table", vp), ("table_f32", i32), ("vocab", i32), ("w_next", vp), ("H", i32), ("eps", f32)]
+
+
 # ---- function signatures ----------------------------------------------------------------------------------
 
 _SIGS = {
     "sl_linear_simt": [C.POINTER(SimtLinearParams), i32, i32, vp],
     "sl_silu_mul_f32": [vp, vp, i32, i32, vp],
     "sl_post_norm": [C.POINTER(PostNormParams), i32, vp],
+    "sl_sum_norm": [C.POINTER(SumNormParams), i32, vp],
+    "sl_angle_table": [vp, vp, vp, i32, i32, vp],
+    "sl_min_gru_step": [vp, i32, i32, i32, vp],
+    "sl_min_gru_chunks": [vp, i32, i32, i32, vp],
     "sl_latent_pre": [vp, i32, i32, vp],
     "sl_latent_rows": [vp, i32, i32, vp],
     "sl_gated_step": [vp, i32, i32, i32, i32, vp],
@@ -219,10 +228,12 @@ _SIGS = {
     "sl_portion_attn_ok": [i32, i32, i32],
     "sl_portion_attn": [vp, i32, i32, vp],
     "sl_grouped_pre": [vp, i32, i32, i32, vp],
+    "sl_grouped_row_pre": [vp, i32, i32, i32, vp],
+    "sl_grouped_row_sums": [vp, vp, i32, i32, vp],
     "sl_grouped_rows": [vp, i32, i32, vp],
     "sl_grouped_decode_ok": [i32, i32],
     "sl_grouped_decode": [vp, i32, vp],
-    "sl_silu_mul_rows": [vp, i32, vp, i32, i32, i32, i32, i32, vp],
+    "sl_gated_act_rows": [vp, i32, vp, i32, vp, i32, i32, i32, i32, i32, vp],
     "sl_short_conv": [vp, vp, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp],
     "sl_delta_step": [vp, i32, i32, i32, vp],
     "sl_delta_chunk_ok": [i32, i32],

@@ -1,15 +1,18 @@
 """Recurrent sub-layer ops of the hybrid families: Gated DeltaNet (Qwen3.5), KDA and manifold
-hyper-connections (glm5_next), GLA and mLSTM (Gidisun).  CUDA tensors run the sm_100a kernels of
-`csrc/recurrent.cu` and `csrc/gated_scan.cu`;
+hyper-connections (glm5_next), GLA and mLSTM (Gidisun), retention and minGRU (Vononex).  CUDA tensors run the sm_100a kernels of
+`csrc/recurrent.cu`, `csrc/gated_scan.cu`, `csrc/gated_chunk.cu` and `csrc/min_gru.cu`;
 CPU tensors run the fp32 definitions in `ops/reference.py` (the oracle of the GPU tests).
 """
 from __future__ import annotations
 
 import ctypes as C
+import math
+from typing import Optional
 
 import torch
 
 from . import reference as R
+from .rotary import Turn
 
 
 class GdnParams(C.Structure):
@@ -93,7 +96,7 @@ def kda_scan(qkv, forget, b, A_log, dt_bias, state, qo_indptr, state_idx, h: int
     return out.to(torch.bfloat16)
 
 
-# ---- gated outer-product recurrences: GLA and mLSTM --------------------------------------------------------------------------
+# ---- gated outer-product recurrences: GLA, mLSTM, retention --------------------------------------------------------------------------
 
 class GatedScanParams(C.Structure):
     _fields_ = [("out", C.c_void_p), ("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("g", C.c_void_p), ("ld", C.c_int),
@@ -101,10 +104,11 @@ class GatedScanParams(C.Structure):
                 ("inv_tau", C.c_float), ("i_b", C.c_void_p), ("f_b", C.c_void_p), ("cap", C.c_float), ("norm_w", C.c_void_p),
                 ("eps", C.c_float), ("S", C.c_void_p), ("n", C.c_void_p), ("m", C.c_void_p), ("qo_indptr", C.c_void_p),
                 ("state_idx", C.c_void_p), ("h", C.c_int), ("dk", C.c_int), ("dv", C.c_int), ("ldg", C.c_int), ("ldo", C.c_int),
-                ("group", C.c_int)]
+                ("group", C.c_int), ("decay", C.c_void_p), ("turn", C.c_void_p), ("ldt", C.c_int), ("rot_dims", C.c_int),
+                ("out_scale", C.c_float)]
 
 
-KIND_GLA, KIND_MLSTM = 0, 1
+KIND_GLA, KIND_MLSTM, KIND_RETENTION = 0, 1, 2
 CHUNK = 64                          # tokens per chunk of the chunked kernels
 CHUNK_MIN_Q = 16                    # longest portion of a step from which on they are used
 CHUNK_SCRATCH_BYTES = 96 << 20      # chunk states of one pass (they stay in L2); longer steps run in several passes
@@ -145,8 +149,8 @@ class ChunkPlan:
 def _gated_params(p_in, h, dk, dv, out, norm_w, eps, qo_indptr, state_idx) -> GatedScanParams:
     esz = p_in.element_size()
     base = p_in.data_ptr()
-    return GatedScanParams(out=out.data_ptr(), q=base, k=base + h * dk * esz, v=base + 2 * h * dk * esz,
-                           g=base + (2 * h * dk + h * dv) * esz, ld=p_in.stride(0), norm_w=norm_w.data_ptr(), eps=float(eps),
+    return GatedScanParams(out=out.data_ptr(), ldo=out.stride(0), q=base, k=base + h * dk * esz, v=base + 2 * h * dk * esz,
+                           g=base + (2 * h * dk + h * dv) * esz, ld=p_in.stride(0), norm_w=_native().ptr(norm_w), eps=float(eps),
                            qo_indptr=qo_indptr.data_ptr(), state_idx=state_idx.data_ptr(), h=h, dk=dk, dv=dv)
 
 
@@ -155,7 +159,7 @@ def _run_gated(kind: int, p: GatedScanParams, proj, out, qo_indptr, plan=None) -
     B = qo_indptr.numel() - 1
     h, dk, dv, dev = p.h, p.dk, p.dv, proj.device
     if (plan is None or plan.longest < CHUNK_MIN_Q or proj.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or p.ld % 8
-            or p.q % 16 or not N.fn("sl_gated_chunk_ok")(kind, dk, dv, p.rank)):
+            or p.q % 16 or p.ldo % 2 or p.out % 4 or not N.fn("sl_gated_chunk_ok")(kind, dk, dv, p.rank)):
         N.call("sl_gated_step", C.byref(p), B, kind, int(proj.dtype == torch.float32), int(out.dtype == torch.float32), N.stream())
         return out
     per_pass = min(plan.count, max(1, CHUNK_SCRATCH_BYTES // (h * dk * dv * 4)))
@@ -231,6 +235,84 @@ def mlstm_mix(proj, gates, i_b, f_b, cap: float, norm_w, eps: float, state, qo_i
             o[r] = R.mlstm_scan(q[r], k[r], v[r], gi[r], gf[r], S[sl], n[sl], m[sl])
     o = R.rmsnorm(o, torch.ones(dv), eps).reshape(T, h * dv) * norm_w * torch.sigmoid(g.reshape(T, h * dv))
     return o.to(out_dtype)
+
+
+def retention_decays(decay) -> torch.Tensor:
+    """[2, heads] fp32 for :func:`retention_mix`: each head's decay and its log2, made once on the host (2^-200 stands for nothing kept)."""
+    if any(not 0.0 <= d for d in decay):
+        raise ValueError("decays must not be negative")
+    return torch.tensor([list(decay), [math.log2(d) if d > 0 else -200.0 for d in decay]], dtype=torch.float32)
+
+
+def retention_mix(proj, decay, turn: Turn, angles, eps: float, state, qo_indptr, state_idx, h: int, dk: int, dv: int, out, scale: float = 1.0,
+                  plan=None) -> None:
+    """Retention over the token ranges of B sequences, up to the output projection: linear attention with a fixed decay per head.
+
+    proj [T, h*dk (q) | h*dk (k) | h*dv (v) | h*dv (output gate)], q and k rows in the adjacent order of `ops/rotary.py` and turned by
+    `turn`; decay from :func:`retention_decays`; state [slots, h, dk, dv] fp32 updated in place.
+    S = decay S + k v^T, o = S^T q dk^-0.5; out [T, h*dv] (rows of any stride) = scale * rms(o) * silu(gate)."""
+    T = proj.shape[0]
+    if proj.is_cuda:
+        p = _gated_params(proj, h, dk, dv, out, None, eps, qo_indptr, state_idx)
+        p.S, p.decay, p.turn, p.ldt, p.rot_dims = state.data_ptr(), decay.data_ptr(), angles.data_ptr() + turn.at * 8, angles.shape[1], turn.dims
+        p.out_scale = scale
+        _run_gated(KIND_RETENTION, p, proj, out, qo_indptr, plan)
+        return
+    q, k, v, g = _qkvg(proj, h, dk, dv)
+    q, k = turn.apply(q, angles), turn.apply(k, angles)
+    keep = decay[0].view(1, h, 1).expand(T, h, dk)
+    o = torch.empty(T, h, dv, dtype=torch.float32)
+    ind = qo_indptr.tolist()
+    for b in range(len(ind) - 1):
+        r = slice(ind[b], ind[b + 1])
+        if ind[b + 1] > ind[b]:
+            o[r] = R.gla_scan(q[r], k[r], v[r], keep[r], state[int(state_idx[b])])
+    o = R.rmsnorm(o, torch.ones(dv), eps) * torch.nn.functional.silu(g) * scale
+    out.copy_(o.reshape(T, h * dv))
+
+
+# ---- element-wise gated recurrence: minGRU -----------------------------------------------------------------------------------
+
+class MinGruParams(C.Structure):
+    _fields_ = [("out", C.c_void_p), ("ldo", C.c_int), ("z", C.c_void_p), ("u", C.c_void_p), ("g", C.c_void_p), ("ld", C.c_int),
+                ("z_b", C.c_void_p), ("u_b", C.c_void_p), ("S", C.c_void_p), ("qo_indptr", C.c_void_p), ("state_idx", C.c_void_p),
+                ("W", C.c_int), ("chunks", C.c_void_p), ("seq_chunks", C.c_void_p), ("maps", C.c_void_p), ("start", C.c_void_p)]
+
+
+def min_gru_mix(proj, bias: Optional[torch.Tensor], state, qo_indptr, state_idx, W: int, out_dtype, plan=None) -> torch.Tensor:
+    """minGRU over the token ranges of B sequences, up to the output projection.
+
+    proj [T, W (z) | W (u) | W (output gate)], bias fp32 [W (z) | W (u)], state [slots, W] fp32 updated in place.
+    z = sigmoid(z), c = u + 1/2 where u >= 0 and sigmoid(u) elsewhere, S = (1 - z) S + z c; returns S * silu(gate) [T, W].
+    With a :class:`ChunkPlan` longer portions run in chunks that are composed."""
+    T = proj.shape[0]
+    if proj.is_cuda:
+        N = _native()
+        out = torch.empty(T, W, dtype=out_dtype, device=proj.device)
+        at = lambda i: proj.data_ptr() + i * W * proj.element_size()
+        p = MinGruParams(out=out.data_ptr(), ldo=out.stride(0), z=at(0), u=at(1), g=at(2), ld=proj.stride(0), z_b=N.ptr(bias),
+                         u_b=0 if bias is None else bias.data_ptr() + 4 * W, S=state.data_ptr(), qo_indptr=qo_indptr.data_ptr(),
+                         state_idx=state_idx.data_ptr(), W=W)
+        B, types = qo_indptr.numel() - 1, (int(proj.dtype == torch.float32), int(out_dtype == torch.float32))
+        if plan is None or plan.longest < CHUNK_MIN_Q:
+            N.call("sl_min_gru_step", C.byref(p), B, *types, N.stream())
+            return out
+        scratch = torch.empty(plan.count * W * 2 + B * W, dtype=torch.float32, device=proj.device)
+        p.chunks, p.seq_chunks = plan.table.data_ptr(), plan.seq_chunks.data_ptr()
+        p.maps, p.start = scratch.data_ptr(), scratch.data_ptr() + plan.count * W * 8
+        N.call("sl_min_gru_chunks", C.byref(p), plan.count, *types, N.stream())
+        return out
+    x = proj[:, :3 * W].to(torch.float32)
+    z, u, g = x[:, :W], x[:, W:2 * W], x[:, 2 * W:]
+    if bias is not None:
+        z, u = z + bias[:W], u + bias[W:]
+    S = torch.empty(T, W, dtype=torch.float32)
+    ind = qo_indptr.tolist()
+    for b in range(len(ind) - 1):
+        r = slice(ind[b], ind[b + 1])
+        if ind[b + 1] > ind[b]:
+            S[r] = R.min_gru_scan(z[r], u[r], state[int(state_idx[b])])
+    return (S * torch.nn.functional.silu(g)).to(out_dtype)
 
 
 def causal_conv1d(x, weight, bias, state, qo_indptr, state_idx, activation: bool = True):

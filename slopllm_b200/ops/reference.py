@@ -88,6 +88,11 @@ def silu_mul(gate_up: torch.Tensor) -> torch.Tensor:
     return torch.nn.functional.silu(g) * u
 
 
+def gated_act(gate_up: torch.Tensor, act: str) -> torch.Tensor:
+    g, u = gate_up.to(torch.float32).chunk(2, dim=-1)
+    return {"silu": torch.nn.functional.silu, "gelu_tanh": lambda x: torch.nn.functional.gelu(x, approximate="tanh")}[act](g) * u
+
+
 # ---- MoE routing --------------------------------------------------------------------------------
 
 
@@ -506,6 +511,18 @@ def gla_scan(q, k, v, decay, state):
     for t in range(q.shape[0]):
         state.mul_(decay[t].unsqueeze(-1)).add_(k[t].unsqueeze(-1) * v[t].unsqueeze(-2))
         out.append(torch.einsum("hkv,hk->hv", state, q[t]))
+    return torch.stack(out)
+
+
+def min_gru_scan(z, u, state):
+    """Element-wise gated recurrence.  z, u [T, W] (gate and candidate before their activations); state [W] advanced in place.
+    Returns the states [T, W]."""
+    z = torch.sigmoid(z)
+    c = torch.where(u >= 0, u + 0.5, torch.sigmoid(u))
+    out = []
+    for t in range(z.shape[0]):
+        state.mul_(1 - z[t]).add_(z[t] * c[t])
+        out.append(state.clone())
     return torch.stack(out)
 
 
