@@ -1,10 +1,11 @@
-"""Prefill and decode throughput of the hybrid families side by side: Zemezen, Gidisun and Qwen3.5 at equal width, heads, head sizes
-and feed-forward, random weights, layers of a real model's size.
+"""Prefill and decode throughput of the hybrid families side by side: Vononex, Zemezen, Gidisun and Qwen3.5 at equal width, heads, head
+sizes and feed-forward, random weights, layers of a real model's size.
 
     python -m slopllm_b200.cli.hybrid_bench [--sizes small,medium,large] [--batches 1,8,64] [--prompt 4096]
 
 Every stack has four layers with a feed-forward each: three recurrent mixers and one attention layer; Zemezen two of its recurrent
-mixers, one windowed and one latent attention layer.  `zemezen_moe` has 32 experts of a quarter of the feed-forward's width in
+mixers, one windowed and one latent attention layer; Vononex two minGRU layers and two in which attention over the whole context and
+retention share the heads (half of them each, so that a layer's projections stay as wide).  `zemezen_moe` has 32 experts of a quarter of the feed-forward's width in
 every layer, of which a token uses four.  Every number is device
 time (CUDA events, three warm-up runs, a 256 MB write in front of every timed run so that nothing is served from L2); decode is
 a replay of the captured step.  Prints one JSON line; `python bench.py --hybrid [sizes]` prints the same.
@@ -58,7 +59,22 @@ def zemezen_config(size: str, moe: bool = False):
                                  ZemezenLayer("attention", attn, *mlp), ZemezenLayer("latent_attention", latent, *mlp)])
 
 
+def vononex_config(size: str):
+    from ..models.vononex import VononexConfig, VononexLayer
+    H, ff, h = SIZES[size]
+    left = {"heads": h // 2, "kv_heads": max(1, h // 8), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "rot": {"base": 1e6, "dims": 128}}
+    right = {"heads": h // 2, "dim": 128, "vdim": 128, "rot": {"base": 1e4, "dims": 128}, "decay": [1 - 2.0 ** (-5 - i % 6) for i in range(h // 2)]}
+    pair, gru = {"left": left, "right": right, "left_scale": 1.0, "right_scale": 1.0}, {"width": H}
+    return VononexConfig(hidden_size=H, vocab_size=VOCAB, rms_norm_eps=1e-6, alpha=2.0,
+                         layers=[VononexLayer("mingru", gru, ff), VononexLayer("parallel", pair, ff), VononexLayer("mingru", gru, ff),
+                                 VononexLayer("parallel", pair, ff)])
+
+
 def build(family: str, size: str, ctx):
+    if family == "vononex":
+        from ..models.vononex import VononexModel, random_vononex_tensors
+        cfg = vononex_config(size)
+        return cfg, VononexModel.from_tensors(cfg, random_vononex_tensors(cfg, 0, device=ctx.device), ctx)
     if family in ("zemezen", "zemezen_moe"):
         from ..models.zemezen import ZemezenModel, random_zemezen_tensors
         cfg = zemezen_config(size, family == "zemezen_moe")
@@ -105,7 +121,7 @@ def run_arm(family: str, size: str, batches, prompt: int, iters: int, flush) -> 
     st, _, _ = eng._pack([s], [ids])
 
     def prefill():
-        for name in ("chunk_plan", "portion_plans"):
+        for name in ("chunk_plan", "portion_plans", "angles"):
             st.extra.pop(name, None)
         return model.forward_hidden(st, eng.cache)
 
@@ -156,7 +172,7 @@ def run(argv=None) -> dict:
     ap.add_argument("--batches", default="1,8,64")
     ap.add_argument("--prompt", type=int, default=4096)
     ap.add_argument("--iters", type=int, default=10)
-    ap.add_argument("--families", default="zemezen,zemezen_moe,gidisun,qwen3_5")
+    ap.add_argument("--families", default="vononex,zemezen,zemezen_moe,gidisun,qwen3_5")
     args = ap.parse_args(argv)
     torch.cuda.set_device(0)
     flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")

@@ -82,12 +82,12 @@ def time_op(fn: Callable[[], object], iters: int, flush: torch.Tensor) -> float:
 
 def mixer_rows(emit, tokens, iters: int, flush, peaks, dev, h: int = 16, dk: int = 128, dv: int = 128, rank: int = 512, rot: int = 64,
                window: int = 1024, context: int = 2048, n_kv: int = 4) -> None:
-    """Token mixers of the hybrid families at 16 heads of 128: channel-wise delta rule, windowed grouped-query attention, GLA, mLSTM and
-    latent attention beside Gated DeltaNet and paged grouped-query attention.  More than 64 tokens: one prompt; fewer: that many sequences of `context` tokens decode one each."""
+    """Token mixers of the hybrid families at 16 heads of 128: retention, minGRU, attention with turned values, channel-wise delta rule,
+    windowed grouped-query attention, GLA, mLSTM and latent attention beside Gated DeltaNet and paged grouped-query attention.  More than 64 tokens: one prompt; fewer: that many sequences of `context` tokens decode one each."""
     import types
     from ..models.glm_moe_dsa import StepState
     from ..ops import delta as DL, delta_chunk as DC, dense as D, get_ops, grouped as G, latent as L, recurrent as RC
-    from ..ops.rotary import rotary_table
+    from ..ops.rotary import AngleTable, rotary_table
     ops = get_ops(types.SimpleNamespace(rms_norm_eps=1e-6), dev)
     g = torch.Generator(device=dev).manual_seed(3)
     rnd = lambda *s, k=1.0: torch.randn(*s, device=dev, generator=g) * k
@@ -119,6 +119,38 @@ def mixer_rows(emit, tokens, iters: int, flush, peaks, dev, h: int = 16, dk: int
         state = (S, rnd(B, h, dk), torch.zeros(B, h, device=dev))
         us = time_op(lambda: RC.mlstm_mix(pr, gates, ib, fb, 15.0, nwh, 1e-6, state, qo, sidx, h, dk, dv, torch.bfloat16, plan), iters, flush)
         emit(roofline_row("mlstm", T, us, io, flops, peaks))
+        # retention, minGRU, attention with whole-row norms and turned values, norm of the sum, biased activation
+        angle = AngleTable()
+        turn, v_turn = angle.turn(dk, 1e4), angle.turn(dv, 1e4)
+        angles, rout = angle.of(st), bf(T, h * dv)
+        us = time_op(lambda: angle.at(st.positions), iters, flush)
+        emit(roofline_row("angle_table", T, us, T * (angles.shape[1] * 8 + 4), 0.0, peaks))
+        decay = RC.retention_decays([1 - 2.0 ** (-5 - i % 6) for i in range(h)]).to(dev)
+        us = time_op(lambda: RC.retention_mix(pr, decay, turn, angles, 1e-6, S, qo, sidx, h, dk, dv, rout, 1.0, plan), iters, flush)
+        emit(roofline_row("retention", T, us, io, flops, peaks))
+        W = h * dv
+        gru, gb, gS = (bf if prompt else rnd)(T, 3 * W), rnd(2 * W), rnd(B, W)
+        us = time_op(lambda: RC.min_gru_mix(gru, gb, gS, qo, sidx, W, torch.bfloat16, plan), iters, flush)
+        emit(roofline_row("min_gru", T, us, T * W * (3 * (2 if prompt else 4) + 2) + 8 * B * W, 0.0, peaks))
+        rs = G.GroupedShape(h, n_kv, 128, 128, 128 ** -0.5, eps=1e-6)
+        rw = G.RowNormWeights(rnd(h * 128), rnd(n_kv * 128), rnd((h + 2 * n_kv) * 128), rnd(h))
+        rproj, rk, rv = (bf if prompt else rnd)(T, (h + 2 * n_kv) * 128), bf(B * width * 64, n_kv, 128), bf(B * width * 64, n_kv, 128)
+        us = time_op(lambda: G.grouped_row_pre(rproj, rs, rw, turn, v_turn, angles, st, rk, rv, torch.bfloat16), iters, flush)
+        emit(roofline_row("grouped_row_pre", T, us, T * 128 * (h + 2 * n_kv) * (2 + (2 if prompt else 4)), 0.0, peaks))
+        rq = G.grouped_row_pre(rproj, rs, rw, turn, v_turn, angles, st, rk, rv, torch.bfloat16)
+        us = time_op(lambda: G.grouped_attention(rq, rs, rw, st, rk, rv, rout, G.Finish(v_turn, angles, 1.0)), iters, flush)
+        every = T * (T + 1) / 2 if prompt else T * kv
+        emit(roofline_row("grouped_attention (full context, turned values)", T, us, 2.0 * (T if prompt else T * kv) * n_kv * 256 + 4.0 * T * h * 128,
+                          4.0 * every * h * 128, peaks))
+        H, sy = h * 128, rnd(T, h * 128)
+        sb, sres = rnd(H), rnd(T, H)
+        us = time_op(lambda: ops.sum_norm(sy, sres, 2.0, sb, sb, None, 1e-6), iters, flush)
+        emit(roofline_row("sum_norm", T, us, T * H * 14.0, 0.0, peaks))
+        gu, act, ab2 = bf(T, 8 * H), bf(T, 4 * H), rnd(8 * H)
+        us = time_op(lambda: ops.gated_act(gu, act, "gelu_tanh", ab2), iters, flush)
+        emit(roofline_row("gated_act (gelu, biases)", T, us, T * H * 24.0, 0.0, peaks))
+        us = time_op(lambda: ops.silu_mul(gu, act), iters, flush)
+        emit(roofline_row("gated_act (silu)", T, us, T * H * 24.0, 0.0, peaks))
         qkv, ab = bf(T, h * (2 * dk + dv)), bf(T, h)
         us = time_op(lambda: RC.gdn_scan(qkv, ab, ab, ib, fb, S, qo, sidx, h, dk, dv), iters, flush)
         emit(roofline_row("gdn (scan alone)", T, us, T * h * (2 * dk + 2 * dv) * 2 + 2 * B * h * dk * dv * 4, flops, peaks))

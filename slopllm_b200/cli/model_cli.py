@@ -23,7 +23,8 @@ from ..parallel.dist import ParallelContext, init_from_env
 def add_model_args(ap: argparse.ArgumentParser) -> None:
     ap.add_argument("--model", default="", help="checkpoint directory or Hugging Face hub id (local cache only)")
     ap.add_argument("--random-init", default="", metavar="SPEC",
-                    help="no checkpoint: random weights of 'tiny', 'glm5[:layers]', 'qwen3-tiny', 'qwen35-tiny', 'gidisun-tiny' or 'zemezen-tiny'")
+                    help="no checkpoint: random weights of 'tiny', 'glm5[:layers]', 'qwen3-tiny', 'qwen35-tiny', 'gidisun-tiny', 'zemezen-tiny' "
+                         "or 'vononex-tiny'")
     ap.add_argument("--dtype", choices=("bfloat16", "float32"), default=None,
                     help="activation and weight type; default bfloat16 on a GPU.  float32 (no reduced-precision products) for the "
                          "families that have it")
@@ -105,7 +106,9 @@ def check_memory_plan(args, ctx: ParallelContext, model_dir: str, model_type: st
     """Before the weights are read: does this rank's share of the model plus the KV pages asked for fit the memory the
     process may use?  A plan that does not fit is reported on stderr (rank 0) and returned; loading still goes ahead, the
     estimate of the workspace is deliberately generous."""
-    if model_type not in ("glm_moe_dsa", "qwen3", "qwen3_5", "gidisun", "zemezen") or ctx.device.type != "cuda":
+    from ..models.registry import hybrid_family
+    family = hybrid_family(model_type)
+    if (family is None and model_type not in ("glm_moe_dsa", "qwen3", "qwen3_5")) or ctx.device.type != "cuda":
         return None
     import sys
     from ..utils.sizing import GIB, plan_dense, plan_memory
@@ -114,16 +117,12 @@ def check_memory_plan(args, ctx: ParallelContext, model_dir: str, model_type: st
         from ..checkpoint.loader import load_config
         p = plan_memory(load_config(model_dir), world=ctx.world, cp=args.cp, ep=args.ep, mtp=args.mtp, batch_size=args.batch_size,
                         chunk_size=args.chunk_size, max_pages=args.max_pages, arena_gb=args.arena, device_gb=total / GIB)
-    elif model_type in ("gidisun", "zemezen"):
+    elif family is not None:
         import json
-        from ..models.gidisun import GidisunConfig
-        from ..models.zemezen import ZemezenConfig
-        from ..utils.sizing import plan_gidisun, plan_zemezen
-        config, planner = (GidisunConfig, plan_gidisun) if model_type == "gidisun" else (ZemezenConfig, plan_zemezen)
         with open(os.path.join(model_dir, "config.json")) as f:
-            hcfg = config.from_dict(json.load(f))
-        p = planner(hcfg, world=ctx.world, batch_size=args.batch_size, chunk_size=args.chunk_size, max_pages=args.max_pages,
-                         arena_gb=args.arena, device_gb=total / GIB, elem=4 if getattr(args, "dtype", None) == "float32" else 2)
+            hcfg = family.config.from_dict(json.load(f))
+        p = family.plan(hcfg, world=ctx.world, batch_size=args.batch_size, chunk_size=args.chunk_size, max_pages=args.max_pages,
+                        arena_gb=args.arena, device_gb=total / GIB, elem=4 if getattr(args, "dtype", None) == "float32" else 2)
     else:
         import json
         from ..models.dense import DenseConfig
@@ -144,14 +143,12 @@ def check_memory_plan(args, ctx: ParallelContext, model_dir: str, model_type: st
 def _random_model(spec: str, ctx: ParallelContext, mtp: int, dtype_name: Optional[str] = None):
     from ..parallel.fused import make_comm
     dtype = torch.bfloat16 if ctx.device.type == "cuda" else torch.float32
-    if spec.startswith("gidisun"):
-        from ..models.gidisun import GidisunConfig, GidisunModel, random_gidisun_tensors
-        cfg = GidisunConfig.tiny()
-        return cfg, GidisunModel.from_tensors(cfg, random_gidisun_tensors(cfg), ctx, getattr(torch, dtype_name) if dtype_name else dtype), cfg.model_type
-    if spec.startswith("zemezen"):
-        from ..models.zemezen import ZemezenConfig, ZemezenModel, random_zemezen_tensors
-        cfg = ZemezenConfig.tiny()
-        return cfg, ZemezenModel.from_tensors(cfg, random_zemezen_tensors(cfg), ctx, getattr(torch, dtype_name) if dtype_name else dtype), cfg.model_type
+    from ..models.registry import hybrid_family
+    family = hybrid_family(spec)
+    if family is not None:
+        cfg = family.config.tiny()
+        model = family.model.from_tensors(cfg, family.random_tensors(cfg), ctx, getattr(torch, dtype_name) if dtype_name else dtype)
+        return cfg, model, cfg.model_type
     if dtype_name is not None and getattr(torch, dtype_name) != dtype:
         raise SystemExit(f"--random-init {spec} does not run in {dtype_name} on {ctx.device.type}")
     tp_world = ctx.world          # weights stay tensor-parallel under context parallelism too

@@ -17,34 +17,28 @@ from ..utils.sizing import GIB, plan_memory
 
 
 def _config(args) -> GlmMoeDsaConfig:
+    from ..models.registry import HYBRID_FAMILIES, hybrid_family, inspect_model
     if args.model:
         from ..checkpoint.loader import load_config
-        from ..models.registry import inspect_model
         from ..utils.model_path import resolve_model_path
         model_dir = resolve_model_path(args.model)
         model_type, _, raw = inspect_model(model_dir)
         if model_type in ("qwen3", "qwen3_5"):
             from ..models.dense import DenseConfig
             return DenseConfig.from_hf_dict(raw)
-        if model_type == "gidisun":
-            from ..models.gidisun import GidisunConfig
-            return GidisunConfig.from_dict(raw)
-        if model_type == "zemezen":
-            from ..models.zemezen import ZemezenConfig
-            return ZemezenConfig.from_dict(raw)
+        family = hybrid_family(model_type)
+        if family is not None:
+            return family.config.from_dict(raw)
         if model_type != "glm_moe_dsa":
-            raise SystemExit(f"plan: the sizing arithmetic covers glm_moe_dsa, qwen3, qwen3_5, gidisun and zemezen; {args.model} is {model_type}")
+            raise SystemExit(f"plan: the sizing arithmetic covers glm_moe_dsa, qwen3, qwen3_5, {', '.join(HYBRID_FAMILIES)}; {args.model} is {model_type}")
         return load_config(model_dir)
     spec = args.random_init or "glm5"
     if spec.startswith("qwen"):
         from ..models.dense import DenseConfig
         return DenseConfig.tiny(hybrid=spec.startswith("qwen35"))
-    if spec.startswith("gidisun"):
-        from ..models.gidisun import GidisunConfig
-        return GidisunConfig.tiny()
-    if spec.startswith("zemezen"):
-        from ..models.zemezen import ZemezenConfig
-        return ZemezenConfig.tiny()
+    family = hybrid_family(spec)
+    if family is not None:
+        return family.config.tiny()
     if spec.startswith("glm5"):
         return GlmMoeDsaConfig.glm5(num_layers=int(spec.split(":")[1]) if ":" in spec else 78)
     return GlmMoeDsaConfig.tiny()
@@ -53,7 +47,7 @@ def _config(args) -> GlmMoeDsaConfig:
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="slopllm_b200.cli.plan", description=__doc__.split("\n")[0])
     ap.add_argument("--model", default="", help="checkpoint directory or hub id (only config.json is read)")
-    ap.add_argument("--random-init", default="", help="glm5[:layers], tiny, qwen3, qwen35, gidisun or zemezen instead of a checkpoint")
+    ap.add_argument("--random-init", default="", help="glm5[:layers], tiny, qwen3, qwen35, gidisun, zemezen or vononex instead of a checkpoint")
     ap.add_argument("--world", type=int, default=1, help="GPUs of one replica")
     ap.add_argument("--cp", action="store_true")
     ap.add_argument("--ep", action="store_true")
@@ -67,8 +61,10 @@ def main(argv=None) -> int:
     args = ap.parse_args(argv)
     cfg = _config(args)
     if not isinstance(cfg, GlmMoeDsaConfig):
-        from ..utils.sizing import plan_dense, plan_gidisun, plan_zemezen
-        planner = {"gidisun": plan_gidisun, "zemezen": plan_zemezen}.get(cfg.model_type, plan_dense)
+        from ..models.registry import hybrid_family
+        from ..utils.sizing import plan_dense
+        family = hybrid_family(cfg.model_type)
+        planner = plan_dense if family is None else family.plan
         p = planner(cfg, world=args.world, batch_size=args.batch_size, chunk_size=args.chunk_size, max_pages=args.max_pages,
                        arena_gb=args.arena, device_gb=args.device_gb)
     else:

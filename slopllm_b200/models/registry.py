@@ -82,6 +82,29 @@ MODEL_REGISTRY: Dict[str, ModelRegistration] = {
 }
 
 
+HYBRID_FAMILIES = ("gidisun", "zemezen", "vononex")      # assembled from the shared mixers
+
+
+@dataclass
+class HybridFamily:
+    config: type              # with `from_dict` (config.json) and `tiny`
+    model: type               # with `from_tensors`
+    random_tensors: Callable  # cfg -> checkpoint tensors
+    plan: Callable            # memory plan, `utils/sizing.py`
+
+
+def hybrid_family(name: str) -> Optional[HybridFamily]:
+    """The parts of a hybrid family by model type or a spec that starts with it ("zemezen-tiny"); None for other families."""
+    import importlib
+    from ..utils import sizing
+    for f in HYBRID_FAMILIES:
+        if name.startswith(f):
+            m = importlib.import_module(f".{f}", __package__)
+            return HybridFamily(getattr(m, f.capitalize() + "Config"), getattr(m, f.capitalize() + "Model"), getattr(m, f"random_{f}_tensors"),
+                                getattr(sizing, f"plan_{f}"))
+    return None
+
+
 def checkpoint_config_dir(model_dir: str) -> str:
     """A CSF container keeps the model's config under `metadata/`."""
     if not os.path.isfile(os.path.join(model_dir, "config.json")) and os.path.isfile(os.path.join(model_dir, "metadata", "config.json")):

@@ -295,3 +295,51 @@ def plan_zemezen(cfg, world: int = 1, batch_size: int = 8, chunk_size: int = 819
         return max(3 * l.ff, experts) + 8 * l.mixer["heads"] * (l.mixer["dim"] + l.mixer.get("vdim", l.mixer["dim"]))
     return _plan_hybrid(cfg, zemezen_weight_bytes(cfg, world, elem), *zemezen_cache_bytes(cfg, world, elem), max(width(l) for l in cfg.layers) // world,
                         world, batch_size, chunk_size, max_pages, arena_gb, device_gb, elem, reserve_gb)
+
+
+# ---- Vononex --------------------------------------------------------------------------------------------------------------
+
+def vononex_weight_bytes(cfg, tp: int = 1, elem: int = 2) -> int:
+    """Per-rank weight bytes, as :func:`gidisun_weight_bytes`; heads, channels and feed-forward rows are sharded with their fp32 biases,
+    norms and decays."""
+    H = cfg.hidden_size
+    b = cfg.vocab_size * H * elem + (cfg.vocab_size // tp) * H * elem + 4 * H
+    for l in cfg.layers:
+        c, ff = l.mixer, l.ff // tp
+        b += 4 * H + 3 * ff * H * elem + (4 * (2 * H + 2 * ff) if ff else 0)
+        if l.type == "mingru":
+            W = c["width"] // tp
+            b += 4 * W * H * elem + 4 * 2 * W
+            continue
+        a, r = c["left"], c["right"]
+        h, kv, hr = a["heads"] // tp, a["kv_heads"] // tp, r["heads"] // tp
+        qk = (h + kv) * a["dim"]
+        b += (qk + (h + kv) * a["vdim"]) * H * elem + 4 * (2 * qk + kv * a["vdim"] + h + H)
+        b += hr * (2 * r["dim"] + 3 * r["vdim"]) * H * elem + 4 * 2 * hr
+    return b
+
+
+def vononex_cache_bytes(cfg, tp: int = 1, elem: int = 2):
+    """(bytes of one 64-token page, bytes of one sequence's recurrent state) on one rank."""
+    page = state = 0
+    for l in cfg.layers:
+        c = l.mixer
+        if l.type == "mingru":
+            state += 4 * (c["width"] // tp)
+        else:
+            a, r = c["left"], c["right"]
+            page += (a["kv_heads"] // tp) * (a["dim"] + a["vdim"]) * elem * PAGE_SIZE
+            state += 4 * (r["heads"] // tp) * r["dim"] * r["vdim"]
+    return page, state
+
+
+def plan_vononex(cfg, world: int = 1, batch_size: int = 8, chunk_size: int = 8192, max_pages: int = 0, arena_gb: float = 0.0,
+                 device_gb: float = 180.0, elem: int = 2, reserve_gb: float = 4.0) -> MemoryPlan:
+    """`plan_memory` for Vononex (tensor parallel only)."""
+    def width(l):
+        if l.type == "mingru":
+            return max(3 * l.ff, 4 * l.mixer["width"])
+        a, r = l.mixer["left"], l.mixer["right"]
+        return max(3 * l.ff, 3 * a["heads"] * (a["dim"] + a["vdim"]) + r["heads"] * (2 * r["dim"] + 3 * r["vdim"]))
+    return _plan_hybrid(cfg, vononex_weight_bytes(cfg, world, elem), *vononex_cache_bytes(cfg, world, elem), max(width(l) for l in cfg.layers) // world,
+                        world, batch_size, chunk_size, max_pages, arena_gb, device_gb, elem, reserve_gb)
