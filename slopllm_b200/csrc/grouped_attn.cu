@@ -107,94 +107,139 @@ struct GroupedRowPreParams {
     int* guard;
 };
 
-template <int VW, typename T>
-__device__ __forceinline__ float2 load_pair(const T* p) {
-    if (VW == 1) return make_float2(to_f(p[0]), 0.f);
-    if (sizeof(T) == 4) return *reinterpret_cast<const float2*>(p);
-    return bf162_to_f2(*reinterpret_cast<const uint32_t*>(p));
-}
-template <int VW, typename T>
-__device__ __forceinline__ void store_pair(T* p, float2 x) {
-    if (VW == 1) put(p, x.x);
-    else if (sizeof(T) == 4) *reinterpret_cast<float2*>(p) = x;
-    else *reinterpret_cast<uint32_t*>(p) = f2_to_bf162(x.x, x.y);
-}
 __device__ __forceinline__ float2 turned(float2 x, float2 cs) { return make_float2(x.x * cs.x - x.y * cs.y, x.y * cs.x + x.x * cs.y); }
 __device__ __forceinline__ float2 turned_back(float2 x, float2 cs) { return make_float2(x.x * cs.x + x.y * cs.y, x.y * cs.x - x.x * cs.y); }
 
-// A block per token.  VW 2: a thread takes pairs (even sizes and strides); 1: single values, whose partner it looks up.
+// VW consecutive values: 1, 2, or 8 (16-byte accesses)
+template <int VW>
+struct Piece { float v[VW]; };
+template <int VW>
+__device__ __forceinline__ Piece<VW> load_piece(const float* p) {
+    Piece<VW> x;
+    if (VW == 1) x.v[0] = *p;
+    else if (VW == 2) *reinterpret_cast<float2*>(x.v) = *reinterpret_cast<const float2*>(p);
+    else
+#pragma unroll
+        for (int i = 0; i < VW; i += 4) *reinterpret_cast<float4*>(x.v + i) = *reinterpret_cast<const float4*>(p + i);
+    return x;
+}
+template <int VW>
+__device__ __forceinline__ Piece<VW> load_piece(const bf16* p) {
+    Piece<VW> x;
+    if (VW == 1) {
+        x.v[0] = to_f(*p);
+    } else {
+        uint32_t w[VW / 2 + 1];
+        if (VW == 8) *reinterpret_cast<uint4*>(w) = *reinterpret_cast<const uint4*>(p);
+        else w[0] = *reinterpret_cast<const uint32_t*>(p);
+#pragma unroll
+        for (int i = 0; i + 1 < VW; i += 2) *reinterpret_cast<float2*>(x.v + i) = bf162_to_f2(w[i / 2]);
+    }
+    return x;
+}
+template <int VW>
+__device__ __forceinline__ void store_piece(float* p, const Piece<VW>& x) {
+    if (VW == 1) *p = x.v[0];
+    else if (VW == 2) *reinterpret_cast<float2*>(p) = *reinterpret_cast<const float2*>(x.v);
+    else
+#pragma unroll
+        for (int i = 0; i < VW; i += 4) *reinterpret_cast<float4*>(p + i) = *reinterpret_cast<const float4*>(x.v + i);
+}
+template <int VW>
+__device__ __forceinline__ void store_piece(bf16* p, const Piece<VW>& x) {
+    if (VW == 1) {
+        put(p, x.v[0]);
+    } else {
+        uint32_t w[VW / 2 + 1];
+#pragma unroll
+        for (int i = 0; i + 1 < VW; i += 2) w[i / 2] = f2_to_bf162(x.v[i], x.v[i + 1]);
+        if (VW == 8) *reinterpret_cast<uint4*>(p) = *reinterpret_cast<const uint4*>(w);
+        else *reinterpret_cast<uint32_t*>(p) = w[0];
+    }
+}
+template <int VW>
+__device__ __forceinline__ void add_piece(Piece<VW>& x, const float* b) {
+    if (b == nullptr) return;
+    const Piece<VW> y = load_piece<VW>(b);
+#pragma unroll
+    for (int i = 0; i < VW; ++i) x.v[i] += y.v[i];
+}
+
+// A block per token, a thread takes pieces of VW values (of one head); with single values it looks up their partners.
 template <int VW, typename TI, typename TO>
-__global__ void __launch_bounds__(256) grouped_row_pre_kernel(GroupedRowPreParams p) {
+__global__ void __launch_bounds__(1024) grouped_row_pre_kernel(GroupedRowPreParams p) {
     pdl_grid_sync();
-    extern __shared__ __align__(8) float row[];          // [heads * dim | kv_heads * dim] with biases
-    __shared__ float part[2][8];
-    const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    extern __shared__ __align__(16) float row[];         // [heads * dim | kv_heads * dim] with biases
+    __shared__ float part[2][32];
+    const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, step = blockDim.x * VW;
     const int nq = p.heads * p.dim, nk = p.kv_heads * p.dim, nv = p.kv_heads * p.vdim, pos = p.positions[t];
     const TI *q = (const TI*)p.q + (size_t)t * p.ld, *k = (const TI*)p.k + (size_t)t * p.ld, *v = (const TI*)p.v + (size_t)t * p.ld;
-    float sq = 0.f, sk = 0.f;
-    for (int i = tid * VW; i < nq + nk; i += 256 * VW) {
-        const bool is_q = i < nq;
-        const int j = is_q ? i : i - nq;
-        const float* b = is_q ? p.q_bias : p.k_bias;
-        float2 x = load_pair<VW>((is_q ? q : k) + j);
-        if (b != nullptr) {
-            x.x += b[j];
-            if (VW == 2) x.y += b[j + 1];
+    const int page = p.page_table[(size_t)p.batch_idx[t] * p.pt_stride + pos / p.page_size];
+    // a row with its biases -> shared, and the sum of its squares
+    auto read = [&](const TI* src, const float* bias, float* dst, int n) {
+        float ss = 0.f;
+#pragma unroll 2
+        for (int i = tid * VW; i < n; i += step) {
+            Piece<VW> x = load_piece<VW>(src + i);
+            add_piece<VW>(x, bias != nullptr ? bias + i : nullptr);
+            store_piece<VW>(dst + i, x);
+#pragma unroll
+            for (int j = 0; j < VW; ++j) ss += x.v[j] * x.v[j];
         }
-        row[i] = x.x;
-        if (VW == 2) row[i + 1] = x.y;
-        (is_q ? sq : sk) += x.x * x.x + (VW == 2 ? x.y * x.y : 0.f);
-    }
-    sq = warp_sum(sq);
-    sk = warp_sum(sk);
+        return warp_sum(ss);
+    };
+    float sq = read(q, p.q_bias, row, nq), sk = read(k, p.k_bias, row + nq, nk);
     if (lane == 0) { part[0][warp] = sq; part[1][warp] = sk; }
     __syncthreads();
     sq = sk = 0.f;
-#pragma unroll
-    for (int i = 0; i < 8; ++i) { sq += part[0][i]; sk += part[1][i]; }
+    for (int i = 0; i < blockDim.x >> 5; ++i) { sq += part[0][i]; sk += part[1][i]; }
     if (p.sums != nullptr) { sq = p.sums[t * 2]; sk = p.sums[t * 2 + 1]; }
     const float iq = 1.f / sqrtf(sq / p.q_count + p.eps), ik = 1.f / sqrtf(sk / p.k_count + p.eps);
-    const int page = p.page_table[(size_t)p.batch_idx[t] * p.pt_stride + pos / p.page_size];
-    const long long slot = (long long)page * p.page_size + pos % p.page_size;
-    const bool cached = guard_ok(p.guard, 28, slot, p.num_slots);
-    TO *kd = (TO*)p.k_cache + (cached ? (size_t)slot * nk : 0), *vd = (TO*)p.v_cache + (cached ? (size_t)slot * nv : 0);
-    TO* qd = (TO*)p.q_out + (size_t)t * nq;
+    // pieces of a head at place d; the partner of a single value is `partner`
+    auto turn_piece = [&](Piece<VW>& x, const float2* turn, int d, int dims, float partner) {
+        if (VW == 1) {
+            if (d < dims) {
+                const float2 cs = turn[d >> 1];
+                x.v[0] = x.v[0] * cs.x + (d & 1 ? partner : -partner) * cs.y;
+            }
+            return;
+        }
+#pragma unroll
+        for (int j = 0; j + 1 < VW; j += 2) {
+            if (d + j >= dims) break;
+            const float2 y = turned(make_float2(x.v[j], x.v[j + 1]), turn[(d + j) >> 1]);
+            x.v[j] = y.x;
+            x.v[j + 1] = y.y;
+        }
+    };
     const float2* qk_turn = p.qk_turn + (size_t)t * p.ldt;
-    for (int i = tid * VW; i < nq + nk; i += 256 * VW) {
-        const bool is_q = i < nq;
-        if (!is_q && !cached) break;
-        const int j = is_q ? i : i - nq, d = j % p.dim;
-        const float* w = is_q ? p.q_norm : p.k_norm;
-        const float inv = (is_q ? iq : ik) * (is_q && p.gain != nullptr ? p.gain[j / p.dim] : 1.f);
-        float2 x = make_float2(row[i] * inv * w[j], VW == 2 ? row[i + 1] * inv * w[j + 1] : 0.f);
-        if (d < p.rot_dims) {
-            const float2 cs = qk_turn[d >> 1];
-            if (VW == 2) {
-                x = turned(x, cs);
-            } else {
-                const int o = d & 1 ? -1 : 1;
-                const float y = row[i + o] * inv * w[j + o];
-                x.x = x.x * cs.x + (d & 1 ? y : -y) * cs.y;
-            }
+    auto finish = [&](const float* src, const float* w, float inv, const float* gain, TO* dst, int n) {
+#pragma unroll 2
+        for (int i = tid * VW; i < n; i += step) {
+            const int h = i / p.dim, d = i - h * p.dim;
+            const float f = gain != nullptr ? inv * gain[h] : inv;
+            Piece<VW> x = load_piece<VW>(src + i);
+            const Piece<VW> g = load_piece<VW>(w + i);
+#pragma unroll
+            for (int j = 0; j < VW; ++j) x.v[j] *= f * g.v[j];
+            const int o = i + (d & 1 ? -1 : 1);
+            turn_piece(x, qk_turn, d, p.rot_dims, VW == 1 && d < p.rot_dims ? src[o] * f * w[o] : 0.f);
+            store_piece<VW>(dst + i, x);
         }
-        store_pair<VW>((is_q ? qd : kd) + j, x);
-    }
-    if (!cached) return;
-    const float2* v_turn = p.v_turn != nullptr ? p.v_turn + (size_t)t * p.ldt : nullptr;
-    auto value = [&](int i) { return to_f(v[i]) + (p.v_bias != nullptr ? p.v_bias[i] : 0.f); };
-    for (int i = tid * VW; i < nv; i += 256 * VW) {
-        const int d = i % p.vdim;
-        float2 x = make_float2(value(i), VW == 2 ? value(i + 1) : 0.f);
-        if (v_turn != nullptr) {
-            const float2 cs = v_turn[d >> 1];
-            if (VW == 2) {
-                x = turned(x, cs);
-            } else {
-                const float y = value(i + (d & 1 ? -1 : 1));
-                x.x = x.x * cs.x + (d & 1 ? y : -y) * cs.y;
-            }
+    };
+    finish(row, p.q_norm, iq, p.gain, (TO*)p.q_out + (size_t)t * nq, nq);
+    const long long slot = (long long)page * p.page_size + pos % p.page_size;
+    if (!guard_ok(p.guard, 28, slot, p.num_slots)) return;
+    finish(row + nq, p.k_norm, ik, nullptr, (TO*)p.k_cache + (size_t)slot * nk, nk);
+    TO* vd = (TO*)p.v_cache + (size_t)slot * nv;
+    for (int i = tid * VW; i < nv; i += step) {
+        Piece<VW> x = load_piece<VW>(v + i);
+        add_piece<VW>(x, p.v_bias != nullptr ? p.v_bias + i : nullptr);
+        if (p.v_turn != nullptr) {
+            const int d = i % p.vdim, o = i + (d & 1 ? -1 : 1);
+            turn_piece(x, p.v_turn + (size_t)t * p.ldt, d, p.vdim, VW == 1 ? to_f(v[o]) + (p.v_bias != nullptr ? p.v_bias[o] : 0.f) : 0.f);
         }
-        store_pair<VW>(vd + i, x);
+        store_piece<VW>(vd + i, x);
     }
 }
 
@@ -530,19 +575,22 @@ SL_API int sl_grouped_row_pre(const GroupedRowPreParams* p, int T, int in_f32, i
     const size_t smem = (size_t)(p->heads + p->kv_heads) * p->dim * sizeof(float);
     if (smem > 200 * 1024) return -1;
     const uintptr_t at = (uintptr_t)p->q | (uintptr_t)p->k | (uintptr_t)p->v;
-    const bool pairs = p->dim % 2 == 0 && p->vdim % 2 == 0 && p->ld % 2 == 0 && at % (in_f32 ? 8 : 4) == 0;
+    auto pieces = [&](int vw) { return p->dim % vw == 0 && p->vdim % vw == 0 && p->ld % vw == 0 && at % (vw == 8 ? 16 : vw * (in_f32 ? 4 : 2)) == 0; };
+    const int vw = pieces(8) ? 8 : pieces(2) ? 2 : 1;
+    // few rows: a thread takes one piece of the row where it can
+    const int threads = T > 148 ? (vw == 8 ? 128 : 256) : max(128, min(1024, (p->heads * p->dim / vw + 31) / 32 * 32));
 #define SL_RP(VW, TI, TO)                                                                                              \
     {                                                                                                                  \
         auto kern = grouped_row_pre_kernel<VW, TI, TO>;                                                                \
         if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);      \
-        sl_launch(kern, T, 256, smem, s, *p);                                                                          \
+        sl_launch(kern, T, threads, smem, s, *p);                                                                      \
     }
     if (out_f32) {
-        if (pairs) SL_RP(2, float, float) else SL_RP(1, float, float)
+        if (vw == 8) SL_RP(8, float, float) else if (vw == 2) SL_RP(2, float, float) else SL_RP(1, float, float)
     } else if (in_f32) {
-        if (pairs) SL_RP(2, float, bf16) else SL_RP(1, float, bf16)
+        if (vw == 8) SL_RP(8, float, bf16) else if (vw == 2) SL_RP(2, float, bf16) else SL_RP(1, float, bf16)
     } else {
-        if (pairs) SL_RP(2, bf16, bf16) else SL_RP(1, bf16, bf16)
+        if (vw == 8) SL_RP(8, bf16, bf16) else if (vw == 2) SL_RP(2, bf16, bf16) else SL_RP(1, bf16, bf16)
     }
 #undef SL_RP
     return SL_LAUNCH_CHECK();

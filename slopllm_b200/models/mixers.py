@@ -194,12 +194,12 @@ class Retention:
 
 @dataclass
 class SideBySide:
-    """Mixers that read the same input and whose outputs are added: one input product makes the rows of all, one output product takes
-    their results side by side."""
+    """Two mixers that read the same input and whose outputs are added: one input product makes the rows of both, which then run at
+    the same time, and one output product takes their results side by side."""
 
     index: int
     kind: str
-    parts: list                      # mixers with `mix`
+    parts: list                      # the mixers (with `mix`)
     rows: List[int]                  # projection rows of each
     outs: List[int]                  # values that each hands to `w_out`
     w_in: LinearWeight
@@ -214,10 +214,10 @@ class SideBySide:
     def __call__(self, model, x, st, cache):
         main = model.ops.linear(x, self.w_in, out_f32=x.shape[0] <= SMALL_T)
         both = torch.empty(x.shape[0], sum(self.outs), dtype=x.dtype, device=x.device)
-        r = o = 0
-        for m, nr, no in zip(self.parts, self.rows, self.outs):
-            m.mix(model, main[:, r:r + nr], None, st, cache, both[:, o:o + no])
-            r, o = r + nr, o + no
+        model.angles.of(st), RC.ChunkPlan.of(st)          # (made in front of the fork: both mixers read them)
+        (a, b), r, o = self.parts, self.rows[0], self.outs[0]
+        model.ops.together(lambda: a.mix(model, main[:, :r], None, st, cache, both[:, :o]),
+                           lambda: b.mix(model, main[:, r:r + self.rows[1]], None, st, cache, both[:, o:]))
         return model.ops.linear(both, self.w_out, out_f32=True)
 
 

@@ -29,6 +29,10 @@ class RefOps:
         self.cfg = cfg
         self.ctx = ctx
 
+    def together(self, first, second):
+        second()
+        first()
+
     # -- elementwise / linear -------------------------------------------------------------
     def embed(self, ids, table):
         return table[ids.to(torch.int64)].to(torch.float32)

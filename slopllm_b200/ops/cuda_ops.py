@@ -54,6 +54,7 @@ class CudaOps:
         self.act_dtype = act_dtype      # fp32: families whose kernels exist in both types (every product on the CUDA cores)
         N.kernels()            # fail loudly when the native library is missing
         self._counters = {}
+        self._side = None               # second stream of `together`
         from ..config import env_str
         # one-launch persistent decode MoE (csrc/moe_persist.cu): opt-in.  Its NVFP4 -> f16 expansion is bound by the
         # conversion rate of the CUDA cores just like the five-launch path, which it does not yet beat below 32 rows
@@ -62,6 +63,18 @@ class CudaOps:
         self._fp4_decode_force = env_str("MOE_FP4_DECODE")          # "0" / "1": never / always the FP4 GEMMs for decode-sized MoE
         self._persist_gsub = 0         # gate/up sub-tiles per tile of the persistent MoE kernel (0: the kernel's default)
         self._persist_trace = None     # u64 [SMs, 96, 4] tile timeline, filled when set (profiling)
+
+    def together(self, first, second) -> None:
+        """Run two pieces of work that do not depend on each other at the same time: `second` on a stream of its own between a fork
+        and a join of the current one (in a capture, a branch of the graph).  What both read must exist before."""
+        here = torch.cuda.current_stream()
+        if self._side is None:
+            self._side = torch.cuda.Stream(here.device)
+        self._side.wait_stream(here)
+        with torch.cuda.stream(self._side):
+            second()
+        first()
+        here.wait_stream(self._side)
 
     # -- helpers ----------------------------------------------------------------------------
     @staticmethod
