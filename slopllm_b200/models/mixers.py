@@ -19,6 +19,8 @@ from ..ops.rotary import RotaryTable, Turn
 from ..utils.tracing import traced
 from .weights import ExpertWeights, LinearWeight
 
+TOGETHER_MAX = 12 << 20      # output values of a step (tokens x width) up to which mixers side by side run at the same time: larger
+                             # ones fill the GPU alone and only get in each other's way
 SMALL_T = 32         # up to this many rows a layer's input projections are one fp32-output product (weight streaming)
 
 
@@ -216,8 +218,12 @@ class SideBySide:
         both = torch.empty(x.shape[0], sum(self.outs), dtype=x.dtype, device=x.device)
         model.angles.of(st), RC.ChunkPlan.of(st)          # (made in front of the fork: both mixers read them)
         (a, b), r, o = self.parts, self.rows[0], self.outs[0]
-        model.ops.together(lambda: a.mix(model, main[:, :r], None, st, cache, both[:, :o]),
-                           lambda: b.mix(model, main[:, r:r + self.rows[1]], None, st, cache, both[:, o:]))
+        first = lambda: a.mix(model, main[:, :r], None, st, cache, both[:, :o])
+        second = lambda: b.mix(model, main[:, r:r + self.rows[1]], None, st, cache, both[:, o:])
+        if both.numel() <= TOGETHER_MAX:
+            model.ops.together(first, second)
+        else:
+            first(), second()
         return model.ops.linear(both, self.w_out, out_f32=True)
 
 

@@ -349,6 +349,19 @@ def test_engine_mixed_batches_and_reused_slots(dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+def test_mixers_of_a_layer_in_turn_give_the_same(dtype, monkeypatch):
+    """A second stream for one of the two mixers changes no result."""
+    from slopllm_b200.models import mixers
+    raw = CONFIGS["tiled"]
+    t = O.random_tensors(raw, 5)
+    ids = random_ids(raw, 150, 8)
+    cuts = portions(150, [70, 3], tail=30)
+    a = feed(make_engine(raw, t, "cuda", dtype), ids, cuts)
+    monkeypatch.setattr(mixers, "TOGETHER_MAX", 0)
+    assert torch.equal(a, feed(make_engine(raw, t, "cuda", dtype), ids, cuts))
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
 def test_long_decoding(dtype):
     """Hundreds of decoded tokens over page borders, in a graph."""
     raw, t = far_key_model()

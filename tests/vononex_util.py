@@ -31,6 +31,8 @@ def configs():
         "wide": O.config([O.parallel_layer(heads=20, kv_heads=1, dim=64, vdim=136, base=1e6, r_heads=2, r_dim=136, r_vdim=160, r_dims=128, ff=96),
                           O.parallel_layer(heads=3, kv_heads=3, dim=160, vdim=200, dims=64, r_heads=6, r_dim=64, r_vdim=96),
                           O.mingru_layer(width=264, ff=64)], width=128, vocab=257),
+        # no attention, so no paged rows at all
+        "recurrent": O.config([O.mingru_layer(width=24, ff=40), O.mingru_layer(width=72)], width=48, vocab=61, alpha=0.5),
     }
 
 
