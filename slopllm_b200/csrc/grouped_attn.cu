@@ -397,18 +397,18 @@ __global__ void __launch_bounds__(DT) grouped_decode_kernel(GroupedAttnParams p)
                 slot = guard_ok(p.guard, 27, s, p.num_slots) ? s : -1;
             }
             bf16 *kd = ks + (st * KT + warp * 16) * ld, *vd = vs + (st * KT + warp * 16) * ldv;
-            for (int i = lane; i < 16 * kpc; i += 32) {
-                const int r = i / kpc, c = i % kpc * 8;
-                const long long s = __shfl_sync(__activemask(), slot, r);
-                if (s >= 0) cp_async16(kd + r * ld + c, kc + (size_t)s * krow + c);
-                else *reinterpret_cast<uint4*>(kd + r * ld + c) = make_uint4(0, 0, 0, 0);
-            }
-            for (int i = lane; i < 16 * vpc; i += 32) {
-                const int r = i / vpc, c = i % vpc * 8;
-                const long long s = __shfl_sync(__activemask(), slot, r);
-                if (s >= 0) cp_async16(vd + r * ldv + c, vc + (size_t)s * vrow + c);
-                else *reinterpret_cast<uint4*>(vd + r * ldv + c) = make_uint4(0, 0, 0, 0);
-            }
+            // (all lanes take part in every shuffle: a lane that left its last round early could not be read)
+            auto copy = [&](bf16* dst, int dld, const bf16* src, size_t row, int pieces) {
+                for (int i0 = 0; i0 < 16 * pieces; i0 += 32) {
+                    const int i = i0 + lane, r = i / pieces, c = i % pieces * 8;
+                    const long long s = __shfl_sync(0xffffffffu, slot, r & 15);
+                    if (r >= 16) continue;
+                    if (s >= 0) cp_async16(dst + r * dld + c, src + (size_t)s * row + c);
+                    else *reinterpret_cast<uint4*>(dst + r * dld + c) = make_uint4(0, 0, 0, 0);
+                }
+            };
+            copy(kd, ld, kc, krow, kpc);
+            copy(vd, ldv, vc, vrow, vpc);
         }
         cp_async_commit();
     };

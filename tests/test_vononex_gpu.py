@@ -171,6 +171,16 @@ def test_one_far_key(vdim, dtype):
     assert rel(a, b) > 0.2                                        # the planted key decides the row
 
 
+@pytest.mark.parametrize("dim", range(8, 137, 8))
+def test_every_size_of_whole_pieces(dim):
+    """Heads of every multiple of eight values, decoded and in portions: rows of a tile are copied by lanes that share them unevenly."""
+    for i, vdim in enumerate((8, 24, 40, 56, 64, 88, 104, 136)):
+        kv = 1 + i % 2
+        for spans in ([(70, 1), (5, 1), (128, 1)], [(20, 70), (66, 2)]):
+            got, want = attention_case(spans, 2 * kv, kv, dim, vdim, dim - 8 * (i % 2) if dim > 8 else dim, torch.bfloat16, seed=vdim)
+            assert rel(got, want) < 1.2e-2, (vdim, spans)
+
+
 def test_decode_key_splits():
     """Long contexts: the keys of one row are shared by several blocks, whose sum is turned back once."""
     for spans in ([(1500, 1), (700, 1)], [(1999, 1)], [(64 * i + 5, 1) for i in range(40)]):
@@ -236,6 +246,15 @@ def test_retention(lens, h, dk, dv, dims, decays, dtype):
             for slot, x in S_want.items():
                 assert rel(S[slot], x) < 1e-5, plan
             assert rel(got, want) < (2e-5 if dtype == torch.float32 else 4e-3), plan
+
+
+@pytest.mark.parametrize("dk", range(8, 137, 8))
+def test_retention_of_every_size_of_whole_pieces(dk):
+    for i, dv in enumerate((8, 24, 40, 56, 64, 88, 136)):
+        args, want, S_want = retention_case([70, 1, 18], 2, dk, dv, dk - 2 * (i % 3), torch.bfloat16, [0.97, 0.999], seed=dv)
+        for plan in (None, RC.ChunkPlan([70, 1, 18], "cuda")):
+            got, S = run_retention(args, torch.bfloat16, plan)
+            assert all(rel(S[slot], x) < 1e-5 for slot, x in S_want.items()) and rel(got, want) < 4e-3, (dv, plan)
 
 
 def test_retention_chunks_follow_the_step_kernel():

@@ -119,7 +119,7 @@ def attention_case(spans, heads, kv, dim, window, keep, dtype, dims=None, sink=N
     return wide[:, :heads * vdim], torch.cat(want)
 
 
-SHAPES = [(4, 2, 16), (6, 2, 40), (3, 3, 128), (20, 1, 64), (16, 2, 96), (2, 1, 256), (4, 2, 12), (1, 1, 8)]
+SHAPES = [(4, 2, 16), (6, 2, 40), (3, 3, 128), (20, 1, 64), (16, 2, 96), (2, 1, 256), (4, 2, 12), (1, 1, 8), (2, 2, 56), (3, 1, 104)]
 SPANS = [[(0, 130), (70, 3), (200, 1), (5, 64)], [(150, 1), (3, 1), (0, 1), (256, 1)], [(127, 2)], [(0, 1)], [(300, 40)]]
 
 
