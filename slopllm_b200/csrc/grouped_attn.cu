@@ -399,12 +399,19 @@ __global__ void __launch_bounds__(DT) grouped_decode_kernel(GroupedAttnParams p)
             bf16 *kd = ks + (st * KT + warp * 16) * ld, *vd = vs + (st * KT + warp * 16) * ldv;
             // (all lanes take part in every shuffle: a lane that left its last round early could not be read)
             auto copy = [&](bf16* dst, int dld, const bf16* src, size_t row, int pieces) {
+                int r = lane / pieces, c = lane - r * pieces;
+                const int dr = 32 / pieces, dc = 32 - dr * pieces;
+#pragma unroll 4
                 for (int i0 = 0; i0 < 16 * pieces; i0 += 32) {
-                    const int i = i0 + lane, r = i / pieces, c = i % pieces * 8;
                     const long long s = __shfl_sync(0xffffffffu, slot, r & 15);
-                    if (r >= 16) continue;
-                    if (s >= 0) cp_async16(dst + r * dld + c, src + (size_t)s * row + c);
-                    else *reinterpret_cast<uint4*>(dst + r * dld + c) = make_uint4(0, 0, 0, 0);
+                    bf16* to = dst + r * dld + c * 8;
+                    if (r < 16) {
+                        if (s >= 0) cp_async16(to, src + (size_t)s * row + c * 8);
+                        else *reinterpret_cast<uint4*>(to) = make_uint4(0, 0, 0, 0);
+                    }
+                    r += dr;
+                    c += dc;
+                    if (c >= pieces) { c -= pieces; ++r; }
                 }
             };
             copy(kd, ld, kc, krow, kpc);
