@@ -1,7 +1,7 @@
 // Grouped-query attention over a paged cache: query / key norm, rotary table, sliding window with kept first tokens, softmax
 // sink, values of their own or the key projections themselves.  (Portions of prompts attend in latent_mma.cu.)
 //
-//  * grouped_pre_kernel: per-head RMS norm and rotate-half of queries and keys; keys and values go into their cache slots.
+//  * grouped_pre_kernel: biases, per-head RMS norm and rotate-half of queries and keys; keys and values go into their cache slots.
 //  * grouped_row_pre_kernel: the same step for norms over the whole query / key rows: biases, norms, rotation of adjacent pairs from
 //    a table of angles, a factor per query head, and values that turn with their position.
 //  * grouped_rows_kernel: independent token rows on the CUDA cores, any sizes, bf16 or fp32.
@@ -32,9 +32,11 @@ struct GroupedPreParams {
     const float* freq; float rot_gain, eps;
     const int* positions; const int* batch_idx; const int* page_table;
     int pt_stride, page_size;
-    void *k_cache, *v_cache; int num_slots;      // [slots, kv_heads, dim], [slots, kv_heads, vdim]
+    void *k_cache, *v_cache; int num_slots;      // [slots, kv_heads, dim], [slots, v_heads, vdim]
     void* q_out;                         // [T, heads, dim]
     int* guard;
+    int v_heads;                         // at most kv_heads
+    const float *q_bias, *k_bias, *v_bias;       // per projection row, or null
 };
 
 // grid (T, ceil((heads + kv_heads) / 8)), block 256: a warp per head
@@ -58,9 +60,10 @@ __global__ void __launch_bounds__(256) grouped_pre_kernel(GroupedPreParams p) {
     float inv = 1.f;
     if (on) {
         const TI* src = (const TI*)(is_q ? p.q : p.k) + (size_t)t * p.ld + (size_t)h * p.dim;
+        const float* bias = is_q ? p.q_bias : p.k_bias;
         float ss = 0.f;
         for (int i = lane; i < p.dim; i += 32) {
-            const float v = to_f(src[i]);
+            const float v = to_f(src[i]) + (bias != nullptr ? bias[h * p.dim + i] : 0.f);
             x[i] = v;
             ss += v * v;
         }
@@ -80,8 +83,9 @@ __global__ void __launch_bounds__(256) grouped_pre_kernel(GroupedPreParams p) {
         if (!guard_ok(p.guard, 25, slot, p.num_slots)) return;
         dst = (TO*)p.k_cache + ((size_t)slot * p.kv_heads + h) * p.dim;
         const TI* vs = (const TI*)p.v + (size_t)t * p.ld + (size_t)h * p.vdim;
-        TO* vd = (TO*)p.v_cache + ((size_t)slot * p.kv_heads + h) * p.vdim;
-        for (int i = lane; i < p.vdim; i += 32) put(vd + i, to_f(vs[i]));
+        TO* vd = (TO*)p.v_cache + ((size_t)slot * p.v_heads + h) * p.vdim;
+        if (h < p.v_heads)
+            for (int i = lane; i < p.vdim; i += 32) put(vd + i, to_f(vs[i]) + (p.v_bias != nullptr ? p.v_bias[h * p.vdim + i] : 0.f));
     }
     for (int i = lane; i < p.dim; i += 32) {
         float v = x[i];
@@ -566,7 +570,7 @@ size_t decode_smem(int dim, int vdim) {
 
 SL_API int sl_grouped_pre(const GroupedPreParams* p, int T, int in_f32, int out_f32, cudaStream_t s) {
     if (T == 0) return 0;
-    if (p->rot_dims > p->dim || p->rot_dims % 2 != 0 || (out_f32 && !in_f32)) return -1;
+    if (p->rot_dims > p->dim || p->rot_dims % 2 != 0 || (out_f32 && !in_f32) || p->v_heads > p->kv_heads) return -1;
     const size_t smem = (size_t)(p->rot_dims + 8 * p->dim) * sizeof(float);
     if (smem > 48 * 1024) return -1;
     const dim3 grid(T, (p->heads + p->kv_heads + 7) / 8);

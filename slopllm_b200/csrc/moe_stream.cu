@@ -1,13 +1,14 @@
 // Mixture of small SwiGLU experts with plain (bf16 or fp32) weights.
 //
-//  * route_softmax_kernel: softmax scores, group-limited choice, a warp per token.
+//  * route_softmax_kernel: softmax scores, group-limited choice by corrected scores, a warp per token.
 //  * expert_gate_up_kernel, expert_down_kernel: a block takes rows of one expert's matrix and streams them past the tokens that
 //    chose the expert, so weights are read once a step and experts that nobody chose are not read at all.
 //      - tensor-core form (bf16, rows of whole 16-byte pieces): 16 rows per block, the reduction is split over the warps;
 //        operands go from global memory to fragments directly (both sides use the same permutation of the reduction index, so a
 //        thread's 16 bytes are two k-steps of its fragment)
 //      - plain form: any sizes, fp32 or bf16
-//  * expert_sum_kernel: weighted sum of a token's routes, added to its output row.
+//  * expert_sum_kernel: weighted sum of a token's routes, added to its output row; identity experts (ids behind the experts') hand the
+//    input through.  identity_experts_kernel adds those alone.
 #include "common.cuh"
 #include "mma_sync.cuh"
 
@@ -24,7 +25,7 @@ constexpr int MAX_GROUPS = 256, ROUTE_WARPS = 4;
 // NPL: experts per lane (E <= 32 * NPL); lane l holds experts l, l + 32, ...
 template <int NPL>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_softmax_kernel(int* __restrict__ ids, float* __restrict__ wts, const float* __restrict__ logits,
-                                                                         int ld, int T, int E, int top, int groups, int keep) {
+                                                                         int ld, const float* __restrict__ correction, int T, int E, int top, int groups, int keep) {
     pdl_grid_sync();
     __shared__ float best[ROUTE_WARPS][MAX_GROUPS];
     __shared__ bool kept[ROUTE_WARPS][MAX_GROUPS];
@@ -49,13 +50,19 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_softmax_kernel(int* __
     const int gsz = E / groups;
 #pragma unroll
     for (int i = 0; i < NPL; ++i) s[i] *= inv;
+    float c[NPL];                                         // what the choice goes by
+#pragma unroll
+    for (int i = 0; i < NPL; ++i) c[i] = s[i] + (correction != nullptr && lane + i * 32 < E ? correction[lane + i * 32] : 0.f);
     if (groups > 1) {
-        for (int g = lane; g < groups; g += 32) best[warp][g] = -1.f;
+        for (int g = lane; g < groups; g += 32) best[warp][g] = -INFINITY;
         __syncwarp();
 #pragma unroll
         for (int i = 0; i < NPL; ++i) {
-            const int e = lane + i * 32;                  // (scores are not negative: their order is that of their bits)
-            if (e < E) atomicMax(reinterpret_cast<int*>(&best[warp][e / gsz]), __float_as_int(s[i]));
+            const int e = lane + i * 32;
+            if (e >= E) continue;
+            // (the order of numbers from zero up is that of their bits, below zero the reverse of it)
+            if (c[i] >= 0.f) atomicMax(reinterpret_cast<int*>(&best[warp][e / gsz]), __float_as_int(c[i] + 0.f));
+            else atomicMin(reinterpret_cast<unsigned*>(&best[warp][e / gsz]), __float_as_uint(c[i]));
         }
         __syncwarp();
         for (int g = lane; g < groups; g += 32) {
@@ -72,11 +79,11 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_softmax_kernel(int* __
         if (e >= E || (groups > 1 && !kept[warp][e / gsz])) taken |= 1u << i;
     }
     for (int r = 0; r < top; ++r) {
-        float v = -1.f;
+        float v = -INFINITY, weight = 0.f;
         int id = 0x7fffffff, mine = 0;
 #pragma unroll
         for (int i = 0; i < NPL; ++i)
-            if (!((taken >> i) & 1u) && s[i] > v) { v = s[i]; id = lane + i * 32; mine = i; }
+            if (!((taken >> i) & 1u) && c[i] > v) { v = c[i]; weight = s[i]; id = lane + i * 32; mine = i; }
         const int my_id = id;
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) {
@@ -84,10 +91,13 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_softmax_kernel(int* __
             const int oid = __shfl_xor_sync(0xffffffffu, id, o);
             if (ov > v || (ov == v && oid < id)) { v = ov; id = oid; }
         }
-        if (my_id == id && id < E) taken |= 1u << mine;
-        if (lane == 0) {
-            ids[(size_t)t * top + r] = id < E ? id : 0;
-            wts[(size_t)t * top + r] = id < E ? v : 0.f;
+        if (my_id == id && id < E) {                      // (one lane: ids differ between the lanes)
+            taken |= 1u << mine;
+            ids[(size_t)t * top + r] = id;
+            wts[(size_t)t * top + r] = weight;
+        } else if (id >= E && lane == 0) {                // (logits that are no numbers)
+            ids[(size_t)t * top + r] = 0;
+            wts[(size_t)t * top + r] = 0.f;
         }
     }
 }
@@ -100,6 +110,7 @@ struct ExpertStreamParams {
     void* act;                           // [T * top, I]
     float* y_route;                      // [T * top, H]
     float* out; int ldo;                 // [T, ldo], added to
+    int identity;                        // ids from E on: the input times the weight is added (else nothing)
 };
 
 constexpr int LIST = 1024;               // routes looked through at a time
@@ -278,24 +289,52 @@ __global__ void __launch_bounds__(256) expert_mma_kernel(ExpertStreamParams p) {
 }
 
 // grid (ceil(H / 256), T)
+template <typename T>
 __global__ void __launch_bounds__(256) expert_sum_kernel(ExpertStreamParams p) {
     pdl_grid_sync();
     const int n = blockIdx.x * 256 + threadIdx.x, t = blockIdx.y;
     if (n >= p.H) return;
     float a = p.out[(size_t)t * p.ldo + n];
 #pragma unroll 8
-    for (int j = 0; j < p.top; ++j) a += p.wts[t * p.top + j] * p.y_route[((size_t)t * p.top + j) * p.H + n];
+    for (int j = 0; j < p.top; ++j) {
+        const float w = p.wts[t * p.top + j];
+        if (p.ids[t * p.top + j] < p.E) a += w * p.y_route[((size_t)t * p.top + j) * p.H + n];
+        else if (p.identity) a += w * to_f(((const T*)p.x)[(size_t)t * p.ldx + n]);
+    }
     p.out[(size_t)t * p.ldo + n] = a;
+}
+
+// out[t] += x[t] * sum of the weights of t's identity experts.  grid (ceil(H / (256 VW)), T)
+template <int VW, typename T>
+__global__ void __launch_bounds__(256) identity_experts_kernel(float* __restrict__ out, int ldo, const T* __restrict__ x, int ldx, const int* __restrict__ ids,
+                                                               const float* __restrict__ wts, int top, int H, int E) {
+    pdl_grid_sync();
+    const int n = (blockIdx.x * 256 + threadIdx.x) * VW, t = blockIdx.y;
+    if (n >= H) return;
+    float w = 0.f;
+    for (int j = 0; j < top; ++j) w += ids[t * top + j] >= E ? wts[t * top + j] : 0.f;
+    if (w == 0.f) return;
+    float* o = out + (size_t)t * ldo + n;
+    const T* v = x + (size_t)t * ldx + n;
+    if (VW == 4) {
+        const uint2 u = *reinterpret_cast<const uint2*>(v);           // (bf16 only)
+        const float2 a = bf162_to_f2(u.x), b = bf162_to_f2(u.y);
+        float4 r = *reinterpret_cast<float4*>(o);
+        r.x += w * a.x; r.y += w * a.y; r.z += w * b.x; r.w += w * b.y;
+        *reinterpret_cast<float4*>(o) = r;
+    } else {
+        *o += w * to_f(*v);
+    }
 }
 
 }  // namespace
 
-// logits fp32 [T, ld].  E <= 1024, groups <= 256 equal runs, top <= experts of the kept groups.
-SL_API int sl_route_softmax(void* ids, void* wts, const void* logits, int ld, int T, int E, int top, int groups, int keep, cudaStream_t s) {
+// logits fp32 [T, ld]; correction fp32 [E] or null.  E <= 1024, groups <= 256 equal runs, top <= experts of the kept groups.
+SL_API int sl_route_softmax(void* ids, void* wts, const void* logits, int ld, const void* correction, int T, int E, int top, int groups, int keep, cudaStream_t s) {
     if (T == 0) return 0;
     if (E < 1 || E > 1024 || groups < 1 || groups > MAX_GROUPS || E % groups != 0 || keep < 1 || keep > groups || top < 1 || top > keep * (E / groups)) return -1;
     const int blocks = (T + ROUTE_WARPS - 1) / ROUTE_WARPS;
-#define SL_RS(N) sl_launch(route_softmax_kernel<N>, blocks, ROUTE_WARPS * 32, 0, s, (int*)ids, (float*)wts, (const float*)logits, ld, T, E, top, groups, keep)
+#define SL_RS(N) sl_launch(route_softmax_kernel<N>, blocks, ROUTE_WARPS * 32, 0, s, (int*)ids, (float*)wts, (const float*)logits, ld, (const float*)correction, T, E, top, groups, keep)
     if (E <= 32) SL_RS(1);
     else if (E <= 64) SL_RS(2);
     else if (E <= 128) SL_RS(4);
@@ -326,6 +365,19 @@ SL_API int sl_expert_stream(const ExpertStreamParams* p, int f32, cudaStream_t s
         sl_launch(expert_gate_up_plain_kernel<bf16>, dim3((p->I + 7) / 8, p->E), 256, 0, s, *p);
         sl_launch(expert_down_plain_kernel<bf16>, dim3((p->H + 7) / 8, p->E), 256, 0, s, *p);
     }
-    sl_launch(expert_sum_kernel, dim3((p->H + 255) / 256, p->T), 256, 0, s, *p);
+    if (f32) sl_launch(expert_sum_kernel<float>, dim3((p->H + 255) / 256, p->T), 256, 0, s, *p);
+    else sl_launch(expert_sum_kernel<bf16>, dim3((p->H + 255) / 256, p->T), 256, 0, s, *p);
+    return SL_LAUNCH_CHECK();
+}
+
+// out fp32 [T, ldo] += x [T, ldx] times the weights of the routes (ids, wts [T, top]) whose id is E or more
+SL_API int sl_identity_experts(float* out, int ldo, const void* x, int ldx, const int* ids, const float* wts, int T, int top, int H, int E, int f32,
+                               cudaStream_t s) {
+    if (T == 0) return 0;
+    if (T > 65535) return -1;
+    const bool v4 = !f32 && H % 4 == 0 && ldo % 4 == 0 && ldx % 4 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)x % 8 == 0;
+    if (f32) sl_launch(identity_experts_kernel<1, float>, dim3((H + 255) / 256, T), 256, 0, s, out, ldo, (const float*)x, ldx, ids, wts, top, H, E);
+    else if (v4) sl_launch(identity_experts_kernel<4, bf16>, dim3((H / 4 + 255) / 256, T), 256, 0, s, out, ldo, (const bf16*)x, ldx, ids, wts, top, H, E);
+    else sl_launch(identity_experts_kernel<1, bf16>, dim3((H + 255) / 256, T), 256, 0, s, out, ldo, (const bf16*)x, ldx, ids, wts, top, H, E);
     return SL_LAUNCH_CHECK();
 }

@@ -15,6 +15,7 @@ from ..ops import experts as EX
 from ..ops import grouped as G
 from ..ops import latent as L
 from ..ops import recurrent as RC
+from ..ops import talking as TK
 from ..ops.rotary import RotaryTable, Turn
 from ..utils.tracing import traced
 from .weights import ExpertWeights, LinearWeight
@@ -268,6 +269,50 @@ class GatedFeedForward:
 
 
 @dataclass
+class FeedForward:
+    """act(up x), projected down."""
+
+    index: int
+    w_in: LinearWeight               # up
+    w_out: LinearWeight
+    act: str = "gelu_tanh"
+
+    @traced(lambda self, *a, **k: f"layer{self.index}.mlp")
+    def __call__(self, model, x, st, cache):
+        up = model.ops.linear(x, self.w_in)
+        act = torch.empty(x.shape[0], up.shape[1], dtype=x.dtype, device=x.device)
+        model.ops.plain_act(up, act, self.act)
+        return model.ops.linear(act, self.w_out, out_f32=True)
+
+
+@dataclass
+class TalkingAttention:
+    """Grouped-query attention inside chunks whose heads' scores are mixed before the softmax, over its own keys and values or those of
+    another layer's cache (`ops/talking.py`)."""
+
+    index: int
+    kv_index: int                    # layer whose cache holds the keys and values
+    shape: TK.TalkingShape
+    w: TK.TalkingWeights
+    w_in: LinearWeight               # q (| k | v, with keys of its own)
+    o_proj: LinearWeight
+
+    @property
+    def spec(self) -> CacheSpec:
+        s = self.shape
+        return CacheSpec(rows={"k": (s.kv_heads, s.dim), "v": (s.v_heads, s.vdim)}) if self.kv_index == self.index else CacheSpec()
+
+    @traced(lambda self, *a, **k: f"layer{self.index}.talking_attention")
+    def __call__(self, model, x, st, cache):
+        s, rows = self.shape, cache.rows[self.kv_index]
+        proj = model.ops.linear(x, self.w_in, out_f32=x.shape[0] <= SMALL_T)
+        q = TK.talking_pre(proj, s, self.w, st, rows["k"], rows["v"], x.dtype)
+        out = torch.empty(x.shape[0], s.out_heads * s.vdim, dtype=x.dtype, device=x.device)
+        TK.talking_attention(q, s, self.w, st, rows["k"], rows["v"], out)
+        return model.ops.linear(out, self.o_proj, out_f32=True)
+
+
+@dataclass
 class ChannelDelta:
     """Gated delta rule with a decay per key channel behind short convolutions (`ops/delta.py`).  Projection rows: q | k | v, and
     with fp32 results low-rank decay input | low-rank gate input | beta."""
@@ -291,16 +336,49 @@ class ChannelDelta:
 
 @dataclass
 class Experts:
-    """Softmax-routed SwiGLU experts (`ops/experts.py`); the router's logits come from the caller's projection."""
+    """Softmax-routed SwiGLU experts (`ops/experts.py`); the router's logits come from the caller's projection.  Router outputs behind the
+    experts' are identity experts, whose output is the input."""
 
     w: ExpertWeights
     top: int
     groups: int = 1
     keep: int = 1
+    correction: Optional[torch.Tensor] = None     # fp32, added to the scores when experts are chosen
+    identity: bool = True                         # this rank adds the identity experts' outputs
 
     def add(self, model, x, logits, out):
-        ids, wts = EX.route_softmax(logits, self.top, self.groups, self.keep)
-        EX.add_experts(x, self.w, ids, wts, out, model.ops)
+        ids, wts = EX.route_softmax(logits, self.top, self.groups, self.keep, self.correction)
+        EX.add_experts(x, self.w, ids, wts, out, model.ops, self.identity and logits.shape[1] > self.w.num_experts)
+
+
+@dataclass
+class RoutedFeedForward:
+    """Routed experts and, if `w_out` is given, a shared expert behind a sigmoid gate: one product makes its rows, the router's logits and
+    the gate."""
+
+    index: int
+    w_in: LinearWeight               # shared gate | shared up and then, with fp32 results, router | gate of the shared expert
+    w_out: Optional[LinearWeight]
+    ff: int                          # width of the shared expert
+    outputs: int                     # of the router
+    experts: Experts
+
+    @traced(lambda self, *a, **k: f"layer{self.index}.moe")
+    def __call__(self, model, x, st, cache):
+        ops, T, m, w = model.ops, x.shape[0], 2 * self.ff, self.w_in.weight
+        if w.dtype == torch.float32 or T <= SMALL_T:
+            y = ops.linear(x, self.w_in, out_f32=True)
+            main, fine = y[:, :m], y[:, m:]
+        else:
+            main, fine = ops.linear(x, LinearWeight(w[:m])) if m else None, ops.linear(x, LinearWeight(w[m:]), out_f32=True)
+        if self.w_out is None:
+            out = torch.zeros(T, x.shape[1], dtype=torch.float32, device=x.device)
+        else:
+            act = torch.empty(T, self.ff, dtype=x.dtype, device=x.device)
+            ops.gated_act(main, act, "silu", row_gate=fine[:, self.outputs])
+            out = ops.linear(act, self.w_out, out_f32=True)
+        self.experts.add(model, x, fine[:, :self.outputs], out)
+        return out
 
 
 @dataclass

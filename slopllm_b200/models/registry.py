@@ -64,6 +64,13 @@ def _load_vononex(model_dir: str, ctx: ParallelContext, mtp: int = 0, dtype=None
     return load_vononex_model(model_dir, ctx, dtype)
 
 
+def _load_pulunex(model_dir: str, ctx: ParallelContext, mtp: int = 0, dtype=None):
+    from .pulunex import load_pulunex_model
+    if dtype is None:
+        dtype = torch.bfloat16 if ctx.device.type == "cuda" else torch.float32
+    return load_pulunex_model(model_dir, ctx, dtype)
+
+
 MODEL_REGISTRY: Dict[str, ModelRegistration] = {
     "glm_moe_dsa": ModelRegistration(True, True, True, True, _load_glm_moe_dsa),
     "glm5_next": ModelRegistration(False, False, False, True, _load_glm5_next),
@@ -79,10 +86,13 @@ MODEL_REGISTRY: Dict[str, ModelRegistration] = {
     "vononex": ModelRegistration(False, False, False, False, _load_vononex, float32=True,
                                  kernel_sources=("elementwise", "gated_chunk", "gated_scan", "gemm_tcgen05", "gemv", "grouped_attn", "latent_mma", "linear_simt",
                                                  "min_gru", "parallel_block", "rotary", "sampling", "sandwich_norm")),
+    "pulunex": ModelRegistration(False, False, False, False, _load_pulunex, float32=True,
+                                 kernel_sources=("elementwise", "gemm_tcgen05", "gemv", "grouped_attn", "linear_simt", "moe_sort", "moe_stream", "parallel_block",
+                                                 "sampling", "sandwich_norm", "talking_attn", "token_shift")),
 }
 
 
-HYBRID_FAMILIES = ("gidisun", "zemezen", "vononex")      # assembled from the shared mixers
+HYBRID_FAMILIES = ("gidisun", "zemezen", "vononex", "pulunex")      # assembled from the shared mixers
 
 
 @dataclass

@@ -1,10 +1,10 @@
 """The decoder loop and the engine hooks shared by the model families whose layers are mixer + feed-forward sublayers over a
 :class:`~slopllm_b200.kv.hybrid.HybridCache`: Qwen3 / Qwen3.5 (`models/dense.py`), Gidisun (`models/gidisun.py`), Zemezen
-(`models/zemezen.py`) and Vononex (`models/vononex.py`).
+(`models/zemezen.py`), Vononex (`models/vononex.py`) and Pulunex (`models/pulunex.py`).
 
 A family builds a flat list of :class:`Sublayer`; the loop runs  x -> run(norm(x)) -> [post norm] -> residual add -> next norm,
 or, in families that normalise the sum,  x -> norm(alpha x + run(x) + bias),  with the residual in fp32, and completes the
-tensor-parallel partial sums in between.
+tensor-parallel partial sums in between.  What a sublayer reads may be mixed with what it read for the previous token.
 """
 from __future__ import annotations
 
@@ -14,7 +14,16 @@ from typing import Callable, List, Optional
 import torch
 
 from ..kv.hybrid import CacheSpec, HybridCache, StateSlots
+from ..ops import shift as SH
 from ..parallel.dist import Comm, ParallelContext
+
+
+@dataclass
+class TokenShift:
+    """The normed input h becomes h + (h of the previous token - h) * mix; the last token's h is the layer's state "shift"."""
+
+    index: int                                 # layer
+    mix: torch.Tensor                          # fp32 [H]
 
 
 @dataclass
@@ -25,6 +34,7 @@ class Sublayer:
                                                # with `alpha` on the sum
     alpha: Optional[float] = None              # factor on the residual of a sublayer whose sum is normalised
     bias: Optional[torch.Tensor] = None        # fp32 [H], added to the complete output (sums that are normalised)
+    shift: Optional[TokenShift] = None         # mixes the normed input with the previous token's
 
 
 def token_ranges(st):
@@ -81,16 +91,29 @@ class DecoderStack:
         sidx = self.states.index if self.states is not None else torch.zeros(qo.numel() - 1, dtype=torch.int32, device=qo.device)
         return qo, sidx
 
-    def _enter(self, st, norm):
+    def _shift(self, shift: Optional[TokenShift], st, cache):
+        if shift is None:
+            return None
+        return SH.Shift(shift.mix, cache.state[shift.index]["shift"], *self.scan_ranges(st), st.batch_idx)
+
+    def _enter(self, st, cache, sub: Sublayer):
         ops, eps = self.ops, self.cfg.rms_norm_eps
+        norm, places = sub.norm, getattr(self.w, "positions", None)
+        if sub.shift is not None or places is not None:
+            return SH.embed_shift_norm(st, self.w.embed, getattr(self.w, "embed_scale", 1.0), places, norm, eps, self._shift(sub.shift, st, cache),
+                                       ops.act_dtype)
         if norm is None:
             return ops.embed_rows(st.input_ids, self.w.embed)
         if self.fp32_norms or self.sublayers[0].post_norm is not None:
             return ops.embed_norm(st.input_ids, self.w.embed, norm, eps)
         return ops.add_rmsnorm(ops.embed(st.input_ids, self.w.embed), None, norm, eps)
 
-    def _join(self, y, residual, sub: Sublayer, norm):
+    def _join(self, y, residual, sub: Sublayer, nxt: Optional[Sublayer], st, cache):
+        """`nxt`: the sublayer that reads the sum (None: the output head)."""
         ops, eps = self.ops, self.cfg.rms_norm_eps
+        norm = self.w.final_norm if nxt is None else nxt.norm
+        if nxt is not None and nxt.shift is not None:
+            return SH.add_shift_norm(st, self.comm.all_reduce(y), residual, norm, eps, self._shift(nxt.shift, st, cache), ops.act_dtype)
         if sub.alpha is not None:
             return ops.sum_norm(self.comm.all_reduce(y), residual, sub.alpha, sub.bias, sub.post_norm, norm, eps)
         if self.fp32_norms or sub.post_norm is not None:
@@ -98,11 +121,10 @@ class DecoderStack:
         return self.comm.allreduce_add_rmsnorm(ops, y, residual, norm, eps)
 
     def forward_hidden(self, st, cache) -> torch.Tensor:
-        x, residual = self._enter(st, self.sublayers[0].norm)
-        for i, sub in enumerate(self.sublayers):
+        x, residual = self._enter(st, cache, self.sublayers[0])
+        for sub, nxt in zip(self.sublayers, [*self.sublayers[1:], None]):
             y = sub.run(x, st, cache)
-            nxt = self.sublayers[i + 1].norm if i + 1 < len(self.sublayers) else self.w.final_norm
-            x, residual = self._join(y, residual, sub, nxt)
+            x, residual = self._join(y, residual, sub, nxt, st, cache)
         return x
 
     def compute_logits(self, hidden: torch.Tensor) -> torch.Tensor:

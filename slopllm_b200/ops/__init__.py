@@ -131,8 +131,12 @@ class RefOps:
     def dense_mlp(self, x, lw, sink=None):
         return R.linear(R.silu_mul(R.linear(x, lw.mlp_w13)), lw.mlp_w2)
 
-    def gated_act(self, gate_up, out, act: str = "silu", bias=None):
-        out.copy_(R.gated_act(gate_up if bias is None else gate_up + bias, act))
+    def gated_act(self, gate_up, out, act: str = "silu", bias=None, row_gate=None):
+        y = R.gated_act(gate_up if bias is None else gate_up + bias, act)
+        out.copy_(y if row_gate is None else y * torch.sigmoid(row_gate.to(torch.float32))[:, None])
+
+    def plain_act(self, x, out, act: str):
+        out.copy_(R.activation(x, act))
 
     def silu_mul(self, gate_up, out):
         self.gated_act(gate_up, out)

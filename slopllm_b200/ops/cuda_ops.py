@@ -16,6 +16,7 @@ from . import native as N
 from . import reference as R
 
 DECODE_MAX_T = 32          # token rows handled by the weight-streaming (GEMV) kernels
+ACTS = {"silu": 0, "gelu_tanh": 1}
 TENSOR_MIN_T = 2           # from this many rows on the streaming kernels use the tensor cores
 
 
@@ -556,12 +557,19 @@ class CudaOps:
         N.call("sl_silu_mul_f32" if gu.dtype == torch.float32 else "sl_silu_mul", act.data_ptr(), gu.data_ptr(), T, I2 // 2, N.stream())
         return self.linear(act, lw.mlp_w2, out_f32=True, sink=sink)
 
-    def gated_act(self, gate_up, out, act: str = "silu", bias=None):
-        """out = act(gate + b) * (up + b') for gate_up [T, 2I] = gate | up, bias fp32 [2I] = b | b' (None: 0) and out [T, I], rows of
-        any stride.  act: "silu" or "gelu_tanh"."""
+    def gated_act(self, gate_up, out, act: str = "silu", bias=None, row_gate=None):
+        """out = act(gate + b) * (up + b') [* sigmoid(g)] for gate_up [T, 2I] = gate | up, bias fp32 [2I] = b | b' (None: 0), out [T, I]
+        and row_gate fp32 [T] = g, rows of any stride.  act: "silu" or "gelu_tanh"."""
         T, I = out.shape
-        N.call("sl_gated_act_rows", out.data_ptr(), out.stride(0), gate_up.data_ptr(), gate_up.stride(0), N.ptr(bias), T, I,
-               {"silu": 0, "gelu_tanh": 1}[act], int(gate_up.dtype == torch.float32), int(out.dtype == torch.float32), N.stream())
+        N.call("sl_gated_act_rows", out.data_ptr(), out.stride(0), gate_up.data_ptr(), gate_up.stride(0), N.ptr(bias), N.ptr(row_gate),
+               0 if row_gate is None else row_gate.stride(0), T, I, ACTS[act], int(gate_up.dtype == torch.float32), int(out.dtype == torch.float32),
+               N.stream())
+
+    def plain_act(self, x, out, act: str):
+        """out = act(x), rows of any stride."""
+        T, I = out.shape
+        N.call("sl_act_rows", out.data_ptr(), out.stride(0), x.data_ptr(), x.stride(0), T, I, ACTS[act], int(x.dtype == torch.float32),
+               int(out.dtype == torch.float32), N.stream())
 
     def silu_mul(self, gate_up, out):
         """out = silu(gate) * up for gate_up [T, 2I] = gate | up and out [T, I], rows of any stride."""

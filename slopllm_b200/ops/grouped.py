@@ -29,7 +29,8 @@ class GroupedPreParams(C.Structure):
                 ("dim", C.c_int), ("vdim", C.c_int), ("rot_dims", C.c_int), ("q_norm", C.c_void_p), ("k_norm", C.c_void_p),
                 ("freq", C.c_void_p), ("rot_gain", C.c_float), ("eps", C.c_float), ("positions", C.c_void_p), ("batch_idx", C.c_void_p),
                 ("page_table", C.c_void_p), ("pt_stride", C.c_int), ("page_size", C.c_int), ("k_cache", C.c_void_p), ("v_cache", C.c_void_p),
-                ("num_slots", C.c_int), ("q_out", C.c_void_p), ("guard", C.c_void_p)]
+                ("num_slots", C.c_int), ("q_out", C.c_void_p), ("guard", C.c_void_p), ("v_heads", C.c_int), ("q_bias", C.c_void_p),
+                ("k_bias", C.c_void_p), ("v_bias", C.c_void_p)]
 
 
 class GroupedAttnParams(C.Structure):
@@ -62,6 +63,7 @@ class GroupedShape:
     keep_first: int = 0
     eps: float = 1e-5
     own_values: bool = True    # False: a value row is the key projection before norm and rotation (vdim == dim)
+    v_heads: Optional[int] = None      # value heads of this rank, where they are not as many as its key heads
 
 
 @dataclass
@@ -69,38 +71,47 @@ class GroupedWeights:
     q_norm: Optional[torch.Tensor]          # fp32 [dim], shared by the heads (None: no norm)
     k_norm: Optional[torch.Tensor]
     sink: Optional[torch.Tensor] = None     # fp32 [heads]
+    bias: Optional[torch.Tensor] = None     # fp32, added to the projection rows
 
 
 def _rms(x, w, eps):
     return x if w is None else x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * w
 
 
-def grouped_pre(proj: torch.Tensor, s: GroupedShape, w: GroupedWeights, rot: RotaryTable, st, k_cache: torch.Tensor,
+def grouped_pre(proj: torch.Tensor, s: GroupedShape, w: GroupedWeights, rot: Optional[RotaryTable], st, k_cache: torch.Tensor,
                 v_cache: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
     """proj [T, heads * dim (q) | kv_heads * dim (k) | kv_heads * vdim (v, if values are their own)] (`dtype` or fp32): norms and
-    rotates queries and keys, writes keys and values into their slots; returns the queries [T, heads, dim] in `dtype`."""
+    rotates queries and keys (`rot` None: does not), writes keys and values into their slots; returns the queries [T, heads, dim] in
+    `dtype`.  Without key heads there are queries only."""
     T, kb = proj.shape[0], s.heads * s.dim
     vb = kb + s.kv_heads * s.dim
+    nv = s.kv_heads if s.v_heads is None else s.v_heads
     if proj.is_cuda:
         N = _native()
         from . import tcgen05
         q = torch.empty(T, s.heads, s.dim, dtype=dtype, device=proj.device)
         at = lambda i: proj.data_ptr() + i * proj.element_size()
-        p = GroupedPreParams(q=at(0), k=at(kb), v=at(vb) if s.own_values else at(kb), ld=proj.stride(0), heads=s.heads, kv_heads=s.kv_heads,
-                             dim=s.dim, vdim=s.vdim, rot_dims=rot.dims, q_norm=N.ptr(w.q_norm), k_norm=N.ptr(w.k_norm),
-                             freq=rot.freq.data_ptr(), rot_gain=rot.gain, eps=s.eps, positions=st.positions.data_ptr(),
+        bias = lambda i: 0 if w.bias is None else w.bias.data_ptr() + 4 * i
+        v_at = vb if s.own_values else kb
+        p = GroupedPreParams(q=at(0), k=at(kb), v=at(v_at), v_heads=nv, q_bias=bias(0), k_bias=bias(kb), v_bias=bias(v_at), ld=proj.stride(0), heads=s.heads, kv_heads=s.kv_heads,
+                             dim=s.dim, vdim=s.vdim, rot_dims=0 if rot is None else rot.dims, q_norm=N.ptr(w.q_norm), k_norm=N.ptr(w.k_norm),
+                             freq=0 if rot is None else rot.freq.data_ptr(), rot_gain=1.0 if rot is None else rot.gain, eps=s.eps, positions=st.positions.data_ptr(),
                              batch_idx=st.batch_idx.data_ptr(), page_table=st.page_table.data_ptr(), pt_stride=st.page_table.stride(0),
                              page_size=st.page_size, k_cache=k_cache.data_ptr(), v_cache=v_cache.data_ptr(), num_slots=k_cache.shape[0],
                              q_out=q.data_ptr(), guard=tcgen05.error_flag(proj.device).data_ptr() + 16)
         N.call("sl_grouped_pre", C.byref(p), T, int(proj.dtype == torch.float32), int(dtype == torch.float32), N.stream())
         return q
+    turn = (lambda y: y) if rot is None else (lambda y: rot.apply(y, st.positions))
     x = proj.to(torch.float32)
-    k = x[:, kb:vb].reshape(T, s.kv_heads, s.dim)
-    v = x[:, vb:vb + s.kv_heads * s.vdim].reshape(T, s.kv_heads, s.vdim) if s.own_values else k
-    slots = _slots(st.positions, st.batch_idx, st.page_table, st.page_size)
-    k_cache[slots] = rot.apply(_rms(k, w.k_norm, s.eps), st.positions).to(k_cache.dtype)
-    v_cache[slots] = v.to(v_cache.dtype)
-    return rot.apply(_rms(x[:, :kb].reshape(T, s.heads, s.dim), w.q_norm, s.eps), st.positions).to(dtype)
+    if w.bias is not None:
+        x = x + w.bias
+    if s.kv_heads:
+        k = x[:, kb:vb].reshape(T, s.kv_heads, s.dim)
+        v = x[:, vb:vb + nv * s.vdim].reshape(T, nv, s.vdim) if s.own_values else k
+        slots = _slots(st.positions, st.batch_idx, st.page_table, st.page_size)
+        k_cache[slots] = turn(_rms(k, w.k_norm, s.eps)).to(k_cache.dtype)
+        v_cache[slots] = v.to(v_cache.dtype)
+    return turn(_rms(x[:, :kb].reshape(T, s.heads, s.dim), w.q_norm, s.eps)).to(dtype)
 
 
 @dataclass

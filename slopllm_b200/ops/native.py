@@ -233,12 +233,16 @@ _SIGS = {
     "sl_grouped_rows": [vp, i32, i32, vp],
     "sl_grouped_decode_ok": [i32, i32],
     "sl_grouped_decode": [vp, i32, vp],
-    "sl_gated_act_rows": [vp, i32, vp, i32, vp, i32, i32, i32, i32, i32, vp],
+    "sl_gated_act_rows": [vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, vp],
+    "sl_act_rows": [vp, i32, vp, i32, i32, i32, i32, i32, i32, vp],
+    "sl_shift_norm": [vp, i32, vp],
+    "sl_talking_rows": [vp, i32, i32, vp],
+    "sl_identity_experts": [vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, vp],
     "sl_short_conv": [vp, vp, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp],
     "sl_delta_step": [vp, i32, i32, i32, vp],
     "sl_delta_chunk_ok": [i32, i32],
     "sl_delta_chunks": [vp, i32, vp],
-    "sl_route_softmax": [vp, vp, vp, i32, i32, i32, i32, i32, i32, vp],
+    "sl_route_softmax": [vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, vp],
     "sl_expert_stream": [vp, i32, vp],
     "sl_latent_decode": [vp, i32, vp],
     "sl_gated_chunk_ok": [i32, i32, i32, i32],

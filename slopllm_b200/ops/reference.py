@@ -88,9 +88,14 @@ def silu_mul(gate_up: torch.Tensor) -> torch.Tensor:
     return torch.nn.functional.silu(g) * u
 
 
+def activation(x: torch.Tensor, act: str) -> torch.Tensor:
+    x = x.to(torch.float32)
+    return {"silu": torch.nn.functional.silu, "gelu_tanh": lambda x: torch.nn.functional.gelu(x, approximate="tanh")}[act](x)
+
+
 def gated_act(gate_up: torch.Tensor, act: str) -> torch.Tensor:
     g, u = gate_up.to(torch.float32).chunk(2, dim=-1)
-    return {"silu": torch.nn.functional.silu, "gelu_tanh": lambda x: torch.nn.functional.gelu(x, approximate="tanh")}[act](g) * u
+    return activation(g, act) * u
 
 
 # ---- MoE routing --------------------------------------------------------------------------------

@@ -81,6 +81,9 @@ class Engine:
         self.cache = (model.allocate_cache(num_pages, max_states or max(64, max_batch)) if hasattr(model, "allocate_cache")
                       else KVCacheTensors.allocate(cfg, num_pages, self.device, len(model.w.layers)))
         self.max_batch = max_batch
+        self.max_positions = int(getattr(cfg, "max_positions", 0) or 0)     # longest sequence of models with learned positions (0: no limit)
+        if self.max_positions:
+            max_seq_len = min(max_seq_len, self.max_positions)
         self.pt_width = -(-max_seq_len // (PAGE_SIZE * self.ctx.cp_world)) + 1
         self.graphs = CaptureManager(enabled=cuda_graph and self.device.type == "cuda")
         self.mtp = mtp
@@ -271,8 +274,14 @@ class Engine:
         self.check_device_errors()           # (the token reads above already synchronised the stream)
         return tokens, (hiddens if want_hidden else None)
 
+    def _check_positions(self, seqs: Seq[Sequence], counts: Seq[int]) -> None:
+        """Refuse, before anything is appended, a step that would pass the model's last position."""
+        if self.max_positions and any(s.length + n > self.max_positions for s, n in zip(seqs, counts)):
+            raise ValueError(f"a sequence would pass the model's {self.max_positions} positions")
+
     def _pack(self, seqs: Seq[Sequence], tokens: Seq[Seq[int]]):
         """Append each sequence's next tokens and lay the portions out as one batch.  Returns (state, ids, positions)."""
+        self._check_positions(seqs, [len(t) for t in tokens])
         ids: List[int] = []
         positions: List[int] = []
         bidx: List[int] = []
@@ -417,6 +426,7 @@ class Engine:
         """Append one token per sequence and run the captured step of this batch size and KV bucket; `finish(hidden)` is
         its last part (`kind` and `variant` name it in the graph's key).  Returns the graph's static output."""
         B = len(seqs)
+        self._check_positions(seqs, [1] * B)
         positions = []
         for s, t in zip(seqs, tokens):
             positions.append(s.length)

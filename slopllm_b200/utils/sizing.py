@@ -343,3 +343,42 @@ def plan_vononex(cfg, world: int = 1, batch_size: int = 8, chunk_size: int = 819
         return max(3 * l.ff, 3 * a["heads"] * (a["dim"] + a["vdim"]) + r["heads"] * (2 * r["dim"] + 3 * r["vdim"]))
     return _plan_hybrid(cfg, vononex_weight_bytes(cfg, world, elem), *vononex_cache_bytes(cfg, world, elem), max(width(l) for l in cfg.layers) // world,
                         world, batch_size, chunk_size, max_pages, arena_gb, device_gb, elem, reserve_gb)
+
+
+# ---- Pulunex --------------------------------------------------------------------------------------------------------------
+
+def pulunex_weight_bytes(cfg, tp: int = 1, elem: int = 2) -> int:
+    """Per-rank weight bytes, as :func:`gidisun_weight_bytes`; queries and keys are whole on every rank (their scores are mixed), value and
+    output heads and feed-forward rows sharded; norms spread over the row, biases, mixtures and corrections are fp32."""
+    H = cfg.hidden_size
+    b = (cfg.vocab_size + cfg.max_positions) * H * elem + (cfg.vocab_size // tp) * H * elem + 4 * H
+    for l in cfg.layers:
+        c = l.mixer
+        h, kv, d, dv = c["heads"], c["kv_heads"], c["dim"], c["vdim"]
+        rows = h * d + (0 if l.kv_from is not None else kv * d + kv // tp * dv)
+        b += rows * (H * elem + 4) + 4 * (h // tp * h + d) + h // tp * dv * H * elem + 4 * 2 * H
+        if l.ff or l.experts is not None:
+            b += 4 * H + 2 * (l.ff // tp) * H * elem
+        if l.experts is not None:
+            e = l.experts
+            n = e.count + e.identity
+            b += (3 * e.count * (e.ff // tp) + 3 * (e.shared_ff // tp) + n + (1 if e.shared_ff else 0)) * H * elem + 4 * n
+    return b
+
+
+def pulunex_cache_bytes(cfg, tp: int = 1, elem: int = 2):
+    """(bytes of one 64-token page, bytes of one sequence's state) on one rank."""
+    page = sum((l.mixer["kv_heads"] * l.mixer["dim"] + l.mixer["kv_heads"] // tp * l.mixer["vdim"]) * elem * PAGE_SIZE
+               for l in cfg.layers if l.kv_from is None)
+    return page, 4 * cfg.hidden_size * len(cfg.layers)
+
+
+def plan_pulunex(cfg, world: int = 1, batch_size: int = 8, chunk_size: int = 8192, max_pages: int = 0, arena_gb: float = 0.0,
+                 device_gb: float = 180.0, elem: int = 2, reserve_gb: float = 4.0) -> MemoryPlan:
+    """`plan_memory` for Pulunex (tensor parallel only)."""
+    def width(l):
+        e = l.experts
+        ff = 2 * l.ff if e is None else 3 * e.shared_ff + e.top * (3 * e.ff + 2 * cfg.hidden_size * world)
+        return max(ff, 3 * l.mixer["heads"] * (l.mixer["dim"] * world + l.mixer["vdim"]))
+    return _plan_hybrid(cfg, pulunex_weight_bytes(cfg, world, elem), *pulunex_cache_bytes(cfg, world, elem), max(width(l) for l in cfg.layers) // world,
+                        world, batch_size, chunk_size, max_pages, arena_gb, device_gb, elem, reserve_gb)
