@@ -5,10 +5,23 @@
 // with positions that see their own chunk of the sequence only.
 //
 //  * talking_rows_kernel: independent token rows on the CUDA cores, any sizes, bf16 or fp32.
+//  * talking_mma_kernel: portions of prompts (up to 16 queries per CTA) and decoding (one), all heads in one CTA, on the tensor cores.
+//    Per tile of keys:  (1) every key head's scores, a 16-row block of (head of the group, query) rows per warp, left in shared memory as
+//    two bf16 terms, hi + lo;  (2) the mixture as a second product, talk x scores, one query and 16 output heads per warp, whose result
+//    holds all keys of the tile for a row: mask and online softmax in registers, weights back to shared memory as hi + lo;  (3) the
+//    weighted values, accumulated in registers by the warps of (1).  Key rows and value rows (all heads of a token are neighbours in the
+//    cache) come by one bulk copy each, the next tile's keys during (2) and (3), its values during (1) and (2).
+//  * talking_merge_kernel: joins the key splits of few queries.
+//
+// Scores and weights lie in blocks of eight keys: [head][key block][query][8 keys], so that a block is one 16-byte row of every matrix
+// that is loaded from there, by query rows (3) as well as by head rows (2).
 #include "common.cuh"
 #include "mma_sync.cuh"
+#include "tcgen05.cuh"
 
 namespace {
+
+constexpr float LOG2E = 1.4426950408889634f;
 
 __device__ __forceinline__ float to_f(float v) { return v; }
 __device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
@@ -25,6 +38,10 @@ struct TalkingParams {
     const float* talk;                   // [out_heads, heads]
     void* out; int ldo;                  // [T, ldo]: output head h at h * vdim
     int* guard;
+    const int4* tiles;                   // portions: first token, tokens, position of the first, page-table row (null: one token each)
+    int splits;
+    float *o_part, *lse_part;            // [T, out_heads, splits, vdim], [T, out_heads, splits] (more than one split)
+    int* err;
 };
 
 constexpr int ROWS_KT = 32, ROWS_THREADS = 256;
@@ -100,6 +117,365 @@ __global__ void __launch_bounds__(ROWS_THREADS) talking_rows_kernel(TalkingParam
     for (int i = tid; i < no; i += ROWS_THREADS) put((T*)p.out + (size_t)t * p.ldo + i, o[i] / l[i / p.vdim]);
 }
 
+// ---- tensor-core form ----------------------------------------------------------------------------------------------------
+
+constexpr int WARPS = 16, MAX_SMEM = 232448;
+
+struct MmaPlan {
+    int bq, kt;                          // queries per CTA, keys per tile (0: the sizes do not fit)
+    int mt;                              // 16-row blocks of a key head's (head, query) rows
+    int ldq, q_swz;                      // bytes of a query row; its 16-byte pieces are permuted by the row's low bits
+    int ldk, ldv;                        // bytes of a key / value row
+    int lds, s_swz;                      // bytes of a head's scores (one plane), likewise
+    int wpv, per_v;                      // warps of a value unit, its 8-wide value tiles per warp
+    int smem, k_at, v_at, s_at, f_at;
+};
+
+MmaPlan make_plan(int heads, int kv_heads, int out_heads, int v_heads, int dim, int vdim, bool decode) {
+    MmaPlan best = {};
+    const int r = heads / kv_heads;
+    if (dim % 8 != 0 || vdim % 8 != 0 || heads > 64 || heads % kv_heads != 0 || out_heads != v_heads * r || out_heads > heads) return best;
+    const int dqp = (dim + 15) / 16 * 16, krow = kv_heads * dim * 2, vrow = v_heads * vdim * 2, mto = (out_heads + 15) / 16;
+    const int hp = heads <= 16 ? 16 : heads <= 32 ? 32 : 64;      // (of the kernel's instances)
+    for (int bq = decode ? 1 : 16; bq >= (decode ? 1 : 2); bq /= 2)
+        for (int kt = 32; kt >= 16; kt /= 2) {
+            MmaPlan m = {};
+            m.bq = bq; m.kt = kt;
+            m.mt = (r * bq + 15) / 16;
+            const int units = v_heads * m.mt;
+            if (units > WARPS || bq * mto > WARPS) continue;
+            m.wpv = WARPS / units;
+            m.per_v = ((vdim / 8 + m.wpv - 1) / m.wpv + 1) / 2 * 2;
+            if (m.per_v > 16) continue;
+            m.q_swz = dqp % 64 == 0 ? 7 : 0;
+            m.ldq = dqp * 2 + (m.q_swz ? 0 : 16);
+            m.ldk = krow + (krow / 16 % 2 == 0 ? 16 : dim % 16 != 0 ? 32 : 0);
+            m.ldv = vrow + (vrow / 16 % 2 == 0 ? 16 : 0);
+            const int blocks = kt / 8 * bq;
+            m.s_swz = blocks % 8 == 0 ? 7 : 0;
+            m.lds = blocks * 16 + (m.s_swz ? 0 : 16);
+            m.k_at = kv_heads * m.mt * 16 * m.ldq;
+            m.v_at = m.k_at + kt * m.ldk;
+            m.s_at = m.v_at + kt * m.ldv;
+            m.f_at = m.s_at + 2 * hp * m.lds;
+            m.smem = m.f_at + out_heads * bq * 4;
+            if (m.smem + 64 > MAX_SMEM) continue;
+            return m;
+        }
+    return best;
+}
+
+__device__ __forceinline__ void bar_sync(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
+
+// grid (splits, tiles), block 512.  KT keys per tile, up to NVT 8-wide value tiles per warp, up to 16 * HT heads.
+template <int KT, int NVT, int HT>
+__global__ void __launch_bounds__(WARPS * 32, 1) talking_mma_kernel(TalkingParams p, MmaPlan m) {
+    pdl_grid_sync();
+    extern __shared__ __align__(128) unsigned char smraw[];
+    __shared__ __align__(8) uint64_t bars[2];                       // keys, values have arrived
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, c4 = lane & 3;
+    const int bq = m.bq, r = p.heads / p.kv_heads, rows = r * bq, unit_rows = m.mt * 16;
+    unsigned char *qs = smraw, *ks = smraw + m.k_at, *vs = smraw + m.v_at, *sh = smraw + m.s_at;
+    const int hp = HT * 16, plane = hp * m.lds;
+    float* fac = reinterpret_cast<float*>(smraw + m.f_at);             // [out_heads][bq]
+    int4 tile;
+    if (p.tiles != nullptr) {
+        tile = p.tiles[blockIdx.y];
+    } else {
+        tile = make_int4(blockIdx.y, 1, p.positions[blockIdx.y], p.batch_idx[blockIdx.y]);
+    }
+    const int tok = tile.x, count = tile.y, pos0 = tile.z, split = blockIdx.x;
+    const int lo = p.chunk > 0 ? pos0 / p.chunk * p.chunk : 0, end = pos0 + count;
+    const int tiles = (end - lo + KT - 1) / KT, per = (tiles + p.splits - 1) / p.splits;
+    const int tb = min(tiles, split * per), te = min(tiles, tb + per);
+    const int* pt = p.page_table + (size_t)tile.w * p.pt_stride;
+    const uint32_t krow = p.kv_heads * p.dim * 2, vrow = p.v_heads * p.vdim * 2;
+
+    auto find = [&](int j) -> long long {                           // cache slot of this lane's key of tile j (warp 0)
+        const int kp = min(lo + j * KT + lane, end - 1);            // (behind the last key: the last once more, never visible)
+        const long long s = (long long)pt[kp / p.page_size] * p.page_size + kp % p.page_size;
+        return guard_ok(p.guard, 32, s, p.num_slots) ? s : 0;
+    };
+    auto fetch = [&](unsigned char* dst, int ld, const void* cache, uint32_t row, uint64_t* bar, long long slot) {
+        if (lane == 0) tc::mbar_expect_tx(bar, KT * row);
+        __syncwarp();
+        if (lane < KT) tc::bulk_load_1d(dst + lane * ld, (const unsigned char*)cache + (size_t)slot * row, row, bar);
+    };
+    if (tid == 0) {
+        tc::mbar_init(&bars[0], 1);
+        tc::mbar_init(&bars[1], 1);
+        tc::mbar_fence_init();
+        tc::fence_proxy_async_smem();
+    }
+    long long slot = 0, slot_next = 0;
+    if (warp == 0) {
+        __syncwarp();
+        if (tb < te) {
+            slot = find(tb);
+            fetch(ks, m.ldk, p.k_cache, krow, &bars[0], slot);
+        }
+    }
+    // queries, zeros behind the last row and the last value; zeros in the scores of heads that are not there
+    const int dp = (p.dim + 15) / 16 * 2;
+    for (int i = tid; i < p.kv_heads * unit_rows * dp; i += WARPS * 32) {
+        const int row = i / dp, c = i - row * dp, unit = row / unit_rows, rho = row - unit * unit_rows, g = rho / bq, qi = rho - g * bq;
+        uint4 x = make_uint4(0, 0, 0, 0);
+        if (rho < rows && qi < count && c * 8 < p.dim)
+            x = *reinterpret_cast<const uint4*>((const bf16*)p.q + ((size_t)(tok + qi) * p.heads + unit * r + g) * p.dim + c * 8);
+        *reinterpret_cast<uint4*>(qs + row * m.ldq + ((c ^ (row & m.q_swz)) << 4)) = x;
+    }
+    for (int i = tid; i < 2 * hp * m.lds / 16; i += WARPS * 32) *reinterpret_cast<uint4*>(sh + i * 16) = make_uint4(0, 0, 0, 0);
+    if (p.dim % 16 != 0)                                            // (the last head's 16-value steps reach into the padding)
+        for (int i = tid; i < KT; i += WARPS * 32) *reinterpret_cast<uint4*>(ks + i * m.ldk + krow) = make_uint4(0, 0, 0, 0);
+    // the mixture: this warp's query and 16 output heads
+    const int mto = (p.out_heads + 15) / 16, qi_mix = warp / mto, h_mix = (warp - qi_mix * mto) * 16;
+    const bool mixes = qi_mix < count;                              // (qi_mix < bq follows)
+    uint32_t tf[HT][4];
+#pragma unroll
+    for (int k = 0; k < HT; ++k)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int h = h_mix + g8 + (i & 1) * 8, g = k * 16 + (i >> 1) * 8 + c4 * 2;
+            float a = 0.f, b = 0.f;
+            if (mixes && h < p.out_heads) {
+                a = g < p.heads ? p.talk[h * p.heads + g] : 0.f;
+                b = g + 1 < p.heads ? p.talk[h * p.heads + g + 1] : 0.f;
+            }
+            tf[k][i] = f2_to_bf162(a, b);
+        }
+    const int q_pos = pos0 + qi_mix, q_lo = p.chunk > 0 ? q_pos / p.chunk * p.chunk : 0;
+    const float scale_log2 = p.scale * LOG2E;
+    float mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.f, 0.f};
+    // the values: this warp's unit and value tiles
+    const int uv = warp / m.wpv, n0 = (warp - uv * m.wpv) * m.per_v, nn = uv < p.v_heads * m.mt ? min(m.per_v, p.vdim / 8 - n0) : 0;
+    const int hv = uv / m.mt, rv = (uv - hv * m.mt) * 16;           // value head, first of the unit's rows
+    float acc[NVT][4];
+#pragma unroll
+    for (int i = 0; i < NVT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    // the row of weights that this lane addresses
+    const int a_rho = min(rv + (lane & 15), rows - 1), a_head = min(hv * r + a_rho / bq, p.out_heads - 1), a_qi = a_rho % bq;
+    const int units_k = p.kv_heads * m.mt, wpq = KT == 32 && units_k * 2 <= WARPS ? 2 : 1;
+    auto s_off = [&](int h, int kb, int qi) { return h * m.lds + ((((kb * bq + qi)) ^ (h & m.s_swz)) << 4); };
+
+    __syncthreads();
+    bool bad = false;
+    for (int j = tb; j < te; ++j) {
+        const uint32_t parity = (j - tb) & 1;
+        if (__syncthreads_or(!tc::mbar_wait(&bars[0], parity))) { bad = true; break; }
+        if (warp == 0) fetch(vs, m.ldv, p.v_cache, vrow, &bars[1], slot);
+        if (warp == 0 && j + 1 < te) slot_next = find(j + 1);
+        // (1) scores
+        for (int i = warp; i < units_k * wpq; i += WARPS) {
+            const int u = i / wpq, kh = u / m.mt, r0 = (u - kh * m.mt) * 16;
+            const int kb0 = wpq == 2 ? (i & 1) * 16 : 0;            // first key
+            const bool both = KT == 32 && wpq == 1;
+            float s[4][4] = {};
+            const int qr = kh * unit_rows + r0 + (lane & 15);
+            const unsigned char* qrow = qs + qr * m.ldq;
+            const unsigned char* krow_s = ks + (kb0 + (lane & 7) + (lane >> 4) * 8) * m.ldk + kh * p.dim * 2 + ((lane >> 3) & 1) * 16;
+#pragma unroll 4
+            for (int c = 0; c < dp; c += 2) {
+                uint32_t a[4], b[4];
+                ldsm_x4(a, qrow + (((c + (lane >> 4)) ^ (qr & m.q_swz)) << 4));
+                ldsm_x4(b, krow_s + c * 16);
+                mma_bf16_16816(s[0], a, b[0], b[1]);
+                mma_bf16_16816(s[1], a, b[2], b[3]);
+                if (both) {
+                    ldsm_x4(b, krow_s + 16 * m.ldk + c * 16);
+                    mma_bf16_16816(s[2], a, b[0], b[1]);
+                    mma_bf16_16816(s[3], a, b[2], b[3]);
+                }
+            }
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int rho = r0 + g8 + e * 8;
+                if (rho >= rows) continue;
+                const int g = rho / bq, qi = rho - g * bq, h = kh * r + g;
+#pragma unroll
+                for (int n = 0; n < 4; ++n) {
+                    if (n >= 2 && !both) break;
+                    uint32_t hi, low;
+                    split_bf162(s[n][e * 2], s[n][e * 2 + 1], hi, low);
+                    unsigned char* at = sh + s_off(h, kb0 / 8 + n, qi) + c4 * 4;
+                    *reinterpret_cast<uint32_t*>(at) = hi;
+                    *reinterpret_cast<uint32_t*>(at + plane) = low;
+                }
+            }
+        }
+        __syncthreads();
+        if (warp == 0 && j + 1 < te) fetch(ks, m.ldk, p.k_cache, krow, &bars[0], slot_next);
+        slot = slot_next;
+        // (2) mixture, mask, softmax
+        if (mixes) {
+            float c[KT / 8][4] = {};
+            const int hr = (lane & 7) + ((lane >> 3) & 1) * 8;
+#pragma unroll
+            for (int k = 0; k < HT; ++k)
+#pragma unroll
+                for (int n = 0; n < KT / 8; n += 2) {
+                    uint32_t b[4];
+                    const unsigned char* at = sh + s_off(k * 16 + hr, n + (lane >> 4), qi_mix);
+                    ldsm_x4_trans(b, at);
+                    mma_bf16_16816(c[n], tf[k], b[0], b[1]);
+                    mma_bf16_16816(c[n + 1], tf[k], b[2], b[3]);
+                    ldsm_x4_trans(b, at + plane);
+                    mma_bf16_16816(c[n], tf[k], b[0], b[1]);
+                    mma_bf16_16816(c[n + 1], tf[k], b[2], b[3]);
+                }
+            if (mto > 1) bar_sync(1 + qi_mix, mto * 32);            // (the weights take the scores' place)
+            else __syncwarp();
+            const int key0 = lo + j * KT + c4 * 2;
+            float top[2] = {mx[0], mx[1]};
+#pragma unroll
+            for (int n = 0; n < KT / 8; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int key = key0 + n * 8 + (e & 1);
+                    c[n][e] = key >= q_lo && key <= q_pos ? c[n][e] * scale_log2 : -INFINITY;
+                    top[e >> 1] = fmaxf(top[e >> 1], c[n][e]);
+                }
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                top[e] = fmaxf(top[e], __shfl_xor_sync(0xffffffffu, top[e], 1));
+                top[e] = fmaxf(top[e], __shfl_xor_sync(0xffffffffu, top[e], 2));
+                const float base = top[e] == -INFINITY ? 0.f : top[e], f = exp2f(mx[e] - base);
+                const int h = h_mix + g8 + e * 8;
+                float l = 0.f;
+#pragma unroll
+                for (int n = 0; n < KT / 8; ++n) {
+                    const float x = exp2f(c[n][e * 2] - base), y = exp2f(c[n][e * 2 + 1] - base);
+                    l += x + y;
+                    if (h < p.out_heads) {
+                        uint32_t hi, low;
+                        split_bf162(x, y, hi, low);
+                        unsigned char* at = sh + s_off(h, n, qi_mix) + c4 * 4;
+                        *reinterpret_cast<uint32_t*>(at) = hi;
+                        *reinterpret_cast<uint32_t*>(at + plane) = low;
+                    }
+                }
+                sum[e] = sum[e] * f + l;
+                mx[e] = top[e];
+                if (c4 == 0 && h < p.out_heads) fac[h * bq + qi_mix] = f;
+            }
+        }
+        if (__syncthreads_or(!tc::mbar_wait(&bars[1], parity))) { bad = true; break; }
+        // (3) values
+        if (nn > 0) {
+            float f[2];
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int rho = rv + g8 + e * 8, g = rho / bq;
+                f[e] = rho < rows && rho - g * bq < count ? fac[hv * rows + rho] : 0.f;
+            }
+#pragma unroll
+            for (int i = 0; i < NVT; ++i) { acc[i][0] *= f[0]; acc[i][1] *= f[0]; acc[i][2] *= f[1]; acc[i][3] *= f[1]; }
+#pragma unroll
+            for (int k = 0; k < KT / 16; ++k) {
+                uint32_t a[4], al[4];
+                const unsigned char* at = sh + s_off(a_head, k * 2 + (lane >> 4), a_qi);
+                ldsm_x4(a, at);
+                ldsm_x4(al, at + plane);
+                const unsigned char* vrow_s = vs + (k * 16 + (lane & 15)) * m.ldv + (hv * p.vdim + n0 * 8 + (lane >> 4) * 8) * 2;
+#pragma unroll
+                for (int i = 0; i < NVT; i += 2) {
+                    if (i >= nn) break;
+                    uint32_t b[4];
+                    if (i + 1 < nn) {
+                        ldsm_x4_trans(b, vrow_s + i * 16);
+                        mma_bf16_16816(acc[i], a, b[0], b[1]);
+                        mma_bf16_16816(acc[i + 1], a, b[2], b[3]);
+                        mma_bf16_16816(acc[i], al, b[0], b[1]);
+                        mma_bf16_16816(acc[i + 1], al, b[2], b[3]);
+                    } else {
+                        ldsm_x2_trans(b[0], b[1], vs + (k * 16 + (lane & 15)) * m.ldv + (hv * p.vdim + (n0 + i) * 8) * 2);
+                        mma_bf16_16816(acc[i], a, b[0], b[1]);
+                        mma_bf16_16816(acc[i], al, b[0], b[1]);
+                    }
+                }
+            }
+        }
+    }
+    if (bad) {                                                      // an expired wait: nothing more is started, copies in flight are let in
+        if (tid == 0) {
+            p.err[0] = 33;
+            tc::mbar_wait(&bars[0], 0, 100000000ull);
+            tc::mbar_wait(&bars[0], 1, 100000000ull);
+            tc::mbar_wait(&bars[1], 0, 100000000ull);
+            tc::mbar_wait(&bars[1], 1, 100000000ull);
+        }
+        return;
+    }
+    __syncthreads();
+    if (mixes) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            sum[e] += __shfl_xor_sync(0xffffffffu, sum[e], 1);
+            sum[e] += __shfl_xor_sync(0xffffffffu, sum[e], 2);
+            const int h = h_mix + g8 + e * 8;
+            if (c4 == 0 && h < p.out_heads) {
+                fac[h * bq + qi_mix] = sum[e] > 0.f ? 1.f / sum[e] : 0.f;
+                if (p.splits > 1)
+                    p.lse_part[((size_t)(tok + qi_mix) * p.out_heads + h) * p.splits + split] = sum[e] > 0.f ? (mx[e] + log2f(sum[e])) / LOG2E : -INFINITY;
+            }
+        }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+        const int rho = rv + g8 + e * 8, g = rho / bq, qi = rho - g * bq;
+        if (nn <= 0 || rho >= rows || qi >= count) continue;
+        const int h = hv * r + g;
+        const float inv = fac[h * bq + qi];
+#pragma unroll
+        for (int i = 0; i < NVT; ++i) {
+            if (i >= nn) break;
+            const int d = (n0 + i) * 8 + c4 * 2;
+            const float x = acc[i][e * 2] * inv, y = acc[i][e * 2 + 1] * inv;
+            if (p.splits == 1) *reinterpret_cast<uint32_t*>((bf16*)p.out + (size_t)(tok + qi) * p.ldo + (size_t)h * p.vdim + d) = f2_to_bf162(x, y);
+            else *reinterpret_cast<float2*>(p.o_part + (((size_t)(tok + qi) * p.out_heads + h) * p.splits + split) * p.vdim + d) = make_float2(x, y);
+        }
+    }
+}
+
+// grid (out_heads, T), block 64: two values per thread and pass
+__global__ void __launch_bounds__(64) talking_merge_kernel(TalkingParams p) {
+    pdl_grid_sync();
+    __shared__ float w[64];
+    const int h = blockIdx.x, t = blockIdx.y, tid = threadIdx.x, lane = tid & 31;
+    const size_t row = (size_t)t * p.out_heads + h;
+    const float a = lane < p.splits ? p.lse_part[row * p.splits + lane] : -INFINITY;
+    const float b = lane + 32 < p.splits ? p.lse_part[row * p.splits + lane + 32] : -INFINITY;
+    const float top = warp_max(fmaxf(a, b));
+    const float ea = a == -INFINITY ? 0.f : expf(a - top), eb = b == -INFINITY ? 0.f : expf(b - top);
+    const float inv = 1.f / warp_sum(ea + eb);
+    if (tid < 32) {
+        w[lane] = ea * inv;
+        w[lane + 32] = eb * inv;
+    }
+    __syncthreads();
+    for (int d = tid * 2; d < p.vdim; d += 128) {
+        float x = 0.f, y = 0.f;
+#pragma unroll 8
+        for (int i = 0; i < p.splits; ++i) {
+            const float2 v = *reinterpret_cast<const float2*>(p.o_part + (row * p.splits + i) * p.vdim + d);
+            x += w[i] * v.x;
+            y += w[i] * v.y;
+        }
+        *reinterpret_cast<uint32_t*>((bf16*)p.out + (size_t)t * p.ldo + (size_t)h * p.vdim + d) = f2_to_bf162(x, y);
+    }
+}
+
+template <int KT, int NVT>
+int launch_mma(const TalkingParams* p, const MmaPlan& m, int tiles, cudaStream_t s) {
+    auto go = [&](auto kern) {
+        cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, m.smem);
+        sl_launch(kern, dim3(p->splits, tiles), WARPS * 32, m.smem, s, *p, m);
+        return SL_LAUNCH_CHECK();
+    };
+    if (p->heads <= 16) return go(talking_mma_kernel<KT, NVT, 1>);
+    return p->heads <= 32 ? go(talking_mma_kernel<KT, NVT, 2>) : go(talking_mma_kernel<KT, NVT, 4>);
+}
+
 bool shape_ok(const TalkingParams* p) {
     return p->heads >= 1 && p->kv_heads >= 1 && p->out_heads >= 1 && p->v_heads >= 1 && p->heads % p->kv_heads == 0 && p->out_heads % p->v_heads == 0 &&
            p->chunk >= 0;
@@ -117,4 +493,35 @@ SL_API int sl_talking_rows(const TalkingParams* p, int T, int f32, cudaStream_t 
         return SL_LAUNCH_CHECK();
     };
     return f32 ? go(talking_rows_kernel<float>) : go(talking_rows_kernel<bf16>);
+}
+
+// Queries per CTA of the tensor-core kernel (decode: 1), 0 when it does not take these sizes.
+SL_API int sl_talking_queries(int heads, int kv_heads, int out_heads, int v_heads, int dim, int vdim, int decode) {
+    if (heads < 1 || kv_heads < 1 || v_heads < 1 || dim < 8 || vdim < 8) return 0;
+    return make_plan(heads, kv_heads, out_heads, v_heads, dim, vdim, decode != 0).bq;
+}
+
+// Keys per tile, as above.
+SL_API int sl_talking_keys(int heads, int kv_heads, int out_heads, int v_heads, int dim, int vdim, int decode) {
+    if (heads < 1 || kv_heads < 1 || v_heads < 1 || dim < 8 || vdim < 8) return 0;
+    return make_plan(heads, kv_heads, out_heads, v_heads, dim, vdim, decode != 0).kt;
+}
+
+// `tiles` query tiles (without p->tiles: tokens) of T tokens.
+SL_API int sl_talking_mma(const TalkingParams* p, int tiles, int T, cudaStream_t s) {
+    if (T == 0 || tiles == 0) return 0;
+    if (!shape_ok(p) || p->dim < 8 || p->vdim < 8 || p->splits < 1 || p->splits > 64 || tiles > 65535 || T > 65535 || p->ldo % 2 != 0 || p->err == nullptr) return -1;
+    if (p->splits > 1 && (p->o_part == nullptr || p->lse_part == nullptr)) return -1;
+    if (((uintptr_t)p->q | (uintptr_t)p->k_cache | (uintptr_t)p->v_cache) % 16 != 0) return -1;
+    const MmaPlan m = make_plan(p->heads, p->kv_heads, p->out_heads, p->v_heads, p->dim, p->vdim, p->tiles == nullptr);
+    if (m.bq == 0) return -1;
+    int rc;
+#define SL_TM(KT) (m.per_v <= 4 ? launch_mma<KT, 4>(p, m, tiles, s) : m.per_v <= 8 ? launch_mma<KT, 8>(p, m, tiles, s) : launch_mma<KT, 16>(p, m, tiles, s))
+    rc = m.kt == 32 ? SL_TM(32) : SL_TM(16);
+#undef SL_TM
+    if (rc == 0 && p->splits > 1) {
+        sl_launch(talking_merge_kernel, dim3(p->out_heads, T), 64, 0, s, *p);
+        rc = SL_LAUNCH_CHECK();
+    }
+    return rc;
 }

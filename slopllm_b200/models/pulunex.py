@@ -139,7 +139,7 @@ def random_pulunex_tensors(cfg: PulunexConfig, seed: int = 0, device="cpu") -> D
     t: Dict[str, torch.Tensor] = {}
 
     def put(name, *shape, k=1.0, shift=0.0):
-        t[name] = (torch.randn(*shape, generator=g, device=device) * k + shift).to(torch.bfloat16)
+        t[name] = (torch.randn(shape, generator=g, device=device) * k + shift).to(torch.bfloat16)
 
     def mat(name, n, k):
         put(name, n, k, k=k ** -0.5)

@@ -237,6 +237,9 @@ _SIGS = {
     "sl_act_rows": [vp, i32, vp, i32, i32, i32, i32, i32, i32, vp],
     "sl_shift_norm": [vp, i32, vp],
     "sl_talking_rows": [vp, i32, i32, vp],
+    "sl_talking_queries": [i32] * 7,
+    "sl_talking_keys": [i32] * 7,
+    "sl_talking_mma": [vp, i32, i32, vp],
     "sl_identity_experts": [vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, vp],
     "sl_short_conv": [vp, vp, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp],
     "sl_delta_step": [vp, i32, i32, i32, vp],

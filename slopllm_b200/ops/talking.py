@@ -28,7 +28,8 @@ class TalkingParams(C.Structure):
     _fields_ = [("q", C.c_void_p), ("k_cache", C.c_void_p), ("v_cache", C.c_void_p), ("num_slots", C.c_int), ("positions", C.c_void_p),
                 ("batch_idx", C.c_void_p), ("page_table", C.c_void_p), ("pt_stride", C.c_int), ("page_size", C.c_int), ("heads", C.c_int),
                 ("kv_heads", C.c_int), ("out_heads", C.c_int), ("v_heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("chunk", C.c_int),
-                ("scale", C.c_float), ("talk", C.c_void_p), ("out", C.c_void_p), ("ldo", C.c_int), ("guard", C.c_void_p)]
+                ("scale", C.c_float), ("talk", C.c_void_p), ("out", C.c_void_p), ("ldo", C.c_int), ("guard", C.c_void_p),
+                ("tiles", C.c_void_p), ("splits", C.c_int), ("o_part", C.c_void_p), ("lse_part", C.c_void_p), ("err", C.c_void_p)]
 
 
 @dataclass
@@ -64,18 +65,68 @@ def talking_pre(proj: torch.Tensor, s: TalkingShape, w: TalkingWeights, st, k_ca
     return grouped_pre(proj, shape, GroupedWeights(w.ones, w.ones, bias=w.bias), None, st, k_cache, v_cache, dtype)
 
 
+SMS = 148
+
+
+def key_splits(work: int, keys: int, tile: int) -> int:
+    """Blocks that share the keys of each of `work` query tiles (one block per SM at a time): the number with the least tiles of keys one
+    after the other, counting one and a half for a block's start and end."""
+    tiles = -(-max(1, keys) // tile)
+    most = max(1, min(64, tiles, 4 * SMS // work))
+    cost = lambda s: -(-work * s // SMS) * (-(-tiles // s) + 1.5) + (1.0 if s > 1 else 0.0)
+    return min(range(1, most + 1), key=cost)
+
+
+class TalkingPlan:
+    """Query tiles of a step's portions, those with the most keys first: (first token, tokens, first position, sequence)."""
+
+    def __init__(self, spans, queries: int, chunk: int, device):
+        tiles, tok = [], 0
+        for b, (start, n) in enumerate(spans):
+            tiles += [(tok + o, min(queries, n - o), start + o, b) for o in range(0, n, queries)]
+            tok += n
+        keys = lambda t: t[2] + t[1] - first_visible(t[2], chunk)
+        tiles.sort(key=keys, reverse=True)
+        self.count, self.longest = len(tiles), keys(tiles[0])
+        self.tiles = torch.tensor(tiles, dtype=torch.int32, device=device)
+
+    @staticmethod
+    def of(st, queries: int, chunk: int) -> "TalkingPlan":
+        plans = st.extra.setdefault("talking_plans", {})
+        if (queries, chunk) not in plans:
+            plans[queries, chunk] = TalkingPlan(st.extra["spans"], queries, chunk, st.input_ids.device)
+        return plans[queries, chunk]
+
+
 def talking_attention(q: torch.Tensor, s: TalkingShape, w: TalkingWeights, st, k_cache, v_cache, out: torch.Tensor) -> None:
     """Attention of every token row over the cached keys it sees, into `out` [T, out_heads * vdim] (rows of any stride)."""
     T = q.shape[0]
     if q.is_cuda:
         N = _native()
         from . import tcgen05
+        err = tcgen05.error_flag(q.device).data_ptr()
         p = TalkingParams(q=q.data_ptr(), k_cache=k_cache.data_ptr(), v_cache=v_cache.data_ptr(), num_slots=k_cache.shape[0],
                           positions=st.positions.data_ptr(), batch_idx=st.batch_idx.data_ptr(), page_table=st.page_table.data_ptr(),
                           pt_stride=st.page_table.stride(0), page_size=st.page_size, heads=s.heads, kv_heads=s.kv_heads, out_heads=s.out_heads,
                           v_heads=s.v_heads, dim=s.dim, vdim=s.vdim, chunk=s.chunk, scale=s.scale, talk=w.talk.data_ptr(), out=out.data_ptr(),
-                          ldo=out.stride(0), guard=tcgen05.error_flag(q.device).data_ptr() + 16)
-        N.call("sl_talking_rows", C.byref(p), T, int(q.dtype == torch.float32), N.stream())
+                          ldo=out.stride(0), guard=err + 16, splits=1, err=err)
+        decode = "spans" not in st.extra
+        sizes = (s.heads, s.kv_heads, s.out_heads, s.v_heads, s.dim, s.vdim, int(decode))
+        queries = N.fn("sl_talking_queries")(*sizes) if q.dtype == torch.bfloat16 and out.stride(0) % 2 == 0 else 0
+        if not queries:
+            N.call("sl_talking_rows", C.byref(p), T, int(q.dtype == torch.float32), N.stream())
+            return
+        if decode:
+            work, keys = T, min(s.chunk or st.max_kv_len, st.max_kv_len)
+        else:
+            plan = TalkingPlan.of(st, queries, s.chunk)
+            work, keys, p.tiles = plan.count, plan.longest, plan.tiles.data_ptr()
+        p.splits = key_splits(work, keys, N.fn("sl_talking_keys")(*sizes))
+        if p.splits > 1:
+            o_part = torch.empty(T, s.out_heads, p.splits, s.vdim, dtype=torch.float32, device=q.device)
+            lse = torch.empty(T, s.out_heads, p.splits, dtype=torch.float32, device=q.device)
+            p.o_part, p.lse_part = o_part.data_ptr(), lse.data_ptr()
+        N.call("sl_talking_mma", C.byref(p), work, T, N.stream())
         return
     for t in range(T):
         pos = int(st.positions[t])

@@ -165,7 +165,7 @@ def random_tensors(raw, seed=0):
     H, t = raw["width"], {}
 
     def put(name, *shape, k=1.0, shift=0.0):
-        t[name] = (torch.randn(*shape, generator=g) * k + shift).to(torch.bfloat16)
+        t[name] = (torch.randn(shape, generator=g) * k + shift).to(torch.bfloat16)
 
     def mat(name, n, k):
         put(name, n, k, k=k ** -0.5)
