@@ -23,8 +23,8 @@ from ..parallel.dist import ParallelContext, init_from_env
 def add_model_args(ap: argparse.ArgumentParser) -> None:
     ap.add_argument("--model", default="", help="checkpoint directory or Hugging Face hub id (local cache only)")
     ap.add_argument("--random-init", default="", metavar="SPEC",
-                    help="no checkpoint: random weights of 'tiny', 'glm5[:layers]', 'qwen3-tiny', 'qwen35-tiny', 'gidisun-tiny', 'zemezen-tiny' "
-                         "or 'vononex-tiny'")
+                    help="no checkpoint: random weights of 'tiny', 'glm5[:layers]', 'qwen3-tiny', 'qwen35-tiny', 'gidisun-tiny', 'zemezen-tiny', "
+                         "'vononex-tiny' or 'pulunex-tiny'")
     ap.add_argument("--dtype", choices=("bfloat16", "float32"), default=None,
                     help="activation and weight type; default bfloat16 on a GPU.  float32 (no reduced-precision products) for the "
                          "families that have it")
@@ -198,6 +198,8 @@ def build_runtime(args, with_scheduler: bool = True) -> Runtime:
         cfg, model = load_registered(reg, model_dir, ctx, args.mtp, getattr(args, "dtype", None))
     if getattr(args, "max_model_len", None) is None:
         args.max_model_len = 65536
+    if getattr(cfg, "max_positions", 0):
+        args.max_model_len = min(args.max_model_len, cfg.max_positions)
     ecfg = EngineConfig(model=args.model or args.random_init, gpus=list(range(ctx.world)), arena_gb=args.arena, cp=args.cp, ep=args.ep,
                         mtp=args.mtp, batch_size=args.batch_size, chunk_size=args.chunk_size, max_pages=args.max_pages,
                         max_host_pages=args.max_host_pages, cuda_graph=not args.no_cuda_graph,

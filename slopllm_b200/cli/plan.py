@@ -47,7 +47,7 @@ def _config(args) -> GlmMoeDsaConfig:
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="slopllm_b200.cli.plan", description=__doc__.split("\n")[0])
     ap.add_argument("--model", default="", help="checkpoint directory or hub id (only config.json is read)")
-    ap.add_argument("--random-init", default="", help="glm5[:layers], tiny, qwen3, qwen35, gidisun, zemezen or vononex instead of a checkpoint")
+    ap.add_argument("--random-init", default="", help="glm5[:layers], tiny, qwen3, qwen35, gidisun, zemezen, vononex or pulunex instead of a checkpoint")
     ap.add_argument("--world", type=int, default=1, help="GPUs of one replica")
     ap.add_argument("--cp", action="store_true")
     ap.add_argument("--ep", action="store_true")

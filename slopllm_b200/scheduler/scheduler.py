@@ -367,6 +367,14 @@ class GenerationScheduler:
             if req.on_finish:
                 req.on_finish(req)
             return
+        limit = getattr(self.engine, "max_positions", 0)
+        if limit:
+            if len(prompt) > limit:
+                req.error, req.finish_reason, req.retired = f"prompt of {len(prompt)} tokens, the model has {limit} positions", "error", True
+                if req.on_finish:
+                    req.on_finish(req)
+                return
+            req.max_tokens = min(req.max_tokens, limit - len(prompt) + 1)      # (the last token is not fed)
         # pages reserved at admission: the prompt plus a bounded look-ahead of output (a request may ask for tens of
         # thousands of tokens and stop after ten; its later pages are found step by step, see `_make_room`)
         need = kv.pages_for(len(prompt) + min(req.max_tokens, self.ADMIT_LOOKAHEAD_TOKENS) + self.engine.mtp + 1)
