@@ -55,7 +55,7 @@ def parse():
     ap.add_argument("--cp-context", type=int, default=131072)
     ap.add_argument("--tiny", action="store_true", help="small model (smoke runs)")
     ap.add_argument("--hybrid", nargs="?", const="small,medium,large", default="", metavar="SIZES",
-                    help="instead of the headline: prefill / decode throughput of the hybrid families (Vononex, Zemezen, Gidisun and Qwen3.5 side by side), one GPU")
+                    help="instead of the headline: prefill / decode throughput of the hybrid families (Pulunex, Vononex, Zemezen, Gidisun and Qwen3.5 side by side), one GPU")
     return ap.parse_args()
 
 

@@ -1,12 +1,13 @@
-"""Prefill and decode throughput of the hybrid families side by side: Vononex, Zemezen, Gidisun and Qwen3.5 at equal width, heads, head
-sizes and feed-forward, random weights, layers of a real model's size.
+"""Prefill and decode throughput of the hybrid families side by side: Pulunex, Vononex, Zemezen, Gidisun and Qwen3.5 at equal width, heads,
+head sizes and feed-forward, random weights, layers of a real model's size.
 
     python -m slopllm_b200.cli.hybrid_bench [--sizes small,medium,large] [--batches 1,8,64] [--prompt 4096]
 
 Every stack has four layers with a feed-forward each: three recurrent mixers and one attention layer; Zemezen two of its recurrent
 mixers, one windowed and one latent attention layer; Vononex two minGRU layers and two in which attention over the whole context and
-retention share the heads (half of them each, so that a layer's projections stay as wide).  `zemezen_moe` has 32 experts of a quarter of the feed-forward's width in
-every layer, of which a token uses four.  Every number is device
+retention share the heads (half of them each, so that a layer's projections stay as wide); Pulunex four layers of talking-heads attention in chunks of 1024, one of which uses another's
+keys (its dense feed-forward has two matrices, the others' three, so it is half as wide again).  `zemezen_moe` and `pulunex_moe` have 32 experts of a quarter of the feed-forward's width in
+every layer, of which a token uses four (Pulunex: of these and four identity experts, beside a shared one of the same width).  Every number is device
 time (CUDA events, three warm-up runs, a 256 MB write in front of every timed run so that nothing is served from L2); decode is
 a replay of the captured step.  Prints one JSON line; `python bench.py --hybrid [sizes]` prints the same.
 """
@@ -70,7 +71,20 @@ def vononex_config(size: str):
                                  VononexLayer("parallel", pair, ff)])
 
 
+def pulunex_config(size: str, moe: bool = False):
+    from ..models.pulunex import PulunexConfig, PulunexExperts, PulunexLayer
+    H, ff, h = SIZES[size]
+    c = {"heads": h, "kv_heads": max(1, h // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": WINDOW}}
+    mlp = (0, PulunexExperts(32, 4, ff // 4, 4, ff // 4)) if moe else (ff * 3 // 2, None)
+    return PulunexConfig(hidden_size=H, vocab_size=VOCAB, rms_norm_eps=1e-6, max_positions=8192,
+                         layers=[PulunexLayer("attention", c if i != 3 else {**c, "kv_from": 2}, *mlp) for i in range(4)])
+
+
 def build(family: str, size: str, ctx):
+    if family in ("pulunex", "pulunex_moe"):
+        from ..models.pulunex import PulunexModel, random_pulunex_tensors
+        cfg = pulunex_config(size, family == "pulunex_moe")
+        return cfg, PulunexModel.from_tensors(cfg, random_pulunex_tensors(cfg, 0, device=ctx.device), ctx)
     if family == "vononex":
         from ..models.vononex import VononexModel, random_vononex_tensors
         cfg = vononex_config(size)
@@ -121,7 +135,7 @@ def run_arm(family: str, size: str, batches, prompt: int, iters: int, flush) -> 
     st, _, _ = eng._pack([s], [ids])
 
     def prefill():
-        for name in ("chunk_plan", "portion_plans", "angles"):
+        for name in ("chunk_plan", "portion_plans", "talking_plans", "angles"):
             st.extra.pop(name, None)
         return model.forward_hidden(st, eng.cache)
 
@@ -172,7 +186,7 @@ def run(argv=None) -> dict:
     ap.add_argument("--batches", default="1,8,64")
     ap.add_argument("--prompt", type=int, default=4096)
     ap.add_argument("--iters", type=int, default=10)
-    ap.add_argument("--families", default="vononex,zemezen,zemezen_moe,gidisun,qwen3_5")
+    ap.add_argument("--families", default="pulunex,pulunex_moe,vononex,zemezen,zemezen_moe,gidisun,qwen3_5")
     args = ap.parse_args(argv)
     torch.cuda.set_device(0)
     flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")

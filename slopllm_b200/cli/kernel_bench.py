@@ -82,11 +82,11 @@ def time_op(fn: Callable[[], object], iters: int, flush: torch.Tensor) -> float:
 
 def mixer_rows(emit, tokens, iters: int, flush, peaks, dev, h: int = 16, dk: int = 128, dv: int = 128, rank: int = 512, rot: int = 64,
                window: int = 1024, context: int = 2048, n_kv: int = 4) -> None:
-    """Token mixers of the hybrid families at 16 heads of 128: retention, minGRU, attention with turned values, channel-wise delta rule,
+    """Token mixers of the hybrid families at 16 heads of 128: talking-heads attention, token shift, retention, minGRU, attention with turned values, channel-wise delta rule,
     windowed grouped-query attention, GLA, mLSTM and latent attention beside Gated DeltaNet and paged grouped-query attention.  More than 64 tokens: one prompt; fewer: that many sequences of `context` tokens decode one each."""
     import types
     from ..models.glm_moe_dsa import StepState
-    from ..ops import delta as DL, delta_chunk as DC, dense as D, get_ops, grouped as G, latent as L, recurrent as RC
+    from ..ops import delta as DL, delta_chunk as DC, dense as D, get_ops, grouped as G, latent as L, recurrent as RC, shift as SH, talking as TK
     from ..ops.rotary import AngleTable, rotary_table
     ops = get_ops(types.SimpleNamespace(rms_norm_eps=1e-6), dev)
     g = torch.Generator(device=dev).manual_seed(3)
@@ -220,6 +220,26 @@ def mixer_rows(emit, tokens, iters: int, flush, peaks, dev, h: int = 16, dk: int
         us = time_op(lambda: D.qk_norm_rope_cache(qk[:, :h * 128], qk[:, h * 128:(h + n_kv) * 128], qk[:, (h + n_kv) * 128:], None, None, st.positions,
                                                   st.batch_idx, pt, 64, kc, vc, h, n_kv, 128, 64, 1e6, 1e-6), iters, flush)
         emit(roofline_row("qk_norm_rope_cache", T, us, 4 * T * (h + 2 * n_kv) * 128, 0.0, peaks))
+        # talking heads in chunks and over the whole context, the join with the token shift, the activation of an ungated feed-forward
+        for what, chunk in (("chunk", window), ("full context", 0)):
+            ts = TK.TalkingShape(h, n_kv, h, n_kv, 128, 128, 128 ** -0.5, chunk, 1e-6)
+            tw = TK.TalkingWeights(rnd((h + 2 * n_kv) * 128), torch.eye(h, device=dev) + rnd(h, h, k=0.1).to(torch.bfloat16).float(), torch.ones(128, device=dev))
+            if chunk:
+                tq = TK.talking_pre(rproj, ts, tw, st, rk, rv, torch.bfloat16)
+                us = time_op(lambda: TK.talking_pre(rproj, ts, tw, st, rk, rv, torch.bfloat16), iters, flush)
+                emit(roofline_row("talking_pre", T, us, T * 128 * (h + 2 * n_kv) * (2 + (2 if prompt else 4)), 0.0, peaks))
+            us = time_op(lambda: TK.talking_attention(tq, ts, tw, st, rk, rv, rout), iters, flush)
+            seen = sum(int(x) - TK.first_visible(int(x), chunk) + 1 for x in st.positions.tolist())
+            emit(roofline_row(f"talking_attention ({what})", T, us, 2.0 * (T if prompt else seen) * n_kv * 256 + 4.0 * T * h * 128,
+                              2.0 * seen * h * (256 + h), peaks))
+        H = h * 128
+        y, res, wf, mix = rnd(T, H), rnd(T, H), rnd(H), rnd(H)
+        shift = SH.Shift(mix, rnd(B, H), qo, sidx, st.batch_idx)
+        us = time_op(lambda: SH.add_shift_norm(st, y, res, wf, 1e-6, shift, torch.bfloat16), iters, flush)
+        emit(roofline_row("shift_norm", T, us, T * H * 14.0 + 8 * B * H, 0.0, peaks))
+        up = bf(T, 4 * H)
+        us = time_op(lambda: ops.plain_act(up, act, "gelu_tanh"), iters, flush)
+        emit(roofline_row("plain_act (gelu)", T, us, T * H * 16.0, 0.0, peaks))
         # norms
         H = h * 128
         y, res, wf, wb = rnd(T, H), rnd(T, H), rnd(H), bf(H)
@@ -318,6 +338,15 @@ def main(argv=None) -> int:
                 uniq = int(torch.unique(ids).numel())
                 row = roofline_row(f"experts_{E}x{I}", T, us, uniq * 3 * I * Hh * 2 + T * Hh * 10, 6.0 * T * top * I * Hh, peaks)
                 row["experts_touched"] = uniq
+                emit(row)
+                z2, c2 = torch.randn(T, E + 8, device=dev, generator=g), torch.randn(E + 8, device=dev, generator=g) * 0.02
+                us = time_op(lambda: EX.route_softmax(z2, top, correction=c2), args.iters, flush)
+                emit(roofline_row(f"route_softmax_{E}+8 (corrected)", T, us, 4.0 * T * (E + 8), 0.0, peaks))
+                ids, wts = EX.route_softmax(z2, top, correction=c2)
+                us = time_op(lambda: EX.add_experts(x, ex, ids, wts, out, ops, True), args.iters, flush)
+                real = int((ids < E).sum())
+                row = roofline_row(f"experts_{E}x{I} beside 8 identity experts", T, us,
+                                   int(torch.unique(ids[ids < E]).numel()) * 3 * I * Hh * 2 + T * Hh * 10, 6.0 * real * I * Hh, peaks)
                 emit(row)
             del ex
     H = cfg.hidden_size
