@@ -126,10 +126,13 @@ struct MmaPlan {
     int mt;                              // 16-row blocks of a key head's (head, query) rows
     int ldq, q_swz;                      // bytes of a query row; its 16-byte pieces are permuted by the row's low bits
     int ldk, ldv;                        // bytes of a key / value row
-    int lds, s_swz;                      // bytes of a head's scores (one plane), likewise
     int wpv, per_v;                      // warps of a value unit, its 8-wide value tiles per warp
     int smem, k_at, v_at, s_at, f_at;
 };
+
+// Bytes of a head's scores (one plane).  Their 16-byte pieces are permuted by the head's low bits where that stays inside.
+__host__ __device__ constexpr int score_swizzle(int kt, int bq) { return kt / 8 * bq % 8 == 0 ? 7 : 0; }
+__host__ __device__ constexpr int score_bytes(int kt, int bq) { return kt / 8 * bq * 16 + (score_swizzle(kt, bq) ? 0 : 16); }
 
 MmaPlan make_plan(int heads, int kv_heads, int out_heads, int v_heads, int dim, int vdim, bool decode) {
     MmaPlan best = {};
@@ -137,13 +140,13 @@ MmaPlan make_plan(int heads, int kv_heads, int out_heads, int v_heads, int dim, 
     if (dim % 8 != 0 || vdim % 8 != 0 || heads > 64 || heads % kv_heads != 0 || out_heads != v_heads * r || out_heads > heads) return best;
     const int dqp = (dim + 15) / 16 * 16, krow = kv_heads * dim * 2, vrow = v_heads * vdim * 2, mto = (out_heads + 15) / 16;
     const int hp = heads <= 16 ? 16 : heads <= 32 ? 32 : 64;      // (of the kernel's instances)
-    for (int bq = decode ? 1 : 16; bq >= (decode ? 1 : 2); bq /= 2)
+    for (int bq = decode ? 1 : 16; bq >= 1; bq = bq > 4 ? bq / 2 : bq - 3)      // 16, 8, 4, 1
         for (int kt = 32; kt >= 16; kt /= 2) {
             MmaPlan m = {};
             m.bq = bq; m.kt = kt;
             m.mt = (r * bq + 15) / 16;
             const int units = v_heads * m.mt;
-            if (units > WARPS || bq * mto > WARPS) continue;
+            if (units > WARPS || bq * mto > WARPS || bq * hp > 256) continue;
             m.wpv = WARPS / units;
             m.per_v = ((vdim / 8 + m.wpv - 1) / m.wpv + 1) / 2 * 2;
             if (m.per_v > 16) continue;
@@ -151,13 +154,10 @@ MmaPlan make_plan(int heads, int kv_heads, int out_heads, int v_heads, int dim, 
             m.ldq = dqp * 2 + (m.q_swz ? 0 : 16);
             m.ldk = krow + (krow / 16 % 2 == 0 ? 16 : dim % 16 != 0 ? 32 : 0);
             m.ldv = vrow + (vrow / 16 % 2 == 0 ? 16 : 0);
-            const int blocks = kt / 8 * bq;
-            m.s_swz = blocks % 8 == 0 ? 7 : 0;
-            m.lds = blocks * 16 + (m.s_swz ? 0 : 16);
             m.k_at = kv_heads * m.mt * 16 * m.ldq;
             m.v_at = m.k_at + kt * m.ldk;
             m.s_at = m.v_at + kt * m.ldv;
-            m.f_at = m.s_at + 2 * hp * m.lds;
+            m.f_at = m.s_at + 2 * hp * score_bytes(kt, bq);
             m.smem = m.f_at + out_heads * bq * 4;
             if (m.smem + 64 > MAX_SMEM) continue;
             return m;
@@ -165,19 +165,26 @@ MmaPlan make_plan(int heads, int kv_heads, int out_heads, int v_heads, int dim, 
     return best;
 }
 
+__device__ __forceinline__ float exp2_hw(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 __device__ __forceinline__ void bar_sync(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
 
-// grid (splits, tiles), block 512.  KT keys per tile, up to NVT 8-wide value tiles per warp, up to 16 * HT heads.
-template <int KT, int NVT, int HT>
+constexpr float RAISE = 8.f;             // a row's reference is raised when its maximum has grown by more than 2^8
+
+// grid (splits, tiles), block 512.  KT keys per tile, up to NVT 8-wide value tiles per warp, up to 16 * HT heads, BQ queries.
+template <int KT, int NVT, int HT, int BQ>
 __global__ void __launch_bounds__(WARPS * 32, 1) talking_mma_kernel(TalkingParams p, MmaPlan m) {
     pdl_grid_sync();
     extern __shared__ __align__(128) unsigned char smraw[];
     __shared__ __align__(8) uint64_t bars[2];                       // keys, values have arrived
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, c4 = lane & 3;
-    const int bq = m.bq, r = p.heads / p.kv_heads, rows = r * bq, unit_rows = m.mt * 16;
+    constexpr int LDS = score_bytes(KT, BQ), SWZ = score_swizzle(KT, BQ), HP = HT * 16, PLANE = HP * LDS;
+    const int r = p.heads / p.kv_heads, rows = r * BQ, unit_rows = m.mt * 16;
     unsigned char *qs = smraw, *ks = smraw + m.k_at, *vs = smraw + m.v_at, *sh = smraw + m.s_at;
-    const int hp = HT * 16, plane = hp * m.lds;
-    float* fac = reinterpret_cast<float*>(smraw + m.f_at);             // [out_heads][bq]
+    float* fac = reinterpret_cast<float*>(smraw + m.f_at);          // [out_heads][BQ]
     int4 tile;
     if (p.tiles != nullptr) {
         tile = p.tiles[blockIdx.y];
@@ -191,9 +198,11 @@ __global__ void __launch_bounds__(WARPS * 32, 1) talking_mma_kernel(TalkingParam
     const int* pt = p.page_table + (size_t)tile.w * p.pt_stride;
     const uint32_t krow = p.kv_heads * p.dim * 2, vrow = p.v_heads * p.vdim * 2;
 
-    auto find = [&](int j) -> long long {                           // cache slot of this lane's key of tile j (warp 0)
-        const int kp = min(lo + j * KT + lane, end - 1);            // (behind the last key: the last once more, never visible)
-        const long long s = (long long)pt[kp / p.page_size] * p.page_size + kp % p.page_size;
+    // warp 0: page of this lane's key of tile j, and the key's cache slot (behind the last key: the last once more, never visible)
+    auto key_of = [&](int j) { return min(lo + j * KT + lane, end - 1); };
+    auto page_of = [&](int j) { return pt[key_of(j) / p.page_size]; };
+    auto slot_of = [&](int j, int page) -> long long {
+        const long long s = (long long)page * p.page_size + key_of(j) % p.page_size;
         return guard_ok(p.guard, 32, s, p.num_slots) ? s : 0;
     };
     auto fetch = [&](unsigned char* dst, int ld, const void* cache, uint32_t row, uint64_t* bar, long long slot) {
@@ -207,29 +216,30 @@ __global__ void __launch_bounds__(WARPS * 32, 1) talking_mma_kernel(TalkingParam
         tc::mbar_fence_init();
         tc::fence_proxy_async_smem();
     }
-    long long slot = 0, slot_next = 0;
+    long long slot = 0;
+    int page_next = 0;
     if (warp == 0) {
         __syncwarp();
         if (tb < te) {
-            slot = find(tb);
+            slot = slot_of(tb, page_of(tb));
             fetch(ks, m.ldk, p.k_cache, krow, &bars[0], slot);
         }
     }
     // queries, zeros behind the last row and the last value; zeros in the scores of heads that are not there
     const int dp = (p.dim + 15) / 16 * 2;
     for (int i = tid; i < p.kv_heads * unit_rows * dp; i += WARPS * 32) {
-        const int row = i / dp, c = i - row * dp, unit = row / unit_rows, rho = row - unit * unit_rows, g = rho / bq, qi = rho - g * bq;
+        const int row = i / dp, c = i - row * dp, unit = row / unit_rows, rho = row - unit * unit_rows, g = rho / BQ, qi = rho % BQ;
         uint4 x = make_uint4(0, 0, 0, 0);
         if (rho < rows && qi < count && c * 8 < p.dim)
             x = *reinterpret_cast<const uint4*>((const bf16*)p.q + ((size_t)(tok + qi) * p.heads + unit * r + g) * p.dim + c * 8);
         *reinterpret_cast<uint4*>(qs + row * m.ldq + ((c ^ (row & m.q_swz)) << 4)) = x;
     }
-    for (int i = tid; i < 2 * hp * m.lds / 16; i += WARPS * 32) *reinterpret_cast<uint4*>(sh + i * 16) = make_uint4(0, 0, 0, 0);
+    for (int i = tid; i < 2 * PLANE / 16; i += WARPS * 32) *reinterpret_cast<uint4*>(sh + i * 16) = make_uint4(0, 0, 0, 0);
     if (p.dim % 16 != 0)                                            // (the last head's 16-value steps reach into the padding)
         for (int i = tid; i < KT; i += WARPS * 32) *reinterpret_cast<uint4*>(ks + i * m.ldk + krow) = make_uint4(0, 0, 0, 0);
     // the mixture: this warp's query and 16 output heads
     const int mto = (p.out_heads + 15) / 16, qi_mix = warp / mto, h_mix = (warp - qi_mix * mto) * 16;
-    const bool mixes = qi_mix < count;                              // (qi_mix < bq follows)
+    const bool mixes = qi_mix < count;                              // (qi_mix < BQ follows)
     uint32_t tf[HT][4];
 #pragma unroll
     for (int k = 0; k < HT; ++k)
@@ -253,9 +263,13 @@ __global__ void __launch_bounds__(WARPS * 32, 1) talking_mma_kernel(TalkingParam
 #pragma unroll
     for (int i = 0; i < NVT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
     // the row of weights that this lane addresses
-    const int a_rho = min(rv + (lane & 15), rows - 1), a_head = min(hv * r + a_rho / bq, p.out_heads - 1), a_qi = a_rho % bq;
+    const int a_rho = min(rv + (lane & 15), rows - 1), a_head = min(hv * r + a_rho / BQ, p.out_heads - 1), a_qi = a_rho % BQ;
     const int units_k = p.kv_heads * m.mt, wpq = KT == 32 && units_k * 2 <= WARPS ? 2 : 1;
-    auto s_off = [&](int h, int kb, int qi) { return h * m.lds + ((((kb * bq + qi)) ^ (h & m.s_swz)) << 4); };
+    auto s_off = [&](int h, int kb, int qi) { return h * LDS + (((kb * BQ + qi) ^ (h & SWZ)) << 4); };
+    const int u_first = warp / wpq, kh_first = u_first / m.mt;
+    bool v_row[2];                                                  // this thread's rows of the unit are those of a query
+#pragma unroll
+    for (int e = 0; e < 2; ++e) v_row[e] = rv + g8 + e * 8 < rows && (rv + g8 + e * 8) % BQ < count;
 
     __syncthreads();
     bool bad = false;
@@ -263,10 +277,10 @@ __global__ void __launch_bounds__(WARPS * 32, 1) talking_mma_kernel(TalkingParam
         const uint32_t parity = (j - tb) & 1;
         if (__syncthreads_or(!tc::mbar_wait(&bars[0], parity))) { bad = true; break; }
         if (warp == 0) fetch(vs, m.ldv, p.v_cache, vrow, &bars[1], slot);
-        if (warp == 0 && j + 1 < te) slot_next = find(j + 1);
+        if (warp == 0 && j + 1 < te) page_next = page_of(j + 1);
         // (1) scores
         for (int i = warp; i < units_k * wpq; i += WARPS) {
-            const int u = i / wpq, kh = u / m.mt, r0 = (u - kh * m.mt) * 16;
+            const int u = i == warp ? u_first : i / wpq, kh = i == warp ? kh_first : u / m.mt, r0 = (u - kh * m.mt) * 16;
             const int kb0 = wpq == 2 ? (i & 1) * 16 : 0;            // first key
             const bool both = KT == 32 && wpq == 1;
             float s[4][4] = {};
@@ -290,7 +304,7 @@ __global__ void __launch_bounds__(WARPS * 32, 1) talking_mma_kernel(TalkingParam
             for (int e = 0; e < 2; ++e) {
                 const int rho = r0 + g8 + e * 8;
                 if (rho >= rows) continue;
-                const int g = rho / bq, qi = rho - g * bq, h = kh * r + g;
+                const int qi = rho % BQ, h = kh * r + rho / BQ;
 #pragma unroll
                 for (int n = 0; n < 4; ++n) {
                     if (n >= 2 && !both) break;
@@ -298,13 +312,15 @@ __global__ void __launch_bounds__(WARPS * 32, 1) talking_mma_kernel(TalkingParam
                     split_bf162(s[n][e * 2], s[n][e * 2 + 1], hi, low);
                     unsigned char* at = sh + s_off(h, kb0 / 8 + n, qi) + c4 * 4;
                     *reinterpret_cast<uint32_t*>(at) = hi;
-                    *reinterpret_cast<uint32_t*>(at + plane) = low;
+                    *reinterpret_cast<uint32_t*>(at + PLANE) = low;
                 }
             }
         }
         __syncthreads();
-        if (warp == 0 && j + 1 < te) fetch(ks, m.ldk, p.k_cache, krow, &bars[0], slot_next);
-        slot = slot_next;
+        if (warp == 0 && j + 1 < te) {
+            slot = slot_of(j + 1, page_next);
+            fetch(ks, m.ldk, p.k_cache, krow, &bars[0], slot);
+        }
         // (2) mixture, mask, softmax
         if (mixes) {
             float c[KT / 8][4] = {};
@@ -318,44 +334,52 @@ __global__ void __launch_bounds__(WARPS * 32, 1) talking_mma_kernel(TalkingParam
                     ldsm_x4_trans(b, at);
                     mma_bf16_16816(c[n], tf[k], b[0], b[1]);
                     mma_bf16_16816(c[n + 1], tf[k], b[2], b[3]);
-                    ldsm_x4_trans(b, at + plane);
+                    ldsm_x4_trans(b, at + PLANE);
                     mma_bf16_16816(c[n], tf[k], b[0], b[1]);
                     mma_bf16_16816(c[n + 1], tf[k], b[2], b[3]);
                 }
             if (mto > 1) bar_sync(1 + qi_mix, mto * 32);            // (the weights take the scores' place)
             else __syncwarp();
-            const int key0 = lo + j * KT + c4 * 2;
-            float top[2] = {mx[0], mx[1]};
+            const int k_first = lo + j * KT, key0 = k_first + c4 * 2;
 #pragma unroll
             for (int n = 0; n < KT / 8; ++n)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int key = key0 + n * 8 + (e & 1);
-                    c[n][e] = key >= q_lo && key <= q_pos ? c[n][e] * scale_log2 : -INFINITY;
-                    top[e >> 1] = fmaxf(top[e >> 1], c[n][e]);
-                }
+                for (int e = 0; e < 4; ++e) c[n][e] *= scale_log2;
+            if (k_first < q_lo || k_first + KT - 1 > q_pos) {       // (a tile inside the query's chunk is seen whole)
+#pragma unroll
+                for (int n = 0; n < KT / 8; ++n)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const int key = key0 + n * 8 + (e & 1);
+                        if (key < q_lo || key > q_pos) c[n][e] = -INFINITY;
+                    }
+            }
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
-                top[e] = fmaxf(top[e], __shfl_xor_sync(0xffffffffu, top[e], 1));
-                top[e] = fmaxf(top[e], __shfl_xor_sync(0xffffffffu, top[e], 2));
-                const float base = top[e] == -INFINITY ? 0.f : top[e], f = exp2f(mx[e] - base);
+                float top = mx[e];
+#pragma unroll
+                for (int n = 0; n < KT / 8; ++n) top = fmaxf(top, fmaxf(c[n][e * 2], c[n][e * 2 + 1]));
+                top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 1));
+                top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 2));
+                if (top <= mx[e] + RAISE) top = mx[e];
+                const float base = top == -INFINITY ? 0.f : top, f = exp2_hw(mx[e] - base);
                 const int h = h_mix + g8 + e * 8;
                 float l = 0.f;
 #pragma unroll
                 for (int n = 0; n < KT / 8; ++n) {
-                    const float x = exp2f(c[n][e * 2] - base), y = exp2f(c[n][e * 2 + 1] - base);
+                    const float x = exp2_hw(c[n][e * 2] - base), y = exp2_hw(c[n][e * 2 + 1] - base);
                     l += x + y;
                     if (h < p.out_heads) {
                         uint32_t hi, low;
                         split_bf162(x, y, hi, low);
                         unsigned char* at = sh + s_off(h, n, qi_mix) + c4 * 4;
                         *reinterpret_cast<uint32_t*>(at) = hi;
-                        *reinterpret_cast<uint32_t*>(at + plane) = low;
+                        *reinterpret_cast<uint32_t*>(at + PLANE) = low;
                     }
                 }
                 sum[e] = sum[e] * f + l;
-                mx[e] = top[e];
-                if (c4 == 0 && h < p.out_heads) fac[h * bq + qi_mix] = f;
+                mx[e] = top;
+                if (c4 == 0 && h < p.out_heads) fac[h * BQ + qi_mix] = f;
             }
         }
         if (__syncthreads_or(!tc::mbar_wait(&bars[1], parity))) { bad = true; break; }
@@ -363,33 +387,41 @@ __global__ void __launch_bounds__(WARPS * 32, 1) talking_mma_kernel(TalkingParam
         if (nn > 0) {
             float f[2];
 #pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const int rho = rv + g8 + e * 8, g = rho / bq;
-                f[e] = rho < rows && rho - g * bq < count ? fac[hv * rows + rho] : 0.f;
-            }
+            for (int e = 0; e < 2; ++e) f[e] = v_row[e] ? fac[hv * rows + rv + g8 + e * 8] : 1.f;
+            if (__any_sync(0xffffffffu, f[0] != 1.f || f[1] != 1.f)) {
 #pragma unroll
-            for (int i = 0; i < NVT; ++i) { acc[i][0] *= f[0]; acc[i][1] *= f[0]; acc[i][2] *= f[1]; acc[i][3] *= f[1]; }
+                for (int i = 0; i < NVT; ++i) { acc[i][0] *= f[0]; acc[i][1] *= f[0]; acc[i][2] *= f[1]; acc[i][3] *= f[1]; }
+            }
 #pragma unroll
             for (int k = 0; k < KT / 16; ++k) {
                 uint32_t a[4], al[4];
                 const unsigned char* at = sh + s_off(a_head, k * 2 + (lane >> 4), a_qi);
                 ldsm_x4(a, at);
-                ldsm_x4(al, at + plane);
-                const unsigned char* vrow_s = vs + (k * 16 + (lane & 15)) * m.ldv + (hv * p.vdim + n0 * 8 + (lane >> 4) * 8) * 2;
-#pragma unroll
-                for (int i = 0; i < NVT; i += 2) {
-                    if (i >= nn) break;
+                ldsm_x4(al, at + PLANE);
+                const unsigned char* v_at = vs + (k * 16 + (lane & 15)) * m.ldv + (hv * p.vdim + n0 * 8) * 2;
+                auto pair = [&](int i) {
                     uint32_t b[4];
-                    if (i + 1 < nn) {
-                        ldsm_x4_trans(b, vrow_s + i * 16);
-                        mma_bf16_16816(acc[i], a, b[0], b[1]);
-                        mma_bf16_16816(acc[i + 1], a, b[2], b[3]);
-                        mma_bf16_16816(acc[i], al, b[0], b[1]);
-                        mma_bf16_16816(acc[i + 1], al, b[2], b[3]);
-                    } else {
-                        ldsm_x2_trans(b[0], b[1], vs + (k * 16 + (lane & 15)) * m.ldv + (hv * p.vdim + (n0 + i) * 8) * 2);
-                        mma_bf16_16816(acc[i], a, b[0], b[1]);
-                        mma_bf16_16816(acc[i], al, b[0], b[1]);
+                    ldsm_x4_trans(b, v_at + (lane >> 4) * 16 + i * 16);
+                    mma_bf16_16816(acc[i], a, b[0], b[1]);
+                    mma_bf16_16816(acc[i + 1], a, b[2], b[3]);
+                    mma_bf16_16816(acc[i], al, b[0], b[1]);
+                    mma_bf16_16816(acc[i + 1], al, b[2], b[3]);
+                };
+                if (nn == NVT) {
+#pragma unroll
+                    for (int i = 0; i < NVT; i += 2) pair(i);
+                } else {
+#pragma unroll
+                    for (int i = 0; i < NVT; i += 2) {
+                        if (i >= nn) break;
+                        if (i + 1 < nn) {
+                            pair(i);
+                        } else {
+                            uint32_t b[2];
+                            ldsm_x2_trans(b[0], b[1], v_at + i * 16);
+                            mma_bf16_16816(acc[i], a, b[0], b[1]);
+                            mma_bf16_16816(acc[i], al, b[0], b[1]);
+                        }
                     }
                 }
             }
@@ -413,7 +445,7 @@ __global__ void __launch_bounds__(WARPS * 32, 1) talking_mma_kernel(TalkingParam
             sum[e] += __shfl_xor_sync(0xffffffffu, sum[e], 2);
             const int h = h_mix + g8 + e * 8;
             if (c4 == 0 && h < p.out_heads) {
-                fac[h * bq + qi_mix] = sum[e] > 0.f ? 1.f / sum[e] : 0.f;
+                fac[h * BQ + qi_mix] = sum[e] > 0.f ? 1.f / sum[e] : 0.f;
                 if (p.splits > 1)
                     p.lse_part[((size_t)(tok + qi_mix) * p.out_heads + h) * p.splits + split] = sum[e] > 0.f ? (mx[e] + log2f(sum[e])) / LOG2E : -INFINITY;
             }
@@ -422,10 +454,9 @@ __global__ void __launch_bounds__(WARPS * 32, 1) talking_mma_kernel(TalkingParam
     __syncthreads();
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
-        const int rho = rv + g8 + e * 8, g = rho / bq, qi = rho - g * bq;
-        if (nn <= 0 || rho >= rows || qi >= count) continue;
-        const int h = hv * r + g;
-        const float inv = fac[h * bq + qi];
+        const int rho = rv + g8 + e * 8, qi = rho % BQ, h = hv * r + rho / BQ;
+        if (nn <= 0 || !v_row[e]) continue;
+        const float inv = fac[h * BQ + qi];
 #pragma unroll
         for (int i = 0; i < NVT; ++i) {
             if (i >= nn) break;
@@ -472,8 +503,17 @@ int launch_mma(const TalkingParams* p, const MmaPlan& m, int tiles, cudaStream_t
         sl_launch(kern, dim3(p->splits, tiles), WARPS * 32, m.smem, s, *p, m);
         return SL_LAUNCH_CHECK();
     };
-    if (p->heads <= 16) return go(talking_mma_kernel<KT, NVT, 1>);
-    return p->heads <= 32 ? go(talking_mma_kernel<KT, NVT, 2>) : go(talking_mma_kernel<KT, NVT, 4>);
+    const int ht = (p->heads + 15) / 16;
+    if (ht == 1) {
+        if (m.bq == 16) return go(talking_mma_kernel<KT, NVT, 1, 16>);
+        if (m.bq == 8) return go(talking_mma_kernel<KT, NVT, 1, 8>);
+        return m.bq == 4 ? go(talking_mma_kernel<KT, NVT, 1, 4>) : go(talking_mma_kernel<KT, NVT, 1, 1>);
+    }
+    if (ht == 2) {
+        if (m.bq == 8) return go(talking_mma_kernel<KT, NVT, 2, 8>);
+        return m.bq == 4 ? go(talking_mma_kernel<KT, NVT, 2, 4>) : go(talking_mma_kernel<KT, NVT, 2, 1>);
+    }
+    return m.bq == 4 ? go(talking_mma_kernel<KT, NVT, 4, 4>) : go(talking_mma_kernel<KT, NVT, 4, 1>);
 }
 
 bool shape_ok(const TalkingParams* p) {
@@ -516,7 +556,7 @@ SL_API int sl_talking_mma(const TalkingParams* p, int tiles, int T, cudaStream_t
     const MmaPlan m = make_plan(p->heads, p->kv_heads, p->out_heads, p->v_heads, p->dim, p->vdim, p->tiles == nullptr);
     if (m.bq == 0) return -1;
     int rc;
-#define SL_TM(KT) (m.per_v <= 4 ? launch_mma<KT, 4>(p, m, tiles, s) : m.per_v <= 8 ? launch_mma<KT, 8>(p, m, tiles, s) : launch_mma<KT, 16>(p, m, tiles, s))
+#define SL_TM(KT) (m.per_v <= 8 ? launch_mma<KT, 8>(p, m, tiles, s) : launch_mma<KT, 16>(p, m, tiles, s))
     rc = m.kt == 32 ? SL_TM(32) : SL_TM(16);
 #undef SL_TM
     if (rc == 0 && p->splits > 1) {
