@@ -141,7 +141,7 @@ MmaPlan make_plan(int heads, int kv_heads, int out_heads, int v_heads, int dim, 
     const int dqp = (dim + 15) / 16 * 16, krow = kv_heads * dim * 2, vrow = v_heads * vdim * 2, mto = (out_heads + 15) / 16;
     const int hp = heads <= 16 ? 16 : heads <= 32 ? 32 : 64;      // (of the kernel's instances)
     for (int bq = decode ? 1 : 16; bq >= 1; bq = bq > 4 ? bq / 2 : bq - 3)      // 16, 8, 4, 1
-        for (int kt = 32; kt >= 16; kt /= 2) {
+        for (int kt = 64; kt >= 16; kt /= 2) {
             MmaPlan m = {};
             m.bq = bq; m.kt = kt;
             m.mt = (r * bq + 15) / 16;
@@ -149,7 +149,7 @@ MmaPlan make_plan(int heads, int kv_heads, int out_heads, int v_heads, int dim, 
             if (units > WARPS || bq * mto > WARPS || bq * hp > 256) continue;
             m.wpv = WARPS / units;
             m.per_v = ((vdim / 8 + m.wpv - 1) / m.wpv + 1) / 2 * 2;
-            if (m.per_v > 16) continue;
+            if (m.per_v > 16 || (kt == 64 && m.per_v > 8)) continue;
             m.q_swz = dqp % 64 == 0 ? 7 : 0;
             m.ldq = dqp * 2 + (m.q_swz ? 0 : 16);
             m.ldk = krow + (krow / 16 % 2 == 0 ? 16 : dim % 16 != 0 ? 32 : 0);
@@ -198,17 +198,26 @@ __global__ void __launch_bounds__(WARPS * 32, 1) talking_mma_kernel(TalkingParam
     const int* pt = p.page_table + (size_t)tile.w * p.pt_stride;
     const uint32_t krow = p.kv_heads * p.dim * 2, vrow = p.v_heads * p.vdim * 2;
 
-    // warp 0: page of this lane's key of tile j, and the key's cache slot (behind the last key: the last once more, never visible)
-    auto key_of = [&](int j) { return min(lo + j * KT + lane, end - 1); };
-    auto page_of = [&](int j) { return pt[key_of(j) / p.page_size]; };
-    auto slot_of = [&](int j, int page) -> long long {
-        const long long s = (long long)page * p.page_size + key_of(j) % p.page_size;
-        return guard_ok(p.guard, 32, s, p.num_slots) ? s : 0;
+    // warp 0: pages of this lane's keys of tile j, and the keys' cache slots (behind the last key: the last once more, never visible)
+    constexpr int KPL = (KT + 31) / 32;                              // keys per lane
+    auto key_of = [&](int j, int i) { return min(lo + j * KT + i * 32 + lane, end - 1); };
+    auto pages_of = [&](int j, int (&page)[KPL]) {
+#pragma unroll
+        for (int i = 0; i < KPL; ++i) page[i] = pt[key_of(j, i) / p.page_size];
     };
-    auto fetch = [&](unsigned char* dst, int ld, const void* cache, uint32_t row, uint64_t* bar, long long slot) {
+    auto slots_of = [&](int j, const int (&page)[KPL], long long (&slot)[KPL]) {
+#pragma unroll
+        for (int i = 0; i < KPL; ++i) {
+            const long long s = (long long)page[i] * p.page_size + key_of(j, i) % p.page_size;
+            slot[i] = guard_ok(p.guard, 32, s, p.num_slots) ? s : 0;
+        }
+    };
+    auto fetch = [&](unsigned char* dst, int ld, const void* cache, uint32_t row, uint64_t* bar, const long long (&slot)[KPL]) {
         if (lane == 0) tc::mbar_expect_tx(bar, KT * row);
         __syncwarp();
-        if (lane < KT) tc::bulk_load_1d(dst + lane * ld, (const unsigned char*)cache + (size_t)slot * row, row, bar);
+#pragma unroll
+        for (int i = 0; i < KPL; ++i)
+            if (lane < KT) tc::bulk_load_1d(dst + (i * 32 + lane) * ld, (const unsigned char*)cache + (size_t)slot[i] * row, row, bar);
     };
     if (tid == 0) {
         tc::mbar_init(&bars[0], 1);
@@ -216,12 +225,13 @@ __global__ void __launch_bounds__(WARPS * 32, 1) talking_mma_kernel(TalkingParam
         tc::mbar_fence_init();
         tc::fence_proxy_async_smem();
     }
-    long long slot = 0;
-    int page_next = 0;
+    long long slot[KPL] = {};
+    int page_next[KPL] = {};
     if (warp == 0) {
         __syncwarp();
         if (tb < te) {
-            slot = slot_of(tb, page_of(tb));
+            pages_of(tb, page_next);
+            slots_of(tb, page_next, slot);
             fetch(ks, m.ldk, p.k_cache, krow, &bars[0], slot);
         }
     }
@@ -264,7 +274,8 @@ __global__ void __launch_bounds__(WARPS * 32, 1) talking_mma_kernel(TalkingParam
     for (int i = 0; i < NVT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
     // the row of weights that this lane addresses
     const int a_rho = min(rv + (lane & 15), rows - 1), a_head = min(hv * r + a_rho / BQ, p.out_heads - 1), a_qi = a_rho % BQ;
-    const int units_k = p.kv_heads * m.mt, wpq = KT == 32 && units_k * 2 <= WARPS ? 2 : 1;
+    const int units_k = p.kv_heads * m.mt;
+    const int wpq = KT >= 64 && units_k * 4 <= WARPS ? 4 : KT >= 32 && units_k * 2 <= WARPS ? 2 : 1, keys_w = KT / wpq;      // warps of a unit, keys of each
     auto s_off = [&](int h, int kb, int qi) { return h * LDS + (((kb * BQ + qi) ^ (h & SWZ)) << 4); };
     const int u_first = warp / wpq, kh_first = u_first / m.mt;
     bool v_row[2];                                                  // this thread's rows of the unit are those of a query
@@ -277,48 +288,52 @@ __global__ void __launch_bounds__(WARPS * 32, 1) talking_mma_kernel(TalkingParam
         const uint32_t parity = (j - tb) & 1;
         if (__syncthreads_or(!tc::mbar_wait(&bars[0], parity))) { bad = true; break; }
         if (warp == 0) fetch(vs, m.ldv, p.v_cache, vrow, &bars[1], slot);
-        if (warp == 0 && j + 1 < te) page_next = page_of(j + 1);
+        if (warp == 0 && j + 1 < te) pages_of(j + 1, page_next);
         // (1) scores
         for (int i = warp; i < units_k * wpq; i += WARPS) {
             const int u = i == warp ? u_first : i / wpq, kh = i == warp ? kh_first : u / m.mt, r0 = (u - kh * m.mt) * 16;
-            const int kb0 = wpq == 2 ? (i & 1) * 16 : 0;            // first key
-            const bool both = KT == 32 && wpq == 1;
-            float s[4][4] = {};
             const int qr = kh * unit_rows + r0 + (lane & 15);
             const unsigned char* qrow = qs + qr * m.ldq;
-            const unsigned char* krow_s = ks + (kb0 + (lane & 7) + (lane >> 4) * 8) * m.ldk + kh * p.dim * 2 + ((lane >> 3) & 1) * 16;
+#pragma unroll
+            for (int x = 0; x < KT; x += 32) {                      // 32 keys (16 if the warp has no more)
+                if (x > 0 && x >= keys_w) break;
+                const int kb0 = (i - u * wpq) * keys_w + x;         // first key
+                const bool both = KT > 16 && x + 16 < keys_w;
+                float s[4][4] = {};
+                const unsigned char* krow_s = ks + (kb0 + (lane & 7) + (lane >> 4) * 8) * m.ldk + kh * p.dim * 2 + ((lane >> 3) & 1) * 16;
 #pragma unroll 4
-            for (int c = 0; c < dp; c += 2) {
-                uint32_t a[4], b[4];
-                ldsm_x4(a, qrow + (((c + (lane >> 4)) ^ (qr & m.q_swz)) << 4));
-                ldsm_x4(b, krow_s + c * 16);
-                mma_bf16_16816(s[0], a, b[0], b[1]);
-                mma_bf16_16816(s[1], a, b[2], b[3]);
-                if (both) {
-                    ldsm_x4(b, krow_s + 16 * m.ldk + c * 16);
-                    mma_bf16_16816(s[2], a, b[0], b[1]);
-                    mma_bf16_16816(s[3], a, b[2], b[3]);
+                for (int c = 0; c < dp; c += 2) {
+                    uint32_t a[4], b[4];
+                    ldsm_x4(a, qrow + (((c + (lane >> 4)) ^ (qr & m.q_swz)) << 4));
+                    ldsm_x4(b, krow_s + c * 16);
+                    mma_bf16_16816(s[0], a, b[0], b[1]);
+                    mma_bf16_16816(s[1], a, b[2], b[3]);
+                    if (both) {
+                        ldsm_x4(b, krow_s + 16 * m.ldk + c * 16);
+                        mma_bf16_16816(s[2], a, b[0], b[1]);
+                        mma_bf16_16816(s[3], a, b[2], b[3]);
+                    }
                 }
-            }
 #pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const int rho = r0 + g8 + e * 8;
-                if (rho >= rows) continue;
-                const int qi = rho % BQ, h = kh * r + rho / BQ;
+                for (int e = 0; e < 2; ++e) {
+                    const int rho = r0 + g8 + e * 8;
+                    if (rho >= rows) continue;
+                    const int qi = rho % BQ, h = kh * r + rho / BQ;
 #pragma unroll
-                for (int n = 0; n < 4; ++n) {
-                    if (n >= 2 && !both) break;
-                    uint32_t hi, low;
-                    split_bf162(s[n][e * 2], s[n][e * 2 + 1], hi, low);
-                    unsigned char* at = sh + s_off(h, kb0 / 8 + n, qi) + c4 * 4;
-                    *reinterpret_cast<uint32_t*>(at) = hi;
-                    *reinterpret_cast<uint32_t*>(at + PLANE) = low;
+                    for (int n = 0; n < 4; ++n) {
+                        if (n >= 2 && !both) break;
+                        uint32_t hi, low;
+                        split_bf162(s[n][e * 2], s[n][e * 2 + 1], hi, low);
+                        unsigned char* at = sh + s_off(h, kb0 / 8 + n, qi) + c4 * 4;
+                        *reinterpret_cast<uint32_t*>(at) = hi;
+                        *reinterpret_cast<uint32_t*>(at + PLANE) = low;
+                    }
                 }
             }
         }
         __syncthreads();
         if (warp == 0 && j + 1 < te) {
-            slot = slot_of(j + 1, page_next);
+            slots_of(j + 1, page_next, slot);
             fetch(ks, m.ldk, p.k_cache, krow, &bars[0], slot);
         }
         // (2) mixture, mask, softmax
@@ -557,7 +572,7 @@ SL_API int sl_talking_mma(const TalkingParams* p, int tiles, int T, cudaStream_t
     if (m.bq == 0) return -1;
     int rc;
 #define SL_TM(KT) (m.per_v <= 8 ? launch_mma<KT, 8>(p, m, tiles, s) : launch_mma<KT, 16>(p, m, tiles, s))
-    rc = m.kt == 32 ? SL_TM(32) : SL_TM(16);
+    rc = m.kt == 64 ? launch_mma<64, 8>(p, m, tiles, s) : m.kt == 32 ? SL_TM(32) : SL_TM(16);
 #undef SL_TM
     if (rc == 0 && p->splits > 1) {
         sl_launch(talking_merge_kernel, dim3(p->out_heads, T), 64, 0, s, *p);
