@@ -204,7 +204,10 @@ def assemble_pulunex_weights(cfg: PulunexConfig, tensors: Dict[str, torch.Tensor
     f32 = lambda t: t.to(torch.float32).to(device).contiguous()
     lin = lambda *parts: LinearWeight(dev(torch.cat(parts, 0) if len(parts) > 1 else parts[0]))
     cols = lambda t: share(t.t()).t()
-    row = lambda name, factor=1.0: f32(get(name).to(torch.float32).reshape(1).expand(H) * factor)
+
+    def row(name, factor=1.0):
+        """A norm's one number, spread over the row."""
+        return f32(get(name).to(torch.float32).expand(H) * factor)
 
     def attention(i, l):
         p, c = f"l{i}.mix.", l.mixer
