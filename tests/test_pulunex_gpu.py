@@ -193,7 +193,8 @@ def tol(dtype):
 
 
 SHAPES = [(4, 2, 16, 16), (6, 2, 40, 24), (3, 3, 128, 128), (20, 1, 64, 136), (2, 1, 256, 200), (4, 2, 9, 14), (1, 1, 8, 2), (1, 1, 8, 8), (6, 3, 24, 48), (5, 5, 13, 10),
-          (32, 8, 128, 128), (64, 8, 24, 16), (40, 4, 16, 136), (16, 16, 16, 32), (32, 32, 16, 16), (48, 3, 56, 24), (33, 11, 8, 8), (12, 12, 128, 64), (8, 4, 32, 256)]
+          (32, 8, 128, 128), (64, 8, 24, 16), (40, 4, 16, 136), (16, 16, 16, 32), (32, 32, 16, 16), (48, 3, 56, 24), (33, 11, 8, 8), (12, 12, 128, 64), (8, 4, 32, 256), (16, 16, 128, 128),
+          (32, 16, 128, 120), (64, 8, 128, 128), (24, 12, 96, 88), (12, 4, 192, 192), (8, 8, 256, 248)]
 SPANS = [[(0, 130), (70, 3), (200, 1), (5, 64)], [(150, 1), (3, 1), (0, 1), (256, 1)], [(127, 2)], [(0, 1)], [(300, 40)], [(0, 2), (64, 2), (63, 1)]]
 
 
